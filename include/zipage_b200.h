@@ -393,6 +393,68 @@ int zp_sample_sharded_emulated(zp_comm* const* comms, int world, const void* con
                                int64_t* const* tokens_outs, int n_rows, int vocab_shard, uint64_t seed,
                                int dtype, void* stream);
 
+/* ---- Decoders with an fp32 residual stream, windowed attention and matrix memories ------------------
+ * No counterpart in the reference (its models are Qwen2/Qwen3/Llama).  The Similorn decoder runs on
+ * these; each takes its constants as parameters. */
+
+/* x[n, :] = table[tokens[n], :] * scale + position vector, fp32, and its copy x_t as T (may be NULL).
+ * Position vector: entries 2i / 2i + 1 = sin / cos of 2 pi positions[n] turns[i]; turns [(hidden + 1)
+ * / 2] fp64 on the device, NULL = no position vector.  Ids outside [0, vocab) are clamped. */
+int zp_embed_position(const int64_t* tokens, const int64_t* positions, const void* table, const double* turns,
+                      float scale, float* x, void* x_t, int n_tokens, int hidden, int64_t vocab, int dtype,
+                      void* stream);
+
+/* out = T(x * rsqrt(mean(x^2) + eps) * (weight + weight_offset)) over fp32 rows x [n_rows, hidden]
+ * with an fp32 weight; weight == NULL: out = T(x). */
+int zp_rms_norm_f32(const float* x, const float* weight, float weight_offset, void* out, int n_rows,
+                    int hidden, float eps, int dtype, void* stream);
+
+/* out = T(0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3)))), n elements; out may be x. */
+int zp_gelu_tanh(const void* x, void* out, int64_t n, int dtype, void* stream);
+
+/* k [n_tokens, Hkv, D], v [n_tokens, Hkv, DV] (common row stride) -> rows slot_mapping[i] of k_cache
+ * [n_slots, Hkv, KP] and v_cache [n_slots, Hkv, VP]; the padding columns are left alone (the caller
+ * zeroes a cache once).  Slots outside [0, n_slots) store nothing. */
+int zp_store_kv_padded(const void* k, const void* v, void* k_cache, void* v_cache,
+                       const int32_t* slot_mapping, int n_tokens, int Hkv, int D, int DV, int KP, int VP,
+                       int64_t row_stride, int64_t n_slots, int dtype, void* stream);
+
+/* Softmax attention of a step's queries over paged keys, with a sliding window and a soft cap:
+ * score = q . k * scale; softcap > 0: score = softcap * tanh(score / softcap); the query at position p
+ * sees the keys j with 0 <= p - j < window (window 0: all j <= p).
+ * q [rows, Hq, D] (row stride), caches [n_pages, BS, Hkv, KP | VP] as zp_store_kv_padded leaves them,
+ * KP and VP multiples of 16, BS a multiple of 64, block_table [B, NBmax].  cu_seqlens_q [B + 1] (absolute
+ * rows of q and out; max_seqlen_q is their largest count) or NULL for one row per sequence;
+ * context_lens [B] counts each sequence's keys including this step's (0: padding row, skipped).
+ * 16-bit caches with KP, VP <= 256 and Hq / Hkv <= 16 take the tensor-core kernels (ZP_IMPL_SIMT: never), whose
+ * one-row form may need a workspace (zp_window_attention_workspace_bytes, span = min(window, NBmax *
+ * BS)).  Scores and softmax weights are fp32. */
+size_t zp_window_attention_workspace_bytes(int B, int Hq, int Hkv, int VP, int span);
+int zp_window_attention(const void* q, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens_q,
+                        const int32_t* context_lens, const int32_t* block_table, void* out, int B,
+                        int max_seqlen_q, int NBmax, int Hq, int Hkv, int D, int DV, int KP, int VP, int BS,
+                        int n_pages, int64_t q_stride, int64_t out_stride, float scale, float softcap,
+                        int window, int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream);
+
+/* One step of a matrix-memory (mLSTM) mixer over a batch of sequences, state to gated output:
+ *   i = cap tanh((gates_i + bias_i) / cap), f = log sigmoid(cap tanh((gates_f + bias_f) / cap))
+ *   m' = max(f + m, i);  S' = exp(f + m - m') S + exp(i - m') k v^T;  n' likewise with k
+ *   o = S'^T q qscale / (max(|n' . q qscale|, exp(-m')) + 1e-6)
+ *   out = T(o / rms(o) * norm_weight * sigmoid(g))          (rms over the head's vdim, eps inside)
+ * token after token of each sequence.  q, k [rows, H * dim], v, g [rows, H * vdim] with one row stride;
+ * gates [rows, 2 H] fp32 (input gates, then forget gates), gate_bias [2 H], norm_weight [H * vdim].
+ * State in fp32: state [n_slots, H, dim, VP] (VP >= vdim, a multiple of 4), state_n [n_slots, H, dim],
+ * state_m [n_slots, H]; slots [B].  cu_seqlens_q / context_lens as in zp_window_attention; a sequence
+ * whose context equals its rows starts from zero, whatever its slot holds.
+ * bf16 with cu_seqlens_q, dim <= 256 and vdim <= 512 takes the chunked tensor-core kernel
+ * (ZP_IMPL_SIMT: never). */
+int zp_mlstm(const void* q, const void* k, const void* v, const void* g, const float* gates,
+             const float* gate_bias, const float* norm_weight, const int32_t* cu_seqlens_q,
+             const int32_t* context_lens, const int32_t* slots, float* state, float* state_n, float* state_m,
+             void* out, int B, int H, int dim, int vdim, int VP, int n_slots, int64_t row_stride,
+             int64_t gates_stride, int64_t out_stride, float qscale, float gate_cap, float eps, int impl,
+             int dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -139,6 +139,39 @@ int zp_sched_compress_due(void* sched, const int32_t* handles, int n, int32_t* o
 int zp_sched_compress_inputs(void* sched, const int32_t* handles, int n, int32_t* tables, int table_width,
                              int32_t* targets, int target_width, int32_t* query_ids, uint8_t* compressed);
 
+/* ---- Portion steps: prompts computed in pieces beside decoded tokens --------------------------------
+ * No counterpart in the reference, whose step is either a prefill of whole prompts or a decode.  For
+ * models without KV compression: each sequence keeps every page, the slot that the reference uses for
+ * the observation window (query_id) names its recurrent state, and a step runs `counts[i]` of the
+ * tokens that sequence i has not computed yet.  The prefix cache is not used.
+ *
+ * zp_sched_schedule_portions picks the sequences and counts of one step: at most token_budget tokens
+ * (more only when more sequences than that wait for a single token each), single tokens first
+ * served; admits waiting sequences while slots, pages and budget last; when pages run out, the
+ * sequence admitted last gives its pages and slot back and is computed again later.  Returns how many. */
+int zp_sched_schedule_portions(void* sched, int token_budget, int32_t* out_handles, int32_t* out_counts, int capacity);
+
+/* The portions ran.  token_ids (may be null): one sampled token per sequence, appended where the
+ * sequence has nothing left to compute.  Returns how many finished, their handles in finished_out. */
+int zp_sched_commit_portions(void* sched, const int32_t* handles, const int32_t* counts, int n, const int32_t* token_ids,
+                             double now, int32_t* finished_out);
+
+/* Given tokens instead of sampled ones (replaying a trace): handle -1 admits a new sequence at once
+ * (a slot and pages must be free), otherwise the tokens follow a running sequence's.  Returns the
+ * handle.  zp_sched_close ends the sequence and gives back what it holds. */
+int zp_sched_feed(void* sched, int handle, const int32_t* token_ids, int n);
+int zp_sched_close(void* sched, int handle);
+
+/* Inputs of one portion step: input_ids / positions / slot_mapping per token, cu_seqlens_q [n + 1],
+ * context_lens [n] (tokens of the sequence including these), slots [n], block_tables [n, table_width]
+ * padded with -1.  Returns the widest table. */
+int zp_sched_portion_inputs(void* sched, const int32_t* handles, const int32_t* counts, int n, int32_t* input_ids,
+                            int32_t* positions, int32_t* slot_mapping, int32_t* cu_seqlens_q, int32_t* context_lens,
+                            int32_t* slots, int32_t* block_tables, int table_width);
+
+/* out[i] = tokens of sequence i that are not computed yet. */
+int zp_sched_pending(void* sched, const int32_t* handles, int n, int32_t* out);
+
 #ifdef __cplusplus
 }
 #endif

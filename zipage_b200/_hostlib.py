@@ -46,6 +46,12 @@ SIGNATURES = {
     "zp_sched_temperatures": (_I, [_P, _P, _I, _P]),
     "zp_sched_prefill_sizes": (_I, [_P, _P, _I, _P]),
     "zp_sched_prefill_inputs": (_I, [_P, _P, _I, _P, _P, _P, _P, _P, _P]),
+    "zp_sched_schedule_portions": (_I, [_P, _I, _P, _P, _I]),
+    "zp_sched_commit_portions": (_I, [_P, _P, _P, _I, _P, _D, _P]),
+    "zp_sched_feed": (_I, [_P, _I, _P, _I]),
+    "zp_sched_close": (_I, [_P, _I]),
+    "zp_sched_portion_inputs": (_I, [_P, _P, _P, _I] + [_P] * 7 + [_I]),
+    "zp_sched_pending": (_I, [_P, _P, _I, _P]),
     "zp_sched_compress_due": (_I, [_P, _P, _I, _P]),
     "zp_sched_compress_inputs": (_I, [_P, _P, _I, _P, _I, _P, _I, _P, _P]),
 }

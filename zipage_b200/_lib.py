@@ -77,6 +77,13 @@ SIGNATURES = {
     "zp_qk_norm_rope_store": (_I, [_P] * 5 + [_F] + [_P] * 7 + [_I, _P] + [_I] * 4 + [_L] * 3 + [_I, _P]),
     "zp_sample": (_I, [_P, _P, _P, _P, _I, _I, C.c_uint64, _I, _P]),
     "zp_prepare_decode": (_I, [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P]),
+    "zp_embed_position": (_I, [_P] * 4 + [_F, _P, _P, _I, _I, _L, _I, _P]),
+    "zp_rms_norm_f32": (_I, [_P, _P, _F, _P, _I, _I, _F, _I, _P]),
+    "zp_gelu_tanh": (_I, [_P, _P, _L, _I, _P]),
+    "zp_store_kv_padded": (_I, [_P] * 5 + [_I] * 6 + [_L, _L, _I, _P]),
+    "zp_window_attention_workspace_bytes": (_Z, [_I] * 5),
+    "zp_window_attention": (_I, [_P] * 7 + [_I] * 11 + [_L, _L, _F, _F, _I, _I, _I, _P, _Z, _P]),
+    "zp_mlstm": (_I, [_P] * 14 + [_I] * 6 + [_L] * 3 + [_F] * 3 + [_I, _I, _P]),
     "zp_comm_create": (_I, [_I, _I, _Z, _I, C.POINTER(_P)]),
     "zp_comm_segment": (_I, [_P, C.POINTER(_P), C.POINTER(_Z)]),
     "zp_comm_ipc_handle": (_I, [_P, _P]),
@@ -103,8 +110,11 @@ def load():
                 f"{LIB_PATH} is missing: build it with `python -m zipage_b200.build` "
                 "(there is no CPU or PyTorch fallback for these kernels)")
         lib = C.CDLL(str(LIB_PATH))
+        whole = LIB_PATH.name == "libzipage_b200.so"      # one family's library exports only its own symbols
         for name, (res, args) in SIGNATURES.items():
-            fn = getattr(lib, name)
+            fn = getattr(lib, name) if whole else getattr(lib, name, None)
+            if fn is None:
+                continue
             fn.restype, fn.argtypes = res, args
         _lib = lib
     return _lib

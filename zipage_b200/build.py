@@ -4,9 +4,14 @@
 parallel) and links them into zipage_b200/libzipage_b200.so next to this file.
 No GPU is needed to build.  Objects are rebuilt only when a source or header
 is newer than the object.
+
+A model family needs only some of the sources: `ensure(part)` hands out the full library when it is
+current and otherwise builds (once) a smaller one from that family's sources.
 """
 from __future__ import annotations
 
+import fcntl
+import hashlib
 import os
 import subprocess
 import sys
@@ -23,15 +28,64 @@ FLAGS = [
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
 ] + os.environ.get("ZIPAGE_NVCC_FLAGS", "").split()
 
+# sources of one model family (stems of csrc/*.cu)
+PARTS = {
+    "similorn": ("zp_api", "zp_host_sched", "zp_mlstm", "zp_mlstm_chunk", "zp_rows", "zp_step", "zp_tc",
+                 "zp_window_attn", "zp_window_attn_mma"),
+}
+
+
+def _headers():
+    return sorted(CSRC.glob("*.cuh")) + sorted((PKG.parent / "include").glob("*.h"))
+
 
 def _newest_header() -> float:
-    hdrs = list(CSRC.glob("*.cuh")) + list((PKG.parent / "include").glob("*.h"))
-    return max(h.stat().st_mtime for h in hdrs)
+    return max(h.stat().st_mtime for h in _headers())
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def _sources(part=None):
+    return sorted(CSRC.glob("*.cu")) if part is None else [CSRC / f"{n}.cu" for n in PARTS[part]]
+
+
+def _digest(part=None) -> str:
+    """What a library was built from: flags, headers and sources by content."""
+    h = hashlib.sha256(" ".join(FLAGS).encode())
+    for f in _headers() + _sources(part):
+        h.update(f.name.encode() + b"\0" + f.read_bytes())
+    return h.hexdigest()
+
+
+def library_path(part=None) -> Path:
+    return LIB if part is None else PKG / f"libzipage_b200_{part}.so"
+
+
+def _stamp(lib: Path) -> Path:
+    return lib.with_suffix(".so.src")
+
+
+def is_current(part=None) -> bool:
+    lib = library_path(part)
+    return lib.exists() and _stamp(lib).exists() and _stamp(lib).read_text() == _digest(part)
+
+
+def ensure(part=None) -> Path:
+    """A library that holds the family's kernels and is current with the sources, compiled if there
+    is none; the bindings load it from here on."""
+    if is_current():
+        part = None
+    elif not is_current(part):
+        with open(PKG / ".build.lock", "w") as lock:
+            fcntl.flock(lock, fcntl.LOCK_EX)
+            if not is_current(part):
+                build(part=part)
+    from . import _hostlib, _lib
+    _lib.LIB_PATH = _hostlib.LIB_PATH = library_path(part)
+    return library_path(part)
+
+
+def build(force: bool = False, verbose: bool = False, part=None) -> Path:
     OBJ.mkdir(exist_ok=True)
-    srcs = sorted(CSRC.glob("*.cu"))
+    srcs, lib = _sources(part), library_path(part)
     hdr_time = _newest_header()
     jobs = []
     for s in srcs:
@@ -53,13 +107,16 @@ def build(force: bool = False, verbose: bool = False) -> Path:
             if r.returncode:
                 raise RuntimeError(f"nvcc failed on {cmd[-3]}")
     objs = [str(OBJ / (s.stem + ".o")) for s in srcs]
-    if jobs or not LIB.exists():
-        cmd = [NVCC, "-shared", "-o", str(LIB), *objs, "-lcudart"]
+    if jobs or not is_current(part):
+        tmp = lib.with_suffix(f".so.{os.getpid()}")
+        cmd = [NVCC, "-shared", "-o", str(tmp), *objs, "-lcudart"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode:
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("link failed")
-    return LIB
+        os.replace(tmp, lib)
+        _stamp(lib).write_text(_digest(part))
+    return lib
 
 
 if __name__ == "__main__":

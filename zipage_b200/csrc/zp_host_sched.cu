@@ -97,6 +97,7 @@ struct List {
 struct Seq {
   Links lk;
   std::vector<int32_t> tokens, table, new_table, to_release;
+  int32_t computed = 0;   // portion steps: tokens whose keys and state exist
   int32_t num_tokens = 0, num_prompt = 0, num_cached = 0, last_token = 0, query_id = -1, max_tokens = 0;
   float temperature = 1.f;
   double time_prefilled = 0, time_finished = 0;
@@ -163,7 +164,7 @@ struct Sched {
   int allocate(Seq& s);
   void deallocate(Seq& s) {                // :119-123
     for (size_t i = s.table.size(); i-- > 0;) deallocate_block(s.table[i]);
-    s.num_cached = 0; s.prefilled = 0; s.table.clear();
+    s.num_cached = 0; s.prefilled = 0; s.computed = 0; s.table.clear();
   }
   void deallocate_to_release(Seq& s) {     // :125-127
     for (size_t i = s.to_release.size(); i-- > 0;) deallocate_block(s.to_release[i]);
@@ -188,6 +189,12 @@ struct Sched {
   int preempt_popped(int h);
   int schedule(int32_t* out, int cap, int32_t* is_prefill);
   int postprocess(const int32_t* hs, int n, const int32_t* toks, double now);
+
+  // ---- portion steps (no counterpart in the reference) ----
+  int grow(Seq& s, int tokens);
+  void finish(int h, double now);
+  int schedule_portions(int token_budget, int32_t* out, int32_t* counts, int cap);
+  int commit_portions(const int32_t* hs, const int32_t* counts, int n, const int32_t* toks, double now);
 };
 
 // ---- BlockManager ------------------------------------------------------------------------------
@@ -461,6 +468,113 @@ int Sched::postprocess(const int32_t* hs, int n, const int32_t* toks, double now
         deallocate_qid(s);
         last_finished.push_back(h);
       }
+    }
+  }
+  return (int)last_finished.size();
+}
+
+// ---- Portion steps ---------------------------------------------------------------------------------
+// Pages for the sequence's first `tokens` tokens; -1 when the pool has too few (nothing is taken).
+int Sched::grow(Seq& s, int tokens) {
+  const int need = (tokens + cfg.block_size - 1) / cfg.block_size - (int)s.table.size();
+  if (need > free_blocks.count) return -1;
+  for (int i = 0; i < need; ++i) {
+    const int id = free_blocks.head;
+    allocate_block(id);
+    s.table.push_back(id);
+  }
+  return 0;
+}
+
+void Sched::finish(int h, double now) {
+  Seq& s = seqs[h];
+  s.time_finished = now;
+  s.status = ZP_SEQ_FINISHED;
+  deallocate(s);
+  running.remove(seqs, h);
+  s.where = 0;
+  deallocate_qid(s);
+}
+
+// One batch of single decoded tokens beside portions of prompts.  Running sequences come in order of
+// admission; every one that waits for a single token gets it, the rest of the budget goes to
+// portions, first of running sequences, then of newly admitted ones (which need a slot and pages for
+// all their tokens).  When a running sequence needs a page and none is free, the one admitted last
+// gives everything back and is computed again later.
+int Sched::schedule_portions(int token_budget, int32_t* out, int32_t* counts, int cap) {
+  int singles = 0, n = 0;
+  for (int i = running.head; i >= 0; i = seqs[i].lk.next) singles += seqs[i].num_tokens - seqs[i].computed == 1;
+  int budget = token_budget > singles ? token_budget - singles : 0, preempted = 0;
+  for (int h = running.head; h >= 0 && n < cap;) {
+    Seq& s = seqs[h];
+    const int pending = s.num_tokens - s.computed;
+    int give = pending == 1 ? 1 : (pending < budget ? pending : budget);
+    while (give > 0 && grow(s, s.computed + give) < 0) {
+      const int victim = running.tail;
+      if (victim == h && running.count == 1 && n == 0)
+        return fail(ZP_SCHED_ERR_STATE, "schedule_portions: %d pages are too few for one sequence of %d tokens",
+                    cfg.num_blocks, s.computed + give);
+      running.remove(seqs, victim);
+      seqs[victim].where = 0;
+      const int rc = preempt_popped(victim);
+      if (rc < 0) return rc;
+      ++preempted;
+      if (victim == h) give = -1;
+    }
+    if (give < 0) break;               // the sequence itself was the last one admitted
+    const int next = s.lk.next;
+    if (give > 0) {
+      out[n] = h; counts[n++] = give;
+      if (pending > 1) budget -= give;
+    }
+    h = next;
+  }
+  while (!preempted && waiting.count && n < cap && budget > 0 && running.count < cfg.max_num_seqs) {
+    const int h = waiting.head;
+    Seq& s = seqs[h];
+    if (free_qids.empty()) break;
+    if (!can_allocate(s)) {
+      if (!running.count)
+        return fail(ZP_SCHED_ERR_STATE, "schedule_portions: a sequence of %d tokens needs more than the pool's %d pages",
+                    s.num_tokens, cfg.num_blocks);
+      break;
+    }
+    grow(s, s.num_tokens);
+    allocate_qid(s);
+    s.status = ZP_SEQ_RUNNING;
+    waiting.pop_front(seqs);
+    running.push_back(seqs, h);
+    s.where = 2;
+    const int give = s.num_tokens < budget ? s.num_tokens : budget;
+    out[n] = h; counts[n++] = give;
+    budget -= give;
+  }
+  return n;
+}
+
+// The portions ran.  A sequence with nothing left to compute takes its sampled token (when there
+// are sampled tokens) and may finish.
+int Sched::commit_portions(const int32_t* hs, const int32_t* counts, int n, const int32_t* toks, double now) {
+  last_finished.clear();
+  for (int i = 0; i < n; ++i) {
+    const int h = hs[i];
+    if (h < 0 || h >= (int)seqs.size()) return fail(ZP_SCHED_ERR_ARG, "commit_portions: bad handle %d", h);
+    Seq& s = seqs[h];
+    if (s.where != 2 || counts[i] < 1 || s.computed + counts[i] > s.num_tokens)
+      return fail(ZP_SCHED_ERR_STATE, "commit_portions: sequence %d cannot have run %d tokens", h, counts[i]);
+    s.computed += counts[i];
+    s.num_cached = s.computed;
+    if (s.computed < s.num_tokens || !toks) continue;
+    const int32_t t = toks[i];
+    s.tokens.push_back(t);
+    s.last_token = t;
+    ++s.num_tokens;
+    s.prefilled = 1;
+    const int done = s.num_tokens - s.num_prompt;
+    if (done == 1) s.time_prefilled = now;
+    if ((!s.ignore_eos && t == cfg.eos) || done >= s.max_tokens) {
+      finish(h, now);
+      last_finished.push_back(h);
     }
   }
   return (int)last_finished.size();
@@ -826,6 +940,109 @@ int zp_sched_compress_inputs(void* sched, const int32_t* handles, int n, int32_t
     compressed[i] = q.compressed;
   }
   return widest;
+}
+
+int zp_sched_schedule_portions(void* sched, int token_budget, int32_t* out_handles, int32_t* out_counts, int capacity) {
+  if (!sched || !out_handles || !out_counts || token_budget < 1 || capacity < 1)
+    return fail(ZP_SCHED_ERR_ARG, "zp_sched_schedule_portions: bad argument");
+  std::unique_lock<std::mutex> lock_(S(sched)->mu);
+  return S(sched)->schedule_portions(token_budget, out_handles, out_counts, capacity);
+}
+
+int zp_sched_commit_portions(void* sched, const int32_t* handles, const int32_t* counts, int n, const int32_t* token_ids,
+                             double now, int32_t* finished_out) {
+  if (!sched || (n > 0 && (!handles || !counts))) return fail(ZP_SCHED_ERR_ARG, "zp_sched_commit_portions: null argument");
+  std::unique_lock<std::mutex> lock_(S(sched)->mu);
+  const int done = S(sched)->commit_portions(handles, counts, n, token_ids, now);
+  if (done > 0 && finished_out) memcpy(finished_out, S(sched)->last_finished.data(), sizeof(int32_t) * done);
+  return done;
+}
+
+int zp_sched_feed(void* sched, int handle, const int32_t* token_ids, int n) {
+  if (!sched || !token_ids || n < 1) return fail(ZP_SCHED_ERR_ARG, "zp_sched_feed: null argument or no tokens");
+  Sched* s = S(sched);
+  std::unique_lock<std::mutex> lock_(s->mu);
+  const bool fresh = handle < 0;
+  if (fresh) {
+    if (s->free_qids.empty()) return fail(ZP_SCHED_ERR_STATE, "zp_sched_feed: all %d slots are taken", s->cfg.max_concurrency);
+    s->seqs.emplace_back();
+    handle = (int)s->seqs.size() - 1;
+  } else if (bad_handle(s, handle) || s->seqs[handle].where != 2) {
+    return fail(ZP_SCHED_ERR_ARG, "zp_sched_feed: sequence %d is not running", handle);
+  }
+  Seq& q = s->seqs[handle];
+  if (s->grow(q, q.num_tokens + n) < 0) {
+    if (fresh) s->seqs.pop_back();
+    return fail(ZP_SCHED_ERR_STATE, "zp_sched_feed: %d free pages are too few for %d more tokens", s->free_blocks.count, n);
+  }
+  if (fresh) {
+    s->allocate_qid(q);
+    q.status = ZP_SEQ_RUNNING;
+    q.max_tokens = INT32_MAX;
+    q.ignore_eos = 1;
+    s->running.push_back(s->seqs, handle);
+    q.where = 2;
+  }
+  q.tokens.insert(q.tokens.end(), token_ids, token_ids + n);
+  q.num_tokens += n;
+  q.num_prompt = q.num_tokens;
+  q.last_token = token_ids[n - 1];
+  return handle;
+}
+
+int zp_sched_close(void* sched, int handle) {
+  if (!sched) return fail(ZP_SCHED_ERR_ARG, "zp_sched_close: null argument");
+  Sched* s = S(sched);
+  std::unique_lock<std::mutex> lock_(s->mu);
+  if (bad_handle(s, handle) || s->seqs[handle].where != 2)
+    return fail(ZP_SCHED_ERR_ARG, "zp_sched_close: sequence %d is not running", handle);
+  s->finish(handle, 0.0);
+  std::vector<int32_t>().swap(s->seqs[handle].tokens);
+  return 0;
+}
+
+int zp_sched_portion_inputs(void* sched, const int32_t* handles, const int32_t* counts, int n, int32_t* input_ids,
+                            int32_t* positions, int32_t* slot_mapping, int32_t* cu_seqlens_q, int32_t* context_lens,
+                            int32_t* slots, int32_t* block_tables, int table_width) {
+  if (!sched || (n > 0 && (!handles || !counts || !input_ids || !positions || !slot_mapping || !cu_seqlens_q ||
+                           !context_lens || !slots || !block_tables)))
+    return fail(ZP_SCHED_ERR_ARG, "zp_sched_portion_inputs: null argument");
+  Sched* s = S(sched);
+  std::unique_lock<std::mutex> lock_(s->mu);
+  const int BS = s->cfg.block_size;
+  int widest = 0, t = 0;
+  if (n > 0) cu_seqlens_q[0] = 0;
+  for (int i = 0; i < n; ++i) {
+    if (bad_handle(s, handles[i])) return fail(ZP_SCHED_ERR_ARG, "zp_sched_portion_inputs: bad handle %d", handles[i]);
+    const Seq& q = s->seqs[handles[i]];
+    const int lo = q.computed, hi = lo + counts[i], nb = (hi + BS - 1) / BS;
+    if (counts[i] < 1 || hi > q.num_tokens || nb > (int)q.table.size() || q.query_id < 0)
+      return fail(ZP_SCHED_ERR_STATE, "zp_sched_portion_inputs: sequence %d cannot run %d tokens", handles[i], counts[i]);
+    if (nb > table_width) return fail(ZP_SCHED_ERR_ARG, "zp_sched_portion_inputs: a table of %d pages, %d columns", nb, table_width);
+    if (nb > widest) widest = nb;
+    for (int p = lo; p < hi; ++p, ++t) {
+      input_ids[t] = q.tokens[p];
+      positions[t] = p;
+      slot_mapping[t] = q.table[p / BS] * BS + p % BS;
+    }
+    cu_seqlens_q[i + 1] = t;
+    context_lens[i] = hi;
+    slots[i] = q.query_id;
+    int32_t* row = block_tables + (size_t)i * table_width;
+    for (int j = 0; j < table_width; ++j) row[j] = j < nb ? q.table[j] : -1;
+  }
+  return widest;
+}
+
+int zp_sched_pending(void* sched, const int32_t* handles, int n, int32_t* out) {
+  if (!sched || (n > 0 && (!handles || !out))) return fail(ZP_SCHED_ERR_ARG, "zp_sched_pending: null argument");
+  Sched* s = S(sched);
+  std::unique_lock<std::mutex> lock_(s->mu);
+  for (int i = 0; i < n; ++i) {
+    if (bad_handle(s, handles[i])) return fail(ZP_SCHED_ERR_ARG, "zp_sched_pending: bad handle %d", handles[i]);
+    out[i] = s->seqs[handles[i]].num_tokens - s->seqs[handles[i]].computed;
+  }
+  return 0;
 }
 
 }  // extern "C"

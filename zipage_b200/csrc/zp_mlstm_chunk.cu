@@ -1,0 +1,376 @@
+// Matrix-memory (mLSTM) mixer over prompt portions, 64 tokens at a time on warp-level tensor-core MMAs
+// (bf16 projections, fp32 state).
+//
+// With F_t the running sum of the log forget gates inside a chunk, u_j = i_j - F_j and
+// M_t = max(m, max_{j<=t} u_j) (m: the running maximum the chunk starts from), the recurrence unrolls to
+//   m_t = M_t + F_t
+//   S_t^T q = exp(m - M_t) S^T q + sum_{j<=t} exp(u_j - M_t) (k_j . q) v_j
+// and the state after the chunk is exp(m - M_C) S + sum_j exp(u_j - M_C) k_j v_j^T; every exponent is
+// <= 0.  n is one more value column whose v is 1.
+//
+// One block per (64-wide value tile, head, sequence) walks the chunks in order.  Its state tile
+// [dim, 64 + 1] stays in fp32 MMA accumulators; only 16-bit operand copies of it pass through shared
+// memory.  Whatever is fp32 in the equations enters a product as a pair of bf16 numbers (hi + lo): the state
+// in S^T q, the decayed scores, and the decayed values of the state update; q, k and v are bf16
+// already.  The blocks of a head form a cluster and exchange per-row sums of squares for the head norm
+// through distributed shared memory, so the normalised, gated output leaves the kernel in one pass.
+#include "zp_mlstm.cuh"
+#include "zp_mma.cuh"
+
+namespace zp {
+
+constexpr int MC_THREADS = 256;
+constexpr int MC_C = 64;            // tokens per chunk
+constexpr int MC_VT = 64;           // value columns per block
+constexpr int MC_RB = 144;          // bytes of a 72-column bf16 row (an odd number of 16-byte chunks)
+
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  const float2 f = __bfloat1622float2(h);
+  lo = pack2<__nv_bfloat16>(a - f.x, b - f.y);
+}
+__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t (&r)[2], const void* smem_row) {
+  const uint32_t a = static_cast<uint32_t>(__cvta_generic_to_shared(smem_row));
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(a));
+}
+
+// B fragments of the 8-column blocks [first, first + 5) (or + 4) of 16 rows of a 72-column tile
+template <typename F>
+__device__ __forceinline__ void for_blocks(const unsigned char* tile, int row0, int half, int lane, F&& fn) {
+  const unsigned char* r = tile + (row0 + (lane & 15)) * MC_RB;
+  uint32_t b[4];
+  ldmatrix_x4_trans(b, r + half * 64 + (lane >> 4) * 16);
+  fn(0, b[0], b[1]); fn(1, b[2], b[3]);
+  ldmatrix_x4_trans(b, r + half * 64 + 32 + (lane >> 4) * 16);
+  fn(2, b[0], b[1]); fn(3, b[2], b[3]);
+  if (half) {
+    uint32_t c[2];
+    ldmatrix_x2_trans(c, r + 128);
+    fn(4, c[0], c[1]);
+  }
+}
+
+// Shared memory, bytes: Q and K tiles, V tile, hi and lo of the state tile, hi and lo of the scores
+// (reused by the decayed values), per-row floats.
+template <int DP> struct ChunkSmem {
+  static constexpr int RB = DP * 2 + 16;
+  static constexpr int Q = 0, K = Q + MC_C * RB, V = K + MC_C * RB, S = V + MC_C * MC_RB, P = S + 2 * DP * MC_RB,
+                       F = P + 2 * MC_C * MC_RB, TOTAL = F + 12 * MC_C * 4;
+};
+
+template <int DP>
+__global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_kernel(const MlstmArgs a) {
+  using T = __nv_bfloat16;
+  using L = ChunkSmem<DP>;
+  constexpr int MB = DP / 64;                    // 16-row blocks of the state tile per warp
+  extern __shared__ __align__(128) unsigned char smem[];
+  const int vt = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
+  const MlstmSeq sq = mlstm_seq(a, b);
+  if (sq.count == 0) return;                     // the same decision in every block of the cluster
+  const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  const int rg = warp & 3, half = warp >> 2;     // 16-row group, column half of every product
+  unsigned char *sQ = smem + L::Q, *sK = smem + L::K, *sV = smem + L::V;
+  unsigned char *sSh = smem + L::S, *sSl = sSh + DP * MC_RB;
+  unsigned char *sPh = smem + L::P, *sPl = sPh + MC_C * MC_RB;
+  float* fl = reinterpret_cast<float*>(smem + L::F);
+  float *sM = fl, *sU = fl + 64, *sA = fl + 128, *sE = fl + 192, *sW = fl + 256, *sDen = fl + 320, *sR = fl + 384;
+  float *sSq = fl + 448;                         // [2 parities][2 halves][64] (read by the cluster)
+  float *sMisc = fl + 704;                       // running maximum, decay of the state over the chunk
+  const int c0 = vt * MC_VT, vcols = min(MC_VT, a.vdim - c0);
+  const int nk16 = (a.dim + 15) / 16;
+  const int64_t head = (int64_t)sq.slot * a.H + h;
+  const T* qb = reinterpret_cast<const T*>(a.q) + (int64_t)h * a.dim;
+  const T* kb = reinterpret_cast<const T*>(a.k) + (int64_t)h * a.dim;
+  const T* vb = reinterpret_cast<const T*>(a.v) + (int64_t)h * a.vdim + c0;
+  const bool vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.row_stride % 8 == 0 &&
+                   ((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) % 16 == 0;
+
+  // columns 64..71 of the value tile: the column of ones that carries n, then zeros
+  for (int i = tid; i < MC_C * 8; i += MC_THREADS)
+    *reinterpret_cast<T*>(sV + (i >> 3) * MC_RB + 128 + (i & 7) * 2) = Elem<T>::from_f32((i & 7) == 0 ? 1.f : 0.f);
+  if (tid == 0) sMisc[0] = sq.fresh ? 0.f : a.m[head];
+
+  float s[MB][5][4];                             // the state tile: rows (rg + 4 i) * 16 + g (+ 8)
+#pragma unroll
+  for (int i = 0; i < MB; ++i)
+#pragma unroll
+    for (int cb = 0; cb < 5; ++cb)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int r = (rg + 4 * i) * 16 + g + (j >> 1) * 8, c = half * 32 + cb * 8 + 2 * tq + (j & 1);
+        float x = 0.f;
+        if (!sq.fresh && r < a.dim) {
+          if (cb < 4) { if (c0 + c < a.VP) x = a.S[(head * a.dim + r) * a.VP + c0 + c]; }
+          else if (c == 64) x = a.n[head * a.dim + r];
+        }
+        s[i][cb][j] = x;
+      }
+
+  auto load_chunk = [&](int t0, int n) {
+    const int64_t row0 = sq.row0 + t0;
+    if (vec) {
+      for (int i = tid; i < MC_C * (DP / 8); i += MC_THREADS) {
+        const int r = i / (DP / 8), c = i % (DP / 8);
+        const int ok = (r < n && c * 8 < a.dim) ? 16 : 0;
+        const int64_t off = ok ? (row0 + r) * a.row_stride + c * 8 : 0;
+        cp_async16(sQ + r * L::RB + c * 16, qb + off, ok);
+        cp_async16(sK + r * L::RB + c * 16, kb + off, ok);
+      }
+      for (int i = tid; i < MC_C * 8; i += MC_THREADS) {
+        const int r = i >> 3, c = i & 7;
+        const int ok = (r < n && c * 8 < vcols) ? 16 : 0;
+        cp_async16(sV + r * MC_RB + c * 16, vb + (ok ? (row0 + r) * a.row_stride + c * 8 : 0), ok);
+      }
+    } else {
+      const T z = Elem<T>::from_f32(0.f);
+      for (int i = tid; i < MC_C * DP; i += MC_THREADS) {
+        const int r = i / DP, c = i % DP;
+        const bool ok = r < n && c < a.dim;
+        *reinterpret_cast<T*>(sQ + r * L::RB + c * 2) = ok ? qb[(row0 + r) * a.row_stride + c] : z;
+        *reinterpret_cast<T*>(sK + r * L::RB + c * 2) = ok ? kb[(row0 + r) * a.row_stride + c] : z;
+      }
+      for (int i = tid; i < MC_C * MC_VT; i += MC_THREADS) {
+        const int r = i >> 6, c = i & 63;
+        *reinterpret_cast<T*>(sV + r * MC_RB + c * 2) = (r < n && c < vcols) ? vb[(row0 + r) * a.row_stride + c] : z;
+      }
+    }
+    cp_async_commit();
+  };
+  // one warp: gates of the chunk, their running sums and maxima (two tokens per lane)
+  auto gates = [&](int t0, int n) {
+    float f[2], u[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int t = 2 * lane + j;
+      const int64_t row = sq.row0 + t0 + t;
+      f[j] = t < n ? log_forget_gate(a, row, h) : 0.f;
+      u[j] = t < n ? log_input_gate(a, row, h) : -INFINITY;
+    }
+    float F = f[0] + f[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const float x = __shfl_up_sync(0xffffffffu, F, o); if (lane >= o) F += x; }
+    const float F1 = F, F0 = F - f[1];
+    u[0] -= F0; u[1] -= F1;
+    float mx = fmaxf(u[0], u[1]);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const float x = __shfl_up_sync(0xffffffffu, mx, o); if (lane >= o) mx = fmaxf(mx, x); }
+    float before = __shfl_up_sync(0xffffffffu, mx, 1);
+    const float m = sMisc[0];
+    before = lane == 0 ? m : fmaxf(m, before);
+    const float M0 = fmaxf(before, u[0]), M1 = fmaxf(M0, u[1]);
+    const float MC = __shfl_sync(0xffffffffu, M1, 31), FC = __shfl_sync(0xffffffffu, F1, 31);
+    const int t = 2 * lane;
+    sM[t] = M0; sM[t + 1] = M1; sU[t] = u[0]; sU[t + 1] = u[1];
+    sA[t] = expf(m - M0); sA[t + 1] = expf(m - M1);
+    sE[t] = expf(-(M0 + F0)); sE[t + 1] = expf(-(M1 + F1));
+    sW[t] = expf(u[0] - MC); sW[t + 1] = expf(u[1] - MC);
+    __syncwarp();
+    if (lane == 0) { sMisc[1] = expf(m - MC); sMisc[0] = MC + FC; }
+  };
+
+  __syncthreads();
+  const int row_a = rg * 16 + g, row_b = row_a + 8;   // this thread's two tokens of the chunk
+  for (int t0 = 0, par = 0; t0 < sq.count; t0 += MC_C, par ^= 1) {
+    const int n = min(MC_C, sq.count - t0);
+    load_chunk(t0, n);
+    if (warp == 0) gates(t0, n);
+    // 16-bit operand copies of the state tile
+#pragma unroll
+    for (int i = 0; i < MB; ++i)
+#pragma unroll
+      for (int cb = 0; cb < 5; ++cb) {
+        if (cb == 4 && !half) continue;
+        const int r = (rg + 4 * i) * 16 + g, off = (half * 32 + cb * 8 + 2 * tq) * 2;
+        uint32_t hi, lo;
+        split_bf16(s[i][cb][0], s[i][cb][1], hi, lo);
+        *reinterpret_cast<uint32_t*>(sSh + r * MC_RB + off) = hi;
+        *reinterpret_cast<uint32_t*>(sSl + r * MC_RB + off) = lo;
+        split_bf16(s[i][cb][2], s[i][cb][3], hi, lo);
+        *reinterpret_cast<uint32_t*>(sSh + (r + 8) * MC_RB + off) = hi;
+        *reinterpret_cast<uint32_t*>(sSl + (r + 8) * MC_RB + off) = lo;
+      }
+    cp_async_wait<0>();
+    __syncthreads();
+
+    float acc[5][4], p[4][4];
+#pragma unroll
+    for (int i = 0; i < 5; ++i) { acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f; }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { p[i][0] = p[i][1] = p[i][2] = p[i][3] = 0.f; }
+    const bool scores = half * 32 <= rg * 16 + 15;     // else every key of this half is later than the rows
+#pragma unroll 2
+    for (int kk = 0; kk < nk16; ++kk) {
+      uint32_t qa[4];
+      ldmatrix_x4(qa, sQ + (rg * 16 + (lane & 15)) * L::RB + kk * 32 + (lane >> 4) * 16);
+      for_blocks(sSh, kk * 16, half, lane, [&](int i, uint32_t b0, uint32_t b1) { mma16816<T>(acc[i], qa, b0, b1); });
+      for_blocks(sSl, kk * 16, half, lane, [&](int i, uint32_t b0, uint32_t b1) { mma16816<T>(acc[i], qa, b0, b1); });
+      if (scores) {
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          uint32_t bf[4];
+          ldmatrix_x4(bf, sK + (half * 32 + np * 16 + (lane & 7) + (lane >> 4) * 8) * L::RB + kk * 32 + ((lane >> 3) & 1) * 16);
+          mma16816<T>(p[2 * np], qa, bf[0], bf[1]);
+          mma16816<T>(p[2 * np + 1], qa, bf[2], bf[3]);
+        }
+      }
+    }
+    if (scores) {
+      const float Ma = sM[row_a], Mb = sM[row_b];
+#pragma unroll
+      for (int nb = 0; nb < 4; ++nb) {
+        const int key = half * 32 + nb * 8 + 2 * tq;
+        const float u0 = sU[key], u1 = sU[key + 1];
+        const float p0 = key <= row_a ? p[nb][0] * a.qscale * __expf(u0 - Ma) : 0.f;
+        const float p1 = key + 1 <= row_a ? p[nb][1] * a.qscale * __expf(u1 - Ma) : 0.f;
+        const float p2 = key <= row_b ? p[nb][2] * a.qscale * __expf(u0 - Mb) : 0.f;
+        const float p3 = key + 1 <= row_b ? p[nb][3] * a.qscale * __expf(u1 - Mb) : 0.f;
+        uint32_t hi, lo;
+        split_bf16(p0, p1, hi, lo);
+        *reinterpret_cast<uint32_t*>(sPh + row_a * MC_RB + key * 2) = hi;
+        *reinterpret_cast<uint32_t*>(sPl + row_a * MC_RB + key * 2) = lo;
+        split_bf16(p2, p3, hi, lo);
+        *reinterpret_cast<uint32_t*>(sPh + row_b * MC_RB + key * 2) = hi;
+        *reinterpret_cast<uint32_t*>(sPl + row_b * MC_RB + key * 2) = lo;
+      }
+    }
+    {
+      const float fa = sA[row_a] * a.qscale, fb = sA[row_b] * a.qscale;
+#pragma unroll
+      for (int i = 0; i < 5; ++i) { acc[i][0] *= fa; acc[i][1] *= fa; acc[i][2] *= fb; acc[i][3] *= fb; }
+    }
+    __syncthreads();
+    for (int kk = 0; kk <= rg; ++kk) {                 // keys 16 kk .. 16 kk + 15 of rows up to 16 rg + 15
+      uint32_t ph[4], pl[4];
+      ldmatrix_x4(ph, sPh + (rg * 16 + (lane & 15)) * MC_RB + kk * 32 + (lane >> 4) * 16);
+      ldmatrix_x4(pl, sPl + (rg * 16 + (lane & 15)) * MC_RB + kk * 32 + (lane >> 4) * 16);
+      for_blocks(sV, kk * 16, half, lane, [&](int i, uint32_t b0, uint32_t b1) {
+        mma16816<T>(acc[i], ph, b0, b1);
+        mma16816<T>(acc[i], pl, b0, b1);
+      });
+    }
+    if (half && tq == 0) { sDen[row_a] = acc[4][0]; sDen[row_b] = acc[4][2]; }   // n . q, decayed like the rest
+    __syncthreads();
+    const float da = 1.f / (fmaxf(fabsf(sDen[row_a]), sE[row_a]) + MLSTM_DEN_EPS);
+    const float db = 1.f / (fmaxf(fabsf(sDen[row_b]), sE[row_b]) + MLSTM_DEN_EPS);
+    float qa2 = 0.f, qb2 = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {                      // (columns past vdim are zero)
+      acc[i][0] *= da; acc[i][1] *= da; acc[i][2] *= db; acc[i][3] *= db;
+      qa2 = fmaf(acc[i][0], acc[i][0], fmaf(acc[i][1], acc[i][1], qa2));
+      qb2 = fmaf(acc[i][2], acc[i][2], fmaf(acc[i][3], acc[i][3], qb2));
+    }
+    qa2 += __shfl_xor_sync(0xffffffffu, qa2, 1); qa2 += __shfl_xor_sync(0xffffffffu, qa2, 2);
+    qb2 += __shfl_xor_sync(0xffffffffu, qb2, 1); qb2 += __shfl_xor_sync(0xffffffffu, qb2, 2);
+    if (tq == 0) { sSq[(par * 2 + half) * 64 + row_a] = qa2; sSq[(par * 2 + half) * 64 + row_b] = qb2; }
+    // decayed values (and the decayed column of ones), over the scores' shared memory
+    for (int i = tid; i < MC_C * 36; i += MC_THREADS) {
+      const int r = i / 36, c = i % 36;
+      const float w = sW[r];
+      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sV + r * MC_RB + c * 4));
+      uint32_t hi, lo;
+      split_bf16(v.x * w, v.y * w, hi, lo);
+      *reinterpret_cast<uint32_t*>(sPh + r * MC_RB + c * 4) = hi;
+      *reinterpret_cast<uint32_t*>(sPl + r * MC_RB + c * 4) = lo;
+    }
+    if (cluster_size() > 1) cluster_sync(); else __syncthreads();
+    if (tid < MC_C) {
+      float ss = 0.f;
+      for (uint32_t r = 0; r < cluster_size(); ++r)
+        ss += ld_cluster(&sSq[par * 128 + tid], r) + ld_cluster(&sSq[par * 128 + 64 + tid], r);
+      sR[tid] = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
+    }
+    const float decay = sMisc[1];
+#pragma unroll
+    for (int i = 0; i < MB; ++i) {
+      if ((rg + 4 * i) * 16 < a.dim) {
+#pragma unroll
+        for (int cb = 0; cb < 5; ++cb) { s[i][cb][0] *= decay; s[i][cb][1] *= decay; s[i][cb][2] *= decay; s[i][cb][3] *= decay; }
+      }
+    }
+    for (int kk = 0; kk * 16 < n; ++kk) {
+      uint32_t ka[MB][4];
+#pragma unroll
+      for (int i = 0; i < MB; ++i)
+        ldmatrix_x4_trans(ka[i], sK + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * L::RB + (rg + 4 * i) * 32 + ((lane >> 3) & 1) * 16);
+      auto add = [&](int cb, uint32_t b0, uint32_t b1) {
+#pragma unroll
+        for (int i = 0; i < MB; ++i) mma16816<T>(s[i][cb], ka[i], b0, b1);
+      };
+      for_blocks(sPh, kk * 16, half, lane, add);
+      for_blocks(sPl, kk * 16, half, lane, add);
+    }
+    __syncthreads();                                   // tiles free for the next chunk; sR visible
+    const float ra = sR[row_a], rb = sR[row_b];
+    const int64_t grow = sq.row0 + t0;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = c0 + half * 32 + i * 8 + 2 * tq;
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const int r = y ? row_b : row_a;
+        if (r >= n) continue;
+        const float rr = y ? rb : ra;
+        const int64_t e = (int64_t)h * a.vdim + c;
+        const T* gp = reinterpret_cast<const T*>(a.g) + (grow + r) * a.row_stride + e;
+        T* op = reinterpret_cast<T*>(a.out) + (grow + r) * a.out_stride + e;
+        float o[2];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+          o[j] = c + j < a.vdim ? acc[i][2 * y + j] * rr * a.norm_weight[e + j] / (1.f + __expf(-Elem<T>::to_f32(gp[j]))) : 0.f;
+        if (vec && a.out_stride % 2 == 0) { if (c < a.vdim) *reinterpret_cast<uint32_t*>(op) = pack2<T>(o[0], o[1]); }
+        else {
+          if (c < a.vdim) op[0] = Elem<T>::from_f32(o[0]);
+          if (c + 1 < a.vdim) op[1] = Elem<T>::from_f32(o[1]);
+        }
+      }
+    }
+  }
+
+  if (cluster_size() > 1) cluster_sync();              // peers may still be reading this block's sums
+#pragma unroll
+  for (int i = 0; i < MB; ++i)
+#pragma unroll
+    for (int cb = 0; cb < 5; ++cb)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int r = (rg + 4 * i) * 16 + g + (j >> 1) * 8, c = half * 32 + cb * 8 + 2 * tq + (j & 1);
+        if (r >= a.dim) continue;
+        if (cb < 4) { if (c0 + c < a.VP) a.S[(head * a.dim + r) * a.VP + c0 + c] = s[i][cb][j]; }
+        else if (c == 64 && vt == 0) a.n[head * a.dim + r] = s[i][cb][j];
+      }
+  if (vt == 0 && tid == 0) a.m[head] = sMisc[0];
+}
+
+bool mlstm_chunk_supports(const MlstmArgs& a, int dtype) {
+  return dtype == ZP_DTYPE_BF16 && a.dim <= 256 && a.vdim <= 8 * MC_VT;
+}
+
+template <int DP>
+static int launch_chunk(const MlstmArgs& a, cudaStream_t st) {
+  auto kern = mlstm_chunk_kernel<DP>;
+  constexpr int smem = ChunkSmem<DP>::TOTAL;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) { set_error("zp_mlstm(chunk): %s", cudaGetErrorString(e)); return ZP_ERR_CUDA; }
+  const int tiles = (a.vdim + MC_VT - 1) / MC_VT;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(tiles, a.H, a.B);
+  cfg.blockDim = dim3(MC_THREADS);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute at[1];
+  at[0].id = cudaLaunchAttributeClusterDimension;
+  at[0].val.clusterDim.x = tiles; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+  cfg.attrs = at; cfg.numAttrs = 1;
+  e = cudaLaunchKernelEx(&cfg, kern, a);
+  if (e != cudaSuccess) { set_error("zp_mlstm(chunk): %s", cudaGetErrorString(e)); return ZP_ERR_CUDA; }
+  return check_launch("zp_mlstm(chunk)");
+}
+
+int mlstm_chunk(const MlstmArgs& a, cudaStream_t st) {
+  if (a.dim <= 64) return launch_chunk<64>(a, st);
+  if (a.dim <= 128) return launch_chunk<128>(a, st);
+  return launch_chunk<256>(a, st);
+}
+
+}  // namespace zp
