@@ -42,7 +42,7 @@ class DecodeGraphRunner:
         pos, ctx, slot, trip, ntrip = prepare_decode(self.num_tokens[:bs], self.block_tables[:bs],
                                                      self.query_ids[:bs], self.qcl, self.block_size)
         set_context(False, slot_mapping=slot, context_lens=ctx, block_tables=self.block_tables[:bs],
-                    query_slot_mapping=trip, query_slot_count=ntrip)
+                    query_slot_mapping=trip, query_slot_count=ntrip, state_slots=self.query_ids[:bs])
         try:
             return self.model(self.input_ids[:bs], pos)
         finally:

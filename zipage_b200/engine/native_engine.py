@@ -9,6 +9,11 @@ decode_sum + compress_sum).  Under tensor parallelism every rank runs this same 
 requests: the sharded sampler leaves every rank with the step's tokens, so the schedulers stay in
 step without any message (the reference pickles the scheduled sequences to its worker ranks every
 step, model_runner.py:151-203).
+
+Models without KV compression (`cache=` given: paged keys and values and recurrent state as the model's
+layers ask for) are served in portion steps instead: one batch of decoded tokens beside portions of
+prompts, run by `run_portions`.  A batch of single tokens goes through the same replayed graphs.
+`feed` / `run_fed` / `close` drive the same step with given tokens (replaying a trace).
 """
 from __future__ import annotations
 
@@ -19,6 +24,7 @@ import numpy as np
 import torch
 
 from .. import _lib as L
+from ..layers.row_ops import project
 from ..layers.step_ops import sample
 from ..utils.context import reset_context, set_context
 from .compressor import Compressor
@@ -48,18 +54,22 @@ def full_state_from_hf(hf_state):
 class NativeEngine:
     def __init__(self, model, lm_head, kv_cache, query_cache, sched_config, compress_cfg, hidden_size,
                  comm=None, max_bs=256, max_model_len=4096, score_cache=None, layer_stride=8,
-                 greedy=False, graph=True, seed=0):
+                 greedy=False, graph=True, seed=0, cache=None):
         self.model, self.lm_head, self.comm = model, lm_head, comm
-        self.device = kv_cache.device
-        self.block_size = int(kv_cache.shape[3])
+        self.cache = cache
+        self.portions = cache is not None
+        self.device = cache.device if self.portions else kv_cache.device
+        self.block_size = cache.block_size if self.portions else int(kv_cache.shape[3])
+        dtype = cache.dtype if self.portions else kv_cache.dtype
         self.qcl = sched_config.query_cache_len
         self.scheduler = Scheduler(sched_config)
-        self.compressor = Compressor(kv_cache, query_cache, score_cache, compress_cfg, layer_stride=layer_stride)
+        self.compressor = None if self.portions else \
+            Compressor(kv_cache, query_cache, score_cache, compress_cfg, layer_stride=layer_stride)
         self.width = (max_model_len + self.block_size - 1) // self.block_size + 1
         self.max_bs = max_bs
         self.runner = DecodeGraphRunner(model, hidden_size, max_bs=max_bs, max_num_blocks=self.width,
                                         query_cache_len=self.qcl, block_size=self.block_size,
-                                        dtype=kv_cache.dtype, device=self.device)
+                                        dtype=dtype, device=self.device)
         self.graph = graph
         if graph:
             self.runner.capture()
@@ -106,6 +116,9 @@ class NativeEngine:
             seed = self.seed * 1000003 + self.step_no
             tok = self.comm.sample(logits, temps, seed=seed) if self.comm is not None else sample(logits, temps, seed=seed)
         self._tokens_host[:n].copy_(tok, non_blocking=True)
+        if self.portions:           # none of this path's kernels waits on a barrier
+            torch.cuda.current_stream().synchronize()
+            return self._tokens_host[:n].numpy().astype(np.int32)
         # a tensor-core kernel whose bounded wait ran out (prefill attention) leaves its code in the
         # device error word: read it with the tokens, on this stream only
         L.check(L.load().zp_device_error_async(L.ptr(self._pin_err), L.stream_ptr()), "device_error")
@@ -136,16 +149,20 @@ class NativeEngine:
 
     @torch.inference_mode()
     def _decode(self, handles):
+        return torch.nn.functional.linear(self._decode_hidden(handles), self.lm_head)
+
+    def _decode_hidden(self, handles):
         n = len(handles)
         d = self.scheduler.decode_inputs(handles, table_width=self.width, out=self._views)
         dev, st = self.device, self._staged
-        hidden = self.runner.run(st["input_ids"][:n].to(dev, non_blocking=True), st["num_tokens"][:n].to(dev, non_blocking=True),
-                                 st["block_tables"][:n, :d["widest"]].to(dev, non_blocking=True),
-                                 st["query_ids"][:n].to(dev, non_blocking=True), eager=not self.graph)
-        return torch.nn.functional.linear(hidden, self.lm_head)
+        return self.runner.run(st["input_ids"][:n].to(dev, non_blocking=True), st["num_tokens"][:n].to(dev, non_blocking=True),
+                               st["block_tables"][:n, :d["widest"]].to(dev, non_blocking=True),
+                               st["query_ids"][:n].to(dev, non_blocking=True), eager=not self.graph)
 
     def step(self):
         """-> (handles that finished, tokens of the step: > 0 prefill tokens, < 0 decode tokens)."""
+        if self.portions:
+            return self._step_portions()
         sched = self.scheduler
         handles, is_prefill = sched.schedule_batch()
         n = len(handles)
@@ -176,6 +193,84 @@ class NativeEngine:
         self.time_record["decode_sum"] += dt
         self.time_record["decode_tokens"] += n
         return done, -n
+
+    # -- portion steps ----------------------------------------------------------------------------
+    def logits(self, hidden):
+        """LM head on rows of hidden states; fp32 where the model asks for it."""
+        if getattr(self.model, "fp32_logits", False):
+            return project(hidden, self.lm_head, fp32=True)
+        return torch.nn.functional.linear(hidden, self.lm_head)
+
+    @torch.inference_mode()
+    def run_portions(self, handles, counts):
+        """Runs `counts[i]` pending tokens of each sequence as one batch.  -> (final hidden states of all
+        its tokens, first row of each sequence).  The caller commits the portions."""
+        n = len(handles)
+        if self.graph and n <= self.max_bs and int(counts.max()) == 1 and int(self.scheduler.pending(handles).max()) == 1:
+            return self._decode_hidden(handles), np.arange(n)
+        order = np.argsort(counts != 1, kind="stable")      # single rows first
+        p = self.scheduler.portion_inputs(np.ascontiguousarray(handles[order]), np.ascontiguousarray(counts[order]),
+                                          self.width)
+        ints = np.concatenate([p[k].ravel() for k in ("input_ids", "positions", "slot_mapping", "cu_seqlens_q",
+                                                      "context_lens", "slots", "block_tables")])
+        dev = torch.from_numpy(ints).to(self.device)        # one copy for the step's inputs
+        t, at = len(p["input_ids"]), 0
+        parts = []
+        for k in (t, t, t, n + 1, n, n, n * p["block_tables"].shape[1]):
+            parts.append(dev[at:at + k])
+            at += k
+        ids, pos, slot_mapping, cu, ctx, slots, tables = parts
+        set_context(True, cu, None, int(counts.max()), 0, slot_mapping,
+                    context_lens=ctx, block_tables=tables.view(n, -1), num_decode=int((counts == 1).sum()),
+                    state_slots=slots)
+        try:
+            hidden = self.model(ids.long(), pos.long())
+        finally:
+            reset_context()
+        first = np.empty(n, dtype=np.int64)
+        first[order] = p["cu_seqlens_q"][:-1]
+        return hidden, first
+
+    def _step_portions(self):
+        sched = self.scheduler
+        handles, counts = sched.schedule_portions()
+        if len(handles) == 0:
+            return handles, 0
+        t0 = time.perf_counter()
+        hidden, first = self.run_portions(handles, counts)
+        rows = first + counts - 1                           # each sequence's newest token
+        if hidden.shape[0] != len(rows) or not np.array_equal(rows, np.arange(len(rows))):
+            hidden = hidden[torch.from_numpy(rows).to(self.device)]
+        with torch.inference_mode():
+            tokens = self._sample(self.logits(hidden), handles)
+        done = sched.commit_portions(handles, counts, tokens)
+        dt = time.perf_counter() - t0
+        decode = int(counts.max()) == 1
+        self.time_record["decode_sum" if decode else "prefill_sum"] += dt
+        if decode:
+            self.time_record["decode_tokens"] += len(handles)
+        return done, -len(handles) if decode else int(counts.sum())
+
+    # given tokens instead of sampled ones
+    def feed(self, tokens, handle=-1):
+        return self.scheduler.feed(tokens, handle)
+
+    @torch.inference_mode()
+    def run_fed(self, handles, counts, want):
+        """Runs everything the fed sequences have pending; `want[i]`: places among sequence i's new
+        tokens.  -> fp32 logits of the wanted places in order, [wanted, vocab] (None: nothing wanted)."""
+        handles, counts = np.asarray(handles, dtype=np.int32), np.asarray(counts, dtype=np.int32)
+        hidden, first = self.run_portions(handles, counts)
+        rows = np.concatenate([first[i] + np.asarray(w, dtype=np.int64) for i, w in enumerate(want)])
+        out = None
+        if len(rows):
+            out = self.logits(hidden[torch.from_numpy(rows).to(self.device)]).float()
+        torch.cuda.current_stream().synchronize()    # the pinned step inputs are rewritten by the next step
+        self.scheduler.commit_portions(handles, counts)
+        return out
+
+    def close(self, handle):
+        self.scheduler.close(handle)
 
     def generate(self, seqs):
         """Runs the requests to completion; -> {handle: completion token ids}."""

@@ -452,3 +452,62 @@ class Scheduler:
             self._obj, _ptr(handles), n, _ptr(out["tables"]), w, _ptr(out["targets"]), nt,
             _ptr(out["query_ids"]), _ptr(out["compressed"])), "compress_inputs")
         return out
+
+    # -- portion steps ---------------------------------------------------------------------------
+    def schedule_portions(self, token_budget=None):
+        """-> (handles, counts): the sequences of one step and how many of their pending tokens it runs."""
+        counts = np.empty(len(self._handles), dtype=np.int32)
+        with self._mutating():
+            n = H.check(self._lib.zp_sched_schedule_portions(self._obj, token_budget or self.max_num_batched_tokens,
+                                                             _ptr(self._handles), _ptr(counts), len(counts)),
+                        "schedule_portions")
+        return self._handles[:n].copy(), counts[:n]
+
+    def commit_portions(self, handles, counts, token_ids=None, now=None):
+        """-> the handles that finished in this call."""
+        toks = None if token_ids is None else np.ascontiguousarray(token_ids, dtype=np.int32)
+        if toks is not None and len(toks) != len(handles):
+            raise ValueError("one token per sequence")
+        done = np.empty(max(len(handles), 1), dtype=np.int32)
+        with self._mutating():
+            n = H.check(self._lib.zp_sched_commit_portions(self._obj, _ptr(handles), _ptr(counts), len(handles),
+                                                           None if toks is None else _ptr(toks),
+                                                           time.time() if now is None else now, _ptr(done)),
+                        "commit_portions")
+        for h in done[:n].tolist():
+            if self._seqs[h] is not None:
+                object.__setattr__(self._seqs[h], "_finished", True)
+        return done[:n]
+
+    def feed(self, tokens, handle=-1):
+        """Given tokens for a running sequence, or for a new one admitted at once (-1); -> its handle."""
+        tok = np.ascontiguousarray(tokens, dtype=np.int32)
+        with self._mutating():
+            h = H.check(self._lib.zp_sched_feed(self._obj, int(handle), _ptr(tok), len(tok)), "feed")
+        if handle < 0:
+            assert h == len(self._seqs)
+            self._seqs.append(None)          # no Sequence object stands behind a fed sequence
+        return h
+
+    def close(self, handle):
+        with self._mutating():
+            H.check(self._lib.zp_sched_close(self._obj, int(handle)), "close")
+
+    def pending(self, handles):
+        handles = np.ascontiguousarray(handles, dtype=np.int32)
+        out = np.empty(max(len(handles), 1), dtype=np.int32)
+        H.check(self._lib.zp_sched_pending(self._obj, _ptr(handles), len(handles), _ptr(out)), "pending")
+        return out[:len(handles)]
+
+    def portion_inputs(self, handles, counts, table_width):
+        """Host arrays of one portion step, see zp_sched_portion_inputs; the table is cut to its widest row."""
+        n, t = len(handles), int(counts.sum())
+        i32 = lambda *s: np.empty(s, np.int32)
+        out = {"input_ids": i32(t), "positions": i32(t), "slot_mapping": i32(t), "cu_seqlens_q": i32(n + 1),
+               "context_lens": i32(n), "slots": i32(n), "block_tables": i32(n, table_width)}
+        w = H.check(self._lib.zp_sched_portion_inputs(
+            self._obj, _ptr(handles), _ptr(counts), n, *(_ptr(out[k]) for k in (
+                "input_ids", "positions", "slot_mapping", "cu_seqlens_q", "context_lens", "slots", "block_tables")),
+            table_width), "portion_inputs")
+        out["block_tables"] = np.ascontiguousarray(out["block_tables"][:, :max(w, 1)])
+        return out

@@ -15,12 +15,15 @@ from ..kernel import _count, store_kvcache, store_query_cache
 from ..utils.context import get_context
 
 _ws_cache: dict = {}
+_ws_kept: list = []   # outgrown buffers stay: a captured graph may still name them
 
 
 def _workspace(device, nbytes):
     key = (device.index, torch.cuda.current_stream().cuda_stream)
     buf = _ws_cache.get(key)
     if buf is None or buf.numel() < nbytes:
+        if buf is not None:
+            _ws_kept.append(buf)
         buf = torch.empty(max(nbytes, 1 << 20), dtype=torch.uint8, device=device)
         _ws_cache[key] = buf
     return buf
@@ -116,3 +119,78 @@ class Attention(nn.Module):
                 context.cu_seqlens_k, self.scale, context.block_tables)
         return paged_decode_attention(q.contiguous().unsqueeze(1), k_cache, v_cache,
                                       context.context_lens, context.block_tables, self.scale)
+
+
+def window_attention(q, k_cache, v_cache, context_lens, block_table, num_heads, head_dim, v_dim, scale,
+                     window=0, softcap=0.0, cu_seqlens_q=None, max_seqlen_q=0, out=None, impl="auto"):
+    """Sliding-window, soft-capped attention over paged caches whose rows are padded to multiples of 16
+    (k_cache [P, BS, Hkv, KP], v_cache [P, BS, Hkv, VP]).  q [rows, Hq * D] may be a column view of a
+    projection.  One row per sequence without `cu_seqlens_q`."""
+    L.require_cuda(q, k_cache, v_cache, context_lens, block_table, cu_seqlens_q)
+    P, BS, Hkv, KP = k_cache.shape
+    VP = v_cache.shape[3]
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and q.stride(1) == 1 and block_table.stride(1) == 1
+    if out is None:
+        out = torch.empty((q.shape[0], num_heads * v_dim), dtype=q.dtype, device=q.device)
+    B, NB = block_table.shape
+    assert block_table.stride(0) == NB or B == 1
+    lib = L.load()
+    ws = None
+    if cu_seqlens_q is None:
+        span = min(window, NB * BS) if window else NB * BS
+        need = lib.zp_window_attention_workspace_bytes(B, num_heads, Hkv, VP, span)
+        ws = _workspace(q.device, need) if need else None
+    L.check(lib.zp_window_attention(
+        L.ptr(q), L.ptr(k_cache), L.ptr(v_cache), L.ptr(cu_seqlens_q), L.ptr(context_lens), L.ptr(block_table),
+        L.ptr(out), B, int(max_seqlen_q), NB, num_heads, Hkv, head_dim, v_dim, KP, VP, BS, P, q.stride(0),
+        out.stride(0), float(scale), float(softcap or 0.0), int(window or 0), L.IMPL[impl], L.dtype_code(q),
+        L.ptr(ws), 0 if ws is None else ws.numel(), L.stream_ptr()), "window_attention")
+    _count(1)
+    return out
+
+
+def store_kv_padded(k, v, k_cache, v_cache, slot_mapping, head_dim, v_dim):
+    """k [N, Hkv * D], v [N, Hkv * DV] (column views of one projection) into padded paged caches."""
+    L.require_cuda(k, v, k_cache, v_cache, slot_mapping)
+    assert k.stride(0) == v.stride(0) and k.stride(1) == v.stride(1) == 1
+    P, BS, Hkv, KP = k_cache.shape
+    L.check(L.load().zp_store_kv_padded(
+        L.ptr(k), L.ptr(v), L.ptr(k_cache), L.ptr(v_cache), L.ptr(slot_mapping), k.shape[0], Hkv, head_dim, v_dim,
+        KP, v_cache.shape[3], k.stride(0), P * BS, L.dtype_code(k), L.stream_ptr()), "store_kv_padded")
+    _count(1)
+
+
+class WindowAttentionMixer(nn.Module):
+    """Grouped-query attention without rotation, with a sliding window and a soft cap on the scores;
+    h -> head outputs [rows, heads * vdim] before the output projection.  `run` selects the cache of
+    this pass when the layer runs several times."""
+
+    def __init__(self, width, heads, kv_heads, dim, vdim, scale, softcap, window, dtype, device):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.softcap, self.window = scale, softcap, window
+        e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
+        self.qkv = e(heads * dim + kv_heads * (dim + vdim), width)
+        self.out_proj = e(width, heads * vdim)
+        self.caches = []                                       # one (k_cache, v_cache) per pass
+
+    def load(self, get):
+        self.qkv.copy_(torch.cat([get(n) for n in "qkv"], 0))
+        self.out_proj.copy_(get("o"))
+
+    def forward(self, h, run):
+        ctx = get_context()
+        x = torch.mm(h, self.qkv.t())
+        nq, nk = self.heads * self.dim, self.kv_heads * self.dim
+        q, k, v = x[:, :nq], x[:, nq:nq + nk], x[:, nq + nk:]
+        kc, vc = self.caches[run]
+        store_kv_padded(k, v, kc, vc, ctx.slot_mapping, self.dim, self.vdim)
+        out = torch.empty((h.shape[0], self.heads * self.vdim), dtype=h.dtype, device=h.device)
+        nd = ctx.decode_rows()
+        shape = (self.heads, self.dim, self.vdim, self.scale, self.window, self.softcap)
+        if nd:
+            window_attention(q, kc, vc, ctx.context_lens[:nd], ctx.block_tables[:nd], *shape, out=out)
+        if ctx.is_prefill and nd < ctx.context_lens.shape[0]:
+            window_attention(q, kc, vc, ctx.context_lens[nd:], ctx.block_tables[nd:], *shape,
+                             cu_seqlens_q=ctx.cu_seqlens_q[nd:], max_seqlen_q=ctx.max_seqlen_q, out=out)
+        return out

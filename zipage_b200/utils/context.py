@@ -3,6 +3,9 @@
 Same fields and accessors as the reference's zipage/utils/context.py:5-52, plus
 `query_slot_count`: a device int32 [1] with the number of valid rows of `query_slot_mapping`
 when that tensor has a fixed capacity (steps built on the device and replayed as a graph).
+Steps that run portions of prompts beside decoded tokens (`is_prefill` with `context_lens`) also carry
+`num_decode`, the number of leading sequences with a single row, and every step of a model with
+recurrent state carries `state_slots`, the slot of each sequence.
 """
 from __future__ import annotations
 
@@ -23,6 +26,12 @@ class Context:
     context_lens: torch.Tensor | None = None
     block_tables: torch.Tensor | None = None
     query_slot_count: torch.Tensor | None = None
+    num_decode: int = 0
+    state_slots: torch.Tensor | None = None
+
+    def decode_rows(self) -> int:
+        """Leading sequences that bring one row each."""
+        return self.num_decode if self.is_prefill else self.context_lens.shape[0]
 
 
 _CONTEXT = Context()
@@ -34,10 +43,11 @@ def get_context() -> Context:
 
 def set_context(is_prefill, cu_seqlens_q=None, cu_seqlens_k=None, max_seqlen_q=0, max_seqlen_k=0,
                 slot_mapping=None, query_slot_mapping=None, context_lens=None, block_tables=None,
-                query_slot_count=None):
+                query_slot_count=None, num_decode=0, state_slots=None):
     global _CONTEXT
     _CONTEXT = Context(is_prefill, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, max_seqlen_k,
-                       slot_mapping, query_slot_mapping, context_lens, block_tables, query_slot_count)
+                       slot_mapping, query_slot_mapping, context_lens, block_tables, query_slot_count,
+                       num_decode, state_slots)
 
 
 def reset_context():
