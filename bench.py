@@ -51,7 +51,7 @@ def parse_args():
                     help="also run the reference ENGINE (baseline/_ref) on a synthetic Qwen3-8B-shaped model, as it "
                          "is and with this library's decode path bound, and report decode tokens/s (adds minutes)")
     ap.add_argument("--also-exact", action="store_true", help="time the exact variant as well")
-    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine"],
+    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine", "similorn"],
                     help="compress (default, the headline op), decode (paged decode attention kernel) or "
                          "step_ops (the element-wise ops of a decoder layer step and the sampler) or "
                          "prefill (varlen causal prefill attention, one layer) or decode_step (the decode "
@@ -1051,6 +1051,207 @@ def run_native_engine(args):
         dist.destroy_process_group()
 
 
+def similorn_kernel_records(args, dev, peaks):
+    """Every kernel of the Similorn decoder at sizes of an 8B-class model's layers (width 4096, attention 32 / 8
+    heads of 128, matrix memories 16 x [128, 256], bf16) beside the like kernel of the Qwen3 path at the same
+    size.  frac = share of the kernel's roofline: the slower of its bytes at the measured copy
+    bandwidth and its products at the measured cuBLAS rate.  Inputs are larger than L2."""
+    import torch
+    from zipage_b200.layers import attention as A
+    from zipage_b200.layers import row_ops as R
+    from zipage_b200.layers import step_ops as P
+    from zipage_b200.layers.mlstm import mlstm_step
+    hbm, tf = peaks.get("hbm_gbs", 6650.0) * 1e9, peaks.get("bf16_tflops", 1590.0) * 1e12
+    bf, W = torch.bfloat16, 4096
+    rnd = lambda *s, dt=bf: torch.empty(s, dtype=dt, device=dev).normal_()
+    recs, launches = {}, 0
+
+    def rec(name, fn, nbytes, flops=0.0, like=None):
+        nonlocal launches
+        for _ in range(args.warmup):
+            fn()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(args.steps):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        ms = e0.elapsed_time(e1) / args.steps
+        launches += args.steps
+        roof = max(nbytes / hbm, flops / tf)
+        recs[name] = {"ms": round(ms, 4), "bound": "hbm" if nbytes / hbm >= flops / tf else "tensor",
+                      "frac": round(roof / (ms * 1e-3), 3), "gbs": round(nbytes / ms / 1e6, 1),
+                      "tflops": round(flops / ms / 1e9, 1)}
+        if like:
+            recs[name]["like"] = like
+            recs[name]["distance_ratio"] = round(recs[like]["frac"] / recs[name]["frac"], 2)
+
+    # prompts: 4 x 4096 tokens
+    B, S = 4, 4096
+    T = B * S
+    i32 = lambda t: t.to(torch.int32).to(dev)
+    cu, ctx = i32(torch.arange(0, T + 1, S)), i32(torch.full((B,), S))
+    q, k, v = rnd(T, HQ, D), rnd(T, HKV, D), rnd(T, HKV, D)
+    fl = 4.0 * D * HQ * B * S * S / 2
+    rec("qwen3 prefill attention", lambda: A.varlen_prefill_attention(q, k, v, S, cu, S, cu),
+        2.0 * T * D * (2 * HQ + 2 * HKV), fl)
+    kc, vc = rnd(T // 64, 64, HKV, D), rnd(T // 64, 64, HKV, D)
+    table = i32(torch.arange(T // 64).view(B, -1))
+    q2, out = q.view(T, -1), torch.empty(T, HQ * D, dtype=bf, device=dev)
+    for win in (4096, 1024):
+        seen = sum(min(p + 1, win) for p in range(S)) * B
+        rec(f"window attention prefill, window {win}",
+            lambda: A.window_attention(q2, kc, vc, ctx, table, HQ, D, D, D ** -0.5, win, 30.0, cu_seqlens_q=cu, max_seqlen_q=S, out=out),
+            2.0 * T * D * (2 * HQ + 2 * HKV), 4.0 * D * HQ * seen, "qwen3 prefill attention")
+    H, dk, dv = 16, 128, 256
+    norm, bias = torch.ones(H * dv, device=dev), torch.zeros(2 * H, device=dev)
+    bias[H:] = 4.0
+    state_of = lambda n: (torch.zeros(n, H, dk, dv, device=dev), torch.zeros(n, H, dk, device=dev), torch.zeros(n, H, device=dev))
+
+    def memory(rows, n, cu=None, ctx=None):
+        x, gates, o = rnd(rows, 2 * H * (dk + dv)), rnd(rows, 2 * H, dt=torch.float32), torch.empty(rows, H * dv, dtype=bf, device=dev)
+        st, slots = state_of(n), i32(torch.arange(n))
+        cols = x[:, :H * dk], x[:, H * dk:2 * H * dk], x[:, 2 * H * dk:2 * H * dk + H * dv], x[:, 2 * H * dk + H * dv:]
+        return lambda: mlstm_step(*cols, gates, bias, norm, st, o, ctx, slots, H, dk, dv, 15.0, 1e-5, cu_seqlens_q=cu)
+    # products of the chunked form (64 tokens): scores and their values (causal half), read-out, update
+    rec("mlstm prefill", memory(T, B, cu, ctx), 2.0 * T * H * (2 * dk + 3 * dv) + 8.0 * T * H,
+        2.0 * T * H * (32 * (dk + dv) + 2 * dk * dv), "qwen3 prefill attention")
+    # decode: 256 sequences
+    n, NB = 256, 9
+    lens = i32(torch.full((n,), NB * 256 - 7))
+    qd = rnd(n, 1, HQ, D)
+    kq, vq = rnd(n * NB, 256, HKV, D), rnd(n * NB, 256, HKV, D)
+    bt = i32(torch.randperm(n * NB).view(n, NB))
+    byt = n * (NB * 256 - 7) * HKV * D * 4.0
+    rec("qwen3 paged decode", lambda: A.paged_decode_attention(qd, kq, vq, lens, bt), byt)
+    qf = qd.view(n, -1)
+    rec("window attention decode, window 4096", lambda: A.window_attention(qf, kq, vq, lens, bt, HQ, D, D, D ** -0.5, 4096, 30.0),
+        byt, 0.0, "qwen3 paged decode")
+    rec("window attention decode, window 1024", lambda: A.window_attention(qf, kq, vq, lens, bt, HQ, D, D, D ** -0.5, 1024, 30.0),
+        n * 1024 * HKV * D * 4.0, 0.0, "qwen3 paged decode")
+    rec("mlstm decode", memory(n, n, None, i32(torch.full((n,), 5))), 8.0 * n * H * dk * dv, 0.0, "qwen3 paged decode")
+    # row ops
+    xr, wr, res = rnd(T, W), torch.ones(W, dtype=bf, device=dev), rnd(T, W)
+    rec("qwen3 add + rms norm", lambda: P.rms_norm(xr, wr, 1e-6, res), 8.0 * T * W)
+    xf, wf = rnd(T, W, dt=torch.float32), torch.zeros(W, device=dev)
+    rec("rms norm of fp32 rows", lambda: R.rms_norm_f32(xf, wf, 1e-5, bf, 1.0), 6.0 * T * W, 0.0, "qwen3 add + rms norm")
+    up = rnd(T, 2 * 12288)
+    rec("qwen3 silu and mul", lambda: P.silu_and_mul(up), 6.0 * T * 12288)
+    up1 = rnd(T, 12288)
+    rec("gelu", lambda: R.gelu_tanh(up1), 4.0 * T * 12288, 0.0, "qwen3 silu and mul")
+    kv = rnd(T, HQ * D + 2 * HKV * D)
+    slot = i32(torch.arange(T))
+    cs = P.rope_cos_sin_cache(D, S, 1e6, dev)
+    w1, pos = torch.ones(D, dtype=bf, device=dev), torch.arange(S, device=dev).repeat(B)
+    rec("qwen3 q/k norm, rotation and store", lambda: P.qk_norm_rope_store(
+        kv, pos, cs, w1, w1, 1e-6, HQ, HKV, D, kc.view(-1, 64, HKV, D), vc.view(-1, 64, HKV, D), slot, return_k=False),
+        2.0 * T * D * (2 * HQ + 4 * HKV))
+    rec("key/value store", lambda: A.store_kv_padded(kv[:, HQ * D:HQ * D + HKV * D], kv[:, HQ * D + HKV * D:], kc, vc, slot, D, D),
+        8.0 * T * HKV * D, 0.0, "qwen3 q/k norm, rotation and store")
+    tok, emb = torch.randint(0, 32768, (T,), device=dev), rnd(32768, W)
+    turns = R.sinusoid_turns(W, dev)
+    rec("embedding and position", lambda: R.embed_position(tok, pos, emb, 2.0, turns, want_t=True), 8.0 * T * W, 0.0, "qwen3 add + rms norm")
+    return recs, launches
+
+
+def run_similorn(args):
+    """Prefill and decode throughput of the Similorn decoder through the serving engine at two widths, random
+    weights, beside Qwen3 blocks of equal width and depth through the same engine; and the kernel table.
+    Similorn: alternating matrix-memory layers and windowed-attention layers with feed-forward, the middle half
+    of the stack run twice; Qwen3: as many blocks as Similorn has layer runs."""
+    import torch
+    from types import SimpleNamespace
+    from zipage_b200.engine.scheduler import SamplingParams, Sequence
+    from zipage_b200.layers.qwen3_block import Qwen3Model
+    from zipage_b200.models.registry import LoadedModel, engine_for
+    from zipage_b200.models.similorn import SimilornConfig, SimilornModel
+    dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
+    torch.cuda.set_device(dev)
+    pk = ROOT / "MEASURED_PEAKS.json"
+    peaks = json.loads(pk.read_text()) if pk.exists() else {}
+    bf = torch.bfloat16
+    torch.manual_seed(3)
+
+    def similorn(width, heads, kv, mheads, ff):
+        mem = {"type": "mlstm", "mixer": {"heads": mheads, "dim": 128, "vdim": width // mheads, "gate_cap": 15.0}, "mlp": None}
+        att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                              "softcap": 30.0, "mask": {"size": 1024}}, "mlp": {"kind": "dense", "ff": ff}}
+        c = SimilornConfig.from_dict({"vocab": 32768, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+                                      "layers": [mem, att] * 4, "loop": {"start": 2, "stop": 6, "times": 2}})
+        m = SimilornModel(c, bf, dev)
+        with torch.no_grad():
+            for n, p in m.named_parameters():
+                if p.dim() > 1:
+                    p.normal_(0, p.shape[1] ** -0.5)
+                else:
+                    p.zero_()
+            for layer in m.layers:
+                if hasattr(layer.mixer, "gate_bias"):
+                    layer.mixer.gate_bias[layer.mixer.heads:] = 4.0
+                    layer.mixer.norm.fill_(1.0)
+        return LoadedModel("Similorn", m, m.head, width, 32768, bf, True), len(m.runs)
+
+    def qwen(width, heads, kv, ff, blocks):
+        c = SimpleNamespace(hidden_size=width, num_attention_heads=heads, num_key_value_heads=kv, head_dim=128, intermediate_size=ff,
+                            hidden_act="silu", rms_norm_eps=1e-6, vocab_size=32768, num_hidden_layers=blocks,
+                            max_position_embeddings=8192, rope_theta=1e6)
+        prev = torch.get_default_dtype()
+        torch.set_default_dtype(bf)
+        try:
+            with dev:
+                m = Qwen3Model(c).eval()
+        finally:
+            torch.set_default_dtype(prev)
+        return LoadedModel("Qwen3ForCausalLM", m, torch.empty(32768, width, dtype=bf, device=dev).normal_(0, 0.02), width, 32768, bf, False)
+
+    R, PROMPT, GEN = 64, 1536, 128
+    g = torch.Generator().manual_seed(1)
+
+    def serve(loaded):
+        eng = engine_for(loaded, max_tokens=R * 2048, max_seqs=R, block_size=256, token_budget=16384, max_model_len=2304,
+                         budget_blocks=8, query_cache_len=32)
+        for rep in range(2):                       # the first pass warms up
+            eng.time_record.clear()
+            reqs = [Sequence(torch.randint(0, 32768, (PROMPT,), generator=g).tolist(), SamplingParams(1.0, GEN if rep else 8, True))
+                    for _ in range(R)]
+            for r in reqs:
+                eng.add_request(r)
+            full = full_s = 0.0
+            while not eng.is_finished():
+                before = eng.time_record["decode_sum"]
+                _, n = eng.step()
+                if n == -R:
+                    full, full_s = full + R, full_s + eng.time_record["decode_sum"] - before
+        tr = eng.time_record
+        return {"prefill_tokens_per_s": round(R * PROMPT / tr["prefill_sum"], 1), "decode_tokens_per_s": round(full / full_s, 1),
+                "decode_ms_per_step": round(full_s / (full / R) * 1e3, 3)}
+
+    res = {}
+    with ClockSampler(dev.index or 0) as clocks:
+        kernels, launches = similorn_kernel_records(args, dev, peaks)
+        torch.cuda.empty_cache()
+        for width, heads, kv, mheads, ff in ((4096, 32, 8, 16, 12288), (2048, 16, 4, 8, 6144)):
+            loaded, runs = similorn(width, heads, kv, mheads, ff)
+            a = serve(loaded)
+            del loaded
+            torch.cuda.empty_cache()
+            b = serve(qwen(width, heads, kv, ff, runs))
+            torch.cuda.empty_cache()
+            res[f"width {width}"] = {"similorn": a, "qwen3": b, "layer_runs": runs}
+    head = res["width 4096"]["similorn"]
+    print(json.dumps({
+        "metric": "similorn_decode_tokens_per_s", "value": head["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+        "steps": args.steps, "warmup": args.warmup, "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True,
+        "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": f"serving engine, {R} requests, prompts of {PROMPT}, {GEN} sampled tokens each; random weights; 12 layer "
+                               "runs (mlstm / windowed attention + feed-forward alternating, the middle half twice) beside 12 Qwen3 blocks",
+                   "l2": "inputs of every kernel are larger than L2"},
+        "serving": res, "kernels": kernels, "gpu_launches": launches, "clocks": clocks.summary(),
+        "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")},
+    }))
+
+
 def run_host_control(args):
     """Host time per decode step of the control plane at `--requests` concurrent requests: the
     native scheduler's array calls (schedule, the runner's input arrays, postprocess) and, when an
@@ -1161,6 +1362,8 @@ def main():
         return run_host_control(args)
     if args.workload == "native_engine":
         return run_native_engine(args)
+    if args.workload == "similorn":
+        return run_similorn(args)
     if args.workload == "prefill":
         return run_prefill(args)
     if args.workload == "decode":

@@ -428,13 +428,16 @@ int zp_store_kv_padded(const void* k, const void* v, void* k_cache, void* v_cach
  * context_lens [B] counts each sequence's keys including this step's (0: padding row, skipped).
  * 16-bit caches with KP, VP <= 256 and Hq / Hkv <= 16 take the tensor-core kernels (ZP_IMPL_SIMT: never), whose
  * one-row form may need a workspace (zp_window_attention_workspace_bytes, span = min(window, NBmax *
- * BS)).  Scores and softmax weights are fp32. */
+ * BS)).  With total_q (rows of q; 0 = not told), bf16 portions with head sizes of 128 and a soft cap of
+ * at most 34 take the tcgen05 kernel (ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED).  Scores and
+ * softmax weights are fp32 in all of them. */
 size_t zp_window_attention_workspace_bytes(int B, int Hq, int Hkv, int VP, int span);
 int zp_window_attention(const void* q, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens_q,
                         const int32_t* context_lens, const int32_t* block_table, void* out, int B,
                         int max_seqlen_q, int NBmax, int Hq, int Hkv, int D, int DV, int KP, int VP, int BS,
                         int n_pages, int64_t q_stride, int64_t out_stride, float scale, float softcap,
-                        int window, int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream);
+                        int window, int total_q, int impl, int dtype, void* workspace, size_t workspace_bytes,
+                        void* stream);
 
 /* One step of a matrix-memory (mLSTM) mixer over a batch of sequences, state to gated output:
  *   i = cap tanh((gates_i + bias_i) / cap), f = log sigmoid(cap tanh((gates_f + bias_f) / cap))

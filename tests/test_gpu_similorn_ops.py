@@ -255,3 +255,23 @@ def test_mlstm_recalls_a_far_token(impl):
     x[3, 2 * dk:2 * dk + dv] *= -1                                 # the checker would notice a lost token
     other, _ = _mlstm_want(x, gates, bias, norm, H, dk, dv, 12.0, 1e-5)
     assert (other[900] - want[900]).abs().max() > 0.5 * want[900].abs().max()
+
+
+@pytest.mark.parametrize("window,softcap", [(1000, 30.0), (0, 20.0), (128, 30.0), (129, 5.0), (65, 34.0)])
+@pytest.mark.parametrize("block", [64, 256])
+def test_window_attention_on_long_portions(window, softcap, block):
+    """Head sizes of 128 (the tcgen05 kernel): many key tiles, a portion after a long prefix, ragged ends; and
+    the mma.sync kernel's numbers stand in for a second opinion through single rows."""
+    from zipage_b200.layers.attention import window_attention
+    H, G, d, S, rows = 4, 2, 128, 1111, 700
+    q, k, v = (_rand(S, h, d, seed=i, dtype=BF) for i, h in enumerate((H, G, G)))
+    k[S - 1 - 64] = q[S - 1].view(G, H // G, d)[:, 0]              # 64 back from the last row
+    kc, vc, t = _paged(k, v, block, 3)
+    want = O.window_attention(q[S - rows:].double(), k.double(), v.double(), d ** -0.5, softcap, window).flatten(1)
+    i32 = lambda a: torch.tensor(a, dtype=torch.int32).cuda()
+    qg = q[S - rows:].reshape(rows, -1).cuda()
+    got = window_attention(qg, kc, vc, i32([S]), t[None].cuda(), H, d, d, d ** -0.5, window, softcap,
+                           cu_seqlens_q=i32([0, rows]), max_seqlen_q=rows, impl="tcgen05")
+    _close(got, want, 6e-3, "tcgen05")
+    one = window_attention(qg[-1:], kc, vc, i32([S]), t[None].cuda(), H, d, d, d ** -0.5, window, softcap)
+    _close(one[0], want[-1], 6e-3, "single row")

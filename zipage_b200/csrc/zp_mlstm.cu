@@ -41,6 +41,16 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_recurrent_kernel(const Mlstm
 
   for (int t = 0; t < sq.count; ++t) {
     const int64_t row = sq.row0 + t;
+    // the first batch of state rows is on its way while the gates are computed
+    float4 s[ML_BATCH];
+    auto load_rows = [&](int r0) {
+#pragma unroll
+      for (int u = 0; u < ML_BATCH; ++u) {
+        const int r = r0 + u * nrg;
+        s[u] = (r < a.dim && !zero) ? *reinterpret_cast<const float4*>(S + (int64_t)r * a.VP) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    };
+    if (mine) load_rows(rg);
     const float gi = log_input_gate(a, row, h), gf = log_forget_gate(a, row, h);
     const float m_new = fmaxf(gf + m, gi);
     const float keep = expf(gf + m - m_new), add = expf(gi - m_new);
@@ -60,12 +70,7 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_recurrent_kernel(const Mlstm
       for (int j = 0; j < 4; ++j)
         v[j] = col + j < a.vdim ? add * Elem<T>::to_f32(vb[row * a.row_stride + (int64_t)h * a.vdim + col + j]) : 0.f;
       for (int r0 = rg; r0 < a.dim; r0 += nrg * ML_BATCH) {
-        float4 s[ML_BATCH];
-#pragma unroll
-        for (int u = 0; u < ML_BATCH; ++u) {
-          const int r = r0 + u * nrg;
-          s[u] = (r < a.dim && !zero) ? *reinterpret_cast<const float4*>(S + (int64_t)r * a.VP) : make_float4(0.f, 0.f, 0.f, 0.f);
-        }
+        if (r0 != rg) load_rows(r0);
 #pragma unroll
         for (int u = 0; u < ML_BATCH; ++u) {
           const int r = r0 + u * nrg;

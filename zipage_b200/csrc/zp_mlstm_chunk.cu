@@ -52,11 +52,12 @@ __device__ __forceinline__ void for_blocks(const unsigned char* tile, int row0, 
 }
 
 // Shared memory, bytes: Q and K tiles, V tile, hi and lo of the state tile, hi and lo of the scores
-// (reused by the decayed values), per-row floats.
+// (reused by the decayed values), the output gate's tile, per-row floats.  A chunk's tiles are requested as
+// soon as the previous chunk has no more use for their place.
 template <int DP> struct ChunkSmem {
   static constexpr int RB = DP * 2 + 16;
   static constexpr int Q = 0, K = Q + MC_C * RB, V = K + MC_C * RB, S = V + MC_C * MC_RB, P = S + 2 * DP * MC_RB,
-                       F = P + 2 * MC_C * MC_RB, TOTAL = F + 12 * MC_C * 4;
+                       G = P + 2 * MC_C * MC_RB, F = G + MC_C * MC_RB, TOTAL = F + 14 * MC_C * 4;
 };
 
 template <int DP>
@@ -77,14 +78,17 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
   float *sM = fl, *sU = fl + 64, *sA = fl + 128, *sE = fl + 192, *sW = fl + 256, *sDen = fl + 320, *sR = fl + 384;
   float *sSq = fl + 448;                         // [2 parities][2 halves][64] (read by the cluster)
   float *sMisc = fl + 704;                       // running maximum, decay of the state over the chunk
+  float* sAct = fl + 768;                        // log input gates, log forget gates of the chunk
+  unsigned char* sG = smem + L::G;
   const int c0 = vt * MC_VT, vcols = min(MC_VT, a.vdim - c0);
   const int nk16 = (a.dim + 15) / 16;
   const int64_t head = (int64_t)sq.slot * a.H + h;
   const T* qb = reinterpret_cast<const T*>(a.q) + (int64_t)h * a.dim;
   const T* kb = reinterpret_cast<const T*>(a.k) + (int64_t)h * a.dim;
   const T* vb = reinterpret_cast<const T*>(a.v) + (int64_t)h * a.vdim + c0;
+  const T* gb = reinterpret_cast<const T*>(a.g) + (int64_t)h * a.vdim + c0;
   const bool vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.row_stride % 8 == 0 &&
-                   ((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) % 16 == 0;
+                   ((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.g) % 16 == 0;
 
   // columns 64..71 of the value tile: the column of ones that carries n, then zeros
   for (int i = tid; i < MC_C * 8; i += MC_THREADS)
@@ -107,46 +111,41 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
         s[i][cb][j] = x;
       }
 
-  auto load_chunk = [&](int t0, int n) {
+  // tiles of the chunk that starts at token t0 (n tokens; none: only the group is committed)
+  auto load_tile = [&](const T* base, unsigned char* dst, int rb, int cols16, int valid_cols, int t0, int n) {
     const int64_t row0 = sq.row0 + t0;
-    if (vec) {
-      for (int i = tid; i < MC_C * (DP / 8); i += MC_THREADS) {
-        const int r = i / (DP / 8), c = i % (DP / 8);
-        const int ok = (r < n && c * 8 < a.dim) ? 16 : 0;
-        const int64_t off = ok ? (row0 + r) * a.row_stride + c * 8 : 0;
-        cp_async16(sQ + r * L::RB + c * 16, qb + off, ok);
-        cp_async16(sK + r * L::RB + c * 16, kb + off, ok);
-      }
-      for (int i = tid; i < MC_C * 8; i += MC_THREADS) {
-        const int r = i >> 3, c = i & 7;
-        const int ok = (r < n && c * 8 < vcols) ? 16 : 0;
-        cp_async16(sV + r * MC_RB + c * 16, vb + (ok ? (row0 + r) * a.row_stride + c * 8 : 0), ok);
-      }
-    } else {
-      const T z = Elem<T>::from_f32(0.f);
-      for (int i = tid; i < MC_C * DP; i += MC_THREADS) {
-        const int r = i / DP, c = i % DP;
-        const bool ok = r < n && c < a.dim;
-        *reinterpret_cast<T*>(sQ + r * L::RB + c * 2) = ok ? qb[(row0 + r) * a.row_stride + c] : z;
-        *reinterpret_cast<T*>(sK + r * L::RB + c * 2) = ok ? kb[(row0 + r) * a.row_stride + c] : z;
-      }
-      for (int i = tid; i < MC_C * MC_VT; i += MC_THREADS) {
-        const int r = i >> 6, c = i & 63;
-        *reinterpret_cast<T*>(sV + r * MC_RB + c * 2) = (r < n && c < vcols) ? vb[(row0 + r) * a.row_stride + c] : z;
+    if (n > 0) {
+      if (vec) {
+        for (int i = tid; i < MC_C * cols16; i += MC_THREADS) {
+          const int r = i / cols16, c = i % cols16;
+          const int ok = (r < n && c * 8 < valid_cols) ? 16 : 0;
+          cp_async16(dst + r * rb + c * 16, base + (ok ? (row0 + r) * a.row_stride + c * 8 : 0), ok);
+        }
+      } else {
+        for (int i = tid; i < MC_C * cols16 * 8; i += MC_THREADS) {
+          const int r = i / (cols16 * 8), c = i % (cols16 * 8);
+          *reinterpret_cast<T*>(dst + r * rb + c * 2) =
+              (r < n && c < valid_cols) ? base[(row0 + r) * a.row_stride + c] : Elem<T>::from_f32(0.f);
+        }
       }
     }
     cp_async_commit();
   };
-  // one warp: gates of the chunk, their running sums and maxima (two tokens per lane)
-  auto gates = [&](int t0, int n) {
-    float f[2], u[2];
-#pragma unroll
-    for (int j = 0; j < 2; ++j) {
-      const int t = 2 * lane + j;
-      const int64_t row = sq.row0 + t0 + t;
-      f[j] = t < n ? log_forget_gate(a, row, h) : 0.f;
-      u[j] = t < n ? log_input_gate(a, row, h) : -INFINITY;
+  // Gate pre-activation of token t0 + (tid & 63): threads 0-63 input gates, 64-127 forget gates.
+  auto gate_raw = [&](int t0, int n) -> float {
+    const int t = tid & 63;
+    return (tid < 128 && t < n) ? a.gates[(sq.row0 + t0 + t) * a.gates_stride + (tid >> 6) * a.H + h] : 0.f;
+  };
+  const float gate_bias = tid < 128 ? a.gate_bias[(tid >> 6) * a.H + h] : 0.f;
+  auto gate_put = [&](float raw, int n) {
+    if (tid < 128) {
+      const float x = soft_cap(raw + gate_bias, a.cap);
+      sAct[tid] = (tid & 63) < n ? (tid < 64 ? x : log_sigmoid(x)) : (tid < 64 ? -INFINITY : 0.f);
     }
+  };
+  // one warp: running sums and maxima of the chunk's gates (two tokens per lane)
+  auto scan = [&]() {
+    float f[2] = {sAct[64 + 2 * lane], sAct[65 + 2 * lane]}, u[2] = {sAct[2 * lane], sAct[2 * lane + 1]};
     float F = f[0] + f[1];
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) { const float x = __shfl_up_sync(0xffffffffu, F, o); if (lane >= o) F += x; }
@@ -169,12 +168,19 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     if (lane == 0) { sMisc[1] = expf(m - MC); sMisc[0] = MC + FC; }
   };
 
+  {
+    const int n = min(MC_C, sq.count);
+    load_tile(qb, sQ, L::RB, DP / 8, a.dim, 0, n);
+    load_tile(kb, sK, L::RB, DP / 8, a.dim, 0, n);
+    load_tile(vb, sV, MC_RB, 8, vcols, 0, n);
+    gate_put(gate_raw(0, n), n);
+  }
   __syncthreads();
   const int row_a = rg * 16 + g, row_b = row_a + 8;   // this thread's two tokens of the chunk
   for (int t0 = 0, par = 0; t0 < sq.count; t0 += MC_C, par ^= 1) {
-    const int n = min(MC_C, sq.count - t0);
-    load_chunk(t0, n);
-    if (warp == 0) gates(t0, n);
+    const int n = min(MC_C, sq.count - t0), t1 = t0 + MC_C, n1 = min(MC_C, sq.count - t1);   // n1 <= 0: the last one
+    if (warp == 0) scan();
+    const float raw_next = gate_raw(t1, n1);
     // 16-bit operand copies of the state tile
 #pragma unroll
     for (int i = 0; i < MB; ++i)
@@ -192,6 +198,7 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
       }
     cp_async_wait<0>();
     __syncthreads();
+    load_tile(gb, sG, MC_RB, 8, vcols, t0, n);
 
     float acc[5][4], p[4][4];
 #pragma unroll
@@ -240,6 +247,7 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
       for (int i = 0; i < 5; ++i) { acc[i][0] *= fa; acc[i][1] *= fa; acc[i][2] *= fb; acc[i][3] *= fb; }
     }
     __syncthreads();
+    load_tile(qb, sQ, L::RB, DP / 8, a.dim, t1, n1);
     for (int kk = 0; kk <= rg; ++kk) {                 // keys 16 kk .. 16 kk + 15 of rows up to 16 rg + 15
       uint32_t ph[4], pl[4];
       ldmatrix_x4(ph, sPh + (rg * 16 + (lane & 15)) * MC_RB + kk * 32 + (lane >> 4) * 16);
@@ -274,6 +282,8 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
       *reinterpret_cast<uint32_t*>(sPl + r * MC_RB + c * 4) = lo;
     }
     if (cluster_size() > 1) cluster_sync(); else __syncthreads();
+    load_tile(vb, sV, MC_RB, 8, vcols, t1, n1);
+    gate_put(raw_next, n1);
     if (tid < MC_C) {
       float ss = 0.f;
       for (uint32_t r = 0; r < cluster_size(); ++r)
@@ -300,7 +310,9 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
       for_blocks(sPh, kk * 16, half, lane, add);
       for_blocks(sPl, kk * 16, half, lane, add);
     }
-    __syncthreads();                                   // tiles free for the next chunk; sR visible
+    cp_async_wait<2>();                                // the gate tile (two younger groups: the next Q and V)
+    __syncthreads();                                   // K free for the next chunk; sR visible
+    load_tile(kb, sK, L::RB, DP / 8, a.dim, t1, n1);
     const float ra = sR[row_a], rb = sR[row_b];
     const int64_t grow = sq.row0 + t0;
 #pragma unroll
@@ -312,12 +324,12 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
         if (r >= n) continue;
         const float rr = y ? rb : ra;
         const int64_t e = (int64_t)h * a.vdim + c;
-        const T* gp = reinterpret_cast<const T*>(a.g) + (grow + r) * a.row_stride + e;
+        const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sG + r * MC_RB + (half * 32 + i * 8 + 2 * tq) * 2));
         T* op = reinterpret_cast<T*>(a.out) + (grow + r) * a.out_stride + e;
         float o[2];
 #pragma unroll
         for (int j = 0; j < 2; ++j)
-          o[j] = c + j < a.vdim ? acc[i][2 * y + j] * rr * a.norm_weight[e + j] / (1.f + __expf(-Elem<T>::to_f32(gp[j]))) : 0.f;
+          o[j] = c + j < a.vdim ? acc[i][2 * y + j] * rr * a.norm_weight[e + j] / (1.f + __expf(-(j ? gv.y : gv.x))) : 0.f;
         if (vec && a.out_stride % 2 == 0) { if (c < a.vdim) *reinterpret_cast<uint32_t*>(op) = pack2<T>(o[0], o[1]); }
         else {
           if (c < a.vdim) op[0] = Elem<T>::from_f32(o[0]);

@@ -123,6 +123,9 @@ bool window_mma_supports(const WinArgs& a);
 int window_prefill_mma(const WinArgs& a, int max_q, int dtype, cudaStream_t st);
 int window_decode_mma(const WinArgs& a, int dtype, cudaStream_t st);
 int window_decode_splits(int B, int Hkv, int span);
+// tcgen05 prefill kernel (zp_window_attn_tc.cu)
+bool window_tc_supports(const WinArgs& a, int total_q, int dtype);
+int window_prefill_tc(const WinArgs& a, int max_q, int total_q, cudaStream_t st);
 
 }  // namespace zp
 
@@ -153,7 +156,7 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
                                    const int32_t* block_table, void* out, int B, int max_seqlen_q, int NBmax,
                                    int Hq, int Hkv, int D, int DV, int KP, int VP, int BS, int n_pages,
                                    int64_t q_stride, int64_t out_stride, float scale, float softcap, int window,
-                                   int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream) {
+                                   int total_q, int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream) {
   if (B == 0 || (cu_seqlens_q && max_seqlen_q == 0)) return ZP_OK;
   ZP_REQUIRE(q && k_cache && v_cache && context_lens && block_table && out, "zp_window_attention: null pointer");
   ZP_REQUIRE(Hkv > 0 && Hq % Hkv == 0, "zp_window_attention: Hq must be a multiple of Hkv");
@@ -169,6 +172,15 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
   a.out_stride = out_stride; a.scale = scale; a.softcap = softcap;
   cudaStream_t st = (cudaStream_t)stream;
   const bool half = dtype == ZP_DTYPE_BF16 || dtype == ZP_DTYPE_F16;
+  // portions long enough to fill 128-row query tiles
+  const bool tc = cu_seqlens_q && zp::window_tc_supports(a, total_q, dtype);
+  if (impl == ZP_IMPL_TCGEN05 && !tc) {
+    zp::set_error("zp_window_attention: the tcgen05 kernel needs bf16 portions, head sizes of 128, 16-byte aligned rows "
+                  "and a soft cap of at most 34");
+    return ZP_ERR_UNSUPPORTED;
+  }
+  if (tc && (impl == ZP_IMPL_TCGEN05 || (impl == ZP_IMPL_AUTO && max_seqlen_q >= 96)))
+    return zp::window_prefill_tc(a, max_seqlen_q, total_q, st);
   if (half && impl != ZP_IMPL_SIMT && zp::window_mma_supports(a)) {
     if (cu_seqlens_q) return zp::window_prefill_mma(a, max_seqlen_q, dtype, st);
     const int reach = NBmax * BS, span = window > 0 && window < reach ? window : reach;

@@ -58,6 +58,7 @@ template <> __device__ __forceinline__ void split2<__half>(float a, float b, uin
 // chunks, which makes the eight rows of an ldmatrix land in different banks
 __host__ __device__ __forceinline__ int row_bytes(int elems) { return elems * 2 + 16; }
 
+// (EXACT kernels: KP = VP = 16 NV16, so every size below is a compile-time constant)
 // 64 rows of one head of the K (V) page that holds key0, rows past n_valid filled with zeros
 __device__ __forceinline__ void load_page_rows(unsigned char* dst, const char* cache, int64_t slot0, int Hkv, int hk,
                                                int elems, int n_valid) {
@@ -71,7 +72,7 @@ __device__ __forceinline__ void load_page_rows(unsigned char* dst, const char* c
   }
 }
 
-template <typename T, int NV16, bool BOUNDED>
+template <typename T, int NV16, bool BOUNDED, bool EXACT>
 __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const WinArgs a) {
   extern __shared__ __align__(128) unsigned char smem[];   // Q | 2 x (K | V)
   const int b = blockIdx.z, h = blockIdx.y;
@@ -79,8 +80,9 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
   const int qi0 = blockIdx.x * WM_TQ;
   if (qi0 >= sq.count) return;
   const int hk = h / (a.Hq / a.Hkv);
+  const int KP = EXACT ? NV16 * 16 : a.KP, VP = EXACT ? NV16 * 16 : a.VP;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
-  const int rbk = row_bytes(a.KP), rbv = row_bytes(a.VP);
+  const int rbk = row_bytes(KP), rbv = row_bytes(VP);
   unsigned char* sQ = smem;
   unsigned char* sKV = smem + WM_TQ * rbk;
   const int stage_bytes = WM_TK * (rbk + rbv);
@@ -93,15 +95,15 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
     const int64_t slot0 = (int64_t)win_page(a, b, key0) * a.BS + key0 % a.BS;
     unsigned char* ks = sKV + stage * stage_bytes;
     const int n_valid = min(WM_TK, sq.ctx - key0);
-    load_page_rows(ks, reinterpret_cast<const char*>(a.k), slot0, a.Hkv, hk, a.KP, n_valid);
-    load_page_rows(ks + WM_TK * rbk, reinterpret_cast<const char*>(a.v), slot0, a.Hkv, hk, a.VP, n_valid);
+    load_page_rows(ks, reinterpret_cast<const char*>(a.k), slot0, a.Hkv, hk, KP, n_valid);
+    load_page_rows(ks + WM_TK * rbk, reinterpret_cast<const char*>(a.v), slot0, a.Hkv, hk, VP, n_valid);
   };
   load_tile(t0, 0);
   cp_async_commit();
   {  // the query tile, its padding columns and missing rows zero
     const T* qp = reinterpret_cast<const T*>(a.q) + (int64_t)(sq.row0 + qi0) * a.q_stride + (int64_t)h * a.D;
     if (a.D % 8 == 0 && a.q_stride % 8 == 0 && (uintptr_t)a.q % 16 == 0) {
-      const int per = a.KP / 8;
+      const int per = KP / 8;
       for (int i = tid; i < WM_TQ * per; i += WM_THREADS) {
         const int r = i / per, c = i - r * per;
         int4 v = make_int4(0, 0, 0, 0);
@@ -109,8 +111,8 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
         st16(sQ + r * rbk + c * 16, v);
       }
     } else {
-      for (int i = tid; i < WM_TQ * a.KP; i += WM_THREADS) {
-        const int r = i / a.KP, c = i - r * a.KP;
+      for (int i = tid; i < WM_TQ * KP; i += WM_THREADS) {
+        const int r = i / KP, c = i - r * KP;
         *reinterpret_cast<T*>(sQ + r * rbk + c * 2) = (r < rows && c < a.D) ? qp[r * a.q_stride + c] : Elem<T>::from_f32(0.f);
       }
     }
@@ -120,7 +122,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
   const int pos0 = p_first + row0, pos1 = pos0 + 8;
   const int lo0 = win_first(a, pos0), lo1 = win_first(a, pos1);
   const int wp0 = p_first + warp * 16, wp1 = wp0 + 15;   // positions of the warp's first and last row
-  const int nv16 = a.VP / 16, nk16 = a.KP / 16;
+  const int nv16 = VP / 16, nk16 = KP / 16;
   float o[2 * NV16][4];
 #pragma unroll
   for (int i = 0; i < 2 * NV16; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
@@ -252,15 +254,16 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
 // group are the 16-row A operand; each of the four warps takes 16 keys of a 64-key tile; warps, then
 // splits, are merged with the (max, sum, weighted output) rule.
 // ---------------------------------------------------------------------------------------------
-template <typename T, int NV16>
+template <typename T, int NV16, bool EXACT>
 __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const WinArgs a) {
   extern __shared__ __align__(128) unsigned char smem[];   // Q (16 rows) | 2 x (K | V); reused by the merge
   const int b = blockIdx.x, hk = blockIdx.y, split = blockIdx.z;
   const WinSeq sq = win_seq(a, b);
   if (sq.count == 0) return;
   const int G = a.Hq / a.Hkv;
+  const int KP = EXACT ? NV16 * 16 : a.KP, VP = EXACT ? NV16 * 16 : a.VP;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
-  const int rbk = row_bytes(a.KP), rbv = row_bytes(a.VP);
+  const int rbk = row_bytes(KP), rbv = row_bytes(VP);
   unsigned char* sQ = smem;
   unsigned char* sKV = smem + 16 * rbk;
   const int stage_bytes = WM_TK * (rbk + rbv);
@@ -274,20 +277,20 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
     const int64_t slot0 = (int64_t)win_page(a, b, key0) * a.BS + key0 % a.BS;
     unsigned char* ks = sKV + stage * stage_bytes;
     const int n_valid = min(WM_TK, sq.ctx - key0);
-    load_page_rows(ks, reinterpret_cast<const char*>(a.k), slot0, a.Hkv, hk, a.KP, n_valid);
-    load_page_rows(ks + WM_TK * rbk, reinterpret_cast<const char*>(a.v), slot0, a.Hkv, hk, a.VP, n_valid);
+    load_page_rows(ks, reinterpret_cast<const char*>(a.k), slot0, a.Hkv, hk, KP, n_valid);
+    load_page_rows(ks + WM_TK * rbk, reinterpret_cast<const char*>(a.v), slot0, a.Hkv, hk, VP, n_valid);
   };
   if (t0 < t1) load_tile(t0, 0);
   cp_async_commit();
   {
     const T* qp = reinterpret_cast<const T*>(a.q) + (int64_t)sq.row0 * a.q_stride + (int64_t)hk * G * a.D;
-    for (int i = tid; i < 16 * a.KP; i += WM_THREADS) {
-      const int r = i / a.KP, c = i - r * a.KP;
+    for (int i = tid; i < 16 * KP; i += WM_THREADS) {
+      const int r = i / KP, c = i - r * KP;
       *reinterpret_cast<T*>(sQ + r * rbk + c * 2) = (r < G && c < a.D) ? qp[r * a.D + c] : Elem<T>::from_f32(0.f);
     }
   }
   const CapConst cc = cap_const(a);
-  const int nv16 = a.VP / 16, nk16 = a.KP / 16;
+  const int nv16 = VP / 16, nk16 = KP / 16;
   float o[2 * NV16][4];
 #pragma unroll
   for (int i = 0; i < 2 * NV16; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
@@ -364,7 +367,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   __syncthreads();
-  const int W = a.VP + 2;
+  const int W = VP + 2;
   float* mbuf = reinterpret_cast<float*>(smem);   // [4 warps][16 rows][VP + 2]: O, m, l
   {
     float* w0 = mbuf + (warp * 16 + g) * W;
@@ -375,21 +378,21 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
         w0[i * 8 + 2 * tq] = o[i][0]; w0[i * 8 + 2 * tq + 1] = o[i][1];
         w1[i * 8 + 2 * tq] = o[i][2]; w1[i * 8 + 2 * tq + 1] = o[i][3];
       }
-    if (tq == 0) { w0[a.VP] = m0; w0[a.VP + 1] = l0; w1[a.VP] = m1; w1[a.VP + 1] = l1; }
+    if (tq == 0) { w0[VP] = m0; w0[VP + 1] = l0; w1[VP] = m1; w1[VP + 1] = l1; }
   }
   __syncthreads();
   for (int i = tid; i < G * a.DV; i += WM_THREADS) {
     const int row = i / a.DV, d = i - row * a.DV;
     float M = -INFINITY;
 #pragma unroll
-    for (int w = 0; w < 4; ++w) M = fmaxf(M, mbuf[(w * 16 + row) * W + a.VP]);
+    for (int w = 0; w < 4; ++w) M = fmaxf(M, mbuf[(w * 16 + row) * W + VP]);
     float num = 0.f, den = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float* rr = mbuf + (w * 16 + row) * W;
-      const float wgt = rr[a.VP] == -INFINITY ? 0.f : ex2(rr[a.VP] - M);
+      const float wgt = rr[VP] == -INFINITY ? 0.f : ex2(rr[VP] - M);
       num = fmaf(wgt, rr[d], num);
-      den = fmaf(wgt, rr[a.VP + 1], den);
+      den = fmaf(wgt, rr[VP + 1], den);
     }
     const int hq = hk * G + row;
     if (a.nsplit == 1) {
@@ -398,7 +401,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
     } else {
       float* pp = a.part + (((int64_t)b * a.Hq + hq) * a.nsplit + split) * W;
       pp[d] = num;
-      if (d == 0) { pp[a.VP] = M; pp[a.VP + 1] = den; }
+      if (d == 0) { pp[VP] = M; pp[VP + 1] = den; }
     }
   }
 }
@@ -452,7 +455,9 @@ template <typename K> static int set_smem(K kern, int bytes, const char* what) {
 
 template <typename T, int NV16, bool BOUNDED>
 static int launch_prefill(const WinArgs& a, int max_q, cudaStream_t st) {
-  auto kern = window_prefill_mma_kernel<T, NV16, BOUNDED>;
+  constexpr bool CAN = NV16 <= 8;      // (larger tiles have no registers left for it)
+  const bool exact = CAN && a.KP == NV16 * 16 && a.VP == NV16 * 16;
+  auto kern = exact ? window_prefill_mma_kernel<T, NV16, BOUNDED, CAN> : window_prefill_mma_kernel<T, NV16, BOUNDED, false>;
   const int smem = prefill_smem(a);
   if (int rc = set_smem(kern, smem, "zp_window_attention(prefill)")) return rc;
   kern<<<dim3((max_q + WM_TQ - 1) / WM_TQ, a.Hq, a.B), WM_THREADS, smem, st>>>(a);
@@ -473,7 +478,8 @@ int window_prefill_mma(const WinArgs& a, int max_q, int dtype, cudaStream_t st) 
 
 template <typename T, int NV16>
 static int launch_decode(const WinArgs& a, cudaStream_t st) {
-  auto kern = window_decode_mma_kernel<T, NV16>;
+  const bool exact = a.KP == NV16 * 16 && a.VP == NV16 * 16;
+  auto kern = exact ? window_decode_mma_kernel<T, NV16, true> : window_decode_mma_kernel<T, NV16, false>;
   const int smem = decode_smem(a);
   if (int rc = set_smem(kern, smem, "zp_window_attention(decode)")) return rc;
   kern<<<dim3(a.B, a.Hkv, a.nsplit), WM_THREADS, smem, st>>>(a);

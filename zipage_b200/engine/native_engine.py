@@ -116,18 +116,18 @@ class NativeEngine:
             seed = self.seed * 1000003 + self.step_no
             tok = self.comm.sample(logits, temps, seed=seed) if self.comm is not None else sample(logits, temps, seed=seed)
         self._tokens_host[:n].copy_(tok, non_blocking=True)
-        if self.portions:           # none of this path's kernels waits on a barrier
-            torch.cuda.current_stream().synchronize()
-            return self._tokens_host[:n].numpy().astype(np.int32)
-        # a tensor-core kernel whose bounded wait ran out (prefill attention) leaves its code in the
-        # device error word: read it with the tokens, on this stream only
+        self._finish_step()
+        return self._tokens_host[:n].numpy().astype(np.int32)
+
+    def _finish_step(self):
+        """Waits for the step.  A tensor-core kernel whose bounded wait ran out (prefill attention) leaves its code
+        in the device error word: read it with the step's results, on this stream only."""
         L.check(L.load().zp_device_error_async(L.ptr(self._pin_err), L.stream_ptr()), "device_error")
         torch.cuda.current_stream().synchronize()
         if int(self._pin_err[0]) != 0:
             code = int(self._pin_err[0])
             L.device_error(reset=True)
             raise L.ZipageError(f"a kernel of this step gave up on a barrier wait (code {code})")
-        return self._tokens_host[:n].numpy().astype(np.int32)
 
     @torch.inference_mode()
     def _prefill(self, handles):
@@ -265,7 +265,7 @@ class NativeEngine:
         out = None
         if len(rows):
             out = self.logits(hidden[torch.from_numpy(rows).to(self.device)]).float()
-        torch.cuda.current_stream().synchronize()    # the pinned step inputs are rewritten by the next step
+        self._finish_step()          # (the pinned step inputs are rewritten by the next one)
         self.scheduler.commit_portions(handles, counts)
         return out
 

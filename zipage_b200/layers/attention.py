@@ -143,7 +143,8 @@ def window_attention(q, k_cache, v_cache, context_lens, block_table, num_heads, 
     L.check(lib.zp_window_attention(
         L.ptr(q), L.ptr(k_cache), L.ptr(v_cache), L.ptr(cu_seqlens_q), L.ptr(context_lens), L.ptr(block_table),
         L.ptr(out), B, int(max_seqlen_q), NB, num_heads, Hkv, head_dim, v_dim, KP, VP, BS, P, q.stride(0),
-        out.stride(0), float(scale), float(softcap or 0.0), int(window or 0), L.IMPL[impl], L.dtype_code(q),
+        out.stride(0), float(scale), float(softcap or 0.0), int(window or 0), q.shape[0], L.IMPL[impl],
+        L.dtype_code(q),
         L.ptr(ws), 0 if ws is None else ws.numel(), L.stream_ptr()), "window_attention")
     _count(1)
     return out
