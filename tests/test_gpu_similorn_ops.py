@@ -275,3 +275,17 @@ def test_window_attention_on_long_portions(window, softcap, block):
     _close(got, want, 6e-3, "tcgen05")
     one = window_attention(qg[-1:], kc, vc, i32([S]), t[None].cuda(), H, d, d, d ** -0.5, window, softcap)
     _close(one[0], want[-1], 6e-3, "single row")
+
+
+def test_mlstm_decode_of_a_large_batch():
+    """Enough sequences for one block per head; two tokens each, odd slots."""
+    H, dk, dv, B = 3, 40, 168, 110
+    x, gates, bias, norm = _mlstm_inputs(H, dk, dv, 2 * B, 2, F32)
+    state, slots = _mlstm_state(B + 1, H, dk, dv), [(7 * b + 3) % B for b in range(B)]
+    got = [_mlstm_run(x[t * B:(t + 1) * B], gates[t * B:(t + 1) * B], bias, norm, state, [t + 1] * B, slots, H, dk, dv, 9.0, 1e-5).cpu()
+           for t in range(2)]
+    for b in (0, 1, 57, 109):
+        want, (S, n, m) = _mlstm_want(x[b::B], gates[b::B], bias, norm, H, dk, dv, 9.0, 1e-5)
+        _close(torch.stack([got[0][b], got[1][b]]), want, 2e-5)
+        _close(state[0][slots[b]], S, 1e-5)
+        _close(state[1][slots[b]], n, 1e-5)

@@ -1,8 +1,9 @@
 // Matrix-memory (mLSTM) mixer, token by token: the decode kernel, also used for prompts in fp32.
 //
-// HBM-bound: a decoded token reads and writes the head's whole fp32 state once.  One block per
-// (value tile, head, sequence); the blocks of a head form a cluster, because the output norm needs the sum
-// of squares over all value dims (exchanged through distributed shared memory).  A thread owns four
+// HBM-bound: a decoded token reads and writes the head's whole fp32 state once.  One block per (head,
+// sequence), or, for small batches, per value tile of a head; the blocks of a head then form a cluster,
+// because the output norm needs the sum of squares over all value dims (exchanged through distributed shared
+// memory).  A thread owns four
 // adjacent value columns and every nrg-th row of the state, so a warp moves whole rows of a tile with
 // 16-byte accesses.  Gates, state update, read-out, normaliser, head norm and output gate are one
 // launch.  With several tokens per sequence the block loops; each thread re-reads only what it wrote.
@@ -11,10 +12,10 @@
 namespace zp {
 
 constexpr int ML_THREADS = 256;
-constexpr int ML_BATCH = 8;    // state rows in flight per thread
+constexpr int ML_BATCH = 4;    // state rows of a batch; two batches are in flight per thread
 
 template <typename T>
-__global__ void __launch_bounds__(ML_THREADS) mlstm_recurrent_kernel(const MlstmArgs a) {
+__global__ void __launch_bounds__(ML_THREADS, 2) mlstm_recurrent_kernel(const MlstmArgs a) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
   __shared__ float xsum[2];      // this block's sum of squares, by token parity
@@ -41,16 +42,18 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_recurrent_kernel(const Mlstm
 
   for (int t = 0; t < sq.count; ++t) {
     const int64_t row = sq.row0 + t;
-    // the first batch of state rows is on its way while the gates are computed
-    float4 s[ML_BATCH];
-    auto load_rows = [&](int r0) {
+    // two batches of state rows alternate: one is updated while the other's loads are in flight, the
+    // first while the gates are computed
+    float4 sa[ML_BATCH], sb[ML_BATCH];
+    const int step = nrg * ML_BATCH;
+    auto load_rows = [&](float4 (&s)[ML_BATCH], int r0) {
 #pragma unroll
       for (int u = 0; u < ML_BATCH; ++u) {
         const int r = r0 + u * nrg;
         s[u] = (r < a.dim && !zero) ? *reinterpret_cast<const float4*>(S + (int64_t)r * a.VP) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
     };
-    if (mine) load_rows(rg);
+    if (mine) load_rows(sa, rg);
     const float gi = log_input_gate(a, row, h), gf = log_forget_gate(a, row, h);
     const float m_new = fmaxf(gf + m, gi);
     const float keep = expf(gf + m - m_new), add = expf(gi - m_new);
@@ -69,8 +72,7 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_recurrent_kernel(const Mlstm
 #pragma unroll
       for (int j = 0; j < 4; ++j)
         v[j] = col + j < a.vdim ? add * Elem<T>::to_f32(vb[row * a.row_stride + (int64_t)h * a.vdim + col + j]) : 0.f;
-      for (int r0 = rg; r0 < a.dim; r0 += nrg * ML_BATCH) {
-        if (r0 != rg) load_rows(r0);
+      auto update_rows = [&](float4 (&s)[ML_BATCH], int r0) {
 #pragma unroll
         for (int u = 0; u < ML_BATCH; ++u) {
           const int r = r0 + u * nrg;
@@ -83,6 +85,12 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_recurrent_kernel(const Mlstm
             *reinterpret_cast<float4*>(S + (int64_t)r * a.VP) = s[u];
           }
         }
+      };
+      for (int r0 = rg; r0 < a.dim; r0 += 2 * step) {
+        load_rows(sb, r0 + step);
+        update_rows(sa, r0);
+        load_rows(sa, r0 + 2 * step);
+        update_rows(sb, r0 + step);
       }
       *reinterpret_cast<float4*>(part + rg * a.VT + 4 * cg) = make_float4(acc[0], acc[1], acc[2], acc[3]);
     }
@@ -129,8 +137,9 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_recurrent_kernel(const Mlstm
 
 template <typename T>
 static int launch_recurrent(MlstmArgs a, cudaStream_t st) {
-  int tiles = (a.VP + 63) / 64;
-  if (tiles > 8) tiles = 8;
+  // a whole head per block, or, when the batch leaves most SMs without one, up to eight value tiles
+  int tiles = (a.VP + 1023) / 1024;
+  while (2 * tiles <= 8 && (int64_t)a.B * a.H * tiles < 148 * 2 && a.VP / tiles > 64) tiles *= 2;
   a.VT = ((a.VP + tiles - 1) / tiles + 3) & ~3;
   tiles = (a.VP + a.VT - 1) / a.VT;
   const int nrg = ML_THREADS / (a.VT / 4);
