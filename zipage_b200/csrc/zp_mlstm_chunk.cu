@@ -14,6 +14,8 @@
 // in S^T q, the decayed scores, and the decayed values of the state update; q, k and v are bf16
 // already.  The blocks of a head form a cluster and exchange per-row sums of squares for the head norm
 // through distributed shared memory, so the normalised, gated output leaves the kernel in one pass.
+#include <type_traits>
+
 #include "zp_mlstm.cuh"
 #include "zp_mma.cuh"
 
@@ -57,7 +59,7 @@ __device__ __forceinline__ void for_blocks(const unsigned char* tile, int row0, 
 template <int DP> struct ChunkSmem {
   static constexpr int RB = DP * 2 + 16;
   static constexpr int Q = 0, K = Q + MC_C * RB, V = K + MC_C * RB, S = V + MC_C * MC_RB, P = S + 2 * DP * MC_RB,
-                       G = P + 2 * MC_C * MC_RB, F = G + MC_C * MC_RB, TOTAL = F + 14 * MC_C * 4;
+                       G = P + 2 * MC_C * MC_RB, F = G + MC_C * MC_RB, TOTAL = F + 25 * MC_C * 4;
 };
 
 template <int DP>
@@ -75,10 +77,12 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
   unsigned char *sSh = smem + L::S, *sSl = sSh + DP * MC_RB;
   unsigned char *sPh = smem + L::P, *sPl = sPh + MC_C * MC_RB;
   float* fl = reinterpret_cast<float*>(smem + L::F);
-  float *sM = fl, *sU = fl + 64, *sA = fl + 128, *sE = fl + 192, *sW = fl + 256, *sDen = fl + 320, *sR = fl + 384;
+  float *sDen = fl + 320, *sR = fl + 384;
+  float* sScan = fl + 896;                       // [2 parities][M, u, A, E, W][64]: see scan()
   float *sSq = fl + 448;                         // [2 parities][2 halves][64] (read by the cluster)
   float *sMisc = fl + 704;                       // running maximum, decay of the state over the chunk
   float* sAct = fl + 768;                        // log input gates, log forget gates of the chunk
+  float* sNorm = fl + 1536;                      // norm weights of the value tile
   unsigned char* sG = smem + L::G;
   const int c0 = vt * MC_VT, vcols = min(MC_VT, a.vdim - c0);
   const int nk16 = (a.dim + 15) / 16;
@@ -111,11 +115,15 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
         s[i][cb][j] = x;
       }
 
+  using Wide = std::integral_constant<int, DP>;
+  using Narrow = std::integral_constant<int, MC_VT>;
   // tiles of the chunk that starts at token t0 (n tokens; none: only the group is committed)
-  auto load_tile = [&](const T* base, unsigned char* dst, int rb, int cols16, int valid_cols, int t0, int n) {
+  auto load_tile = [&](auto width, const T* base, unsigned char* dst, int valid_cols, int t0, int n) {
+    constexpr int cols16 = decltype(width)::value / 8, rb = decltype(width)::value == DP ? L::RB : MC_RB;
     const int64_t row0 = sq.row0 + t0;
     if (n > 0) {
       if (vec) {
+        _Pragma("unroll")
         for (int i = tid; i < MC_C * cols16; i += MC_THREADS) {
           const int r = i / cols16, c = i % cols16;
           const int ok = (r < n && c * 8 < valid_cols) ? 16 : 0;
@@ -144,7 +152,8 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     }
   };
   // one warp: running sums and maxima of the chunk's gates (two tokens per lane)
-  auto scan = [&]() {
+  auto scan = [&](int par) {
+    float *sM = sScan + par * 320, *sU = sM + 64, *sA = sM + 128, *sE = sM + 192, *sW = sM + 256;
     float f[2] = {sAct[64 + 2 * lane], sAct[65 + 2 * lane]}, u[2] = {sAct[2 * lane], sAct[2 * lane + 1]};
     float F = f[0] + f[1];
 #pragma unroll
@@ -165,22 +174,30 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     sE[t] = expf(-(M0 + F0)); sE[t + 1] = expf(-(M1 + F1));
     sW[t] = expf(u[0] - MC); sW[t + 1] = expf(u[1] - MC);
     __syncwarp();
-    if (lane == 0) { sMisc[1] = expf(m - MC); sMisc[0] = MC + FC; }
+    if (lane == 0) { sMisc[1 + par] = expf(m - MC); sMisc[0] = MC + FC; }
   };
 
   {
     const int n = min(MC_C, sq.count);
-    load_tile(qb, sQ, L::RB, DP / 8, a.dim, 0, n);
-    load_tile(kb, sK, L::RB, DP / 8, a.dim, 0, n);
-    load_tile(vb, sV, MC_RB, 8, vcols, 0, n);
+    load_tile(Wide{}, qb, sQ, a.dim, 0, n);
+    load_tile(Wide{}, kb, sK, a.dim, 0, n);
+    load_tile(Narrow{}, vb, sV, vcols, 0, n);
     gate_put(gate_raw(0, n), n);
+    for (int i = tid; i < MC_VT; i += MC_THREADS) sNorm[i] = i < vcols ? a.norm_weight[(int64_t)h * a.vdim + c0 + i] : 0.f;
+    __syncthreads();
+    if (warp == 0) scan(0);
+    __syncthreads();
+    const int n1 = min(MC_C, sq.count - MC_C);
+    gate_put(gate_raw(MC_C, n1), n1);
   }
   __syncthreads();
+  const float inv_vdim = 1.f / (float)a.vdim;
   const int row_a = rg * 16 + g, row_b = row_a + 8;   // this thread's two tokens of the chunk
   for (int t0 = 0, par = 0; t0 < sq.count; t0 += MC_C, par ^= 1) {
     const int n = min(MC_C, sq.count - t0), t1 = t0 + MC_C, n1 = min(MC_C, sq.count - t1);   // n1 <= 0: the last one
-    if (warp == 0) scan();
-    const float raw_next = gate_raw(t1, n1);
+    const int t2 = t1 + MC_C, n2 = min(MC_C, sq.count - t2);
+    const float raw_next = gate_raw(t2, n2);           // (used two chunks ahead)
+    const float *sM = sScan + par * 320, *sU = sM + 64, *sA = sM + 128, *sE = sM + 192, *sW = sM + 256;
     // 16-bit operand copies of the state tile
 #pragma unroll
     for (int i = 0; i < MB; ++i)
@@ -198,7 +215,7 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
       }
     cp_async_wait<0>();
     __syncthreads();
-    load_tile(gb, sG, MC_RB, 8, vcols, t0, n);
+    load_tile(Narrow{}, gb, sG, vcols, t0, n);
 
     float acc[5][4], p[4][4];
 #pragma unroll
@@ -241,13 +258,14 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
         *reinterpret_cast<uint32_t*>(sPl + row_b * MC_RB + key * 2) = lo;
       }
     }
+    else if (warp == 4) scan(par ^ 1);                 // a warp without scores prepares the next chunk's gates
     {
       const float fa = sA[row_a] * a.qscale, fb = sA[row_b] * a.qscale;
 #pragma unroll
       for (int i = 0; i < 5; ++i) { acc[i][0] *= fa; acc[i][1] *= fa; acc[i][2] *= fb; acc[i][3] *= fb; }
     }
     __syncthreads();
-    load_tile(qb, sQ, L::RB, DP / 8, a.dim, t1, n1);
+    load_tile(Wide{}, qb, sQ, a.dim, t1, n1);
     for (int kk = 0; kk <= rg; ++kk) {                 // keys 16 kk .. 16 kk + 15 of rows up to 16 rg + 15
       uint32_t ph[4], pl[4];
       ldmatrix_x4(ph, sPh + (rg * 16 + (lane & 15)) * MC_RB + kk * 32 + (lane >> 4) * 16);
@@ -259,8 +277,8 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     }
     if (half && tq == 0) { sDen[row_a] = acc[4][0]; sDen[row_b] = acc[4][2]; }   // n . q, decayed like the rest
     __syncthreads();
-    const float da = 1.f / (fmaxf(fabsf(sDen[row_a]), sE[row_a]) + MLSTM_DEN_EPS);
-    const float db = 1.f / (fmaxf(fabsf(sDen[row_b]), sE[row_b]) + MLSTM_DEN_EPS);
+    const float da = __fdividef(1.f, fmaxf(fabsf(sDen[row_a]), sE[row_a]) + MLSTM_DEN_EPS);
+    const float db = __fdividef(1.f, fmaxf(fabsf(sDen[row_b]), sE[row_b]) + MLSTM_DEN_EPS);
     float qa2 = 0.f, qb2 = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {                      // (columns past vdim are zero)
@@ -272,9 +290,10 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     qb2 += __shfl_xor_sync(0xffffffffu, qb2, 1); qb2 += __shfl_xor_sync(0xffffffffu, qb2, 2);
     if (tq == 0) { sSq[(par * 2 + half) * 64 + row_a] = qa2; sSq[(par * 2 + half) * 64 + row_b] = qb2; }
     // decayed values (and the decayed column of ones), over the scores' shared memory
-    for (int i = tid; i < MC_C * 36; i += MC_THREADS) {
-      const int r = i / 36, c = i % 36;
-      const float w = sW[r];
+    const float w = sW[tid >> 2];
+#pragma unroll
+    for (int i = 0; i < 9; ++i) {
+      const int r = tid >> 2, c = (tid & 3) + 4 * i;
       const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sV + r * MC_RB + c * 4));
       uint32_t hi, lo;
       split_bf16(v.x * w, v.y * w, hi, lo);
@@ -282,15 +301,15 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
       *reinterpret_cast<uint32_t*>(sPl + r * MC_RB + c * 4) = lo;
     }
     if (cluster_size() > 1) cluster_sync(); else __syncthreads();
-    load_tile(vb, sV, MC_RB, 8, vcols, t1, n1);
-    gate_put(raw_next, n1);
+    load_tile(Narrow{}, vb, sV, vcols, t1, n1);
+    gate_put(raw_next, n2);
     if (tid < MC_C) {
       float ss = 0.f;
       for (uint32_t r = 0; r < cluster_size(); ++r)
         ss += ld_cluster(&sSq[par * 128 + tid], r) + ld_cluster(&sSq[par * 128 + 64 + tid], r);
-      sR[tid] = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
+      sR[tid] = rsqrtf(ss * inv_vdim + a.eps);
     }
-    const float decay = sMisc[1];
+    const float decay = sMisc[1 + par];
 #pragma unroll
     for (int i = 0; i < MB; ++i) {
       if ((rg + 4 * i) * 16 < a.dim) {
@@ -312,7 +331,7 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     }
     cp_async_wait<2>();                                // the gate tile (two younger groups: the next Q and V)
     __syncthreads();                                   // K free for the next chunk; sR visible
-    load_tile(kb, sK, L::RB, DP / 8, a.dim, t1, n1);
+    load_tile(Wide{}, kb, sK, a.dim, t1, n1);
     const float ra = sR[row_a], rb = sR[row_b];
     const int64_t grow = sq.row0 + t0;
 #pragma unroll
@@ -326,10 +345,9 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
         const int64_t e = (int64_t)h * a.vdim + c;
         const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sG + r * MC_RB + (half * 32 + i * 8 + 2 * tq) * 2));
         T* op = reinterpret_cast<T*>(a.out) + (grow + r) * a.out_stride + e;
-        float o[2];
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-          o[j] = c + j < a.vdim ? acc[i][2 * y + j] * rr * a.norm_weight[e + j] / (1.f + __expf(-(j ? gv.y : gv.x))) : 0.f;
+        const float2 nw = *reinterpret_cast<const float2*>(sNorm + half * 32 + i * 8 + 2 * tq);
+        const float o[2] = {acc[i][2 * y] * rr * nw.x * __fdividef(1.f, 1.f + __expf(-gv.x)),
+                            acc[i][2 * y + 1] * rr * nw.y * __fdividef(1.f, 1.f + __expf(-gv.y))};
         if (vec && a.out_stride % 2 == 0) { if (c < a.vdim) *reinterpret_cast<uint32_t*>(op) = pack2<T>(o[0], o[1]); }
         else {
           if (c < a.vdim) op[0] = Elem<T>::from_f32(o[0]);
