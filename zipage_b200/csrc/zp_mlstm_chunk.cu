@@ -24,8 +24,11 @@ namespace zp {
 constexpr int MC_THREADS = 256;
 constexpr int MC_C = 64;            // tokens per chunk
 constexpr int MC_VT = 64;           // value columns per block
+constexpr float MC_LOG2E = 1.4426950408889634f;
 constexpr int MC_RB = 144;          // bytes of a 72-column bf16 row (an odd number of 16-byte chunks)
 
+__device__ __forceinline__ float exp2_(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float rcp_approx(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
   hi = *reinterpret_cast<const uint32_t*>(&h);
@@ -85,7 +88,6 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
   float* sNorm = fl + 1536;                      // norm weights of the value tile
   unsigned char* sG = smem + L::G;
   const int c0 = vt * MC_VT, vcols = min(MC_VT, a.vdim - c0);
-  const int nk16 = (a.dim + 15) / 16;
   const int64_t head = (int64_t)sq.slot * a.H + h;
   const T* qb = reinterpret_cast<const T*>(a.q) + (int64_t)h * a.dim;
   const T* kb = reinterpret_cast<const T*>(a.k) + (int64_t)h * a.dim;
@@ -152,6 +154,7 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     }
   };
   // one warp: running sums and maxima of the chunk's gates (two tokens per lane)
+  const float log2_qscale = log2f(a.qscale);
   auto scan = [&](int par) {
     float *sM = sScan + par * 320, *sU = sM + 64, *sA = sM + 128, *sE = sM + 192, *sW = sM + 256;
     float f[2] = {sAct[64 + 2 * lane], sAct[65 + 2 * lane]}, u[2] = {sAct[2 * lane], sAct[2 * lane + 1]};
@@ -169,8 +172,10 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     const float M0 = fmaxf(before, u[0]), M1 = fmaxf(M0, u[1]);
     const float MC = __shfl_sync(0xffffffffu, M1, 31), FC = __shfl_sync(0xffffffffu, F1, 31);
     const int t = 2 * lane;
-    sM[t] = M0; sM[t + 1] = M1; sU[t] = u[0]; sU[t + 1] = u[1];
-    sA[t] = expf(m - M0); sA[t + 1] = expf(m - M1);
+    // (exponents in log2 units, the query scale folded into the row's)
+    sM[t] = fmaf(M0, MC_LOG2E, -log2_qscale); sM[t + 1] = fmaf(M1, MC_LOG2E, -log2_qscale);
+    sU[t] = u[0] * MC_LOG2E; sU[t + 1] = u[1] * MC_LOG2E;
+    sA[t] = expf(m - M0) * a.qscale; sA[t + 1] = expf(m - M1) * a.qscale;
     sE[t] = expf(-(M0 + F0)); sE[t + 1] = expf(-(M1 + F1));
     sW[t] = expf(u[0] - MC); sW[t + 1] = expf(u[1] - MC);
     __syncwarp();
@@ -223,8 +228,8 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
 #pragma unroll
     for (int i = 0; i < 4; ++i) { p[i][0] = p[i][1] = p[i][2] = p[i][3] = 0.f; }
     const bool scores = half * 32 <= rg * 16 + 15;     // else every key of this half is later than the rows
-#pragma unroll 2
-    for (int kk = 0; kk < nk16; ++kk) {
+#pragma unroll
+    for (int kk = 0; kk < DP / 16; ++kk) {
       uint32_t qa[4];
       ldmatrix_x4(qa, sQ + (rg * 16 + (lane & 15)) * L::RB + kk * 32 + (lane >> 4) * 16);
       for_blocks(sSh, kk * 16, half, lane, [&](int i, uint32_t b0, uint32_t b1) { mma16816<T>(acc[i], qa, b0, b1); });
@@ -244,11 +249,11 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
 #pragma unroll
       for (int nb = 0; nb < 4; ++nb) {
         const int key = half * 32 + nb * 8 + 2 * tq;
-        const float u0 = sU[key], u1 = sU[key + 1];
-        const float p0 = key <= row_a ? p[nb][0] * a.qscale * __expf(u0 - Ma) : 0.f;
-        const float p1 = key + 1 <= row_a ? p[nb][1] * a.qscale * __expf(u1 - Ma) : 0.f;
-        const float p2 = key <= row_b ? p[nb][2] * a.qscale * __expf(u0 - Mb) : 0.f;
-        const float p3 = key + 1 <= row_b ? p[nb][3] * a.qscale * __expf(u1 - Mb) : 0.f;
+        const float2 u = *reinterpret_cast<const float2*>(sU + key);
+        const float p0 = key <= row_a ? p[nb][0] * exp2_(u.x - Ma) : 0.f;
+        const float p1 = key + 1 <= row_a ? p[nb][1] * exp2_(u.y - Ma) : 0.f;
+        const float p2 = key <= row_b ? p[nb][2] * exp2_(u.x - Mb) : 0.f;
+        const float p3 = key + 1 <= row_b ? p[nb][3] * exp2_(u.y - Mb) : 0.f;
         uint32_t hi, lo;
         split_bf16(p0, p1, hi, lo);
         *reinterpret_cast<uint32_t*>(sPh + row_a * MC_RB + key * 2) = hi;
@@ -260,13 +265,15 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     }
     else if (warp == 4) scan(par ^ 1);                 // a warp without scores prepares the next chunk's gates
     {
-      const float fa = sA[row_a] * a.qscale, fb = sA[row_b] * a.qscale;
+      const float fa = sA[row_a], fb = sA[row_b];
 #pragma unroll
       for (int i = 0; i < 5; ++i) { acc[i][0] *= fa; acc[i][1] *= fa; acc[i][2] *= fb; acc[i][3] *= fb; }
     }
     __syncthreads();
     load_tile(Wide{}, qb, sQ, a.dim, t1, n1);
-    for (int kk = 0; kk <= rg; ++kk) {                 // keys 16 kk .. 16 kk + 15 of rows up to 16 rg + 15
+#pragma unroll
+    for (int kk = 0; kk < MC_C / 16; ++kk) {           // keys 16 kk .. 16 kk + 15 of rows up to 16 rg + 15
+      if (kk > rg) break;
       uint32_t ph[4], pl[4];
       ldmatrix_x4(ph, sPh + (rg * 16 + (lane & 15)) * MC_RB + kk * 32 + (lane >> 4) * 16);
       ldmatrix_x4(pl, sPl + (rg * 16 + (lane & 15)) * MC_RB + kk * 32 + (lane >> 4) * 16);
@@ -277,8 +284,8 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
     }
     if (half && tq == 0) { sDen[row_a] = acc[4][0]; sDen[row_b] = acc[4][2]; }   // n . q, decayed like the rest
     __syncthreads();
-    const float da = __fdividef(1.f, fmaxf(fabsf(sDen[row_a]), sE[row_a]) + MLSTM_DEN_EPS);
-    const float db = __fdividef(1.f, fmaxf(fabsf(sDen[row_b]), sE[row_b]) + MLSTM_DEN_EPS);
+    const float da = rcp_approx(fmaxf(fabsf(sDen[row_a]), sE[row_a]) + MLSTM_DEN_EPS);
+    const float db = rcp_approx(fmaxf(fabsf(sDen[row_b]), sE[row_b]) + MLSTM_DEN_EPS);
     float qa2 = 0.f, qb2 = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {                      // (columns past vdim are zero)
@@ -317,7 +324,9 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
         for (int cb = 0; cb < 5; ++cb) { s[i][cb][0] *= decay; s[i][cb][1] *= decay; s[i][cb][2] *= decay; s[i][cb][3] *= decay; }
       }
     }
-    for (int kk = 0; kk * 16 < n; ++kk) {
+#pragma unroll
+    for (int kk = 0; kk < MC_C / 16; ++kk) {
+      if (kk * 16 >= n) break;
       uint32_t ka[MB][4];
 #pragma unroll
       for (int i = 0; i < MB; ++i)
@@ -346,8 +355,8 @@ __global__ void __launch_bounds__(MC_THREADS, DP <= 128 ? 2 : 1) mlstm_chunk_ker
         const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sG + r * MC_RB + (half * 32 + i * 8 + 2 * tq) * 2));
         T* op = reinterpret_cast<T*>(a.out) + (grow + r) * a.out_stride + e;
         const float2 nw = *reinterpret_cast<const float2*>(sNorm + half * 32 + i * 8 + 2 * tq);
-        const float o[2] = {acc[i][2 * y] * rr * nw.x * __fdividef(1.f, 1.f + __expf(-gv.x)),
-                            acc[i][2 * y + 1] * rr * nw.y * __fdividef(1.f, 1.f + __expf(-gv.y))};
+        const float o[2] = {acc[i][2 * y] * rr * nw.x * rcp_approx(1.f + exp2_(-MC_LOG2E * gv.x)),
+                            acc[i][2 * y + 1] * rr * nw.y * rcp_approx(1.f + exp2_(-MC_LOG2E * gv.y))};
         if (vec && a.out_stride % 2 == 0) { if (c < a.vdim) *reinterpret_cast<uint32_t*>(op) = pack2<T>(o[0], o[1]); }
         else {
           if (c < a.vdim) op[0] = Elem<T>::from_f32(o[0]);
