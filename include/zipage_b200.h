@@ -449,14 +449,15 @@ int zp_window_attention(const void* q, const void* k_cache, const void* v_cache,
  * State in fp32: state [n_slots, H, dim, VP] (VP >= vdim, a multiple of 4), state_n [n_slots, H, dim],
  * state_m [n_slots, H]; slots [B].  cu_seqlens_q / context_lens as in zp_window_attention; a sequence
  * whose context equals its rows starts from zero, whatever its slot holds.
- * bf16 with cu_seqlens_q, dim <= 256 and vdim <= 512 takes the chunked tensor-core kernel
- * (ZP_IMPL_SIMT: never). */
+ * bf16 with cu_seqlens_q, dim <= 256 and vdim <= 512 takes a chunked tensor-core kernel (ZP_IMPL_SIMT:
+ * never); with total_rows (rows of q, k, v, g; 0 = not told), dim 128, vdim a multiple of 128 and at least
+ * 64 rows per sequence on average its tcgen05 form (ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED). */
 int zp_mlstm(const void* q, const void* k, const void* v, const void* g, const float* gates,
              const float* gate_bias, const float* norm_weight, const int32_t* cu_seqlens_q,
              const int32_t* context_lens, const int32_t* slots, float* state, float* state_n, float* state_m,
              void* out, int B, int H, int dim, int vdim, int VP, int n_slots, int64_t row_stride,
-             int64_t gates_stride, int64_t out_stride, float qscale, float gate_cap, float eps, int impl,
-             int dtype, void* stream);
+             int64_t gates_stride, int64_t out_stride, float qscale, float gate_cap, float eps, int total_rows,
+             int impl, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

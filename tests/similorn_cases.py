@@ -35,6 +35,9 @@ CONFIGS = {
                       width=80, vocab=64),
     "one_pass_over_all": config([attention(5, 5, 48, 16, 65, softcap=30.0, ff=40), mlstm(2, 20, 28, cap=30.0)], width=72,
                                 vocab=203, loop=(0, 2, 1), embed_scale=9.5),
+    # head sizes of the tcgen05 kernels
+    "large_heads": config([mlstm(1, 128, 128), attention(2, 1, 128, 128, 100, softcap=30.0, ff=64), mlstm(2, 128, 256)], width=64,
+                          vocab=90, loop=(1, 3, 2)),
     "odd_sizes": config([mlstm(3, 17, 23), attention(3, 1, 13, 19, 77, ff=61)], width=58, vocab=101, loop=(1, 2, 2)),
 }
 

@@ -106,7 +106,7 @@ def test_every_cut_gives_the_same_logits(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("name", ["mixed", "loop_in_the_middle", "odd_sizes"])
+@pytest.mark.parametrize("name", ["mixed", "loop_in_the_middle", "odd_sizes", "large_heads"])
 def test_mixed_batches_with_reused_pages_and_slots(name, dtype):
     """Random batches of portions beside single tokens; requests pause, end and make room for others in
     a pool just large enough, so that pages and slots change hands."""

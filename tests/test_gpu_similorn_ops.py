@@ -289,3 +289,36 @@ def test_mlstm_decode_of_a_large_batch():
         _close(torch.stack([got[0][b], got[1][b]]), want, 2e-5)
         _close(state[0][slots[b]], S, 1e-5)
         _close(state[1][slots[b]], n, 1e-5)
+
+
+@pytest.mark.parametrize("dv", [128, 256, 512])
+@pytest.mark.parametrize("lengths", [(128,), (1, 300), (257, 128, 40)])
+def test_mlstm_tcgen05_portions(dv, lengths):
+    """Key size 128: 128-token chunks on tcgen05, one portion after another (whole chunks, ragged ends, two
+    tokens), against the recurrence; what the other rows of the batch hold must not matter."""
+    H, dk, cap, eps = 2, 128, 8.0, 1e-4
+    data = [_mlstm_inputs(H, dk, dv, n, 40 + n, BF) for n in lengths]
+    for d in data:
+        d[2].copy_(data[0][2]), d[3].copy_(data[0][3])
+    want = [_mlstm_want(*d, H, dk, dv, cap, eps) for d in data]
+    B = len(lengths)
+    state, slots = _mlstm_state(B + 1, H, dk, dv), [(i + 1) % (B + 1) for i in range(B)]
+    got = [[] for _ in lengths]
+    cuts = [[0] * B, [min(n, 130) for n in lengths], [min(n, 132) for n in lengths], list(lengths)]
+    for a, b in zip(cuts, cuts[1:]):
+        live = [i for i in range(B) if b[i] > a[i]]
+        if not live:
+            continue
+        rows = [b[i] - a[i] for i in live]
+        x, g = (torch.cat([data[i][j][a[i]:b[i]] for i in live] + [torch.full_like(data[0][j][:1], float("nan"))]) for j in (0, 1))
+        cu = [0] + torch.tensor(rows).cumsum(0).tolist()
+        o = _mlstm_run(x, g, *data[0][2:], state, [b[i] for i in live], [slots[i] for i in live], H, dk, dv, cap, eps, cu=cu,
+                       impl="tcgen05")
+        for k, i in enumerate(live):
+            got[i].append(o[cu[k]:cu[k + 1]].cpu())
+    for i in range(B):
+        _close(torch.cat(got[i]), want[i][0], 6e-3, f"outputs {i}")
+        S, n, m = want[i][1]
+        _close(state[0][slots[i]], S, 1e-4, f"S {i}")
+        _close(state[1][slots[i]], n, 1e-4, f"n {i}")
+        assert (state[2][slots[i]].cpu().double() - m).abs().max() < 1e-3

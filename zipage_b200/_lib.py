@@ -83,7 +83,7 @@ SIGNATURES = {
     "zp_store_kv_padded": (_I, [_P] * 5 + [_I] * 6 + [_L, _L, _I, _P]),
     "zp_window_attention_workspace_bytes": (_Z, [_I] * 5),
     "zp_window_attention": (_I, [_P] * 7 + [_I] * 11 + [_L, _L, _F, _F, _I, _I, _I, _I, _P, _Z, _P]),
-    "zp_mlstm": (_I, [_P] * 14 + [_I] * 6 + [_L] * 3 + [_F] * 3 + [_I, _I, _P]),
+    "zp_mlstm": (_I, [_P] * 14 + [_I] * 6 + [_L] * 3 + [_F] * 3 + [_I, _I, _I, _P]),
     "zp_comm_create": (_I, [_I, _I, _Z, _I, C.POINTER(_P)]),
     "zp_comm_segment": (_I, [_P, C.POINTER(_P), C.POINTER(_Z)]),
     "zp_comm_ipc_handle": (_I, [_P, _P]),

@@ -30,7 +30,7 @@ FLAGS = [
 
 # sources of one model family (stems of csrc/*.cu)
 PARTS = {
-    "similorn": ("zp_api", "zp_host_sched", "zp_mlstm", "zp_mlstm_chunk", "zp_rows", "zp_step", "zp_tc",
+    "similorn": ("zp_api", "zp_host_sched", "zp_mlstm", "zp_mlstm_chunk", "zp_mlstm_tc", "zp_rows", "zp_step", "zp_tc",
                  "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
 }
 

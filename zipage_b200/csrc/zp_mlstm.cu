@@ -161,6 +161,9 @@ static int launch_recurrent(MlstmArgs a, cudaStream_t st) {
 // chunked tensor-core prefill (zp_mlstm_chunk.cu)
 bool mlstm_chunk_supports(const MlstmArgs& a, int dtype);
 int mlstm_chunk(const MlstmArgs& a, cudaStream_t st);
+// its tcgen05 form (zp_mlstm_tc.cu)
+bool mlstm_tc_supports(const MlstmArgs& a, int total_rows, int dtype);
+int mlstm_tc(const MlstmArgs& a, int total_rows, cudaStream_t st);
 
 }  // namespace zp
 
@@ -169,7 +172,7 @@ extern "C" int zp_mlstm(const void* q, const void* k, const void* v, const void*
                         const int32_t* context_lens, const int32_t* slots, float* state, float* state_n,
                         float* state_m, void* out, int B, int H, int dim, int vdim, int VP, int n_slots,
                         int64_t row_stride, int64_t gates_stride, int64_t out_stride, float qscale, float gate_cap,
-                        float eps, int impl, int dtype, void* stream) {
+                        float eps, int total_rows, int impl, int dtype, void* stream) {
   if (B == 0) return ZP_OK;
   ZP_REQUIRE(q && k && v && g && gates && gate_bias && norm_weight && context_lens && slots && state && state_n &&
                  state_m && out, "zp_mlstm: null pointer");
@@ -184,6 +187,14 @@ extern "C" int zp_mlstm(const void* q, const void* k, const void* v, const void*
   a.row_stride = row_stride; a.gates_stride = gates_stride; a.out_stride = out_stride;
   a.qscale = qscale; a.cap = gate_cap; a.eps = eps;
   cudaStream_t st = (cudaStream_t)stream;
+  const bool tc = cu_seqlens_q && zp::mlstm_tc_supports(a, total_rows, dtype);
+  if (impl == ZP_IMPL_TCGEN05 && !tc) {
+    zp::set_error("zp_mlstm: the tcgen05 kernel needs bf16 portions, a key size of 128, a value size that is a multiple of "
+                  "128 and 16-byte aligned rows");
+    return ZP_ERR_UNSUPPORTED;
+  }
+  // (chunks of 128 tokens: not for portions of a few)
+  if (tc && (impl == ZP_IMPL_TCGEN05 || (impl == ZP_IMPL_AUTO && total_rows >= 64 * B))) return zp::mlstm_tc(a, total_rows, st);
   if (cu_seqlens_q && impl != ZP_IMPL_SIMT && zp::mlstm_chunk_supports(a, dtype)) return zp::mlstm_chunk(a, st);
   ZP_DISPATCH_DTYPE(dtype, T, { return zp::launch_recurrent<T>(a, st); });
   return ZP_OK;

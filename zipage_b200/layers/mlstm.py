@@ -29,7 +29,7 @@ def mlstm_step(q, k, v, g, gates, gate_bias, norm_weight, state, out, context_le
         L.ptr(q), L.ptr(k), L.ptr(v), L.ptr(g), L.ptr(gates), L.ptr(gate_bias), L.ptr(norm_weight),
         L.ptr(cu_seqlens_q), L.ptr(context_lens), L.ptr(slots), L.ptr(S), L.ptr(n), L.ptr(m), L.ptr(out),
         B, heads, dim, vdim, S.shape[3], S.shape[0], q.stride(0), gates.stride(0), out.stride(0),
-        float(dim ** -0.5 if qscale is None else qscale), float(gate_cap), float(eps), L.IMPL[impl],
+        float(dim ** -0.5 if qscale is None else qscale), float(gate_cap), float(eps), q.shape[0], L.IMPL[impl],
         L.dtype_code(out), L.stream_ptr()), "mlstm")
     _count(1)
     return out
