@@ -337,6 +337,11 @@ mlstm_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         fence_async();
         if (!csync(924)) { ok = false; break; }
       }
+      if (r < n) {                                 // the output gate is read at the end of the chunk
+        const T* gp = reinterpret_cast<const T*>(a.g) + (sq.row0 + (int64_t)c * 128 + r) * a.row_stride + (int64_t)h * a.vdim + c0 + cq * 32;
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(gp));
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(gp + 16));
+      }
       // n . q over this thread's 32 key dims
       if (!mbar_wait(&sh.full[slot(tq)], phase(tq), abortp, err, 925)) { ok = false; break; }
       float nq = 0.f;
