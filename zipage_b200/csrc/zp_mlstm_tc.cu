@@ -119,6 +119,21 @@ __device__ __forceinline__ bool mt_wait_cluster(uint64_t* bar, uint32_t parity, 
   return false;
 }
 
+// 4 x 4 transpose of 16-byte chunks within groups of four lanes: v[i] of lane t <- v[t] of lane i.  Turns
+// "one row per lane" into "four lanes per row", so that global accesses touch whole 64-byte row pieces.
+__device__ __forceinline__ void mt_transpose4(int4 (&v)[4], int lane) {
+  auto swap = [&](int4& x, int4& y, int mask, bool upper) {
+    int4 snd = upper ? x : y, rcv;
+    rcv.x = __shfl_xor_sync(0xffffffffu, snd.x, mask); rcv.y = __shfl_xor_sync(0xffffffffu, snd.y, mask);
+    rcv.z = __shfl_xor_sync(0xffffffffu, snd.z, mask); rcv.w = __shfl_xor_sync(0xffffffffu, snd.w, mask);
+    if (upper) x = rcv; else y = rcv;
+  };
+  swap(v[0], v[1], 1, lane & 1);
+  swap(v[2], v[3], 1, lane & 1);
+  swap(v[0], v[2], 2, lane & 2);
+  swap(v[1], v[3], 2, lane & 2);
+}
+
 struct MtParams { MlstmArgs a; int* error_word; };
 
 __global__ void __launch_bounds__(MT_THREADS, 1)
@@ -337,11 +352,6 @@ mlstm_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         fence_async();
         if (!csync(924)) { ok = false; break; }
       }
-      if (r < n) {                                 // the output gate is read at the end of the chunk
-        const T* gp = reinterpret_cast<const T*>(a.g) + (sq.row0 + (int64_t)c * 128 + r) * a.row_stride + (int64_t)h * a.vdim + c0 + cq * 32;
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(gp));
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(gp + 16));
-      }
       // n . q over this thread's 32 key dims
       if (!mbar_wait(&sh.full[slot(tq)], phase(tq), abortp, err, 925)) { ok = false; break; }
       float nq = 0.f;
@@ -465,6 +475,13 @@ mlstm_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
       for (int i = 0; i < 32; ++i) { o[i] *= den; ss = fmaf(o[i], o[i], ss); }
       sh.ssq[cq][r] = ss;
+      // the output gate, four lanes per row (lane t of a group: chunk t of the group's rows)
+      int4 gt[4];
+      const int lrow = q * 32 + (lane & ~3);
+      const int64_t lrow0 = sq.row0 + (int64_t)c * 128 + lrow, lcol = (int64_t)h * a.vdim + c0 + cq * 32 + (lane & 3) * 8;
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        gt[i] = lrow + i < n ? ld16(reinterpret_cast<const T*>(a.g) + (lrow0 + i) * a.row_stride + lcol) : make_int4(0, 0, 0, 0);
       if (!csync(932)) { ok = false; break; }
       ss = (sh.ssq[0][r] + sh.ssq[1][r]) + (sh.ssq[2][r] + sh.ssq[3][r]);
       if (tiles > 1) {
@@ -482,27 +499,26 @@ mlstm_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         ss = all;
       }
       const float rr = rsqrtf(ss / (float)a.vdim + a.eps);
-      if (r < n) {
-        const int64_t row = sq.row0 + c * 128 + r, e = (int64_t)h * a.vdim + c0 + cq * 32;
-        const T* gp = reinterpret_cast<const T*>(a.g) + row * a.row_stride + e;
-        T* op = reinterpret_cast<T*>(a.out) + row * a.out_stride + e;
+      mt_transpose4(gt, lane);                     // to this thread's own row
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int4 g = ld16(gp + 8 * i);
-          const int gg[4] = {g.x, g.y, g.z, g.w};
-          uint32_t w[4];
+      for (int i = 0; i < 4; ++i) {
+        const int gg[4] = {gt[i].x, gt[i].y, gt[i].z, gt[i].w};
+        uint32_t w[4];
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const float2 gv = mt_pair((uint32_t)gg[j]);
-            const float2 nw = *reinterpret_cast<const float2*>(&sh.norm[cq * 32 + 8 * i + 2 * j]);
-            const float x = o[8 * i + 2 * j] * rr * nw.x * mt_rcp(1.f + mt_ex2(-MT_LOG2E * gv.x));
-            const float z = o[8 * i + 2 * j + 1] * rr * nw.y * mt_rcp(1.f + mt_ex2(-MT_LOG2E * gv.y));
-            const __nv_bfloat162 pr = __floats2bfloat162_rn(x, z);
-            w[j] = *reinterpret_cast<const uint32_t*>(&pr);
-          }
-          st16(op + 8 * i, make_int4((int)w[0], (int)w[1], (int)w[2], (int)w[3]));
+        for (int j = 0; j < 4; ++j) {
+          const float2 gv = mt_pair((uint32_t)gg[j]);
+          const float2 nw = *reinterpret_cast<const float2*>(&sh.norm[cq * 32 + 8 * i + 2 * j]);
+          const float x = o[8 * i + 2 * j] * rr * nw.x * mt_rcp(1.f + mt_ex2(-MT_LOG2E * gv.x));
+          const float z = o[8 * i + 2 * j + 1] * rr * nw.y * mt_rcp(1.f + mt_ex2(-MT_LOG2E * gv.y));
+          const __nv_bfloat162 pr = __floats2bfloat162_rn(x, z);
+          w[j] = *reinterpret_cast<const uint32_t*>(&pr);
         }
+        gt[i] = make_int4((int)w[0], (int)w[1], (int)w[2], (int)w[3]);
       }
+      mt_transpose4(gt, lane);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (lrow + i < n) st16(reinterpret_cast<T*>(a.out) + (lrow0 + i) * a.out_stride + lcol, gt[i]);
     }
     if (ok) {
 #pragma unroll
