@@ -47,6 +47,10 @@ extern "C" {
 #define ZP_IMPL_SIMT 1
 #define ZP_IMPL_TCGEN05 2
 
+/* activations applied by a product's epilogue */
+#define ZP_ACT_NONE 0
+#define ZP_ACT_RELU_SQUARED 1
+
 const char* zp_last_error(void);
 int zp_version(void);
 
@@ -458,6 +462,65 @@ int zp_mlstm(const void* q, const void* k, const void* v, const void* g, const f
              void* out, int B, int H, int dim, int vdim, int VP, int n_slots, int64_t row_stride,
              int64_t gates_stride, int64_t out_stride, float qscale, float gate_cap, float eps, int total_rows,
              int impl, int dtype, void* stream);
+
+/* ---- Latent attention, mixtures of experts, layers with parallel sublayers --------------------------
+ * No counterpart in the reference.  The Dobedra decoder runs on these; each takes its constants as parameters. */
+
+/* The boundary between two layers, per fp32 row of x [n_rows, hidden], in place:
+ *   x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k weights[k] * y[pos[k]])
+ *   out1 = T(layer norm of x * w1 + bias1), out2 likewise  (variance = mean of the squared deviations)
+ * a, b [n_rows, hidden] of T, ls_* [hidden] fp32 (NULL = ones), gate: one fp32 number per row at stride
+ * gate_stride (NULL = 1); y [y_rows, hidden] of T with pos, weights [n_rows, top] (top 0: none, at most 64).
+ * a, b, out1 and out2 may be NULL; with no summand x is only read. */
+int zp_join_norms(float* x, const void* a, const float* ls_a, const void* b, const float* ls_b, const float* gate,
+                  int64_t gate_stride, const void* y, int64_t y_rows, const int32_t* pos, const float* weights,
+                  int top, const float* w1, const float* bias1, void* out1, const float* w2, const float* bias2,
+                  void* out2, int n_rows, int hidden, float eps, int dtype, void* stream);
+
+/* gate | up [n_rows, 2 width] -> T(gelu_tanh(gate) * up) [n_rows, width] */
+int zp_gelu_tanh_and_mul(const void* x, void* out, int n_rows, int width, int dtype, void* stream);
+/* out = T(max(x, 0)^2), n elements; out may be x */
+int zp_relu_squared(const void* x, void* out, int64_t n, int dtype, void* stream);
+/* z = cap tanh(z / cap), n fp32 elements in place */
+int zp_soft_cap(float* z, int64_t n, float cap, void* stream);
+
+/* Down projections y [n_tokens, q_rank + kv_rank + rot] (row stride) of latent attention:
+ *   cq [n_tokens, q_rank] = RMS norm of the first part with q_weight,
+ *   cache row slot_mapping[i] of [n_slots, KP] (and row i of dense [n_tokens, KP], may be NULL) =
+ *     [RMS norm of the second part with kv_weight | the third part rotated | padding]
+ * Rotation: the pair (2t, 2t + 1) turns by 2 pi positions[i] turns[t], turns [rot / 2] fp64 on the device.
+ * kv_rank 0: only cq.  The cache's padding columns are left alone (dense's become zero); slots outside
+ * [0, n_slots) store nothing. */
+int zp_latent_prepare(const void* y, int64_t row_stride, const int64_t* positions, const double* turns,
+                      const float* q_weight, const float* kv_weight, void* cq, void* cache, void* dense,
+                      const int32_t* slot_mapping, int n_tokens, int q_rank, int kv_rank, int rot, int KP,
+                      int64_t n_slots, float eps, int dtype, void* stream);
+
+/* The last rot entries of every head of q [n_tokens, H, dim + rot] (row stride) rotated as above: in place
+ * (q_lat NULL), or into q_lat [n_tokens, H, KP] at kv_rank, with q_lat's padding set to zero and its first
+ * kv_rank entries left to the caller. */
+int zp_latent_rotate_q(void* q, int64_t row_stride, const int64_t* positions, const double* turns, void* q_lat,
+                       int n_tokens, int H, int dim, int rot, int kv_rank, int KP, int dtype, void* stream);
+
+/* dense row cu_seqlens_k[b] + j = cache row of position j of sequence b, for all total =
+ * cu_seqlens_k[B] rows.  cache [n_pages, BS, row_bytes], row_bytes a multiple of 16. */
+int zp_gather_rows(const void* cache, const int32_t* block_table, const int32_t* cu_seqlens_k, void* dense, int B,
+                   int NBmax, int BS, int n_pages, int row_bytes, int total, void* stream);
+
+/* Routing: logits [n_tokens, n_experts] fp32 (row stride, at most 1024 experts), s = softmax over all
+ * experts; the top largest of a token (ties: the lower expert) with weights s, not renormalised.
+ * weights, experts, places [n_tokens, top]; the n_tokens * top pairs sorted by expert: expert e has the places
+ * offsets[e] .. offsets[e + 1] ([n_experts + 1]), rows[place] = its token.  counts [n_experts]: scratch. */
+int zp_moe_route(const float* logits, int64_t row_stride, int n_tokens, int n_experts, int top, float* weights,
+                 int32_t* experts, int32_t* places, int32_t* rows, int32_t* offsets, int32_t* counts, void* stream);
+
+/* out[p, n] = act(sum_k x[r(p), k] weight[e, n, k]) for the places p of every expert e (offsets as above, at
+ * most n_places in all); r(p) = rows[p], or p when rows is NULL.  x [src_rows, k] (row stride), weight
+ * [n_experts, n_out, k], out [n_places, n_out]; fp32 accumulation.  bf16 with k and x_stride multiples of 8
+ * takes the tcgen05 kernel (ZP_IMPL_SIMT: never; ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED). */
+int zp_grouped_gemm(const void* x, int64_t x_stride, const int32_t* rows, int src_rows, const void* weight,
+                    const int32_t* offsets, void* out, int n_places, int n_experts, int n_out, int k, int act,
+                    int impl, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

@@ -32,6 +32,8 @@ FLAGS = [
 PARTS = {
     "similorn": ("zp_api", "zp_host_sched", "zp_mlstm", "zp_mlstm_chunk", "zp_mlstm_tc", "zp_rows", "zp_step", "zp_tc",
                  "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
+    "dobedra": ("zp_api", "zp_host_sched", "zp_latent", "zp_moe", "zp_moe_tc", "zp_rows", "zp_step", "zp_tc",
+                "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
 }
 
 

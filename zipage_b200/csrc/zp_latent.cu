@@ -1,0 +1,174 @@
+// Row kernels of latent attention (keys and values of all heads are products of one small cached latent):
+//   * from a token's down projections: the query latent RMS-normed, the key/value latent RMS-normed, the
+//     shared key part rotated, both written to the token's cache row (and to a dense row),
+//   * rotation of the queries' rotated part, in place or into the rows that meet the latents directly,
+//   * the dense copy of sequences' cached rows.
+// Norms, angles and rotations are fp32; angles come from fp64 turns per position, reduced to a fraction of
+// a turn before the conversion.
+#include "zp_common.cuh"
+
+namespace zp {
+
+constexpr int LP_THREADS = 128;
+
+// cos and sin of position * turns (in turns)
+__device__ __forceinline__ void turn_cs(int64_t pos, double turns, float& c, float& s) {
+  const double t = (double)pos * turns;
+  sincospif(2.f * (float)(t - rint(t)), &s, &c);
+}
+
+// v (n entries) -> T(v * rsqrt(mean(v^2) + eps) * w) at each of dst0 / dst1 (may be NULL)
+template <typename T>
+__device__ __forceinline__ void rms_part(const T* __restrict__ v, int n, const float* __restrict__ w, float eps, T* dst0, T* dst1,
+                                         float* red, bool vec) {
+  constexpr int EPV = 16 / sizeof(T);
+  float ss = 0.f;
+  if (vec) {
+    for (int c = threadIdx.x * EPV; c < n; c += LP_THREADS * EPV) {
+      const int4 raw = ld16(v + c);
+      const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+      for (int j = 0; j < EPV; ++j) { const float f = Elem<T>::to_f32(e[j]); ss = fmaf(f, f, ss); }
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += LP_THREADS) { const float f = Elem<T>::to_f32(v[c]); ss = fmaf(f, f, ss); }
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+  if (vec) {
+    for (int c = threadIdx.x * EPV; c < n; c += LP_THREADS * EPV) {
+      const int4 raw = ld16(v + c);
+      const T* e = reinterpret_cast<const T*>(&raw);
+      int4 o;
+      T* oe = reinterpret_cast<T*>(&o);
+#pragma unroll
+      for (int j = 0; j < EPV; ++j) oe[j] = Elem<T>::from_f32(Elem<T>::to_f32(e[j]) * r * w[c + j]);
+      if (dst0) st16(dst0 + c, o);
+      if (dst1) st16(dst1 + c, o);
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += LP_THREADS) {
+      const T o = Elem<T>::from_f32(Elem<T>::to_f32(v[c]) * r * w[c]);
+      if (dst0) dst0[c] = o;
+      if (dst1) dst1[c] = o;
+    }
+  }
+}
+
+// One block per token: y [q_rank | kv_rank | rot] -> cq, cache row [kv_rank | rot | padding] and dense row.
+template <typename T>
+__global__ void __launch_bounds__(LP_THREADS)
+latent_prepare_kernel(const T* __restrict__ y, int64_t ld, const int64_t* __restrict__ positions,
+                      const double* __restrict__ turns, const float* __restrict__ wq, const float* __restrict__ wkv,
+                      T* __restrict__ cq, T* __restrict__ cache, T* __restrict__ dense, const int32_t* __restrict__ slot_mapping,
+                      int q_rank, int kv_rank, int rot, int KP, int64_t n_slots, float eps, int vec_q, int vec_kv) {
+  __shared__ float red[32];
+  const int64_t i = blockIdx.x;
+  const T* row = y + i * ld;
+  rms_part<T>(row, q_rank, wq, eps, cq + i * q_rank, (T*)nullptr, red, vec_q);
+  if (kv_rank == 0) return;
+  row += q_rank;
+  const int64_t slot = slot_mapping[i];
+  T* c0 = slot >= 0 && slot < n_slots ? cache + slot * KP : nullptr;
+  T* c1 = dense ? dense + i * KP : nullptr;
+  rms_part<T>(row, kv_rank, wkv, eps, c0, c1, red, vec_kv);
+  const int64_t pos = positions[i];
+  for (int t = threadIdx.x; 2 * t < rot; t += LP_THREADS) {
+    float c, s;
+    turn_cs(pos, turns[t], c, s);
+    const float u = Elem<T>::to_f32(row[kv_rank + 2 * t]), v = Elem<T>::to_f32(row[kv_rank + 2 * t + 1]);
+    const T a = Elem<T>::from_f32(u * c - v * s), b = Elem<T>::from_f32(v * c + u * s);
+    if (c0) { c0[kv_rank + 2 * t] = a; c0[kv_rank + 2 * t + 1] = b; }
+    if (c1) { c1[kv_rank + 2 * t] = a; c1[kv_rank + 2 * t + 1] = b; }
+  }
+  if (c1)
+    for (int t = kv_rank + rot + threadIdx.x; t < KP; t += LP_THREADS) c1[t] = Elem<T>::from_f32(0.f);
+}
+
+// One block per token: the last `rot` entries of each head of q [H, dim + rot] turned; written in place, or
+// (q_lat given) to entries kv_rank .. kv_rank + rot of q_lat [H, KP], whose padding becomes zero.
+template <typename T>
+__global__ void __launch_bounds__(LP_THREADS)
+latent_rotate_q_kernel(T* __restrict__ q, int64_t ld, const int64_t* __restrict__ positions, const double* __restrict__ turns,
+                       T* __restrict__ q_lat, int H, int dim, int rot, int kv_rank, int KP) {
+  extern __shared__ float2 cs[];
+  const int64_t i = blockIdx.x, pos = positions[i];
+  const int half = rot / 2;
+  for (int t = threadIdx.x; t < half; t += LP_THREADS) turn_cs(pos, turns[t], cs[t].x, cs[t].y);
+  __syncthreads();
+  T* row = q + i * ld;
+  for (int k = threadIdx.x; k < H * half; k += LP_THREADS) {
+    const int h = k / half, t = k - h * half;
+    T* p = row + h * (dim + rot) + dim + 2 * t;
+    const float u = Elem<T>::to_f32(p[0]), v = Elem<T>::to_f32(p[1]);
+    T* o = q_lat ? q_lat + (i * H + h) * KP + kv_rank + 2 * t : p;
+    o[0] = Elem<T>::from_f32(u * cs[t].x - v * cs[t].y);
+    o[1] = Elem<T>::from_f32(v * cs[t].x + u * cs[t].y);
+  }
+  if (q_lat) {
+    const int pad = KP - kv_rank - rot;
+    for (int k = threadIdx.x; k < H * pad; k += LP_THREADS)
+      q_lat[(i * H + k / pad) * KP + kv_rank + rot + k % pad] = Elem<T>::from_f32(0.f);
+  }
+}
+
+// One warp per row of dense [total, KP]: key cu_k[b] + j <- position j of sequence b.
+__global__ void __launch_bounds__(256)
+gather_rows_kernel(const int4* __restrict__ cache, const int32_t* __restrict__ table, const int32_t* __restrict__ cu_k,
+                   int4* __restrict__ dense, int B, int NBmax, int BS, int n_pages, int vecs, int total) {
+  const int i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (i >= total) return;
+  int lo = 0, hi = B - 1;                 // last b with cu_k[b] <= i
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_k[mid] <= i) lo = mid; else hi = mid - 1;
+  }
+  const int j = i - cu_k[lo];
+  const int page = min(max(table[(int64_t)lo * NBmax + min(j / BS, NBmax - 1)], 0), n_pages - 1);
+  const int4* src = cache + ((int64_t)page * BS + j % BS) * vecs;
+  for (int c = lane; c < vecs; c += 32) dense[(int64_t)i * vecs + c] = src[c];
+}
+
+}  // namespace zp
+
+extern "C" int zp_latent_prepare(const void* y, int64_t row_stride, const int64_t* positions, const double* turns,
+                                 const float* q_weight, const float* kv_weight, void* cq, void* cache, void* dense,
+                                 const int32_t* slot_mapping, int n_tokens, int q_rank, int kv_rank, int rot, int KP,
+                                 int64_t n_slots, float eps, int dtype, void* stream) {
+  if (n_tokens == 0) return ZP_OK;
+  ZP_REQUIRE(y && q_weight && cq, "zp_latent_prepare: null pointer");
+  ZP_REQUIRE(q_rank > 0 && kv_rank >= 0 && rot >= 0 && rot % 2 == 0, "zp_latent_prepare: bad sizes");
+  ZP_REQUIRE(kv_rank == 0 || (positions && kv_weight && cache && slot_mapping && KP >= kv_rank + rot && (rot == 0 || turns)),
+             "zp_latent_prepare: a key/value latent without its cache, weight or positions");
+  const int epv = 16 / (int)zp::dtype_size(dtype);
+  const int vec_q = q_rank % epv == 0 && row_stride % epv == 0 && ((uintptr_t)y | (uintptr_t)cq) % 16 == 0;
+  const int vec_kv = vec_q && kv_rank % epv == 0 && KP % epv == 0 && ((uintptr_t)cache | (uintptr_t)dense) % 16 == 0;
+  ZP_DISPATCH_DTYPE(dtype, T, {
+    zp::latent_prepare_kernel<T><<<n_tokens, zp::LP_THREADS, 0, (cudaStream_t)stream>>>(
+        (const T*)y, row_stride, positions, turns, q_weight, kv_weight, (T*)cq, (T*)cache, (T*)dense, slot_mapping, q_rank, kv_rank,
+        rot, KP, n_slots, eps, vec_q, vec_kv);
+  });
+  return zp::check_launch("zp_latent_prepare");
+}
+
+extern "C" int zp_latent_rotate_q(void* q, int64_t row_stride, const int64_t* positions, const double* turns, void* q_lat,
+                                  int n_tokens, int H, int dim, int rot, int kv_rank, int KP, int dtype, void* stream) {
+  if (n_tokens == 0 || (rot == 0 && !q_lat)) return ZP_OK;
+  ZP_REQUIRE(q && positions && (turns || rot == 0), "zp_latent_rotate_q: null pointer");
+  ZP_REQUIRE(H > 0 && dim >= 0 && rot >= 0 && rot % 2 == 0 && rot <= 4096 && (!q_lat || KP >= kv_rank + rot), "zp_latent_rotate_q: bad sizes");
+  ZP_DISPATCH_DTYPE(dtype, T, {
+    zp::latent_rotate_q_kernel<T><<<n_tokens, zp::LP_THREADS, rot / 2 * sizeof(float2), (cudaStream_t)stream>>>(
+        (T*)q, row_stride, positions, turns, (T*)q_lat, H, dim, rot, kv_rank, KP);
+  });
+  return zp::check_launch("zp_latent_rotate_q");
+}
+
+extern "C" int zp_gather_rows(const void* cache, const int32_t* block_table, const int32_t* cu_seqlens_k, void* dense, int B,
+                              int NBmax, int BS, int n_pages, int row_bytes, int total, void* stream) {
+  if (total == 0 || B == 0) return ZP_OK;
+  ZP_REQUIRE(cache && block_table && cu_seqlens_k && dense, "zp_gather_rows: null pointer");
+  ZP_REQUIRE(NBmax > 0 && BS > 0 && n_pages > 0 && row_bytes > 0 && row_bytes % 16 == 0 && ((uintptr_t)cache | (uintptr_t)dense) % 16 == 0,
+             "zp_gather_rows: rows must be whole 16-byte pieces");
+  zp::gather_rows_kernel<<<(total + 7) / 8, 256, 0, (cudaStream_t)stream>>>(
+      (const int4*)cache, block_table, cu_seqlens_k, (int4*)dense, B, NBmax, BS, n_pages, row_bytes / 16, total);
+  return zp::check_launch("zp_gather_rows");
+}

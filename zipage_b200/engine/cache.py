@@ -1,5 +1,5 @@
-"""Device memory of models that describe what each layer keeps: paged keys and values, and recurrent
-state in slots.  Pages and slots are handed out by the native scheduler (block tables, query_id);
+"""Device memory of models that describe what each layer keeps: paged keys and values or latents, and
+recurrent state in slots.  Pages and slots are handed out by the native scheduler (block tables, query_id);
 this only owns the storage.
 
 A page id or slot means the same row range in every entry, so one block table and one slot number per
@@ -26,6 +26,24 @@ class KVSpec:
 
     def bytes(self, pages, block_size, slots, itemsize):
         return pages * block_size * self.kv_heads * ((self.dim + 15) // 16 + (self.vdim + 15) // 16) * 16 * itemsize
+
+
+@dataclass(frozen=True)
+class LatentSpec:
+    """One row per token for all heads of a latent-attention layer: the latent and the rotated key part, padded
+    to a multiple of 16 elements (the padding stays zero)."""
+    rank: int
+    rot: int
+
+    @property
+    def row(self):
+        return (self.rank + self.rot + 15) // 16 * 16
+
+    def allocate(self, pages, block_size, slots, dtype, device):
+        return (torch.zeros((pages, block_size, 1, self.row), dtype=dtype, device=device),)
+
+    def bytes(self, pages, block_size, slots, itemsize):
+        return pages * block_size * self.row * itemsize
 
 
 @dataclass(frozen=True)

@@ -24,7 +24,7 @@ import numpy as np
 import torch
 
 from .. import _lib as L
-from ..layers.row_ops import project
+from ..layers.row_ops import project, soft_cap_
 from ..layers.step_ops import sample
 from ..utils.context import reset_context, set_context
 from .compressor import Compressor
@@ -196,9 +196,11 @@ class NativeEngine:
 
     # -- portion steps ----------------------------------------------------------------------------
     def logits(self, hidden):
-        """LM head on rows of hidden states; fp32 where the model asks for it."""
+        """LM head on rows of hidden states; fp32, and soft-capped, where the model asks for it."""
         if getattr(self.model, "fp32_logits", False):
-            return project(hidden, self.lm_head, fp32=True)
+            z = project(hidden, self.lm_head, fp32=True)
+            cap = getattr(self.model, "logit_softcap", 0.0)
+            return soft_cap_(z, cap) if cap else z
         return torch.nn.functional.linear(hidden, self.lm_head)
 
     @torch.inference_mode()

@@ -1,0 +1,114 @@
+"""Feed-forward blocks whose result joins the residual stream at the layer boundary (`row_ops.join_norms`):
+a gated dense block and a mixture of experts, on libzipage_b200 kernels and the library's matrix product.
+
+Each block returns the keyword arguments that `join_norms` takes for its result, so that the experts'
+weighting, the shared expert's gate and the sum are part of that launch.
+"""
+from __future__ import annotations
+
+import torch
+from torch import nn
+
+from .. import _lib as L
+from ..kernel import _count
+from .row_ops import project
+
+
+def gelu_tanh_and_mul(x):
+    """gate | up [N, 2 F] -> gelu_tanh(gate) * up [N, F]."""
+    L.require_cuda(x)
+    assert x.is_contiguous()
+    N, F = x.shape[0], x.shape[1] // 2
+    out = torch.empty((N, F), dtype=x.dtype, device=x.device)
+    L.check(L.load().zp_gelu_tanh_and_mul(L.ptr(x), L.ptr(out), N, F, L.dtype_code(x), L.stream_ptr()), "gelu_tanh_and_mul")
+    _count(1)
+    return out
+
+
+def relu_squared_(x):
+    L.require_cuda(x)
+    assert x.is_contiguous()
+    L.check(L.load().zp_relu_squared(L.ptr(x), L.ptr(x), x.numel(), L.dtype_code(x), L.stream_ptr()), "relu_squared")
+    _count(1)
+    return x
+
+
+def moe_route(logits, n_experts, top):
+    """logits [N, >= n_experts] fp32 -> (weights [N, top] fp32, experts [N, top], places [N, top],
+    rows [N * top], offsets [n_experts + 1]): softmax over all experts, the `top` largest of a token, and
+    the (token, expert) pairs sorted by expert."""
+    L.require_cuda(logits)
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    N, dev = logits.shape[0], logits.device
+    w = torch.empty((N, top), dtype=torch.float32, device=dev)
+    ints = torch.empty(3 * N * top + 2 * n_experts + 1, dtype=torch.int32, device=dev)
+    experts, places, rows, offsets, counts = ints.split([N * top] * 3 + [n_experts + 1, n_experts])
+    L.check(L.load().zp_moe_route(L.ptr(logits), logits.stride(0), N, n_experts, top, L.ptr(w), L.ptr(experts), L.ptr(places),
+                                  L.ptr(rows), L.ptr(offsets), L.ptr(counts), L.stream_ptr()), "moe_route")
+    _count(1 if N <= 512 else 2)
+    return w, experts.view(N, top), places.view(N, top), rows, offsets
+
+
+def grouped_gemm(x, weight, offsets, n_places, rows=None, act=None, impl="auto"):
+    """out[p] = act(x[rows[p]] @ weight[e].T) for the places p of every expert e; x [src, K] (rows None:
+    place p is row p), weight [E, n_out, K]."""
+    L.require_cuda(x, weight, offsets, rows)
+    E, n_out, K = weight.shape
+    assert x.stride(1) == 1 and weight.is_contiguous() and x.dtype == weight.dtype and x.shape[1] == K
+    out = torch.empty((n_places, n_out), dtype=x.dtype, device=x.device)
+    L.check(L.load().zp_grouped_gemm(L.ptr(x), x.stride(0), L.ptr(rows), x.shape[0], L.ptr(weight), L.ptr(offsets), L.ptr(out),
+                                     n_places, E, n_out, K, L.ACT[act], L.IMPL[impl], L.dtype_code(x), L.stream_ptr()),
+            "grouped_gemm")
+    _count(1)
+    return out
+
+
+class GatedFF(nn.Module):
+    """W_down (gelu_tanh(W_gate h) * (W_up h))."""
+
+    def __init__(self, width, ff, dtype, device):
+        super().__init__()
+        e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
+        self.gate_up, self.down = e(2 * ff, width), e(width, ff)
+
+    def load(self, get):
+        self.gate_up.copy_(torch.cat([get("gate"), get("up")], 0))
+        self.down.copy_(get("down"))
+
+    def forward(self, h):
+        return {"b": project(gelu_tanh_and_mul(project(h, self.gate_up)), self.down)}
+
+
+class MixtureFF(nn.Module):
+    """`top` of `experts` squared-ReLU blocks per token, weighted by their softmax scores, and (shared_ff > 0)
+    a shared block scaled by a sigmoid gate.  The gate's row is the router product's last row."""
+
+    def __init__(self, width, experts, top, ff, shared_ff, dtype, device):
+        super().__init__()
+        self.experts, self.top, self.shared = experts, top, shared_ff > 0
+        e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
+        self.router = e(experts + int(self.shared), width)
+        self.up, self.down = e(experts, ff, width), e(experts, width, ff)
+        if self.shared:
+            self.shared_up, self.shared_down = e(shared_ff, width), e(width, shared_ff)
+
+    def load(self, get):
+        for i in range(self.experts):
+            self.up[i].copy_(get(f"e{i}.up"))
+            self.down[i].copy_(get(f"e{i}.down"))
+        self.router[:self.experts].copy_(get("router"))
+        if self.shared:
+            self.router[self.experts:].copy_(get("shared.sg"))
+            self.shared_up.copy_(get("shared.up"))
+            self.shared_down.copy_(get("shared.down"))
+
+    def forward(self, h):
+        N = h.shape[0]
+        z = project(h, self.router, fp32=True)
+        w, _, places, rows, offsets = moe_route(z, self.experts, self.top)
+        mid = grouped_gemm(h, self.up, offsets, N * self.top, rows=rows, act="relu_squared")
+        out = {"y": grouped_gemm(mid, self.down, offsets, N * self.top), "pos": places, "weights": w}
+        if self.shared:
+            out["b"] = project(relu_squared_(project(h, self.shared_up)), self.shared_down)
+            out["gate"] = z[:, self.experts]
+        return out

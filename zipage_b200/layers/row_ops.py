@@ -1,6 +1,6 @@
 """Row ops of decoders whose residual stream stays in fp32 between 16-bit matrix products.
 
-`embed_position`, `rms_norm_f32` and `gelu_tanh` are single launches of libzipage_b200 kernels;
+`embed_position`, `rms_norm_f32`, `join_norms`, `soft_cap_` and `gelu_tanh` are single launches of libzipage_b200 kernels;
 `project` and `project_add` are the library's matrix product with fp32 accumulation and, where the
 result joins the fp32 stream, an fp32 result (the residual add is the product's epilogue).
 """
@@ -43,6 +43,33 @@ def rms_norm_f32(x, weight, eps, dtype, offset=0.0):
                                      float(eps), L.dtype_code(out), L.stream_ptr()), "rms_norm_f32")
     _count(1)
     return out
+
+
+def join_norms(x, norms, eps, dtype, a=None, ls_a=None, b=None, ls_b=None, gate=None, y=None, pos=None, weights=None):
+    """The boundary between layers with parallel sublayers.  x fp32 [N, width], in place:
+    x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k weights[:, k] * y[pos[:, k]]); then one layer norm of x per
+    (weight, bias) of `norms` (at most two), each as `dtype`."""
+    L.require_cuda(x, a, ls_a, b, ls_b, gate, y, pos, weights, *(t for n in norms for t in n))
+    assert x.dtype == torch.float32 and x.is_contiguous() and len(norms) <= 2
+    assert all(t is None or t.dtype == dtype and t.is_contiguous() for t in (a, b, y))
+    outs = [torch.empty(x.shape, dtype=dtype, device=x.device) for _ in norms]
+    flat = [p for n, o in zip(norms, outs) for p in (L.ptr(n[0]), L.ptr(n[1]), L.ptr(o))]
+    flat += [None] * (6 - len(flat))
+    L.check(L.load().zp_join_norms(
+        L.ptr(x), L.ptr(a), L.ptr(ls_a), L.ptr(b), L.ptr(ls_b), L.ptr(gate), 0 if gate is None else gate.stride(0), L.ptr(y),
+        0 if y is None else y.shape[0], L.ptr(pos), L.ptr(weights), 0 if y is None else pos.shape[1], *flat, x.shape[0],
+        x.shape[1], float(eps), L.ZP_DTYPE[dtype], L.stream_ptr()), "join_norms")
+    _count(1)
+    return outs
+
+
+def soft_cap_(z, cap):
+    """z = cap tanh(z / cap), fp32, in place."""
+    L.require_cuda(z)
+    assert z.dtype == torch.float32 and z.is_contiguous()
+    L.check(L.load().zp_soft_cap(L.ptr(z), z.numel(), float(cap), L.stream_ptr()), "soft_cap")
+    _count(1)
+    return z
 
 
 def gelu_tanh(x):

@@ -74,6 +74,15 @@ def _similorn(config, weights, dtype, device):
     return LoadedModel("Similorn", model, model.head, cfg.width, cfg.vocab, dtype, portions=True)
 
 
+@register("Dobedra", part="dobedra")
+def _dobedra(config, weights, dtype, device):
+    from .dobedra import DobedraConfig, DobedraModel
+    cfg = DobedraConfig.from_dict(config)
+    model = DobedraModel(cfg, dtype, device)
+    model.load_weights(weights)
+    return LoadedModel("Dobedra", model, model.head, cfg.width, cfg.vocab, dtype, portions=True)
+
+
 @register("Qwen3ForCausalLM")
 def _qwen3(config, weights, dtype, device):
     from ..engine.native_engine import full_state_from_hf
