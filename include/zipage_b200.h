@@ -502,6 +502,29 @@ int zp_latent_prepare(const void* y, int64_t row_stride, const int64_t* position
 int zp_latent_rotate_q(void* q, int64_t row_stride, const int64_t* positions, const double* turns, void* q_lat,
                        int n_tokens, int H, int dim, int rot, int kv_rank, int KP, int dtype, void* stream);
 
+/* Softmax attention of queries that meet cached latents directly: score = q . cache row * scale (KP entries, both
+ * paddings zero), value = the row's first R entries, the query at position p sees every key j <= p.
+ * q [rows, H, KP], cache [n_pages, BS, KP], out [rows, H, R] contiguous; rows, positions and contexts as in
+ * zp_window_attention (total_rows: rows of q).  KP a multiple of 16, R <= 512.  bf16 with KP <= 640 takes the tcgen05
+ * kernel (ZP_IMPL_SIMT: never; ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED), which may need a workspace
+ * (span = NBmax * BS, max_seqlen_q = 1 without cu_seqlens_q).  Scores and softmax weights are fp32. */
+size_t zp_latent_attention_workspace_bytes(int total_rows, int B, int max_seqlen_q, int H, int R, int span);
+int zp_latent_attention(const void* q, const void* cache, const int32_t* cu_seqlens_q, const int32_t* context_lens,
+                        const int32_t* block_table, void* out, int B, int max_seqlen_q, int total_rows, int NBmax, int H,
+                        int R, int KP, int BS, int n_pages, float scale, int impl, int dtype, void* workspace,
+                        size_t workspace_bytes, void* stream);
+
+/* Causal softmax attention of prompt portions over expanded keys and values (tcgen05, bf16): score = (q[:dim] .
+ * key + q[dim:] . latent[kv_rank : kv_rank + rot]) * scale.  q [total_q, H, dim + rot] (row stride), kv [total_k,
+ * H * dim keys | H * vdim values] contiguous, latent [total_k, KP] contiguous, out [total_q, H, vdim] (row stride).
+ * Sequence b has the rows cu_seqlens_q[b] .. and the keys cu_seqlens_k[b] ..; its rows are its newest tokens.
+ * Sizes: zp_latent_prefill_supported (1 = yes): multiples of 8, vdim <= 128, at most four 64-entry key blocks. */
+int zp_latent_prefill_supported(int dim, int rot, int vdim, int kv_rank, int KP, int dtype);
+int zp_latent_prefill(const void* q, int64_t q_stride, const void* kv, const void* latent, const int32_t* cu_seqlens_q,
+                      const int32_t* cu_seqlens_k, void* out, int64_t out_stride, int B, int max_seqlen_q, int total_q,
+                      int total_k, int H, int dim, int rot, int vdim, int kv_rank, int KP, float scale, int dtype,
+                      void* stream);
+
 /* dense row cu_seqlens_k[b] + j = cache row of position j of sequence b, for all total =
  * cu_seqlens_k[B] rows.  cache [n_pages, BS, row_bytes], row_bytes a multiple of 16. */
 int zp_gather_rows(const void* cache, const int32_t* block_table, const int32_t* cu_seqlens_k, void* dense, int B,

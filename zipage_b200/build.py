@@ -32,7 +32,7 @@ FLAGS = [
 PARTS = {
     "similorn": ("zp_api", "zp_host_sched", "zp_mlstm", "zp_mlstm_chunk", "zp_mlstm_tc", "zp_rows", "zp_step", "zp_tc",
                  "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
-    "dobedra": ("zp_api", "zp_host_sched", "zp_latent", "zp_moe", "zp_moe_tc", "zp_rows", "zp_step", "zp_tc",
+    "dobedra": ("zp_api", "zp_host_sched", "zp_latent", "zp_latent_decode_tc", "zp_latent_prefill_tc", "zp_moe", "zp_moe_tc", "zp_rows", "zp_step", "zp_tc",
                 "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
 }
 

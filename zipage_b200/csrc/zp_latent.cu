@@ -5,7 +5,7 @@
 //   * the dense copy of sequences' cached rows.
 // Norms, angles and rotations are fp32; angles come from fp64 turns per position, reduced to a fraction of
 // a turn before the conversion.
-#include "zp_common.cuh"
+#include "zp_latent.cuh"
 
 namespace zp {
 
@@ -171,4 +171,43 @@ extern "C" int zp_gather_rows(const void* cache, const int32_t* block_table, con
   zp::gather_rows_kernel<<<(total + 7) / 8, 256, 0, (cudaStream_t)stream>>>(
       (const int4*)cache, block_table, cu_seqlens_k, (int4*)dense, B, NBmax, BS, n_pages, row_bytes / 16, total);
   return zp::check_launch("zp_gather_rows");
+}
+
+extern "C" size_t zp_latent_attention_workspace_bytes(int total_rows, int B, int max_seqlen_q, int H, int R, int span) {
+  if (total_rows < 1 || B < 1 || max_seqlen_q < 1 || H < 1) return 0;
+  const int ns = zp::latent_decode_splits(B, max_seqlen_q, H, span);
+  return ns > 1 ? (size_t)total_rows * H * ns * (R + 2) * sizeof(float) : 0;
+}
+
+extern "C" int zp_latent_attention(const void* q, const void* cache, const int32_t* cu_seqlens_q, const int32_t* context_lens,
+                                   const int32_t* block_table, void* out, int B, int max_seqlen_q, int total_rows, int NBmax, int H,
+                                   int R, int KP, int BS, int n_pages, float scale, int impl, int dtype, void* workspace,
+                                   size_t workspace_bytes, void* stream) {
+  if (B == 0 || (cu_seqlens_q && max_seqlen_q == 0)) return ZP_OK;
+  ZP_REQUIRE(q && cache && context_lens && block_table && out, "zp_latent_attention: null pointer");
+  ZP_REQUIRE(H > 0 && R > 0 && R <= 512 && R <= KP && KP % 16 == 0 && KP <= 2048, "zp_latent_attention: %d of %d entries", R, KP);
+  ZP_REQUIRE(BS > 0 && BS % 64 == 0 && NBmax > 0 && n_pages > 0 && B <= 65535 && total_rows > 0, "zp_latent_attention: bad sizes");
+  const int max_q = cu_seqlens_q ? max_seqlen_q : 1;
+  zp::LatentArgs a;
+  a.q = q; a.cache = cache; a.cu_q = cu_seqlens_q; a.context_lens = context_lens; a.table = block_table; a.out = out;
+  a.part = nullptr; a.B = B; a.NBmax = NBmax; a.H = H; a.R = R; a.KP = KP; a.BS = BS; a.n_pages = n_pages;
+  a.pairs = (int64_t)total_rows * H; a.scale = scale;
+  const bool tc = zp::latent_decode_tc_supports(a, dtype) && (int64_t)max_q * H <= 65535 * 16ll;
+  if (impl == ZP_IMPL_TCGEN05 && !tc) {
+    zp::set_error("zp_latent_attention: the tcgen05 kernel needs bf16, rows of at most 640 entries and 16-byte aligned tensors");
+    return ZP_ERR_UNSUPPORTED;
+  }
+  if (tc && impl != ZP_IMPL_SIMT) {
+    a.nsplit = zp::latent_decode_splits(B, max_q, H, NBmax * BS);
+    if (a.nsplit > 1) {
+      const size_t need = (size_t)a.pairs * a.nsplit * (R + 2) * sizeof(float);
+      ZP_REQUIRE(workspace && workspace_bytes >= need, "zp_latent_attention: workspace of %zu bytes, %zu needed", workspace_bytes, need);
+      a.part = reinterpret_cast<float*>(workspace);
+    }
+    return zp::latent_decode_tc(a, max_q, total_rows, (cudaStream_t)stream);
+  }
+  // one shared key/value head whose values are the first R entries of its keys
+  return zp_window_attention(q, cache, cache, cu_seqlens_q, context_lens, block_table, out, B, max_seqlen_q, NBmax, H, 1, KP, R, KP,
+                             KP, BS, n_pages, (int64_t)H * KP, (int64_t)H * R, scale, 0.f, 0, total_rows, ZP_IMPL_SIMT, dtype,
+                             nullptr, 0, stream);
 }

@@ -43,6 +43,19 @@ int make_tensor_map_5d(CUtensorMap* out, CUtensorMapDataType dt, const void* bas
   return ZP_OK;
 }
 
+int make_tensor_map_rows(CUtensorMap* out, CUtensorMapDataType dt, const void* base, uint64_t cols, uint64_t rows,
+                         uint64_t row_stride_elems, size_t elem_size) {
+  EncodeTiledFn fn = encode_fn();
+  if (!fn) { set_error("cuTensorMapEncodeTiled is not available from this driver"); return ZP_ERR_CUDA; }
+  const cuuint64_t gdim[2] = {cols, rows}, gstr[1] = {row_stride_elems * elem_size};
+  const cuuint32_t bx[2] = {64, 1}, es[2] = {1, 1};
+  CUresult r = fn(out, dt, 2, const_cast<void*>(base), gdim, gstr, bx, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) { set_error("cuTensorMapEncodeTiled failed with code %d (%llu rows of %llu)", (int)r,
+                                     (unsigned long long)rows, (unsigned long long)cols); return ZP_ERR_CUDA; }
+  return ZP_OK;
+}
+
 int* device_error_word() {
   int* p = nullptr;
   if (cudaGetSymbolAddress(reinterpret_cast<void**>(&p), g_error_word) != cudaSuccess) return nullptr;

@@ -223,6 +223,10 @@ __device__ __forceinline__ void umma_k128(uint32_t d_tmem, uint32_t a_addr, uint
 int make_tensor_map_5d(CUtensorMap* out, CUtensorMapDataType dt, const void* base, const uint64_t dims[5],
                        const uint64_t strides_elems[4], const uint32_t box[5], size_t elem_size);
 
+// 2-D map over rows of `cols` elements for four-row gathers (box: one row of 64 elements), 128-byte swizzle.
+int make_tensor_map_rows(CUtensorMap* out, CUtensorMapDataType dt, const void* base, uint64_t cols, uint64_t rows,
+                         uint64_t row_stride_elems, size_t elem_size);
+
 // Device error word shared by the tensor-core kernels (0 = no error).
 int* device_error_word();
 
