@@ -92,7 +92,7 @@ SIGNATURES = {
     "zp_latent_prepare": (_I, [_P, _L] + [_P] * 8 + [_I] * 5 + [_L, _F, _I, _P]),
     "zp_latent_rotate_q": (_I, [_P, _L] + [_P] * 3 + [_I] * 7 + [_P]),
     "zp_latent_attention_workspace_bytes": (_Z, [_I] * 6),
-    "zp_latent_attention": (_I, [_P] * 6 + [_I] * 8 + [_F, _I, _I, _P, _Z, _P]),
+    "zp_latent_attention": (_I, [_P] * 6 + [_I] * 9 + [_F, _I, _I, _P, _Z, _P]),
     "zp_latent_prefill_supported": (_I, [_I] * 6),
     "zp_latent_prefill": (_I, [_P, _L] + [_P] * 5 + [_L] + [_I] * 10 + [_F, _I, _P]),
     "zp_gather_rows": (_I, [_P] * 4 + [_I] * 6 + [_P]),

@@ -213,18 +213,20 @@ class NativeEngine:
         order = np.argsort(counts != 1, kind="stable")      # single rows first
         p = self.scheduler.portion_inputs(np.ascontiguousarray(handles[order]), np.ascontiguousarray(counts[order]),
                                           self.width)
+        nd = int((counts == 1).sum())
+        cu_k = np.concatenate([[0], np.cumsum(p["context_lens"][nd:], dtype=np.int32)]).astype(np.int32)
         ints = np.concatenate([p[k].ravel() for k in ("input_ids", "positions", "slot_mapping", "cu_seqlens_q",
-                                                      "context_lens", "slots", "block_tables")])
+                                                      "context_lens", "slots", "block_tables")] + [cu_k])
         dev = torch.from_numpy(ints).to(self.device)        # one copy for the step's inputs
         t, at = len(p["input_ids"]), 0
         parts = []
-        for k in (t, t, t, n + 1, n, n, n * p["block_tables"].shape[1]):
+        for k in (t, t, t, n + 1, n, n, n * p["block_tables"].shape[1], n - nd + 1):
             parts.append(dev[at:at + k])
             at += k
-        ids, pos, slot_mapping, cu, ctx, slots, tables = parts
-        set_context(True, cu, None, int(counts.max()), 0, slot_mapping,
-                    context_lens=ctx, block_tables=tables.view(n, -1), num_decode=int((counts == 1).sum()),
-                    state_slots=slots)
+        ids, pos, slot_mapping, cu, ctx, slots, tables, cu_k_dev = parts
+        set_context(True, cu, cu_k_dev, int(counts.max()), 0, slot_mapping,
+                    context_lens=ctx, block_tables=tables.view(n, -1), num_decode=nd,
+                    state_slots=slots, total_k=int(cu_k[-1]))
         try:
             hidden = self.model(ids.long(), pos.long())
         finally:

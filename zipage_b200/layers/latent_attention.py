@@ -18,7 +18,7 @@ from torch import nn
 from .. import _lib as L
 from ..kernel import _count
 from ..utils.context import get_context
-from .attention import window_attention
+from .attention import _workspace
 from .row_ops import project
 
 
@@ -66,6 +66,45 @@ def gather_rows(cache, block_table, cu_seqlens_k, total):
     return out
 
 
+def latent_attention(q_lat, cache, context_lens, block_table, rank, scale, cu_seqlens_q=None, max_seqlen_q=1, out=None, impl="auto"):
+    """q_lat [rows, H, KP] over cached rows [P, BS, 1, KP] whose first `rank` entries are the values -> [rows, H, rank].
+    One row per sequence without `cu_seqlens_q`."""
+    L.require_cuda(q_lat, cache, context_lens, block_table, cu_seqlens_q)
+    N, H, KP = q_lat.shape
+    P, BS, _, row = cache.shape
+    B, NB = block_table.shape
+    assert q_lat.is_contiguous() and cache.is_contiguous() and row == KP and block_table.is_contiguous()
+    if out is None:
+        out = torch.empty((N, H, rank), dtype=q_lat.dtype, device=q_lat.device)
+    assert out.is_contiguous()
+    lib = L.load()
+    need = lib.zp_latent_attention_workspace_bytes(N, B, max_seqlen_q, H, rank, NB * BS)
+    ws = _workspace(q_lat.device, need) if need else None
+    L.check(lib.zp_latent_attention(
+        L.ptr(q_lat), L.ptr(cache), L.ptr(cu_seqlens_q), L.ptr(context_lens), L.ptr(block_table), L.ptr(out), B,
+        int(max_seqlen_q), N, NB, H, rank, KP, BS, P, float(scale), L.IMPL[impl], L.dtype_code(q_lat), L.ptr(ws),
+        0 if ws is None else ws.numel(), L.stream_ptr()), "latent_attention")
+    _count(1)
+    return out
+
+
+def latent_prefill(q, kv, latent, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, out, heads, dim, rot, vdim, rank, scale):
+    """Causal attention of q [rows, heads * (dim + rot)] over kv [keys, heads * (dim + vdim)] (keys of all heads, then
+    values) and the rotated parts in latent [keys, KP] at `rank`; writes out [rows, heads * vdim]."""
+    L.require_cuda(q, kv, latent, cu_seqlens_q, cu_seqlens_k, out)
+    assert q.stride(1) == out.stride(1) == 1 and kv.is_contiguous() and latent.is_contiguous()
+    L.check(L.load().zp_latent_prefill(
+        L.ptr(q), q.stride(0), L.ptr(kv), L.ptr(latent), L.ptr(cu_seqlens_q), L.ptr(cu_seqlens_k), L.ptr(out), out.stride(0),
+        cu_seqlens_q.numel() - 1, int(max_seqlen_q), q.shape[0], kv.shape[0], heads, dim, rot, vdim, rank, latent.shape[1],
+        float(scale), L.dtype_code(q), L.stream_ptr()), "latent_prefill")
+    _count(1)
+    return out
+
+
+# portions whose longest has at least this many tokens take the expanded form
+EXPAND_FROM = 64
+
+
 class LatentAttentionMixer(nn.Module):
     """h -> W_o of the head outputs [rows, width].  `shares`: the layer keeps nothing of its own and reads another
     layer's cache (`cache` is bound to that one's)."""
@@ -95,28 +134,50 @@ class LatentAttentionMixer(nn.Module):
 
     def forward(self, h, positions):
         ctx = get_context()
+        N, nd = h.shape[0], ctx.decode_rows()
+        expand = ctx.is_prefill and nd < ctx.context_lens.shape[0] and self._expands(h, ctx)
+        dense = None
+        if expand and not self.shares and ctx.total_k == N - nd:      # no earlier context: the step's own rows are the keys
+            dense = torch.empty((N, self.cache.shape[3]), dtype=h.dtype, device=h.device)
+            ctx.scratch[id(self.cache)] = dense[nd:]
         cq = latent_prepare(project(h, self.down), positions, self.turns, self.q_norm, self.kv_norm, self.cache,
-                            ctx.slot_mapping, self.q_rank, 0 if self.shares else self.kv_rank, self.rot, self.eps)
+                            ctx.slot_mapping, self.q_rank, 0 if self.shares else self.kv_rank, self.rot, self.eps, dense)
         q = project(cq, self.q_up)
-        out = torch.empty((h.shape[0], self.heads * self.vdim), dtype=h.dtype, device=h.device)
-        self._direct(q, positions, out, ctx)
+        out = torch.empty((N, self.heads * self.vdim), dtype=h.dtype, device=h.device)
+        if expand:
+            if nd:
+                self._direct(q[:nd], positions[:nd], out[:nd], ctx, nd, False)
+            self._expanded(q[nd:], positions[nd:], out[nd:], ctx, nd)
+        else:
+            self._direct(q, positions, out, ctx, nd, ctx.is_prefill and nd < ctx.context_lens.shape[0])
         return project(out, self.out_proj)
 
-    def _direct(self, q, positions, out, ctx):
+    def _expands(self, h, ctx):
+        return ctx.max_seqlen_q >= EXPAND_FROM and ctx.cu_seqlens_k is not None and L.load().zp_latent_prefill_supported(
+            self.dim, self.rot, self.vdim, self.kv_rank, self.cache.shape[3], L.dtype_code(h)) == 1
+
+    def _expanded(self, q, positions, out, ctx, nd):
+        latent = ctx.scratch.get(id(self.cache))        # (layers that share latents share their dense copy)
+        if latent is None:
+            latent = ctx.scratch[id(self.cache)] = gather_rows(self.cache, ctx.block_tables[nd:], ctx.cu_seqlens_k, ctx.total_k)
+        kv = project(latent[:, :self.kv_rank], self.kv_up)
+        latent_rotate_q(q, positions, self.turns, self.heads, self.dim, self.rot)
+        latent_prefill(q, kv, latent, ctx.cu_seqlens_q[nd:] - nd if nd else ctx.cu_seqlens_q, ctx.cu_seqlens_k, ctx.max_seqlen_q, out,
+                       self.heads, self.dim, self.rot, self.vdim, self.kv_rank, self.scale)
+
+    def _direct(self, q, positions, out, ctx, nd, portions):
+        """`nd` leading rows are sequences of one row each; with `portions`, the rest are portions."""
         H, R, N = self.heads, self.kv_rank, q.shape[0]
         q_lat = torch.empty((N, H, self.cache.shape[3]), dtype=q.dtype, device=q.device)
         latent_rotate_q(q, positions, self.turns, H, self.dim, self.rot, q_lat, R)
         nk = H * self.dim
         torch.bmm(q.view(N, H, -1)[:, :, :self.dim].transpose(0, 1), self.kv_up[:nk].view(H, self.dim, R),
                   out=q_lat.transpose(0, 1)[:, :, :R])
-        o_lat = torch.empty((N, H * R), dtype=q.dtype, device=q.device)
-        nd = ctx.decode_rows()
-        args = (H, q_lat.shape[2], R, self.scale)
-        ql = q_lat.view(N, -1)
+        o_lat = torch.empty((N, H, R), dtype=q.dtype, device=q.device)
         if nd:
-            window_attention(ql, self.cache, self.cache, ctx.context_lens[:nd], ctx.block_tables[:nd], *args, out=o_lat)
-        if ctx.is_prefill and nd < ctx.context_lens.shape[0]:
-            window_attention(ql, self.cache, self.cache, ctx.context_lens[nd:], ctx.block_tables[nd:], *args,
+            latent_attention(q_lat, self.cache, ctx.context_lens[:nd], ctx.block_tables[:nd], R, self.scale, out=o_lat)
+        if portions:
+            latent_attention(q_lat, self.cache, ctx.context_lens[nd:], ctx.block_tables[nd:], R, self.scale,
                              cu_seqlens_q=ctx.cu_seqlens_q[nd:], max_seqlen_q=ctx.max_seqlen_q, out=o_lat)
-        torch.bmm(o_lat.view(N, H, R).transpose(0, 1), self.kv_up[nk:].view(H, self.vdim, R).transpose(1, 2),
+        torch.bmm(o_lat.transpose(0, 1), self.kv_up[nk:].view(H, self.vdim, R).transpose(1, 2),
                   out=out.view(N, H, self.vdim).transpose(0, 1))
