@@ -51,7 +51,7 @@ def parse_args():
                     help="also run the reference ENGINE (baseline/_ref) on a synthetic Qwen3-8B-shaped model, as it "
                          "is and with this library's decode path bound, and report decode tokens/s (adds minutes)")
     ap.add_argument("--also-exact", action="store_true", help="time the exact variant as well")
-    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine", "similorn"],
+    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine", "similorn", "dobedra"],
                     help="compress (default, the headline op), decode (paged decode attention kernel) or "
                          "step_ops (the element-wise ops of a decoder layer step and the sampler) or "
                          "prefill (varlen causal prefill attention, one layer) or decode_step (the decode "
@@ -1051,6 +1051,84 @@ def run_native_engine(args):
         dist.destroy_process_group()
 
 
+class KernelTable:
+    """Timed kernels: share of each one's roofline (the slower of its bytes at the measured copy bandwidth and its
+    products at the measured cuBLAS rate) and how many times farther from it than the like kernel."""
+
+    def __init__(self, args, peaks):
+        self.args, self.recs, self.launches = args, {}, 0
+        self.hbm, self.tf = peaks.get("hbm_gbs", 6650.0) * 1e9, peaks.get("bf16_tflops", 1590.0) * 1e12
+
+    def __call__(self, name, fn, nbytes, flops=0.0, like=None):
+        import torch
+        for _ in range(self.args.warmup):
+            fn()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(self.args.steps):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        ms = e0.elapsed_time(e1) / self.args.steps
+        self.launches += self.args.steps
+        roof = max(nbytes / self.hbm, flops / self.tf)
+        r = self.recs[name] = {"ms": round(ms, 4), "bound": "hbm" if nbytes / self.hbm >= flops / self.tf else "tensor",
+                               "frac": round(roof / (ms * 1e-3), 3), "gbs": round(nbytes / ms / 1e6, 1),
+                               "tflops": round(flops / ms / 1e9, 1)}
+        if like:
+            r["like"] = like
+            r["distance_ratio"] = round(self.recs[like]["frac"] / r["frac"], 2)
+
+
+def qwen_of_size(dev, width, heads, kv, ff, blocks):
+    """Qwen3 blocks with random weights, as the engine takes them."""
+    import torch
+    from types import SimpleNamespace
+    from zipage_b200.layers.qwen3_block import Qwen3Model
+    from zipage_b200.models.registry import LoadedModel
+    bf = torch.bfloat16
+    c = SimpleNamespace(hidden_size=width, num_attention_heads=heads, num_key_value_heads=kv, head_dim=128, intermediate_size=ff,
+                        hidden_act="silu", rms_norm_eps=1e-6, vocab_size=32768, num_hidden_layers=blocks,
+                        max_position_embeddings=8192, rope_theta=1e6)
+    prev = torch.get_default_dtype()
+    torch.set_default_dtype(bf)
+    try:
+        with dev:
+            m = Qwen3Model(c).eval()
+    finally:
+        torch.set_default_dtype(prev)
+    return LoadedModel("Qwen3ForCausalLM", m, torch.empty(32768, width, dtype=bf, device=dev).normal_(0, 0.02), width, 32768, bf, False)
+
+
+SERVE = (64, 1536, 128)      # requests, prompt tokens, generated tokens of the model workloads
+
+
+def serve_model(loaded, g):
+    """Prefill and full-batch decode throughput of one model through the serving engine."""
+    import torch
+    from zipage_b200.engine.scheduler import SamplingParams, Sequence
+    from zipage_b200.models.registry import engine_for
+    R, PROMPT, GEN = SERVE
+    eng = engine_for(loaded, max_tokens=R * 2048, max_seqs=R, block_size=256, token_budget=16384, max_model_len=2304,
+                     budget_blocks=8, query_cache_len=32)
+    for rep in range(2):                       # the first pass warms up
+        eng.time_record.clear()
+        reqs = [Sequence(torch.randint(0, 32768, (PROMPT,), generator=g).tolist(), SamplingParams(1.0, GEN if rep else 8, True))
+                for _ in range(R)]
+        for r in reqs:
+            eng.add_request(r)
+        full = full_s = 0.0
+        while not eng.is_finished():
+            before = eng.time_record["decode_sum"]
+            _, n = eng.step()
+            if n == -R:
+                full, full_s = full + R, full_s + eng.time_record["decode_sum"] - before
+    tr = eng.time_record
+    return {"prefill_tokens_per_s": round(R * PROMPT / tr["prefill_sum"], 1), "decode_tokens_per_s": round(full / full_s, 1),
+            "decode_ms_per_step": round(full_s / (full / R) * 1e3, 3)}
+
+
 def similorn_kernel_records(args, dev, peaks):
     """Every kernel of the Similorn decoder at sizes of an 8B-class model's layers (width 4096, attention 32 / 8
     heads of 128, matrix memories 16 x [128, 256], bf16) beside the like kernel of the Qwen3 path at the same
@@ -1061,31 +1139,9 @@ def similorn_kernel_records(args, dev, peaks):
     from zipage_b200.layers import row_ops as R
     from zipage_b200.layers import step_ops as P
     from zipage_b200.layers.mlstm import mlstm_step
-    hbm, tf = peaks.get("hbm_gbs", 6650.0) * 1e9, peaks.get("bf16_tflops", 1590.0) * 1e12
     bf, W = torch.bfloat16, 4096
     rnd = lambda *s, dt=bf: torch.empty(s, dtype=dt, device=dev).normal_()
-    recs, launches = {}, 0
-
-    def rec(name, fn, nbytes, flops=0.0, like=None):
-        nonlocal launches
-        for _ in range(args.warmup):
-            fn()
-        torch.cuda.synchronize()
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        e0.record()
-        for _ in range(args.steps):
-            fn()
-        e1.record()
-        torch.cuda.synchronize()
-        ms = e0.elapsed_time(e1) / args.steps
-        launches += args.steps
-        roof = max(nbytes / hbm, flops / tf)
-        recs[name] = {"ms": round(ms, 4), "bound": "hbm" if nbytes / hbm >= flops / tf else "tensor",
-                      "frac": round(roof / (ms * 1e-3), 3), "gbs": round(nbytes / ms / 1e6, 1),
-                      "tflops": round(flops / ms / 1e9, 1)}
-        if like:
-            recs[name]["like"] = like
-            recs[name]["distance_ratio"] = round(recs[like]["frac"] / recs[name]["frac"], 2)
+    rec = KernelTable(args, peaks)
 
     # prompts: 4 x 4096 tokens
     B, S = 4, 4096
@@ -1152,7 +1208,7 @@ def similorn_kernel_records(args, dev, peaks):
     tok, emb = torch.randint(0, 32768, (T,), device=dev), rnd(32768, W)
     turns = R.sinusoid_turns(W, dev)
     rec("embedding and position", lambda: R.embed_position(tok, pos, emb, 2.0, turns, want_t=True), 8.0 * T * W, 0.0, "qwen3 add + rms norm")
-    return recs, launches
+    return rec.recs, rec.launches
 
 
 def run_similorn(args):
@@ -1161,10 +1217,7 @@ def run_similorn(args):
     Similorn: alternating matrix-memory layers and windowed-attention layers with feed-forward, the middle half
     of the stack run twice; Qwen3: as many blocks as Similorn has layer runs."""
     import torch
-    from types import SimpleNamespace
-    from zipage_b200.engine.scheduler import SamplingParams, Sequence
-    from zipage_b200.layers.qwen3_block import Qwen3Model
-    from zipage_b200.models.registry import LoadedModel, engine_for
+    from zipage_b200.models.registry import LoadedModel
     from zipage_b200.models.similorn import SimilornConfig, SimilornModel
     dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
     torch.cuda.set_device(dev)
@@ -1192,40 +1245,8 @@ def run_similorn(args):
                     layer.mixer.norm.fill_(1.0)
         return LoadedModel("Similorn", m, m.head, width, 32768, bf, True), len(m.runs)
 
-    def qwen(width, heads, kv, ff, blocks):
-        c = SimpleNamespace(hidden_size=width, num_attention_heads=heads, num_key_value_heads=kv, head_dim=128, intermediate_size=ff,
-                            hidden_act="silu", rms_norm_eps=1e-6, vocab_size=32768, num_hidden_layers=blocks,
-                            max_position_embeddings=8192, rope_theta=1e6)
-        prev = torch.get_default_dtype()
-        torch.set_default_dtype(bf)
-        try:
-            with dev:
-                m = Qwen3Model(c).eval()
-        finally:
-            torch.set_default_dtype(prev)
-        return LoadedModel("Qwen3ForCausalLM", m, torch.empty(32768, width, dtype=bf, device=dev).normal_(0, 0.02), width, 32768, bf, False)
-
-    R, PROMPT, GEN = 64, 1536, 128
+    R, PROMPT, GEN = SERVE
     g = torch.Generator().manual_seed(1)
-
-    def serve(loaded):
-        eng = engine_for(loaded, max_tokens=R * 2048, max_seqs=R, block_size=256, token_budget=16384, max_model_len=2304,
-                         budget_blocks=8, query_cache_len=32)
-        for rep in range(2):                       # the first pass warms up
-            eng.time_record.clear()
-            reqs = [Sequence(torch.randint(0, 32768, (PROMPT,), generator=g).tolist(), SamplingParams(1.0, GEN if rep else 8, True))
-                    for _ in range(R)]
-            for r in reqs:
-                eng.add_request(r)
-            full = full_s = 0.0
-            while not eng.is_finished():
-                before = eng.time_record["decode_sum"]
-                _, n = eng.step()
-                if n == -R:
-                    full, full_s = full + R, full_s + eng.time_record["decode_sum"] - before
-        tr = eng.time_record
-        return {"prefill_tokens_per_s": round(R * PROMPT / tr["prefill_sum"], 1), "decode_tokens_per_s": round(full / full_s, 1),
-                "decode_ms_per_step": round(full_s / (full / R) * 1e3, 3)}
 
     res = {}
     with ClockSampler(dev.index or 0) as clocks:
@@ -1233,10 +1254,10 @@ def run_similorn(args):
         torch.cuda.empty_cache()
         for width, heads, kv, mheads, ff in ((4096, 32, 8, 16, 12288), (2048, 16, 4, 8, 6144)):
             loaded, runs = similorn(width, heads, kv, mheads, ff)
-            a = serve(loaded)
+            a = serve_model(loaded, g)
             del loaded
             torch.cuda.empty_cache()
-            b = serve(qwen(width, heads, kv, ff, runs))
+            b = serve_model(qwen_of_size(dev, width, heads, kv, ff, runs), g)
             torch.cuda.empty_cache()
             res[f"width {width}"] = {"similorn": a, "qwen3": b, "layer_runs": runs}
     head = res["width 4096"]["similorn"]
@@ -1247,6 +1268,184 @@ def run_similorn(args):
         "config": {"workload": f"serving engine, {R} requests, prompts of {PROMPT}, {GEN} sampled tokens each; random weights; 12 layer "
                                "runs (mlstm / windowed attention + feed-forward alternating, the middle half twice) beside 12 Qwen3 blocks",
                    "l2": "inputs of every kernel are larger than L2"},
+        "serving": res, "kernels": kernels, "gpu_launches": launches, "clocks": clocks.summary(),
+        "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")},
+    }))
+
+
+def dobedra_kernel_records(args, dev, peaks):
+    """Every kernel of the Dobedra decoder at sizes of an 8B-class model's layers (width 4096, 32 heads of 128 + 64 | 128,
+    latents of 512 + 64, queries through 1536; 64 experts of 1024, six a token; bf16) beside the like kernel of
+    the Qwen3 path at the same width and heads.  Inputs are larger than L2 wherever the kernel streams."""
+    import torch
+    from zipage_b200.layers import attention as A
+    from zipage_b200.layers import feed_forward as F
+    from zipage_b200.layers import latent_attention as LA
+    from zipage_b200.layers import row_ops as R
+    from zipage_b200.layers import step_ops as P
+    bf, W = torch.bfloat16, 4096
+    rnd = lambda *s, dt=bf: torch.empty(s, dtype=dt, device=dev).normal_()
+    i32 = lambda t: t.to(torch.int32).to(dev)
+    rec = KernelTable(args, peaks)
+    H, dim, rot, vdim, QR, KR = 32, 128, 64, 128, 1536, 512
+    KP = KR + rot
+
+    # prompts: 4 x 4096 tokens
+    B, S = 4, 4096
+    T = B * S
+    cu, pos = i32(torch.arange(0, T + 1, S)), torch.arange(S, device=dev).repeat(B)
+    pairs = B * S * S / 2
+    q, k, v = rnd(T, HQ, D), rnd(T, HKV, D), rnd(T, HKV, D)
+    rec("qwen3 prefill attention", lambda: A.varlen_prefill_attention(q, k, v, S, cu, S, cu), 2.0 * T * D * (2 * HQ + 2 * HKV),
+        4.0 * D * HQ * pairs)
+    ql, kv, lat = rnd(T, H * (dim + rot)), rnd(T, H * (dim + vdim)), rnd(T, KP)
+    out = torch.empty(T, H * vdim, dtype=bf, device=dev)
+    rec("latent prefill attention", lambda: LA.latent_prefill(ql, kv, lat, cu, cu, S, out, H, dim, rot, vdim, KR, (dim + rot) ** -0.5),
+        2.0 * T * (H * (2 * dim + rot + 2 * vdim) + rot), 2.0 * (dim + rot + vdim) * H * pairs, "qwen3 prefill attention")
+    del q, k, v, kv
+    # decode: 256 sequences (Qwen3) and 128 (a latent row serves every head: fewer bytes per sequence)
+    n, NB = 256, 9
+    ctx = NB * 256 - 7
+    lens = i32(torch.full((n,), ctx))
+    qd, kq, vq = rnd(n, 1, HQ, D), rnd(n * NB, 256, HKV, D), rnd(n * NB, 256, HKV, D)
+    bt = i32(torch.randperm(n * NB).view(n, NB))
+    rec("qwen3 paged decode", lambda: A.paged_decode_attention(qd, kq, vq, lens, bt), n * ctx * HKV * D * 4.0)
+    del kq, vq
+    cache = rnd(n * NB, 256, 1, KP)
+    for seqs, heads in ((256, 16), (256, 32), (64, 32), (256, 128)):
+        qa, oa = rnd(seqs, heads, KP), torch.empty(seqs, heads, KR, dtype=bf, device=dev)
+        rec(f"latent decode attention, {heads} heads, {seqs} sequences",
+            lambda: LA.latent_attention(qa, cache, lens[:seqs], bt[:seqs], KR, 0.07, out=oa),
+            seqs * (ctx * KP + heads * (KP + KR)) * 2.0, 2.0 * seqs * heads * ctx * (KP + KR), "qwen3 paged decode")
+    # row ops
+    xr, wr, res = rnd(T, W), torch.ones(W, dtype=bf, device=dev), rnd(T, W)
+    rec("qwen3 add + rms norm", lambda: P.rms_norm(xr, wr, 1e-6, res), 8.0 * T * W)
+    x, vec = rnd(T, W, dt=torch.float32), [torch.ones(W, device=dev) for _ in range(6)]
+    norms = [(vec[0], vec[1]), (vec[2], vec[3])]
+    a, b = rnd(T, W), rnd(T, W)
+    rec("layer boundary, dense", lambda: R.join_norms(x, norms, 1e-5, bf, a=a, ls_a=vec[4], b=b, ls_b=vec[5]), 16.0 * T * W, 0.0,
+        "qwen3 add + rms norm")
+    E, top, ff = 64, 6, 1024
+    y, places = rnd(T * top, W), i32(torch.randperm(T * top)).view(T, top)
+    wts, gate = torch.rand(T, top, device=dev), rnd(T, 1, dt=torch.float32)[:, 0]
+    rec("layer boundary, experts", lambda: R.join_norms(x, norms, 1e-5, bf, a=a, ls_a=vec[4], b=b, ls_b=vec[5], gate=gate, y=y, pos=places,
+                                                        weights=wts), (16.0 + 2 * top) * T * W, 0.0, "qwen3 add + rms norm")
+    del y, a, b
+    up = rnd(T, 2 * 12288)
+    rec("qwen3 silu and mul", lambda: P.silu_and_mul(up), 6.0 * T * 12288)
+    rec("gelu and mul", lambda: F.gelu_tanh_and_mul(up), 6.0 * T * 12288, 0.0, "qwen3 silu and mul")
+    rec("squared relu", lambda: F.relu_squared_(up), 8.0 * T * 12288, 0.0, "qwen3 silu and mul")
+    z = rnd(2048, 32768, dt=torch.float32)
+    rec("soft cap of the logits", lambda: R.soft_cap_(z, 30.0), 8.0 * z.numel(), 0.0, "qwen3 silu and mul")
+    del up, z
+    qkv = rnd(T, HQ * D + 2 * HKV * D)
+    slot = i32(torch.arange(T))
+    cs = P.rope_cos_sin_cache(D, S, 1e6, dev)
+    w1 = torch.ones(D, dtype=bf, device=dev)
+    kc, vc = rnd(T // 64, 64, HKV, D), rnd(T // 64, 64, HKV, D)
+    rec("qwen3 q/k norm, rotation and store", lambda: P.qk_norm_rope_store(
+        qkv, pos, cs, w1, w1, 1e-6, HQ, HKV, D, kc, vc, slot, return_k=False), 2.0 * T * D * (2 * HQ + 4 * HKV))
+    yd, turns = rnd(T, QR + KP), LA.rotary_turns(rot, 1e6, dev)
+    wq, wk = torch.ones(QR, device=dev), torch.ones(KR, device=dev)
+    like = "qwen3 q/k norm, rotation and store"
+    rec("latent norms, rotation and store", lambda: LA.latent_prepare(yd, pos, turns, wq, wk, cache, slot, QR, KR, rot, 1e-5),
+        2.0 * T * 2 * (QR + KP), 0.0, like)
+    rec("query rotation in place", lambda: LA.latent_rotate_q(ql, pos, turns, H, dim, rot), 2.0 * T * H * rot * 2, 0.0, like)
+    rec("gather of cached rows", lambda: LA.gather_rows(cache, bt[:58], torch.arange(0, 58 * 2304, 2260, device=dev, dtype=torch.int32)[:59],
+                                                        58 * 2260), 4.0 * 58 * 2260 * KP, 0.0, like)
+    # experts
+    zl = rnd(T, E + 1, dt=torch.float32)
+    rec("routing", lambda: F.moe_route(zl, E, top), 4.0 * T * (E + 1) + T * top * 20.0)
+    dn = rnd(T, W)
+    wd = rnd(6 * 1024, W)
+    rec("cuBLAS product of a dense feed-forward", lambda: torch.mm(dn, wd.t()), 2.0 * (T * W + wd.numel() + T * wd.shape[0]),
+        2.0 * T * wd.numel())
+    wu, wdn = rnd(E, ff, W), rnd(E, W, ff)
+    _, _, _, prow, off = F.moe_route(zl, E, top)
+    M = T * top
+    mid = rnd(M, ff)
+    like = "cuBLAS product of a dense feed-forward"
+    rec("experts up, prompts", lambda: F.grouped_gemm(dn, wu, off, M, rows=prow, act="relu_squared"), 2.0 * (T * W + wu.numel() + M * ff),
+        2.0 * M * W * ff, like)
+    rec("experts down, prompts", lambda: F.grouped_gemm(mid, wdn, off, M), 2.0 * (M * ff + wu.numel() + M * W), 2.0 * M * W * ff, like)
+    # decode: 64 tokens reach nearly all experts; their weights stream through
+    t = 64
+    sets = [rnd(E, ff, W) for _ in range(2)]
+    _, _, _, prow2, off2 = F.moe_route(zl[:t], E, top)
+    used = int((off2[1:] > off2[:-1]).sum())
+    wbig = rnd(65536, W)
+    rec("cuBLAS product, 64 tokens", lambda: torch.mm(dn[:t], wbig.t()), 2.0 * (wbig.numel() + t * (W + 65536)), 2.0 * t * wbig.numel())
+    like = "cuBLAS product, 64 tokens"
+    turn = [0]
+
+    def decode_up():
+        turn[0] ^= 1
+        F.grouped_gemm(dn[:t], sets[turn[0]], off2, t * top, rows=prow2, act="relu_squared")
+
+    def decode_down():
+        turn[0] ^= 1
+        F.grouped_gemm(mid[:t * top], sets[turn[0]].view(E, W, ff), off2, t * top)
+    rec("experts up, 64 tokens", decode_up, 2.0 * (used * ff * W + t * W + t * top * ff), 0.0, like)
+    rec("experts down, 64 tokens", decode_down, 2.0 * (used * ff * W + t * top * (W + ff)), 0.0, like)
+    rec("routing, 64 tokens", lambda: F.moe_route(zl[:t], E, top), 4.0 * t * (E + 1) + t * top * 20.0)
+    return rec.recs, rec.launches
+
+
+def dobedra_of_size(dev, width, heads, q_rank, ff, experts, top, eff, layers=12):
+    """A Dobedra decoder with random weights: the first layer dense, the others with experts, every second layer attending to
+    the latents of the one before."""
+    import torch
+    from zipage_b200.models.dobedra import DobedraConfig, DobedraModel
+    from zipage_b200.models.registry import LoadedModel
+    mix = lambda i: {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": 512, "scale": 192 ** -0.5,
+                     "rot": {"base": 1e6, "dims": 64}, **({"kv_from": i - 1} if i % 2 else {})}
+    mlp = lambda i: {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": eff}, "shared": {"ff": 2 * eff}} if i else \
+        {"kind": "dense", "ff": ff}
+    c = DobedraConfig.from_dict({"vocab": 32768, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+                                 "layers": [{"type": "latent_attention", "mixer": mix(i), "mlp": mlp(i)} for i in range(layers)]})
+    m = DobedraModel(c, torch.bfloat16, dev)
+    with torch.no_grad():
+        for n, p in m.named_parameters():
+            if p.dim() > 1:
+                p.normal_(0, p.shape[-1] ** -0.5)
+            else:
+                p.zero_() if "bias" in n else p.fill_(1.0)
+    return LoadedModel("Dobedra", m, m.head, width, 32768, torch.bfloat16, True)
+
+
+def run_dobedra(args):
+    """Prefill and decode throughput of the Dobedra decoder through the serving engine at two widths, random weights, beside
+    Qwen3 blocks of equal width, depth and heads whose feed-forward is as wide as what a token's experts and the shared
+    block add up to; and the kernel table."""
+    import torch
+    dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
+    torch.cuda.set_device(dev)
+    pk = ROOT / "MEASURED_PEAKS.json"
+    peaks = json.loads(pk.read_text()) if pk.exists() else {}
+    torch.manual_seed(3)
+    R, PROMPT, GEN = SERVE
+    g = torch.Generator().manual_seed(1)
+    res = {}
+    with ClockSampler(dev.index or 0) as clocks:
+        kernels, launches = dobedra_kernel_records(args, dev, peaks)
+        torch.cuda.empty_cache()
+        for width, heads, kv, q_rank, ff, experts, top, eff in ((4096, 32, 8, 1536, 8192, 64, 6, 1024), (2048, 16, 4, 768, 4096, 64, 6, 512)):
+            loaded = dobedra_of_size(dev, width, heads, q_rank, ff, experts, top, eff)
+            a = serve_model(loaded, g)
+            del loaded
+            torch.cuda.empty_cache()
+            b = serve_model(qwen_of_size(dev, width, heads, kv, ff, 12), g)
+            torch.cuda.empty_cache()
+            res[f"width {width}"] = {"dobedra": a, "qwen3": b, "layers": 12}
+    head = res["width 4096"]["dobedra"]
+    print(json.dumps({
+        "metric": "dobedra_decode_tokens_per_s", "value": head["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+        "steps": args.steps, "warmup": args.warmup, "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True,
+        "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": f"serving engine, {R} requests, prompts of {PROMPT}, {GEN} sampled tokens each; random weights; 12 layers "
+                               "(latent attention, every second one sharing the latents before it; 64 experts, six a token, and a shared "
+                               "one) beside 12 Qwen3 blocks",
+                   "l2": "inputs of the streaming kernels are larger than L2"},
         "serving": res, "kernels": kernels, "gpu_launches": launches, "clocks": clocks.summary(),
         "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")},
     }))
@@ -1364,6 +1563,8 @@ def main():
         return run_native_engine(args)
     if args.workload == "similorn":
         return run_similorn(args)
+    if args.workload == "dobedra":
+        return run_dobedra(args)
     if args.workload == "prefill":
         return run_prefill(args)
     if args.workload == "decode":
