@@ -11,9 +11,9 @@
 // which fp32 sums and bf16 pairs carry without loss, so nearly always once per span.
 // M = 128 also for 64-key tiles: the upper lanes of S^T come from whatever follows in shared memory and are not read.
 //
-// Roles (384 threads, one block per SM): warp 0 = TMA producer and TMEM owner, warp 1 = MMA issuer (it takes
-// whichever of the next tile's scores and this tile's values is ready), warps 4-11 = softmax in lane quadrants
-// 0-1 (thread <-> key, two warps split the columns), rescaling and output in all four (lane <-> latent entry).
+// Roles (384 threads, one block per SM): warp 0 = TMA producer and TMEM owner, warp 1 issues the score products, warp
+// 2 the value products, warps 4-11 = softmax in lane quadrants 0-1 (thread <-> key, two warps split the columns),
+// rescaling and output in all four (lane <-> latent entry).
 // Shared memory: the queries, stages of 128-entry chunks (64 rows each), two P tiles.  Every wait is bounded.
 #include "zp_latent.cuh"
 #include "zp_tc.cuh"
@@ -37,15 +37,6 @@ struct __align__(16) LdShared {
   int abort_flag;
 };
 
-__device__ __forceinline__ bool ld_test(uint64_t* bar, uint32_t parity) {
-  uint32_t ok;
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-      "selp.u32 %0, 1, 0, p;\n\t}"
-      : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
-  return ok != 0;
-}
 __device__ __forceinline__ uint64_t ld_desc_mn(uint32_t addr, uint32_t lbo) {   // MN-major, 64-entry blocks lbo apart
   const uint32_t lo = ((addr >> 4) & 0x3FFFu) | ((lbo >> 4) << 16);
   const uint32_t hi = (1024u >> 4) | (1u << 14) | (2u << 29);
@@ -109,6 +100,7 @@ __device__ __forceinline__ bool ld_meet_any(bool v) {
 struct LdParams {
   LatentArgs a;
   int nb, nc, nv, stages;     // 64-entry blocks of a row; 128-entry chunks; chunks that hold values; stages
+  int pairs;                  // a row is whole blocks, and a chunk is one load
   int* error_word;
 };
 
@@ -133,7 +125,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   unsigned char* stage0 = qbuf + p.nb * NC * 128;
   unsigned char* pbuf = stage0 + p.stages * p.nc * LD_CHUNK;     // two tiles of 64 keys x 128 bytes
   LdShared& sh = *reinterpret_cast<LdShared*>(pbuf + 2 * LD_SUB);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = warp_index(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     mbar_init(&sh.qfull, 1);
     for (int s = 0; s < p.stages; ++s)
@@ -160,68 +152,80 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   volatile int* abortp = &sh.abort_flag;
 
   if (warp == 0) {
-    if (lane == 0 && n > 0) {
+    if (n > 0 && elect_one()) {
       prefetch_tensormap(&tmQ);
       prefetch_tensormap(&tmC);
       mbar_arrive_expect_tx(&sh.qfull, (uint32_t)(p.nb * NC * 128));
       for (int k = 0; k < p.nb; ++k) tma_load_5d(qbuf + k * NC * 128, &tmQ, &sh.qfull, k * 64, (int)flat0, 0, 0, 0);
       bool ok = true;
+      int s = 0, parity = 1;
+      unsigned char* dst = stage0;
       for (int j = 0; ok && j < n; ++j) {
-        const int key0 = (t0 + j) * 64, page = lat_page(a, b, key0), s = j % p.stages, k = j / p.stages;
-        for (int c = 0; c < p.nc; ++c) {
-          if (!mbar_wait<true>(&sh.empty[s][c], (k & 1) ^ 1, abortp, p.error_word, 901)) { ok = false; break; }
-          const int subs = min(2, p.nb - 2 * c);
-          unsigned char* dst = stage0 + (s * p.nc + c) * LD_CHUNK;
-          mbar_arrive_expect_tx(&sh.full[s][c], (uint32_t)(subs * LD_SUB));
-          for (int u = 0; u < subs; ++u) tma_load_5d(dst + u * LD_SUB, &tmC, &sh.full[s][c], (2 * c + u) * 64, 0, key0 % a.BS, page, 0);
+        const int key0 = (t0 + j) * 64, page = lat_page(a, b, key0), off = key0 % a.BS;
+        for (int c = 0; c < p.nc; ++c, dst += LD_CHUNK) {
+          if (!mbar_wait<true>(&sh.empty[s][c], parity, abortp, p.error_word, 901)) { ok = false; break; }
+          if (p.pairs) {          // both halves of the chunk at once (one past the row's end is filled with zeros)
+            mbar_arrive_expect_tx(&sh.full[s][c], LD_CHUNK);
+            tma_load_5d(dst, &tmC, &sh.full[s][c], 0, off, 2 * c, page, 0);
+          } else {
+            const int subs = min(2, p.nb - 2 * c);
+            mbar_arrive_expect_tx(&sh.full[s][c], (uint32_t)(subs * LD_SUB));
+            for (int u = 0; u < subs; ++u) tma_load_5d(dst + u * LD_SUB, &tmC, &sh.full[s][c], (2 * c + u) * 64, off, 0, page, 0);
+          }
         }
+        if (++s == p.stages) { s = 0; parity ^= 1; dst = stage0; }
       }
     }
   } else if (warp == 1) {
-    if (lane == 0 && n > 0) {
+    if (n > 0 && elect_one()) {               // scores
       constexpr uint32_t ID_S = idesc_f16(1, 128, NC);
-      constexpr uint32_t ID_O = idesc_f16(1, 128, 2 * NC) | (1u << 15) | (1u << 16);   // both operands MN-major
       bool ok = mbar_wait(&sh.qfull, 0, abortp, p.error_word, 902);
-      const uint32_t q_addr = smem_u32(qbuf), st_addr = smem_u32(stage0), p_addr = smem_u32(pbuf);
-      int js = 0, cs = 0, jp = 0;           // next tile and chunk of scores, next tile of values
-      uint32_t idle = 0;
-      while (ok && jp < n) {
-        bool moved = false;
-        if (js < n) {
-          const int s = js % p.stages, sb = js & 1;
-          if ((cs > 0 || ld_test(&sh.sempty[sb], ((js >> 1) & 1) ^ 1)) && ld_test(&sh.full[s][cs], (js / p.stages) & 1)) {
-            fence_after_sync();
-            const uint32_t c_addr = st_addr + (s * p.nc + cs) * LD_CHUNK;
-            const int subs = min(2, p.nb - 2 * cs);
-            for (int u = 0; u < subs; ++u) {
-              const uint64_t ad = smem_desc_sw128(c_addr + u * LD_SUB), bd = smem_desc_sw128(q_addr + (2 * cs + u) * NC * 128);
-#pragma unroll
-              for (int ks = 0; ks < 4; ++ks) umma_f16(tmem + sb * NC, ad + 2u * ks, bd + 2u * ks, ID_S, (cs | u | ks) ? 1u : 0u);
-            }
-            if (cs >= p.nv) umma_commit(&sh.empty[s][cs]);
-            if (++cs == p.nc) { umma_commit(&sh.sfull[sb]); cs = 0; ++js; }
-            moved = true;
-          }
-        }
-        if (jp < js && ld_test(&sh.pfull[jp & 1], (jp >> 1) & 1)) {
+      const uint64_t q_desc = smem_desc_sw128(smem_u32(qbuf));
+      uint64_t c_desc = smem_desc_sw128(smem_u32(stage0));
+      int s = 0, parity = 0;
+      for (int j = 0; ok && j < n; ++j) {
+        const uint32_t d = tmem + (j & 1) * NC;
+        if (!mbar_wait(&sh.sempty[j & 1], ((j >> 1) & 1) ^ 1, abortp, p.error_word, 903)) break;
+        uint64_t bd = q_desc;
+        for (int c = 0; c < p.nc; ++c, c_desc += LD_CHUNK >> 4, bd += 2 * NC * 8) {
+          if (!mbar_wait(&sh.full[s][c], parity, abortp, p.error_word, 904)) { ok = false; break; }
           fence_after_sync();
-          const int s = jp % p.stages;
-          const uint32_t pt = p_addr + (jp & 1) * LD_SUB;
-          for (int m = 0; m < p.nv; ++m) {
-            const uint32_t c_addr = st_addr + (s * p.nc + m) * LD_CHUNK;
+          umma_f16(d, c_desc, bd, ID_S, c ? 1u : 0u);
 #pragma unroll
-            for (int ks = 0; ks < 4; ++ks)
-              umma_f16(tmem + O_COL + m * 2 * NC, ld_desc_mn(c_addr + ks * 2048, LD_SUB), ld_desc_mn(pt + ks * 2048, LD_SUB), ID_O,
-                       (jp | ks) ? 1u : 0u);
-            umma_commit(&sh.empty[s][m]);
+          for (int ks = 1; ks < 4; ++ks) umma_f16(d, c_desc + 2u * ks, bd + 2u * ks, ID_S, 1u);
+          if (2 * c + 1 < p.nb) {
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks) umma_f16(d, c_desc + (LD_SUB >> 4) + 2u * ks, bd + NC * 8 + 2u * ks, ID_S, 1u);
           }
-          umma_commit(&sh.pempty[jp & 1]);
-          ++jp;
-          moved = true;
+          if (c >= p.nv) umma_commit(&sh.empty[s][c]);
         }
-        if (moved) idle = 0;
-        else if (*abortp) ok = false;
-        else if (++idle > WAIT_LIMIT * 4u) { *abortp = 1; atomicCAS(p.error_word, 0, 903); ok = false; }
+        if (!ok) break;
+        umma_commit(&sh.sfull[j & 1]);
+        if (++s == p.stages) { s = 0; parity ^= 1; c_desc = smem_desc_sw128(smem_u32(stage0)); }
+      }
+    }
+  } else if (warp == 2) {
+    if (n > 0 && elect_one()) {               // values
+      constexpr uint32_t ID_O = idesc_f16(1, 128, 2 * NC) | (1u << 15) | (1u << 16);   // both operands MN-major
+      const uint64_t p_desc = ld_desc_mn(smem_u32(pbuf), LD_SUB);
+      uint64_t c_desc = ld_desc_mn(smem_u32(stage0), LD_SUB);
+      bool ok = true;
+      int s = 0;
+      for (int j = 0; j < n; ++j) {
+        if (!mbar_wait(&sh.pfull[j & 1], (j >> 1) & 1, abortp, p.error_word, 905)) { ok = false; break; }
+        fence_after_sync();
+        const uint64_t pd = p_desc + (j & 1) * (LD_SUB >> 4);
+        uint64_t ad = c_desc;
+        for (int m = 0; m < p.nv; ++m, ad += LD_CHUNK >> 4) {
+          const uint32_t d = tmem + O_COL + m * 2 * NC;
+          umma_f16(d, ad, pd, ID_O, j ? 1u : 0u);
+#pragma unroll
+          for (int ks = 1; ks < 4; ++ks) umma_f16(d, ad + (2048 >> 4) * ks, pd + (2048 >> 4) * ks, ID_O, 1u);
+          umma_commit(&sh.empty[s][m]);
+        }
+        umma_commit(&sh.pempty[j & 1]);
+        c_desc += (uint32_t)(p.nc * (LD_CHUNK >> 4));
+        if (++s == p.stages) { s = 0; c_desc = ld_desc_mn(smem_u32(stage0), LD_SUB); }
       }
       if (ok) umma_commit(&sh.obar);
     }
@@ -232,16 +236,16 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     const float sl2 = a.scale * LD_LOG2E;
     const int tid = threadIdx.x - 128;
     bool ok = true;
-    float l[CW];
+    float l[CW], ref[CW];
 #pragma unroll
-    for (int i = 0; i < CW; ++i) l[i] = 0.f;
+    for (int i = 0; i < CW; ++i) { l[i] = 0.f; ref[i] = -INFINITY; }
     for (int j = 0; j < n; ++j) {
       const int key0 = (t0 + j) * 64, sb = j & 1;
       float x[CW];
       bool over = false;
       const bool whole = key0 + 63 <= p_first && ncol == NC;
       if (q < 2) {
-        ok = ld_wait(&sh.sfull[sb], (j >> 1) & 1, abortp, p.error_word, 904);
+        ok = ld_wait(&sh.sfull[sb], (j >> 1) & 1, abortp, p.error_word, 907);
         if (ok) {
           fence_after_sync();
           LdTmem<CW>::ld(lane_base + sb * NC + ch * CW, x);
@@ -252,7 +256,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           for (int i = 0; i < CW; ++i) {
             x[i] *= sl2;
             if (!whole && key0 + key > sh.lim[ch * CW + i]) x[i] = -INFINITY;
-            over |= x[i] > sh.ref[ch * CW + i] + LD_LAZY;
+            over |= x[i] > ref[i] + LD_LAZY;
           }
         }
       }
@@ -274,11 +278,11 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         ld_meet_any(false);
         if (q < 2) {
 #pragma unroll
-          for (int i = 0; i < CW; ++i) l[i] *= sh.fac[ch * CW + i];
+          for (int i = 0; i < CW; ++i) { l[i] *= sh.fac[ch * CW + i]; ref[i] = sh.ref[ch * CW + i]; }
         }
         if (j > 0) {
           // every product into O so far has completed once the previous tile's P is free again
-          if (ok) ok = ld_wait(&sh.pempty[(j - 1) & 1], ((j - 1) >> 1) & 1, abortp, p.error_word, 905);
+          if (ok) ok = ld_wait(&sh.pempty[(j - 1) & 1], ((j - 1) >> 1) & 1, abortp, p.error_word, 908);
           if (ok) {
             fence_after_sync();
             for (int m = 0; m < p.nv; ++m)
@@ -296,7 +300,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         ld_meet_any(false);                              // fac and tmax may be rewritten
       }
       if (q < 2 && ok) {
-        if (j >= 2) ok = ld_wait(&sh.pempty[sb], ((j >> 1) & 1) ^ 1, abortp, p.error_word, 906);
+        if (j >= 2) ok = ld_wait(&sh.pempty[sb], ((j >> 1) & 1) ^ 1, abortp, p.error_word, 909);
         if (ok) {
           unsigned char* row = pbuf + sb * LD_SUB + key * 128;
           uint32_t hi[CW / 2], lo[CW / 2];
@@ -305,7 +309,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             float w[2];
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
-              w[u] = x[i + u] == -INFINITY ? 0.f : ld_ex2(x[i + u] - sh.ref[ch * CW + i + u]);
+              w[u] = x[i + u] == -INFINITY ? 0.f : ld_ex2(x[i + u] - ref[i + u]);
               l[i + u] += w[u];
             }
             const __nv_bfloat162 h = __floats2bfloat162_rn(w[0], w[1]);
@@ -326,7 +330,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (ok && first < 64) {
           const int s = j % p.stages;
           for (int c = 0; ok && c < p.nv; ++c) {
-            ok = ld_wait(&sh.full[s][c], (j / p.stages) & 1, abortp, p.error_word, 907);
+            ok = ld_wait(&sh.full[s][c], (j / p.stages) & 1, abortp, p.error_word, 910);
             unsigned char* t = stage0 + (s * p.nc + c) * LD_CHUNK;
             if (key >= first) {
               for (int i = 0; i < 8; ++i) st16(t + ch * LD_SUB + key * 128 + (i << 4), make_int4(0, 0, 0, 0));
@@ -347,7 +351,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (lane == 0) sh.lsum[q][ch * CW + i] = s;
       }
     }
-    if (ok && n > 0) ok = ld_wait(&sh.obar, 0, abortp, p.error_word, 908);
+    if (ok && n > 0) ok = ld_wait(&sh.obar, 0, abortp, p.error_word, 911);
     ld_meet_any(false);
     if (ok) {
       fence_after_sync();
@@ -442,6 +446,7 @@ template <int NC> static int ld_launch(const LatentArgs& a, int max_q, int total
   LdParams p;
   p.a = a;
   p.nb = (a.KP + 63) / 64;
+  p.pairs = a.KP % 64 == 0;
   p.nc = (p.nb + 1) / 2;
   p.nv = (a.R + 127) / 128;
   p.error_word = device_error_word();
@@ -460,9 +465,10 @@ template <int NC> static int ld_launch(const LatentArgs& a, int max_q, int total
   }
   {
     const uint64_t page = (uint64_t)a.BS * a.KP;
-    const uint64_t dims[5] = {(uint64_t)a.KP, 1, (uint64_t)a.BS, (uint64_t)a.n_pages, 1};
-    const uint64_t strides[4] = {(uint64_t)a.KP, (uint64_t)a.KP, page, page * a.n_pages};
-    const uint32_t box[5] = {64, 1, 64, 1, 1};
+    // whole 64-entry blocks: [block][key][entry] boxes of two blocks; else one block's box, cut at the row's end
+    const uint64_t dims[5] = {p.pairs ? 64u : (uint64_t)a.KP, (uint64_t)a.BS, p.pairs ? (uint64_t)p.nb : 1u, (uint64_t)a.n_pages, 1};
+    const uint64_t strides[4] = {(uint64_t)a.KP, p.pairs ? 64u : (uint64_t)a.KP, page, page * a.n_pages};
+    const uint32_t box[5] = {64, 64, p.pairs ? 2u : 1u, 1, 1};
     if (int rc = make_tensor_map_5d(&tmC, UmmaFmt<__nv_bfloat16>::tm, a.cache, dims, strides, box, 2)) return rc;
   }
   cudaError_t e = cudaFuncSetAttribute(latent_decode_tc_kernel<NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);

@@ -103,7 +103,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_
   unsigned char* qbuf = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   unsigned char* ring = qbuf + nbq * LF_BLK;
   LfShared& sh = *reinterpret_cast<LfShared*>(ring + p.ring * LF_BLK);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = warp_index(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     mbar_init(&sh.qfull, 1);
     for (int i = 0; i < p.ring; ++i) { mbar_init(&sh.full[i], 1); mbar_init(&sh.empty[i], 1); }
@@ -125,7 +125,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_
   volatile int* abortp = &sh.abort_flag;
 
   if (warp == 0) {
-    if (lane == 0) {
+    if (elect_one()) {
       mbar_arrive_expect_tx(&sh.qfull, (uint32_t)(nbq * LF_BLK));
       for (int i = 0; i < p.nbn; ++i) tma_load_5d(qbuf + i * LF_BLK, &tmQn, &sh.qfull, i * 64, h, q0 + qi0, 0, 0);
       for (int i = 0; i < p.nbr; ++i) tma_load_5d(qbuf + (p.nbn + i) * LF_BLK, &tmQr, &sh.qfull, i * 64, h, q0 + qi0, 0, 0);
@@ -145,7 +145,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
+    if (elect_one()) {
       constexpr uint32_t ID_S = idesc_f16(1, 128, 128);
       constexpr uint32_t ID_O = idesc_f16(1, 128, 64) | (1u << 16);   // V MN-major, one 64-entry block at a time
       bool ok = mbar_wait(&sh.qfull, 0, abortp, p.error_word, 922);

@@ -65,7 +65,7 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_con
   extern __shared__ unsigned char smem_raw[];
   unsigned char* ring = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   GtShared& sh = *reinterpret_cast<GtShared*>(ring + p.stages * STAGE);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = warp_index(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     for (int s = 0; s < p.stages; ++s) { mbar_init(&sh.full[s], 1); mbar_init(&sh.empty[s], 1); }
     for (int i = 0; i < 2; ++i) { mbar_init(&sh.afull[i], 1); mbar_init(&sh.aempty[i], 4); }
@@ -127,7 +127,7 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_con
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
+    if (elect_one()) {
       constexpr uint32_t ID = idesc_f16(1, 128, BN);
       bool ok = true;
       int slot = 0, round = 0, i = 0;
