@@ -5,10 +5,13 @@
 // places, BN outputs), whose length it derives from the experts' offsets on the device, so the launch is the
 // same whatever the routing chose (graphs).
 //
-// Roles (192 threads): warp 0 = TMA producer: one load for the weights, and for the rows a four-row gather per
-// lane, of which only those with places are issued (a decode step brings a few rows per expert, and the rest of the
-// 128-row operand is whatever the stage held: rows do not mix); warp 1 = MMA issuer, accumulating in TMEM, two
-// tiles in turn; warps 2-5 = epilogue (thread <-> TMEM lane <-> place): activation, rounding, store.  Every wait is bounded.
+// Roles: warp 0 = TMA producer; warp 1 = MMA issuer, accumulating in TMEM, two tiles in turn; warps 2-5 = epilogue
+// (thread <-> TMEM lane <-> place): activation, rounding, store.  Every wait is bounded.  How the rows arrive:
+//   GT_FEW     four-row gathers, one per lane, of which only those with places are issued (a decode step brings a few rows
+//              per expert, and the rest of the 128-row operand is whatever the stage held: rows do not mix);
+//   GT_TILE    one 128-row load (rows that already lie in the order of the places);
+//   GT_GATHER  four more warps copy the rows' 16-byte pieces with cp.async (a gather load fetches rows at a
+//              small part of a tile load's rate), publishing a stage two stages later, when its copies have landed.
 #include "zp_moe.cuh"
 #include "zp_tc.cuh"
 
@@ -16,7 +19,8 @@ namespace zp {
 
 using namespace tc;
 
-constexpr int GT_THREADS = 192;
+enum { GT_FEW = 0, GT_TILE = 1, GT_GATHER = 2 };
+constexpr int GT_LAG = 2;                 // stages between the issue of a stage's copies and its publication
 constexpr int GT_A = 16384;               // 128 rows x 64 entries
 constexpr int GT_MAXS = 8, GT_MAXE = 1024;
 
@@ -58,8 +62,21 @@ template <int BN> __device__ __forceinline__ GtTile gt_tile(const GtParams& p, c
   return r;
 }
 
-template <int BN, bool RELU2>
-__global__ void __launch_bounds__(GT_THREADS, 1)
+__device__ __forceinline__ void gt_copy16(uint32_t dst, const void* src, int bytes) {   // the rest of 16 bytes becomes zero
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+// the copies of the stage issued GT_LAG stages ago (or, LEFT = 0, all) have landed: tell the tensor cores
+template <int LEFT> __device__ __forceinline__ void gt_publish(uint64_t* bar, int lane) {
+  asm volatile("cp.async.wait_group %0;" ::"n"(LEFT) : "memory");
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  __syncwarp();
+  if (lane == 0) mbar_arrive(bar);
+}
+
+template <int MODE> constexpr int gt_threads() { return MODE == GT_GATHER ? 320 : 192; }
+
+template <int BN, bool RELU2, int MODE>
+__global__ void __launch_bounds__(gt_threads<MODE>(), 1)
 grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW, const GtParams p) {
   constexpr int STAGE = GT_A + BN * 128;
   extern __shared__ unsigned char smem_raw[];
@@ -67,7 +84,7 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_con
   GtShared& sh = *reinterpret_cast<GtShared*>(ring + p.stages * STAGE);
   const int warp = warp_index(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int s = 0; s < p.stages; ++s) { mbar_init(&sh.full[s], 1); mbar_init(&sh.empty[s], 1); }
+    for (int s = 0; s < p.stages; ++s) { mbar_init(&sh.full[s], MODE == GT_GATHER ? 5 : 1); mbar_init(&sh.empty[s], 1); }
     for (int i = 0; i < 2; ++i) { mbar_init(&sh.afull[i], 1); mbar_init(&sh.aempty[i], 4); }
     sh.abort_flag = 0;
     fence_mbar_init();
@@ -98,32 +115,48 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_con
   const int total = sh.mtiles[p.a.E] * p.ntn;
 
   if (warp == 0) {
-    bool ok = true;
-    int slot = 0, round = 0;
-    for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
-      const GtTile tl = gt_tile<BN>(p, sh, t);
-      const int groups = (tl.count + 3) >> 2;
-      int4 r;
-      {
-        int v[4];
+    if constexpr (MODE == GT_FEW) {
+      bool ok = true;
+      int slot = 0, round = 0;
+      for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
+        const GtTile tl = gt_tile<BN>(p, sh, t);
+        const int groups = (tl.count + 3) >> 2;
+        int4 r;
+        {
+          int v[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int at = tl.first + min(4 * lane + i, tl.count - 1);
-          v[i] = p.a.rows ? min(max(p.a.rows[at], 0), p.a.src_rows - 1) : at;
+          for (int i = 0; i < 4; ++i) {
+            const int at = tl.first + min(4 * lane + i, tl.count - 1);
+            v[i] = p.a.rows ? min(max(p.a.rows[at], 0), p.a.src_rows - 1) : at;
+          }
+          r = make_int4(v[0], v[1], v[2], v[3]);
         }
-        r = make_int4(v[0], v[1], v[2], v[3]);
+        for (int k = 0; k < p.kb; ++k) {
+          ok = __all_sync(0xffffffffu, mbar_wait(&sh.empty[slot], (round & 1) ^ 1, abortp, p.error_word, 941));
+          if (!ok) break;
+          unsigned char* dst = ring + slot * STAGE;
+          if (elect_one()) {
+            mbar_arrive_expect_tx(&sh.full[slot], (uint32_t)(groups * 512 + BN * 128));
+            tma_load_5d(dst + GT_A, &tmW, &sh.full[slot], k * 64, tl.n0, tl.e, 0, 0);
+          }
+          __syncwarp();
+          if (lane < groups) gt_gather4(dst + lane * 512, &tmX, &sh.full[slot], k * 64, r);
+          if (++slot == p.stages) { slot = 0; ++round; }
+        }
       }
-      for (int k = 0; k < p.kb; ++k) {
-        ok = __all_sync(0xffffffffu, mbar_wait(&sh.empty[slot], (round & 1) ^ 1, abortp, p.error_word, 941));
-        if (!ok) break;
-        unsigned char* dst = ring + slot * STAGE;
-        if (lane == 0) {
-          mbar_arrive_expect_tx(&sh.full[slot], (uint32_t)(groups * 512 + BN * 128));
+    } else if (elect_one()) {
+      bool ok = true;
+      int slot = 0, round = 0;
+      for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
+        const GtTile tl = gt_tile<BN>(p, sh, t);
+        for (int k = 0; k < p.kb; ++k) {
+          if (!mbar_wait(&sh.empty[slot], (round & 1) ^ 1, abortp, p.error_word, 941)) { ok = false; break; }
+          unsigned char* dst = ring + slot * STAGE;
+          mbar_arrive_expect_tx(&sh.full[slot], (uint32_t)((MODE == GT_TILE ? GT_A : 0) + BN * 128));
+          if (MODE == GT_TILE) tma_load_5d(dst, &tmX, &sh.full[slot], k * 64, tl.first, 0, 0, 0);
           tma_load_5d(dst + GT_A, &tmW, &sh.full[slot], k * 64, tl.n0, tl.e, 0, 0);
+          if (++slot == p.stages) { slot = 0; ++round; }
         }
-        __syncwarp();
-        if (lane < groups) gt_gather4(dst + lane * 512, &tmX, &sh.full[slot], k * 64, r);
-        if (++slot == p.stages) { slot = 0; ++round; }
       }
     }
   } else if (warp == 1) {
@@ -147,6 +180,43 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_con
         }
         if (ok) umma_commit(&sh.afull[acc]);
       }
+    }
+  } else if (warp >= 6) {                      // (GT_GATHER) eight lanes a row, four rows an instruction
+    const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(p.a.x);
+    const int r0 = (warp - 6) * 32 + (lane >> 3), piece = lane & 7;
+    bool ok = true;
+    int slot = 0, round = 0, late = 0, pending = 0;          // late: the slot to publish next
+    for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
+      const GtTile tl = gt_tile<BN>(p, sh, t);
+      const __nv_bfloat16* src[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int at = tl.first + min(r0 + 4 * i, tl.count - 1);
+        src[i] = x + (int64_t)min(max(p.a.rows[at], 0), p.a.src_rows - 1) * p.a.x_stride + piece * 8;
+      }
+      for (int k = 0; k < p.kb; ++k) {
+        ok = __all_sync(0xffffffffu, mbar_wait(&sh.empty[slot], (round & 1) ^ 1, abortp, p.error_word, 945));
+        if (!ok) break;
+        const uint32_t dst = smem_u32(ring + slot * STAGE);
+        const int bytes = k * 64 + piece * 8 < p.a.K ? 16 : 0;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int r = r0 + 4 * i;
+          gt_copy16(dst + r * 128 + ((piece ^ (r & 7)) << 4), bytes ? src[i] + k * 64 : x, bytes);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (++pending > GT_LAG) {
+          gt_publish<GT_LAG>(&sh.full[late], lane);
+          --pending;
+          if (++late == p.stages) late = 0;
+        }
+        if (++slot == p.stages) { slot = 0; ++round; }
+      }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    for (; ok && pending > 0; --pending) {
+      gt_publish<0>(&sh.full[late], lane);
+      if (++late == p.stages) late = 0;
     }
   } else {
     const int q = warp & 3, row = q * 32 + lane;
@@ -209,7 +279,7 @@ bool grouped_tc_supports(const GroupedArgs& a, int dtype) {
          ((uintptr_t)a.x | (uintptr_t)a.w | (uintptr_t)a.out) % 16 == 0;
 }
 
-template <int BN, bool RELU2> static int gt_launch(const GroupedArgs& a, cudaStream_t st) {
+template <int BN, bool RELU2, int MODE> static int gt_launch(const GroupedArgs& a, cudaStream_t st) {
   constexpr int STAGE = GT_A + BN * 128;
   GtParams p;
   p.a = a;
@@ -221,7 +291,14 @@ template <int BN, bool RELU2> static int gt_launch(const GroupedArgs& a, cudaStr
   if (!p.error_word) { set_error("zp_grouped_gemm(tcgen05): no device error word"); return ZP_ERR_CUDA; }
   const int smem = 1024 + p.stages * STAGE + (int)sizeof(GtShared);
   CUtensorMap tmX, tmW;
-  if (int rc = make_tensor_map_rows(&tmX, UmmaFmt<__nv_bfloat16>::tm, a.x, (uint64_t)a.K, (uint64_t)a.src_rows, (uint64_t)a.x_stride, 2)) return rc;
+  if (MODE == GT_TILE) {
+    const uint64_t all = (uint64_t)a.src_rows * a.x_stride;
+    const uint64_t dims[5] = {(uint64_t)a.K, (uint64_t)a.src_rows, 1, 1, 1}, strides[4] = {(uint64_t)a.x_stride, all, all, all};
+    const uint32_t box[5] = {64, 128, 1, 1, 1};
+    if (int rc = make_tensor_map_5d(&tmX, UmmaFmt<__nv_bfloat16>::tm, a.x, dims, strides, box, 2)) return rc;
+  } else {
+    if (int rc = make_tensor_map_rows(&tmX, UmmaFmt<__nv_bfloat16>::tm, a.x, (uint64_t)a.K, (uint64_t)a.src_rows, (uint64_t)a.x_stride, 2)) return rc;
+  }
   {
     const uint64_t per = (uint64_t)a.Nout * a.K;
     const uint64_t dims[5] = {(uint64_t)a.K, (uint64_t)a.Nout, (uint64_t)a.E, 1, 1};
@@ -229,19 +306,24 @@ template <int BN, bool RELU2> static int gt_launch(const GroupedArgs& a, cudaStr
     const uint32_t box[5] = {64, BN, 1, 1, 1};
     if (int rc = make_tensor_map_5d(&tmW, UmmaFmt<__nv_bfloat16>::tm, a.w, dims, strides, box, 2)) return rc;
   }
-  const auto kern = grouped_gemm_tc_kernel<BN, RELU2>;
+  const auto kern = grouped_gemm_tc_kernel<BN, RELU2, MODE>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) { set_error("zp_grouped_gemm(tcgen05): %s", cudaGetErrorString(e)); return ZP_ERR_CUDA; }
   const int64_t most = ((int64_t)a.places / 128 + (a.places < a.E ? a.places : a.E)) * p.ntn;   // tiles, at most
-  kern<<<(int)(most < 148 ? (most < 1 ? 1 : most) : 148), GT_THREADS, smem, st>>>(tmX, tmW, p);
+  kern<<<(int)(most < 148 ? (most < 1 ? 1 : most) : 148), gt_threads<MODE>(), smem, st>>>(tmX, tmW, p);
   return check_launch("zp_grouped_gemm(tcgen05)");
+}
+
+template <int BN, bool RELU2> static int gt_pick(const GroupedArgs& a, bool many, cudaStream_t st) {
+  if (!many) return gt_launch<BN, RELU2, GT_FEW>(a, st);
+  return a.rows ? gt_launch<BN, RELU2, GT_GATHER>(a, st) : gt_launch<BN, RELU2, GT_TILE>(a, st);
 }
 
 int grouped_gemm_tc(const GroupedArgs& a, cudaStream_t st) {
   // few places per expert: the weights stream through, and narrower tiles spread them better over the SMs
-  const bool wide = a.places >= 64 * (int64_t)a.E && a.Nout > 128;
-  if (a.act == ZP_ACT_RELU_SQUARED) return wide ? gt_launch<256, true>(a, st) : gt_launch<128, true>(a, st);
-  return wide ? gt_launch<256, false>(a, st) : gt_launch<128, false>(a, st);
+  const bool many = a.places >= 32 * (int64_t)a.E, wide = many && a.Nout > 128;
+  if (a.act == ZP_ACT_RELU_SQUARED) return wide ? gt_pick<256, true>(a, many, st) : gt_pick<128, true>(a, many, st);
+  return wide ? gt_pick<256, false>(a, many, st) : gt_pick<128, false>(a, many, st);
 }
 
 }  // namespace zp
