@@ -394,26 +394,43 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   }
 }
 
-// out [pair, R] from the spans' unnormalised sums, references and row sums
+// out [pair, R] from the spans' unnormalised sums, references and row sums; one block per pair, four entries a thread
 __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a) {
   // rows that no sequence of this call names (another call's, or padding) keep what they hold
+  __shared__ float w[32];
   const int b = blockIdx.y, i = blockIdx.x;
   const LatSeq sq = lat_seq(a, b);
   if (i >= sq.count * a.H) return;
   const int64_t pair = (int64_t)sq.row0 * a.H + i;
-  const float* ml = a.part + (int64_t)a.pairs * a.nsplit * a.R + pair * a.nsplit * 2;
-  float m = -INFINITY;
-  for (int s = 0; s < a.nsplit; ++s) m = fmaxf(m, ml[2 * s]);
-  float l = 0.f;
-  for (int s = 0; s < a.nsplit; ++s) l += ml[2 * s] == -INFINITY ? 0.f : ld_ex2(ml[2 * s] - m) * ml[2 * s + 1];
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int d = threadIdx.x; d < a.R; d += 128) {
-    float o = 0.f;
-    for (int s = 0; s < a.nsplit; ++s) {
-      const float w = ml[2 * s] == -INFINITY ? 0.f : ld_ex2(ml[2 * s] - m);
-      if (w > 0.f) o = fmaf(w, a.part[(pair * a.nsplit + s) * a.R + d], o);
+  if (threadIdx.x < 32) {                   // (at most 32 spans)
+    const float* ml = a.part + (int64_t)a.pairs * a.nsplit * a.R + pair * a.nsplit * 2;
+    const bool in = (int)threadIdx.x < a.nsplit;
+    const float2 v = in ? make_float2(ml[2 * threadIdx.x], ml[2 * threadIdx.x + 1]) : make_float2(-INFINITY, 0.f);
+    const float m = warp_max(v.x), f = v.x == -INFINITY ? 0.f : ld_ex2(v.x - m), l = warp_sum(f * v.y);
+    w[threadIdx.x] = l > 0.f ? f / l : 0.f;
+  }
+  __syncthreads();
+  const float* part = a.part + pair * a.nsplit * a.R;
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + pair * a.R;
+  if (a.R % 4 == 0) {
+    for (int d = threadIdx.x * 4; d < a.R; d += 512) {
+      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+      for (int s = 0; s < a.nsplit; ++s) {
+        const float4 v = *reinterpret_cast<const float4*>(part + (int64_t)s * a.R + d);
+        const float f = w[s];
+        if (f > 0.f) { o.x = fmaf(f, v.x, o.x); o.y = fmaf(f, v.y, o.y); o.z = fmaf(f, v.z, o.z); o.w = fmaf(f, v.w, o.w); }
+      }
+      const __nv_bfloat162 r[2] = {__floats2bfloat162_rn(o.x, o.y), __floats2bfloat162_rn(o.z, o.w)};
+      *reinterpret_cast<uint2*>(out + d) = *reinterpret_cast<const uint2*>(r);
     }
-    reinterpret_cast<__nv_bfloat16*>(a.out)[pair * a.R + d] = __float2bfloat16_rn(o * inv);
+  } else {
+    for (int d = threadIdx.x; d < a.R; d += 128) {
+      float o = 0.f;
+      for (int s = 0; s < a.nsplit; ++s)
+        if (w[s] > 0.f) o = fmaf(w[s], part[(int64_t)s * a.R + d], o);
+      out[d] = __float2bfloat16_rn(o);
+    }
   }
 }
 

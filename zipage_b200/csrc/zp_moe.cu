@@ -11,15 +11,25 @@ namespace zp {
 
 constexpr int RT_MAXE = 1024;
 
-// Scores of one token by one warp: lane holds experts lane, lane + 32, ...  Ties: the lower expert.
-// emit(k, expert, score) is called by lane 0.
+// fp32 -> unsigned with the same order (NaNs of either sign sort above or below all numbers)
+__device__ __forceinline__ unsigned order_key(float v) {
+  const unsigned u = __float_as_uint(v);
+  return (u & 0x80000000u) ? ~u : u | 0x80000000u;
+}
+
+// The `top` largest of one token's logits by one warp: lane holds experts lane, lane + 32, ...  Ties: the lower
+// expert.  Choice k is returned by lane k % 32 of round k / 32 (emit(k, expert, score) is called by that lane,
+// all lanes of a round at once).
 template <int VPL, typename F>
 __device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, int top, F&& emit) {
   const int lane = threadIdx.x & 31;
   float v[VPL], mx = -INFINITY;
+  unsigned key[VPL];                        // 0: taken, or no expert
 #pragma unroll
   for (int i = 0; i < VPL; ++i) {
-    v[i] = lane + 32 * i < E ? z[lane + 32 * i] : -INFINITY;
+    const bool in = lane + 32 * i < E;
+    v[i] = in ? z[lane + 32 * i] : -INFINITY;
+    key[i] = in ? max(order_key(v[i]), 1u) : 0u;
     mx = fmaxf(mx, v[i]);
   }
   mx = warp_max(mx);
@@ -27,22 +37,26 @@ __device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, 
 #pragma unroll
   for (int i = 0; i < VPL; ++i) sum += lane + 32 * i < E ? expf(v[i] - mx) : 0.f;
   sum = warp_sum(sum);
-  unsigned taken = 0;                       // bit i: this lane's i-th expert is chosen already
-  for (int k = 0; k < top; ++k) {
-    float bv = -INFINITY;
-    int bi = 0x7fffffff;
+  for (int k0 = 0; k0 < top; k0 += 32) {
+    int mine = 0;
+    float score = 0.f;
+    for (int k = k0; k < min(top, k0 + 32); ++k) {
+      unsigned bk = 0, bi = 0xffffffffu;
+      float bv = 0.f;
 #pragma unroll
-    for (int i = 0; i < VPL; ++i)
-      if (!((taken >> i) & 1u) && lane + 32 * i < E && (bi == 0x7fffffff || v[i] > bv)) { bv = v[i]; bi = lane + 32 * i; }
+      for (int i = 0; i < VPL; ++i)
+        if (key[i] > bk) { bk = key[i]; bi = lane + 32 * i; bv = v[i]; }
+      const unsigned best = __reduce_max_sync(0xffffffffu, bk);
+      const unsigned at = __reduce_min_sync(0xffffffffu, bk == best ? bi : 0xffffffffu);
+      bv = __shfl_sync(0xffffffffu, bv, at & 31);
+      if ((int)(at & 31) == lane) {
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (oi != 0x7fffffff && (bi == 0x7fffffff || ov > bv || (ov == bv && oi < bi))) { bv = ov; bi = oi; }
+        for (int i = 0; i < VPL; ++i)
+          if ((int)(at >> 5) == i) key[i] = 0u;
+      }
+      if (lane == k - k0) { mine = (int)at; score = bv; }
     }
-    if (bi == 0x7fffffff) bi = 0;           // (top <= E: only a row of NaNs gets here)
-    if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
-    if (lane == 0) emit(k, bi, expf(bv - mx) / sum);
+    if (lane < top - k0) emit(k0 + lane, mine, expf(score - mx) / sum);
   }
 }
 
@@ -74,20 +88,24 @@ struct RouteArgs {
   int32_t *rows, *offsets, *counts;
 };
 
-// One block does everything (ONE), or several blocks choose and count and route_place_kernel places.
+// One block does everything (ONE; at most RT_ONE pairs), or several blocks choose and count and route_place_kernel places.
+constexpr int RT_ONE = 4096;
 template <int VPL, bool ONE>
 __global__ void __launch_bounds__(ONE ? 1024 : 256) route_kernel(const RouteArgs a) {
   __shared__ int hist[RT_MAXE], offs[RT_MAXE + 1];
+  __shared__ int2 picks[ONE ? RT_ONE : 1];                     // expert and rank within it
   for (int e = threadIdx.x; e < a.E; e += blockDim.x) hist[e] = 0;
   __syncthreads();
-  const int nw = blockDim.x >> 5, per = ONE ? a.N : 64;        // tokens of a block
+  const int nw = blockDim.x >> 5, per = ONE ? a.N : 32;        // tokens of a block
   const int t0 = blockIdx.x * per, t1 = min(a.N, t0 + per);
   for (int t = t0 + (threadIdx.x >> 5); t < t1; t += nw)
     top_experts<VPL>(a.logits + (int64_t)t * a.ld, a.E, a.top, [&](int k, int e, float s) {
       const int64_t at = (int64_t)t * a.top + k;
       a.wts[at] = s;
       a.idx[at] = e;
-      a.pos[at] = atomicAdd(&hist[e], 1);
+      const int rank = atomicAdd(&hist[e], 1);
+      if constexpr (ONE) picks[at] = make_int2(e, rank);
+      else a.pos[at] = rank;
     });
   __syncthreads();
   if constexpr (ONE) {
@@ -95,7 +113,7 @@ __global__ void __launch_bounds__(ONE ? 1024 : 256) route_kernel(const RouteArgs
     __syncthreads();
     for (int e = threadIdx.x; e <= a.E; e += blockDim.x) a.offsets[e] = offs[e];
     for (int i = threadIdx.x; i < a.N * a.top; i += blockDim.x) {
-      const int p = offs[a.idx[i]] + a.pos[i];
+      const int p = offs[picks[i].x] + picks[i].y;
       a.pos[i] = p;
       a.rows[p] = i / a.top;
     }
@@ -121,12 +139,12 @@ __global__ void __launch_bounds__(256) route_place_kernel(const RouteArgs a) {
 }
 
 template <int VPL> static int launch_route(const RouteArgs& a, cudaStream_t st) {
-  if (a.N <= 512) {
+  if (a.N <= 512 && a.N * a.top <= RT_ONE) {
     route_kernel<VPL, true><<<1, 1024, 0, st>>>(a);
   } else {
     cudaError_t e = cudaMemsetAsync(a.counts, 0, (size_t)a.E * sizeof(int), st);
     if (e != cudaSuccess) { set_error("zp_moe_route: %s", cudaGetErrorString(e)); return ZP_ERR_CUDA; }
-    route_kernel<VPL, false><<<(a.N + 63) / 64, 256, 0, st>>>(a);
+    route_kernel<VPL, false><<<(a.N + 31) / 32, 256, 0, st>>>(a);
     const int64_t want = ((int64_t)a.N * a.top + 255) / 256;
     route_place_kernel<<<(int)(want < 592 ? want : 592), 256, 0, st>>>(a);
   }

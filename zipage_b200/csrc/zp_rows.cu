@@ -186,29 +186,24 @@ __device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) {
 }
 __device__ __forceinline__ float4 splat4(float s) { return make_float4(s, s, s, s); }
 
+// What joins x at entry c of a row: `add` gathers it, so that the loads of all of a thread's entries can be in
+// flight before the first of them is stored.
 template <typename T, int V>
-__device__ __forceinline__ float4 join_entry(const JoinArgs& p, int64_t row, int c, const float* swts, const int32_t* spos, float g) {
+__device__ __forceinline__ float4 join_add(const JoinArgs& p, int64_t row, int c, const float* swts, const int32_t* spos, float g) {
   using L = JoinVec<T, V>;
-  float4 v = L::ldf(p.x, row * p.H + c);
   float4 add = splat4(0.f);
-  bool any = false;
   if (p.a) {
     add = L::ld(p.a, row * p.H + c);
     if (p.ls_a) { const float4 s = L::ldf(p.ls_a, c); add = make_float4(add.x * s.x, add.y * s.y, add.z * s.z, add.w * s.w); }
-    any = true;
   }
   if (p.b || p.y) {
     float4 f = splat4(0.f);
+#pragma unroll 4
     for (int k = 0; k < p.top; ++k) f = fma4(splat4(swts[k]), L::ld(p.y, (int64_t)spos[k] * p.H + c), f);
     if (p.b) f = fma4(splat4(g), L::ld(p.b, row * p.H + c), f);
     add = fma4(p.ls_b ? L::ldf(p.ls_b, c) : splat4(1.f), f, add);
-    any = true;
   }
-  if (any) {
-    v = make_float4(v.x + add.x, v.y + add.y, v.z + add.z, v.w + add.w);
-    L::stf(p.x, row * p.H + c, v);
-  }
-  return v;
+  return add;
 }
 template <typename T, int V>
 __device__ __forceinline__ void join_norm(const JoinArgs& p, int64_t row, int c, float4 d, float r) {
@@ -233,16 +228,27 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
     __syncthreads();
   }
   const float g = p.gate ? 1.f / (1.f + expf(-p.gate[row * p.gate_stride])) : 1.f;
-  const bool norm = p.out1 || p.out2;
+  const bool norm = p.out1 || p.out2, any = p.a || p.b || p.y;
   if constexpr (VPT > 0) {
     const int nvec = p.H / 4;
+    using L = JoinVec<T, 4>;
     float4 v[VPT];
     float s = 0.f;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = threadIdx.x + i * 256;
       if (c < nvec) {
-        v[i] = join_entry<T, 4>(p, row, 4 * c, swts, spos, g);
+        const float4 x = L::ldf(p.x, row * p.H + 4 * c);
+        if (!any) { v[i] = x; continue; }
+        const float4 d = join_add<T, 4>(p, row, 4 * c, swts, spos, g);
+        v[i] = make_float4(x.x + d.x, x.y + d.y, x.z + d.z, x.w + d.w);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      if (c < nvec) {
+        if (any) L::stf(p.x, row * p.H + 4 * c, v[i]);
         s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
       }
     }
@@ -266,7 +272,11 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
     }
   } else {
     float s = 0.f;
-    for (int c = threadIdx.x; c < p.H; c += blockDim.x) s += join_entry<T, 1>(p, row, c, swts, spos, g).x;
+    for (int c = threadIdx.x; c < p.H; c += blockDim.x) {
+      float v = p.x[row * p.H + c];
+      if (any) p.x[row * p.H + c] = v += join_add<T, 1>(p, row, c, swts, spos, g).x;
+      s += v;
+    }
     if (!norm) return;
     const float mean = block_sum(s, red) / (float)p.H;
     float ss = 0.f;

@@ -45,7 +45,7 @@ def moe_route(logits, n_experts, top):
     experts, places, rows, offsets, counts = ints.split([N * top] * 3 + [n_experts + 1, n_experts])
     L.check(L.load().zp_moe_route(L.ptr(logits), logits.stride(0), N, n_experts, top, L.ptr(w), L.ptr(experts), L.ptr(places),
                                   L.ptr(rows), L.ptr(offsets), L.ptr(counts), L.stream_ptr()), "moe_route")
-    _count(1 if N <= 512 else 2)
+    _count(1 if N <= 512 and N * top <= 4096 else 2)
     return w, experts.view(N, top), places.view(N, top), rows, offsets
 
 
@@ -81,13 +81,14 @@ class GatedFF(nn.Module):
 
 class MixtureFF(nn.Module):
     """`top` of `experts` squared-ReLU blocks per token, weighted by their softmax scores, and (shared_ff > 0)
-    a shared block scaled by a sigmoid gate.  The gate's row is the router product's last row."""
+    a shared block scaled by a sigmoid gate.  The gate's row follows the experts' in the router product."""
 
     def __init__(self, width, experts, top, ff, shared_ff, dtype, device):
         super().__init__()
         self.experts, self.top, self.shared = experts, top, shared_ff > 0
         e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
-        self.router = e(experts + int(self.shared), width)
+        # rows: experts, the gate, zeros up to a multiple of 8 (aligned rows of logits)
+        self.router = e((experts + int(self.shared) + 7) // 8 * 8, width)
         self.up, self.down = e(experts, ff, width), e(experts, width, ff)
         if self.shared:
             self.shared_up, self.shared_down = e(shared_ff, width), e(width, shared_ff)
@@ -96,9 +97,10 @@ class MixtureFF(nn.Module):
         for i in range(self.experts):
             self.up[i].copy_(get(f"e{i}.up"))
             self.down[i].copy_(get(f"e{i}.down"))
+        self.router.zero_()
         self.router[:self.experts].copy_(get("router"))
         if self.shared:
-            self.router[self.experts:].copy_(get("shared.sg"))
+            self.router[self.experts:self.experts + 1].copy_(get("shared.sg"))
             self.shared_up.copy_(get("shared.up"))
             self.shared_down.copy_(get("shared.down"))
 

@@ -162,7 +162,9 @@ class LatentAttentionMixer(nn.Module):
             latent = ctx.scratch[id(self.cache)] = gather_rows(self.cache, ctx.block_tables[nd:], ctx.cu_seqlens_k, ctx.total_k)
         kv = project(latent[:, :self.kv_rank], self.kv_up)
         latent_rotate_q(q, positions, self.turns, self.heads, self.dim, self.rot)
-        latent_prefill(q, kv, latent, ctx.cu_seqlens_q[nd:] - nd if nd else ctx.cu_seqlens_q, ctx.cu_seqlens_k, ctx.max_seqlen_q, out,
+        if "cu_q" not in ctx.scratch:                   # rows counted from the first portion's
+            ctx.scratch["cu_q"] = ctx.cu_seqlens_q[nd:] - nd if nd else ctx.cu_seqlens_q
+        latent_prefill(q, kv, latent, ctx.scratch["cu_q"], ctx.cu_seqlens_k, ctx.max_seqlen_q, out,
                        self.heads, self.dim, self.rot, self.vdim, self.kv_rank, self.scale)
 
     def _direct(self, q, positions, out, ctx, nd, portions):
