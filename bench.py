@@ -1303,20 +1303,22 @@ def dobedra_kernel_records(args, dev, peaks):
     rec("latent prefill attention", lambda: LA.latent_prefill(ql, kv, lat, cu, cu, S, out, H, dim, rot, vdim, KR, (dim + rot) ** -0.5),
         2.0 * T * (H * (2 * dim + rot + 2 * vdim) + rot), 2.0 * (dim + rot + vdim) * H * pairs, "qwen3 prefill attention")
     del q, k, v, kv
-    # decode: 256 sequences (Qwen3) and 128 (a latent row serves every head: fewer bytes per sequence)
+    # decode
     n, NB = 256, 9
     ctx = NB * 256 - 7
     lens = i32(torch.full((n,), ctx))
     qd, kq, vq = rnd(n, 1, HQ, D), rnd(n * NB, 256, HKV, D), rnd(n * NB, 256, HKV, D)
     bt = i32(torch.randperm(n * NB).view(n, NB))
-    rec("qwen3 paged decode", lambda: A.paged_decode_attention(qd, kq, vq, lens, bt), n * ctx * HKV * D * 4.0)
+    for seqs in (256, 64):
+        rec(f"qwen3 paged decode, {seqs} sequences", lambda: A.paged_decode_attention(qd[:seqs], kq, vq, lens[:seqs], bt[:seqs]),
+            seqs * ctx * HKV * D * 4.0)
     del kq, vq
     cache = rnd(n * NB, 256, 1, KP)
-    for seqs, heads in ((256, 16), (256, 32), (64, 32), (256, 128)):
+    for seqs, heads in ((256, 16), (256, 32), (64, 16), (64, 32)):
         qa, oa = rnd(seqs, heads, KP), torch.empty(seqs, heads, KR, dtype=bf, device=dev)
         rec(f"latent decode attention, {heads} heads, {seqs} sequences",
             lambda: LA.latent_attention(qa, cache, lens[:seqs], bt[:seqs], KR, 0.07, out=oa),
-            seqs * (ctx * KP + heads * (KP + KR)) * 2.0, 2.0 * seqs * heads * ctx * (KP + KR), "qwen3 paged decode")
+            seqs * (ctx * KP + heads * (KP + KR)) * 2.0, 2.0 * seqs * heads * ctx * (KP + KR), f"qwen3 paged decode, {seqs} sequences")
     # row ops
     xr, wr, res = rnd(T, W), torch.ones(W, dtype=bf, device=dev), rnd(T, W)
     rec("qwen3 add + rms norm", lambda: P.rms_norm(xr, wr, 1e-6, res), 8.0 * T * W)

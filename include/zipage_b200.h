@@ -427,7 +427,7 @@ int zp_store_kv_padded(const void* k, const void* v, void* k_cache, void* v_cach
  * score = q . k * scale; softcap > 0: score = softcap * tanh(score / softcap); the query at position p
  * sees the keys j with 0 <= p - j < window (window 0: all j <= p).
  * q [rows, Hq, D] (row stride), caches [n_pages, BS, Hkv, KP | VP] as zp_store_kv_padded leaves them,
- * KP and VP multiples of 16, BS a multiple of 64, block_table [B, NBmax].  cu_seqlens_q [B + 1] (absolute
+ * KP and VP multiples of 16 (DV <= 1024), BS a multiple of 64, block_table [B, NBmax].  cu_seqlens_q [B + 1] (absolute
  * rows of q and out; max_seqlen_q is their largest count) or NULL for one row per sequence;
  * context_lens [B] counts each sequence's keys including this step's (0: padding row, skipped).
  * 16-bit caches with KP, VP <= 256 and Hq / Hkv <= 16 take the tensor-core kernels (ZP_IMPL_SIMT: never), whose
@@ -505,7 +505,7 @@ int zp_latent_rotate_q(void* q, int64_t row_stride, const int64_t* positions, co
 /* Softmax attention of queries that meet cached latents directly: score = q . cache row * scale (KP entries, both
  * paddings zero), value = the row's first R entries, the query at position p sees every key j <= p.
  * q [rows, H, KP], cache [n_pages, BS, KP], out [rows, H, R] contiguous; rows, positions and contexts as in
- * zp_window_attention (total_rows: rows of q).  KP a multiple of 16, R <= 512.  bf16 with KP <= 640 takes the tcgen05
+ * zp_window_attention (total_rows: rows of q).  KP a multiple of 16, R <= 1024.  bf16 with KP <= 640 and R <= 512 takes the tcgen05
  * kernel (ZP_IMPL_SIMT: never; ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED), which may need a workspace
  * (span = NBmax * BS, max_seqlen_q = 1 without cu_seqlens_q).  Scores and softmax weights are fp32. */
 size_t zp_latent_attention_workspace_bytes(int total_rows, int B, int max_seqlen_q, int H, int R, int span);

@@ -119,6 +119,17 @@ def test_decode_over_latents_long_spans_and_moving_references():
         _close(got, want, torch.bfloat16)
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_rows_too_long_for_the_tensor_core_kernel(dtype):
+    from zipage_b200._lib import ZipageError
+    from zipage_b200.layers.latent_attention import latent_attention
+    cache, table, q, want, scale = _latent_case(3, 900, 40, [130, 7], [1, 1], dtype, seed=4)
+    args = _dev(q), _dev(cache), _dev(torch.tensor([130, 7], dtype=torch.int32)), _dev(table), 900, scale
+    _close(latent_attention(*args), want, dtype)
+    with pytest.raises(ZipageError):
+        latent_attention(*args, impl="tcgen05")
+
+
 @pytest.mark.parametrize("place", [0, 63, 64, 447, 448, 500])
 def test_one_far_key_decides(place):
     """A key whose score stands out by 30: the output is its value, wherever it lies and however the span is cut."""

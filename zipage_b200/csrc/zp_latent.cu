@@ -185,7 +185,7 @@ extern "C" int zp_latent_attention(const void* q, const void* cache, const int32
                                    size_t workspace_bytes, void* stream) {
   if (B == 0 || (cu_seqlens_q && max_seqlen_q == 0)) return ZP_OK;
   ZP_REQUIRE(q && cache && context_lens && block_table && out, "zp_latent_attention: null pointer");
-  ZP_REQUIRE(H > 0 && R > 0 && R <= 512 && R <= KP && KP % 16 == 0 && KP <= 2048, "zp_latent_attention: %d of %d entries", R, KP);
+  ZP_REQUIRE(H > 0 && R > 0 && R <= 1024 && R <= KP && KP % 16 == 0 && KP <= 2048, "zp_latent_attention: %d of %d entries", R, KP);
   ZP_REQUIRE(BS > 0 && BS % 64 == 0 && NBmax > 0 && n_pages > 0 && B <= 65535 && total_rows > 0, "zp_latent_attention: bad sizes");
   const int max_q = cu_seqlens_q ? max_seqlen_q : 1;
   zp::LatentArgs a;

@@ -100,7 +100,7 @@ __device__ __forceinline__ bool ld_meet_any(bool v) {
 struct LdParams {
   LatentArgs a;
   int nb, nc, nv, stages;     // 64-entry blocks of a row; 128-entry chunks; chunks that hold values; stages
-  int pairs;                  // a row is whole blocks, and a chunk is one load
+  int pairs;                  // a row is whole blocks, and a chunk (the queries) is one load
   int* error_word;
 };
 
@@ -156,7 +156,9 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       prefetch_tensormap(&tmQ);
       prefetch_tensormap(&tmC);
       mbar_arrive_expect_tx(&sh.qfull, (uint32_t)(p.nb * NC * 128));
-      for (int k = 0; k < p.nb; ++k) tma_load_5d(qbuf + k * NC * 128, &tmQ, &sh.qfull, k * 64, (int)flat0, 0, 0, 0);
+      if (p.pairs) tma_load_5d(qbuf, &tmQ, &sh.qfull, 0, (int)flat0, 0, 0, 0);
+      else
+        for (int k = 0; k < p.nb; ++k) tma_load_5d(qbuf + k * NC * 128, &tmQ, &sh.qfull, k * 64, (int)flat0, 0, 0, 0);
       bool ok = true;
       int s = 0, parity = 1;
       unsigned char* dst = stage0;
@@ -353,8 +355,16 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     }
     if (ok && n > 0) ok = ld_wait(&sh.obar, 0, abortp, p.error_word, 911);
     ld_meet_any(false);
+    // O^T to rows in shared memory (the stages are free), then whole rows to global memory
     if (ok) {
       fence_after_sync();
+      const bool whole = a.nsplit == 1;
+      float inv[CW];
+#pragma unroll
+      for (int i = 0; i < CW; ++i) {
+        const float s = sh.lsum[0][ch * CW + i] + sh.lsum[1][ch * CW + i];
+        inv[i] = whole ? (s > 0.f ? 1.f / s : 0.f) : 1.f;
+      }
       for (int m = 0; m < p.nv; ++m) {
         float o[CW], o2[CW];
         if (n > 0) {
@@ -366,18 +376,27 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (d < a.R) {
 #pragma unroll
           for (int i = 0; i < CW; ++i) {
-            const int c = ch * CW + i;
-            if (c < ncol) {
-              const float v = n > 0 ? o[i] + o2[i] : 0.f;
-              if (a.nsplit == 1) {
-                const float s = sh.lsum[0][c] + sh.lsum[1][c];
-                reinterpret_cast<__nv_bfloat16*>(a.out)[(flat0 + c) * a.R + d] = __float2bfloat16_rn(s > 0.f ? v / s : 0.f);
-              } else {
-                a.part[((flat0 + c) * a.nsplit + split) * a.R + d] = v;
-              }
-            }
+            const float v = n > 0 ? (o[i] + o2[i]) * inv[i] : 0.f;
+            const int at = (ch * CW + i) * a.R + d;
+            if (whole) reinterpret_cast<__nv_bfloat16*>(stage0)[at] = __float2bfloat16_rn(v);
+            else reinterpret_cast<float*>(stage0)[at] = v;
           }
         }
+      }
+    }
+    ld_meet_any(false);
+    if (ok) {
+      const int row = a.R * (a.nsplit == 1 ? 2 : 4);      // bytes
+      char* dst = a.nsplit == 1 ? reinterpret_cast<char*>(a.out) + flat0 * row
+                                : reinterpret_cast<char*>(a.part) + (flat0 * a.nsplit + split) * row;
+      const int64_t step = (int64_t)row * a.nsplit;       // between the columns' rows
+      if (row % 16 == 0) {
+        const int per = row / 16;
+        for (int i = tid; i < ncol * per; i += 256) st16(dst + (i / per) * step + (i % per) * 16, ld16(stage0 + i * 16));
+      } else {
+        const int per = row / 2;
+        for (int i = tid; i < ncol * per; i += 256)
+          *reinterpret_cast<uint16_t*>(dst + (i / per) * step + (i % per) * 2) = *reinterpret_cast<const uint16_t*>(stage0 + i * 2);
       }
       if (a.nsplit > 1 && tid < ncol) {
         float* ml = a.part + (int64_t)a.pairs * a.nsplit * a.R + ((flat0 + tid) * a.nsplit + split) * 2;
@@ -475,9 +494,9 @@ template <int NC> static int ld_launch(const LatentArgs& a, int max_q, int total
   CUtensorMap tmQ, tmC;
   const uint64_t pairs = (uint64_t)total_rows * a.H;
   {
-    const uint64_t dims[5] = {(uint64_t)a.KP, pairs, 1, 1, 1};
-    const uint64_t strides[4] = {(uint64_t)a.KP, pairs * a.KP, pairs * a.KP, pairs * a.KP};
-    const uint32_t box[5] = {64, NC, 1, 1, 1};
+    const uint64_t dims[5] = {p.pairs ? 64u : (uint64_t)a.KP, pairs, p.pairs ? (uint64_t)p.nb : 1u, 1, 1};
+    const uint64_t strides[4] = {(uint64_t)a.KP, p.pairs ? 64u : pairs * a.KP, pairs * a.KP, pairs * a.KP};
+    const uint32_t box[5] = {64, NC, p.pairs ? (uint32_t)p.nb : 1u, 1, 1};
     if (int rc = make_tensor_map_5d(&tmQ, UmmaFmt<__nv_bfloat16>::tm, a.q, dims, strides, box, 2)) return rc;
   }
   {

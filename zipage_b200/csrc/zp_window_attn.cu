@@ -114,7 +114,8 @@ static int launch_simt(const WinArgs& a, int max_q, cudaStream_t st) {
   if (a.DV <= 64) window_attn_simt_kernel<T, 2><<<grid, WS_WARPS * 32, smem, st>>>(a);
   else if (a.DV <= 128) window_attn_simt_kernel<T, 4><<<grid, WS_WARPS * 32, smem, st>>>(a);
   else if (a.DV <= 256) window_attn_simt_kernel<T, 8><<<grid, WS_WARPS * 32, smem, st>>>(a);
-  else window_attn_simt_kernel<T, 16><<<grid, WS_WARPS * 32, smem, st>>>(a);
+  else if (a.DV <= 512) window_attn_simt_kernel<T, 16><<<grid, WS_WARPS * 32, smem, st>>>(a);
+  else window_attn_simt_kernel<T, 32><<<grid, WS_WARPS * 32, smem, st>>>(a);
   return check_launch("zp_window_attention");
 }
 
@@ -161,7 +162,7 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
   ZP_REQUIRE(q && k_cache && v_cache && context_lens && block_table && out, "zp_window_attention: null pointer");
   ZP_REQUIRE(Hkv > 0 && Hq % Hkv == 0, "zp_window_attention: Hq must be a multiple of Hkv");
   ZP_REQUIRE(BS > 0 && BS % 64 == 0, "zp_window_attention: page size must be a multiple of 64");
-  ZP_REQUIRE(D > 0 && D <= KP && DV > 0 && DV <= VP && KP % 16 == 0 && VP % 16 == 0 && DV <= 512 && VP <= 2048 && KP <= 2048,
+  ZP_REQUIRE(D > 0 && D <= KP && DV > 0 && DV <= VP && KP % 16 == 0 && VP % 16 == 0 && DV <= 1024 && VP <= 2048 && KP <= 2048,
              "zp_window_attention: head sizes %d / %d (padded %d / %d) not supported", D, DV, KP, VP);
   ZP_REQUIRE(NBmax > 0 && n_pages > 0 && B <= 65535, "zp_window_attention: bad sizes");
   ZP_REQUIRE(((uintptr_t)k_cache | (uintptr_t)v_cache) % 16 == 0, "zp_window_attention: caches must be 16-byte aligned");

@@ -16,6 +16,7 @@ from ..engine.cache import LatentSpec
 from ..layers.feed_forward import GatedFF, MixtureFF
 from ..layers.latent_attention import LatentAttentionMixer
 from ..layers.row_ops import embed_position, join_norms
+from ..utils.context import get_context
 
 
 @dataclass(frozen=True)
@@ -56,7 +57,7 @@ class DobedraConfig:
 
 
 class DobedraLayer(nn.Module):
-    def __init__(self, c: DobedraConfig, lc: LayerConfig, dtype, device):
+    def __init__(self, c: DobedraConfig, lc: LayerConfig, dtype, device, side=None):
         super().__init__()
         m, f = lc.mixer, lc.mlp
         self.kv_from = m.get("kv_from")
@@ -70,6 +71,7 @@ class DobedraLayer(nn.Module):
             self.ff = MixtureFF(c.width, f["router"]["experts"], f["router"]["top"], f["expert"]["ff"],
                                 (f.get("shared") or {}).get("ff", 0), dtype, device)
         v = lambda: nn.Parameter(torch.empty(c.width, dtype=torch.float32, device=device), requires_grad=False)
+        self.side = side
         self.norm1, self.bias1, self.scale1 = v(), v(), v()
         self.norm2, self.bias2, self.scale2 = (v(), v(), v()) if self.ff is not None else (None, None, None)
 
@@ -91,6 +93,16 @@ class DobedraLayer(nn.Module):
     def forward(self, h, positions):
         """h: the outputs of `norms`.  -> this layer's summands, as `join_norms` takes them."""
         parts = {"ls_a": self.scale1, "ls_b": self.scale2}
+        if self.ff is not None and self.side is not None and not get_context().is_prefill:
+            # a decode step's launches are short: the two sublayers run side by side (the next layer's fork waits for
+            # this layer's boundary, so memory that crosses the streams is not reused before its last reader)
+            main = torch.cuda.current_stream()
+            self.side.wait_stream(main)
+            with torch.cuda.stream(self.side):
+                parts.update(self.ff(h[1]))
+            parts["a"] = self.mixer(h[0], positions)
+            main.wait_stream(self.side)
+            return parts
         if self.ff is not None:
             parts.update(self.ff(h[1]))
         parts["a"] = self.mixer(h[0], positions)
@@ -105,7 +117,8 @@ class DobedraModel(nn.Module):
         self.config, self.dtype, self.logit_softcap = c, dtype, c.softcap
         e = lambda *s, dt=dtype: nn.Parameter(torch.empty(*s, dtype=dt, device=device), requires_grad=False)
         self.embed = e(c.vocab, c.width)
-        self.layers = nn.ModuleList([DobedraLayer(c, lc, dtype, device) for lc in c.layers])
+        side = torch.cuda.Stream(device) if device.type == "cuda" else None
+        self.layers = nn.ModuleList([DobedraLayer(c, lc, dtype, device, side) for lc in c.layers])
         self.norm, self.norm_bias = e(c.width, dt=torch.float32), e(c.width, dt=torch.float32)
         self.head = e(c.vocab, c.width)
         self.trail = None      # optional list: the residual stream after every layer
