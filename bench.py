@@ -1059,15 +1059,26 @@ class KernelTable:
         self.args, self.recs, self.launches = args, {}, 0
         self.hbm, self.tf = peaks.get("hbm_gbs", 6650.0) * 1e9, peaks.get("bf16_tflops", 1590.0) * 1e12
 
-    def __call__(self, name, fn, nbytes, flops=0.0, like=None):
+    def __call__(self, name, fn, nbytes, flops=0.0, like=None, graph=False):
+        """graph: the calls as one replayed graph, for kernels shorter than a call's host time."""
         import torch
+
+        def run():
+            for _ in range(self.args.steps):
+                fn()
         for _ in range(self.args.warmup):
             fn()
         torch.cuda.synchronize()
+        if graph:
+            g = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(g):
+                run()
+            run = g.replay
+            run()
+            torch.cuda.synchronize()
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         e0.record()
-        for _ in range(self.args.steps):
-            fn()
+        run()
         e1.record()
         torch.cuda.synchronize()
         ms = e0.elapsed_time(e1) / self.args.steps
@@ -1357,7 +1368,7 @@ def dobedra_kernel_records(args, dev, peaks):
                                                         58 * 2260), 4.0 * 58 * 2260 * KP, 0.0, like)
     # experts
     zl = rnd(T, E + 1, dt=torch.float32)
-    rec("routing", lambda: F.moe_route(zl, E, top), 4.0 * T * (E + 1) + T * top * 20.0)
+    rec("routing, prompts", lambda: F.moe_route(zl, E, top), 4.0 * T * (E + 1) + T * top * 20.0, graph=True)
     dn = rnd(T, W)
     wd = rnd(6 * 1024, W)
     rec("cuBLAS product of a dense feed-forward", lambda: torch.mm(dn, wd.t()), 2.0 * (T * W + wd.numel() + T * wd.shape[0]),
@@ -1389,7 +1400,7 @@ def dobedra_kernel_records(args, dev, peaks):
         F.grouped_gemm(mid[:t * top], sets[turn[0]].view(E, W, ff), off2, t * top)
     rec("experts up, 64 tokens", decode_up, 2.0 * (used * ff * W + t * W + t * top * ff), 0.0, like)
     rec("experts down, 64 tokens", decode_down, 2.0 * (used * ff * W + t * top * (W + ff)), 0.0, like)
-    rec("routing, 64 tokens", lambda: F.moe_route(zl[:t], E, top), 4.0 * t * (E + 1) + t * top * 20.0)
+    rec("routing, 64 tokens", lambda: F.moe_route(zl[:t], E, top), 4.0 * t * (E + 1) + t * top * 20.0, graph=True)
     return rec.recs, rec.launches
 
 
