@@ -2,7 +2,7 @@
 
 Written for clarity, not speed: keys and values of every head spelled out, dense masks, one expert at a
 time, no cache.  Everything is computed in the dtype of the inputs (float64 unless a caller asks
-otherwise), so a comparison shows the error of the kernels and not of the checker.  Shares no code with
+otherwise), so a comparison shows the error of the kernels and not of this file.  Shares no code with
 the product path.
 """
 from __future__ import annotations

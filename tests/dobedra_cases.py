@@ -40,7 +40,7 @@ CONFIGS = {
                                 layer(1, 80, 16, 120, 40, 96, dense(48), kv_from=1),
                                 layer(3, 56, 32, 64, 32, 120, moe(6, 2, 48), kv_from=0, base=1e6),
                                 layer(9, 32, 16, 24, 48, 96, None, kv_from=1)], width=104, vocab=97, eps=1e-2, softcap=5.0),
-    "large_heads": config([layer(20, 128, 64, 128, 96, 256, moe(12, 2, 72, 128)),
+    "large_heads": config([layer(20, 128, 64, 128, 96, 256, moe(11, 2, 72, 128)),
                            layer(40, 64, 64, 96, 64, 256, dense(128), kv_from=0)], width=192, vocab=90, softcap=30.0),
     # sizes that are not multiples of eight: kernels for any size
     "odd_sizes": config([layer(3, 13, 6, 11, 21, 19, moe(5, 2, 27, 13)), layer(2, 9, 6, 15, 17, 19, dense(23), kv_from=0),

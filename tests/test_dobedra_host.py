@@ -1,4 +1,4 @@
-"""Dobedra without a GPU: configuration, registry, what the layers keep, and the checker's own consistency."""
+"""Dobedra without a GPU: configuration, registry, what the layers keep, and the oracle's own consistency."""
 import json
 
 import pytest
@@ -89,7 +89,7 @@ def test_argument_errors_come_back_as_errors():
 
 
 def test_oracle_moving_the_key_product_to_the_queries_changes_nothing():
-    """The attention over expanded keys equals the one over latents (the checker's two readings agree)."""
+    """The attention over expanded keys equals the one over latents (two readings of the same mechanism)."""
     g = torch.Generator().manual_seed(0)
     r = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
     T, H, R, dim, rot, vd = 9, 3, 8, 5, 4, 6

@@ -72,7 +72,7 @@ def _latent_case(H, R, rot, ctxs, counts, dtype, seed=0, qk=1.0, steep=0.0, BS=6
     return cache, table, torch.cat(qs), torch.cat(want), scale
 
 
-SIZES = [(6, 64, 16), (1, 48, 16), (16, 128, 8), (20, 160, 24), (40, 512, 64), (3, 96, 30), (5, 512, 0), (130, 64, 4)]
+SIZES = [(7, 64, 16), (1, 48, 16), (16, 128, 8), (20, 160, 24), (40, 512, 64), (3, 96, 30), (5, 512, 0), (130, 64, 4)]
 
 
 @pytest.mark.parametrize("impl", ["simt", "tcgen05"])
@@ -151,7 +151,7 @@ def test_one_far_key_decides(place):
 def test_rows_past_the_context_do_not_count():
     """What a page holds after the sequence's last key is another request's, here NaN."""
     from zipage_b200.layers.latent_attention import latent_attention
-    cache, table, q, want, scale = _latent_case(6, 64, 16, [70], [1], torch.bfloat16, seed=5)
+    cache, table, q, want, scale = _latent_case(7, 64, 24, [70], [1], torch.bfloat16, seed=5)
     cache[table[0, 1].item(), 6:] = float("nan")
     got = latent_attention(_dev(q), _dev(cache), _dev(torch.tensor([70], dtype=torch.int32)), _dev(table), 64, scale, impl="tcgen05")
     _check_device()
@@ -159,7 +159,7 @@ def test_rows_past_the_context_do_not_count():
 
 
 # -- expanded keys and values ----------------------------------------------------------------------------
-@pytest.mark.parametrize("H,dim,rot,vdim,R", [(6, 64, 16, 64, 64), (2, 128, 64, 128, 512), (3, 48, 8, 32, 96), (4, 96, 32, 120, 128),
+@pytest.mark.parametrize("H,dim,rot,vdim,R", [(7, 64, 16, 56, 72), (2, 128, 64, 128, 512), (3, 48, 8, 32, 96), (4, 96, 32, 120, 128),
                                               (1, 192, 64, 72, 40), (2, 8, 0, 8, 64)])
 def test_prompts_over_expanded_keys(H, dim, rot, vdim, R):
     from zipage_b200.layers.latent_attention import latent_prefill
@@ -190,7 +190,7 @@ def test_prompts_over_expanded_keys(H, dim, rot, vdim, R):
 
 # -- row ops ---------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("q_rank,R,rot", [(40, 64, 16), (33, 21, 6), (256, 512, 64)])
+@pytest.mark.parametrize("q_rank,R,rot", [(40, 72, 16), (33, 21, 6), (256, 512, 64)])
 def test_latent_rows(q_rank, R, rot, dtype):
     from zipage_b200.layers.latent_attention import gather_rows, latent_prepare, latent_rotate_q, rotary_turns
     g = _gen(1)
@@ -246,7 +246,7 @@ def test_angles_stay_exact_far_from_the_start():
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("W", [256, 58, 2052, 8192, 9000])
+@pytest.mark.parametrize("W", [260, 58, 2052, 8192, 9000])
 def test_join_norms(W, dtype):
     from zipage_b200.layers.row_ops import join_norms
     g = _gen(W)
@@ -291,7 +291,7 @@ def test_activations_and_soft_cap(F, dtype):
 
 
 # -- experts -----------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("N,E,top", [(1, 12, 2), (7, 5, 5), (300, 64, 6), (513, 12, 2), (3000, 300, 8), (700, 1, 1), (600, 33, 1)])
+@pytest.mark.parametrize("N,E,top", [(1, 11, 2), (7, 5, 5), (300, 64, 6), (513, 11, 2), (3000, 300, 8), (700, 1, 1), (600, 33, 1)])
 def test_routing(N, E, top):
     from zipage_b200.layers.feed_forward import moe_route
     z = _r(_gen(N), N, E + 3, k=3.0)
@@ -317,7 +317,7 @@ def test_routing_ties_take_the_lower_expert():
 
 
 @pytest.mark.parametrize("impl,dtype", [("simt", torch.float32), ("simt", torch.bfloat16), ("tcgen05", torch.bfloat16)])
-@pytest.mark.parametrize("K,n_out,counts", [(96, 256, [3, 0, 130, 1, 0, 64]), (256, 96, [1] * 40 + [0]), (64, 40, [0, 0, 5]),
+@pytest.mark.parametrize("K,n_out,counts", [(112, 264, [3, 0, 130, 1, 0, 64]), (264, 112, [1] * 40 + [0]), (64, 40, [0, 0, 5]),
                                             (200, 520, [300, 128, 256, 0, 1]), (2048, 128, [2, 129]), (72, 77, [9, 4])])
 def test_grouped_products(K, n_out, counts, impl, dtype):
     from zipage_b200.layers.feed_forward import grouped_gemm
