@@ -50,6 +50,9 @@ extern "C" {
 /* activations applied by a product's epilogue */
 #define ZP_ACT_NONE 0
 #define ZP_ACT_RELU_SQUARED 1
+#define ZP_ACT_SILU_MUL 2
+#define ZP_SCORE_SOFTMAX 0
+#define ZP_SCORE_SIGMOID 1
 
 const char* zp_last_error(void);
 int zp_version(void);
@@ -423,24 +426,28 @@ int zp_store_kv_padded(const void* k, const void* v, void* k_cache, void* v_cach
                        const int32_t* slot_mapping, int n_tokens, int Hkv, int D, int DV, int KP, int VP,
                        int64_t row_stride, int64_t n_slots, int dtype, void* stream);
 
-/* Softmax attention of a step's queries over paged keys, with a sliding window and a soft cap:
+/* Softmax attention of a step's queries over paged keys, with masks, a soft cap, a sink and an output gate:
  * score = q . k * scale; softcap > 0: score = softcap * tanh(score / softcap); the query at position p
- * sees the keys j with 0 <= p - j < window (window 0: all j <= p).
+ * sees the keys j <= p, of these with window > 0 only p - j < window, with chunk > 0 only floor(j / chunk) =
+ * floor(p / chunk).  sink [Hq] (or NULL): the softmax's denominator also has exp(sink[h]).  The result is
+ * multiplied by out_scale and, with gate_mode 1 (2), by sigmoid(gate), gate [rows, Hq] ([rows, Hq * DV]) of T
+ * with its own row stride.
  * q [rows, Hq, D] (row stride), caches [n_pages, BS, Hkv, KP | VP] as zp_store_kv_padded leaves them,
  * KP and VP multiples of 16 (DV <= 1024), BS a multiple of 64, block_table [B, NBmax].  cu_seqlens_q [B + 1] (absolute
  * rows of q and out; max_seqlen_q is their largest count) or NULL for one row per sequence;
  * context_lens [B] counts each sequence's keys including this step's (0: padding row, skipped).
  * 16-bit caches with KP, VP <= 256 and Hq / Hkv <= 16 take the tensor-core kernels (ZP_IMPL_SIMT: never), whose
- * one-row form may need a workspace (zp_window_attention_workspace_bytes, span = min(window, NBmax *
- * BS)).  With total_q (rows of q; 0 = not told), bf16 portions with head sizes of 128 and a soft cap of
- * at most 34 take the tcgen05 kernel (ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED).  Scores and
+ * one-row form may need a workspace (zp_window_attention_workspace_bytes, span = the most keys a row
+ * sees).  With total_q (rows of q; 0 = not told), bf16 portions with head sizes up to 128 (multiples of 8) and no
+ * soft cap or one of at most 69 take the tcgen05 kernel (ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED).  Scores and
  * softmax weights are fp32 in all of them. */
 size_t zp_window_attention_workspace_bytes(int B, int Hq, int Hkv, int VP, int span);
 int zp_window_attention(const void* q, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens_q,
                         const int32_t* context_lens, const int32_t* block_table, void* out, int B,
                         int max_seqlen_q, int NBmax, int Hq, int Hkv, int D, int DV, int KP, int VP, int BS,
                         int n_pages, int64_t q_stride, int64_t out_stride, float scale, float softcap,
-                        int window, int total_q, int impl, int dtype, void* workspace, size_t workspace_bytes,
+                        int window, int chunk, const float* sink, const void* gate, int64_t gate_stride, int gate_mode,
+                        float out_scale, int total_q, int impl, int dtype, void* workspace, size_t workspace_bytes,
                         void* stream);
 
 /* One step of a matrix-memory (mLSTM) mixer over a batch of sequences, state to gated output:
@@ -468,14 +475,15 @@ int zp_mlstm(const void* q, const void* k, const void* v, const void* g, const f
 
 /* The boundary between two layers, per fp32 row of x [n_rows, hidden], in place:
  *   x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k weights[k] * y[pos[k]])
- *   out1 = T(layer norm of x * w1 + bias1), out2 likewise  (variance = mean of the squared deviations)
+ *   out1 = T(norm of x * w1 + bias1), out2 likewise  (layer norm: variance = mean of the squared deviations; rms 1: no
+ *   mean taken off)
  * a, b [n_rows, hidden] of T, ls_* [hidden] fp32 (NULL = ones), gate: one fp32 number per row at stride
- * gate_stride (NULL = 1); y [y_rows, hidden] of T with pos, weights [n_rows, top] (top 0: none, at most 64).
+ * gate_stride (NULL = 1); y [y_rows, hidden] of T with pos, weights [n_rows, top] (weights NULL = ones; top 0: none, at most 64).
  * a, b, out1 and out2 may be NULL; with no summand x is only read. */
 int zp_join_norms(float* x, const void* a, const float* ls_a, const void* b, const float* ls_b, const float* gate,
                   int64_t gate_stride, const void* y, int64_t y_rows, const int32_t* pos, const float* weights,
                   int top, const float* w1, const float* bias1, void* out1, const float* w2, const float* bias2,
-                  void* out2, int n_rows, int hidden, float eps, int dtype, void* stream);
+                  void* out2, int n_rows, int hidden, float eps, int rms, int dtype, void* stream);
 
 /* gate | up [n_rows, 2 width] -> T(gelu_tanh(gate) * up) [n_rows, width] */
 int zp_gelu_tanh_and_mul(const void* x, void* out, int n_rows, int width, int dtype, void* stream);
@@ -531,19 +539,63 @@ int zp_gather_rows(const void* cache, const int32_t* block_table, const int32_t*
                    int NBmax, int BS, int n_pages, int row_bytes, int total, void* stream);
 
 /* Routing: logits [n_tokens, n_experts] fp32 (row stride, at most 1024 experts), s = softmax over all
- * experts; the top largest of a token (ties: the lower expert) with weights s, not renormalised.
+ * experts (ZP_SCORE_SOFTMAX) or sigmoid (ZP_SCORE_SIGMOID); the top largest of a token (ties: the lower expert) with weights s, not renormalised.
  * weights, experts, places [n_tokens, top]; the n_tokens * top pairs sorted by expert: expert e has the places
- * offsets[e] .. offsets[e + 1] ([n_experts + 1]), rows[place] = its token.  counts [n_experts]: scratch. */
+ * offsets[e] .. offsets[e + 1] ([n_experts + 1]), rows[place] = its token.  counts [n_experts]: scratch.
+ * place_weights [n_tokens * top] (may be NULL): the weights in the order of the places. */
 int zp_moe_route(const float* logits, int64_t row_stride, int n_tokens, int n_experts, int top, float* weights,
-                 int32_t* experts, int32_t* places, int32_t* rows, int32_t* offsets, int32_t* counts, void* stream);
+                 int32_t* experts, int32_t* places, int32_t* rows, int32_t* offsets, int32_t* counts, float* place_weights,
+                 int score, void* stream);
 
 /* out[p, n] = act(sum_k x[r(p), k] weight[e, n, k]) for the places p of every expert e (offsets as above, at
  * most n_places in all); r(p) = rows[p], or p when rows is NULL.  x [src_rows, k] (row stride), weight
- * [n_experts, n_out, k], out [n_places, n_out]; fp32 accumulation.  bf16 with k and x_stride multiples of 8
+ * [n_experts, n_out, k], out [n_places, n_out]; fp32 accumulation.  ZP_ACT_SILU_MUL: the rows of weight alternate between
+ * 16 gates and 16 ups (n_out a multiple of 32), out [n_places, n_out / 2] = silu(s gate) * (s up) with s = row_scale[p]
+ * (NULL = 1): the product of an input that is scaled by s.  bf16 with k and x_stride multiples of 8
  * takes the tcgen05 kernel (ZP_IMPL_SIMT: never; ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED). */
 int zp_grouped_gemm(const void* x, int64_t x_stride, const int32_t* rows, int src_rows, const void* weight,
-                    const int32_t* offsets, void* out, int n_places, int n_experts, int n_out, int k, int act,
-                    int impl, int dtype, void* stream);
+                    const int32_t* offsets, const float* row_scale, void* out, int n_places, int n_experts, int n_out, int k,
+                    int act, int impl, int dtype, void* stream);
+
+/* ---- Rotary attention with norms and caches, gated delta rule ----------------------------------------
+ * No counterpart in the reference.  The Tukarax decoder runs on these; each takes its constants as parameters. */
+
+/* q [n_tokens, Hq, D] in place, k [n_tokens, Hkv, D] -> rows slot_mapping[i] of k_cache [n_slots, Hkv, KP]: optional RMS norm
+ * per head (q_weight, k_weight [D] fp32, NULL = none), then the pairs of the first dims entries turned by
+ * 2 pi positions[i] turns[t] (turns [dims / 2] fp64 on the device), cosine and sine multiplied by mul.  Pair t: entries
+ * 2t, 2t + 1 (interleaved) or t, t + dims / 2.  v [n_tokens, Hkv, DV] -> v_cache [n_slots, Hkv, VP] as it is; v may be k.
+ * q, k and v have one row stride.  Padding columns are left alone; slots outside [0, n_slots) store nothing. */
+int zp_rotate_store(void* q, const void* k, const void* v, int64_t row_stride, const int64_t* positions,
+                    const double* turns, int dims, int interleaved, float mul, const float* q_weight,
+                    const float* k_weight, float eps, void* k_cache, void* v_cache, const int32_t* slot_mapping,
+                    int n_tokens, int Hq, int Hkv, int D, int DV, int KP, int VP, int64_t n_slots, int dtype,
+                    void* stream);
+
+/* out[t, c] = silu(sum_j weight[taps - 1 - j, c] x[t - j, c]) over the portions of a step: sequence b has the rows
+ * cu_seqlens_q[b] .. of x [rows, channels] (row stride) and out; earlier inputs come from ring [n_slots, taps, channels], where
+ * position p lies in row p % taps, and are zero before position 0.  The portion's last inputs go into the ring.
+ * weight [taps, channels] fp32, at most 8 taps; context_lens counts each sequence's tokens including these. */
+int zp_short_conv(const void* x, int64_t x_stride, const float* weight, void* ring, const int32_t* cu_seqlens_q,
+                  const int32_t* context_lens, const int32_t* slots, void* out, int64_t out_stride, int B,
+                  int max_seqlen_q, int channels, int taps, int n_slots, int dtype, void* stream);
+
+/* One step of a gated delta rule over a batch of sequences, per head h of H with unit keys and queries (q, k / sqrt(sum of
+ * squares + 1e-6)) of head h / (H / G):
+ *   g = exp(-exp(A_log) softplus(a + dt_bias)), b = sigmoid(beta), S <- g S, u = b (v - S^T k), S <- S + k u^T, o = S^T q dim^-0.5
+ *   out = T(o / rms(o) * norm_weight * silu(gate) * out_scale)          (rms over the head's vdim, eps inside)
+ * x [rows, q (G dim) | k (G dim) | v (H vdim)], gate [rows, H vdim], ab [rows, a (H) | beta (H)] fp32, out [rows, H vdim], each with
+ * its own row stride; A_log, dt_bias [H], norm_weight [vdim] fp32; state [n_slots, H, dim, VP] fp32 (VP >= vdim, a
+ * multiple of 4).  cu_seqlens_q, context_lens, slots as in zp_mlstm.  taps > 0 (single rows only): x is the input of the
+ * convolution of zp_short_conv, which is then part of the launch; taps 0: x has been through it.
+ * bf16 portions with head sizes up to 128 (multiples of 8) and at least 8 rows per sequence on average take the chunked tcgen05
+ * kernels (ZP_IMPL_SIMT: never; ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED), which need a workspace. */
+size_t zp_gated_delta_workspace_bytes(int total_rows, int B, int H);
+int zp_gated_delta(const void* x, int64_t x_stride, const void* gate, int64_t gate_stride, const float* ab,
+                   int64_t ab_stride, const float* A_log, const float* dt_bias, const float* norm_weight,
+                   const float* conv_weight, void* ring, int taps, const int32_t* cu_seqlens_q,
+                   const int32_t* context_lens, const int32_t* slots, float* state, void* out, int64_t out_stride,
+                   int B, int H, int G, int dim, int vdim, int VP, int n_slots, float eps, float out_scale,
+                   int total_rows, int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream);
 
 #ifdef __cplusplus
 }

@@ -14,7 +14,9 @@ _PKG = Path(__file__).resolve().parent
 LIB_PATH = _PKG / "libzipage_b200.so"
 
 ZP_DTYPE = {torch.bfloat16: 0, torch.float32: 1, torch.float16: 2}
-ACT = {None: 0, "relu_squared": 1}
+ACT = {None: 0, "relu_squared": 1, "silu_mul": 2}
+SCORE = {"softmax": 0, "sigmoid": 1}
+GATE = {None: 0, "head": 1, "entry": 2}
 IMPL = {"auto": 0, "simt": 1, "tcgen05": 2}
 
 
@@ -83,9 +85,9 @@ SIGNATURES = {
     "zp_gelu_tanh": (_I, [_P, _P, _L, _I, _P]),
     "zp_store_kv_padded": (_I, [_P] * 5 + [_I] * 6 + [_L, _L, _I, _P]),
     "zp_window_attention_workspace_bytes": (_Z, [_I] * 5),
-    "zp_window_attention": (_I, [_P] * 7 + [_I] * 11 + [_L, _L, _F, _F, _I, _I, _I, _I, _P, _Z, _P]),
+    "zp_window_attention": (_I, [_P] * 7 + [_I] * 11 + [_L, _L, _F, _F, _I, _I, _P, _P, _L, _I, _F, _I, _I, _I, _P, _Z, _P]),
     "zp_mlstm": (_I, [_P] * 14 + [_I] * 6 + [_L] * 3 + [_F] * 3 + [_I, _I, _I, _P]),
-    "zp_join_norms": (_I, [_P] * 6 + [_L, _P, _L, _P, _P, _I] + [_P] * 6 + [_I, _I, _F, _I, _P]),
+    "zp_join_norms": (_I, [_P] * 6 + [_L, _P, _L, _P, _P, _I] + [_P] * 6 + [_I, _I, _F, _I, _I, _P]),
     "zp_gelu_tanh_and_mul": (_I, [_P, _P, _I, _I, _I, _P]),
     "zp_relu_squared": (_I, [_P, _P, _L, _I, _P]),
     "zp_soft_cap": (_I, [_P, _L, _F, _P]),
@@ -96,8 +98,12 @@ SIGNATURES = {
     "zp_latent_prefill_supported": (_I, [_I] * 6),
     "zp_latent_prefill": (_I, [_P, _L] + [_P] * 5 + [_L] + [_I] * 10 + [_F, _I, _P]),
     "zp_gather_rows": (_I, [_P] * 4 + [_I] * 6 + [_P]),
-    "zp_moe_route": (_I, [_P, _L, _I, _I, _I] + [_P] * 7),
-    "zp_grouped_gemm": (_I, [_P, _L, _P, _I, _P, _P, _P] + [_I] * 7 + [_P]),
+    "zp_moe_route": (_I, [_P, _L, _I, _I, _I] + [_P] * 7 + [_I, _P]),
+    "zp_grouped_gemm": (_I, [_P, _L, _P, _I, _P, _P, _P, _P] + [_I] * 7 + [_P]),
+    "zp_rotate_store": (_I, [_P, _P, _P, _L, _P, _P, _I, _I, _F, _P, _P, _F, _P, _P, _P] + [_I] * 7 + [_L, _I, _P]),
+    "zp_short_conv": (_I, [_P, _L] + [_P] * 6 + [_L] + [_I] * 6 + [_P]),
+    "zp_gated_delta_workspace_bytes": (_Z, [_I] * 3),
+    "zp_gated_delta": (_I, [_P, _L, _P, _L, _P, _L] + [_P] * 5 + [_I] + [_P] * 5 + [_L] + [_I] * 7 + [_F, _F, _I, _I, _I, _P, _Z, _P]),
     "zp_comm_create": (_I, [_I, _I, _Z, _I, C.POINTER(_P)]),
     "zp_comm_segment": (_I, [_P, C.POINTER(_P), C.POINTER(_Z)]),
     "zp_comm_ipc_handle": (_I, [_P, _P]),

@@ -1,4 +1,4 @@
-// Mixture of experts: routing (softmax scores over all experts, the largest `top` of a token) with the
+// Mixture of experts: routing (softmax scores over all experts or sigmoid scores, the largest `top` of a token) with the
 // bookkeeping that sorts (token, expert) pairs by expert, and matrix products of the sorted rows with their
 // expert's weights.  This file has the routing kernels, the SIMT product for fp32 and odd sizes, and the entry
 // points; zp_moe_tc.cu has the tensor-core product.
@@ -21,7 +21,7 @@ __device__ __forceinline__ unsigned order_key(float v) {
 // expert.  Choice k is returned by lane k % 32 of round k / 32 (emit(k, expert, score) is called by that lane,
 // all lanes of a round at once).
 template <int VPL, typename F>
-__device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, int top, F&& emit) {
+__device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, int top, bool sigmoid, F&& emit) {
   const int lane = threadIdx.x & 31;
   float v[VPL], mx = -INFINITY;
   unsigned key[VPL];                        // 0: taken, or no expert
@@ -56,7 +56,7 @@ __device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, 
       }
       if (lane == k - k0) { mine = (int)at; score = bv; }
     }
-    if (lane < top - k0) emit(k0 + lane, mine, expf(score - mx) / sum);
+    if (lane < top - k0) emit(k0 + lane, mine, sigmoid ? 1.f / (1.f + expf(-score)) : expf(score - mx) / sum);
   }
 }
 
@@ -86,6 +86,8 @@ struct RouteArgs {
   float* wts;          // [N, top]
   int32_t *idx, *pos;  // [N, top]; between the two kernels pos holds ranks within the expert
   int32_t *rows, *offsets, *counts;
+  float* place_wts;    // [N * top] or NULL: the weights in the order of the places
+  int sigmoid;
 };
 
 // One block does everything (ONE; at most RT_ONE pairs), or several blocks choose and count and route_place_kernel places.
@@ -99,7 +101,7 @@ __global__ void __launch_bounds__(ONE ? 1024 : 256) route_kernel(const RouteArgs
   const int nw = blockDim.x >> 5, per = ONE ? a.N : 32;        // tokens of a block
   const int t0 = blockIdx.x * per, t1 = min(a.N, t0 + per);
   for (int t = t0 + (threadIdx.x >> 5); t < t1; t += nw)
-    top_experts<VPL>(a.logits + (int64_t)t * a.ld, a.E, a.top, [&](int k, int e, float s) {
+    top_experts<VPL>(a.logits + (int64_t)t * a.ld, a.E, a.top, a.sigmoid != 0, [&](int k, int e, float s) {
       const int64_t at = (int64_t)t * a.top + k;
       a.wts[at] = s;
       a.idx[at] = e;
@@ -116,6 +118,7 @@ __global__ void __launch_bounds__(ONE ? 1024 : 256) route_kernel(const RouteArgs
       const int p = offs[picks[i].x] + picks[i].y;
       a.pos[i] = p;
       a.rows[p] = i / a.top;
+      if (a.place_wts) a.place_wts[p] = a.wts[i];
     }
   } else {
     for (int e = threadIdx.x; e < a.E; e += blockDim.x) offs[e] = hist[e] ? atomicAdd(&a.counts[e], hist[e]) : 0;
@@ -135,6 +138,7 @@ __global__ void __launch_bounds__(256) route_place_kernel(const RouteArgs a) {
     const int p = offs[a.idx[i]] + a.pos[i];
     a.pos[i] = p;
     a.rows[p] = (int32_t)(i / a.top);
+    if (a.place_wts) a.place_wts[p] = a.wts[i];
   }
 }
 
@@ -200,6 +204,20 @@ template <typename T> __global__ void __launch_bounds__(256) grouped_gemm_simt_k
     }
     __syncthreads();
   }
+  if (a.act == ZP_ACT_SILU_MUL) {      // threads 0-3 of eight hold gates, the other four the matching entries of `up`
+    const int col = (n0 >> 1) + (tx >> 3) * 16 + (tx & 3) * 4;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float f = 4 * ty + i < count && a.row_scale ? a.row_scale[first + 4 * ty + i] : 1.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float up = __shfl_down_sync(0xffffffffu, acc[i][j], 4) * f, g = acc[i][j] * f;
+        if ((tx & 4) == 0 && 4 * ty + i < count && col + j < a.Nout / 2)
+          reinterpret_cast<T*>(a.out)[(int64_t)(first + 4 * ty + i) * (a.Nout / 2) + col + j] = Elem<T>::from_f32(g / (1.f + expf(-g)) * up);
+      }
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -214,12 +232,15 @@ template <typename T> __global__ void __launch_bounds__(256) grouped_gemm_simt_k
 }  // namespace zp
 
 extern "C" int zp_moe_route(const float* logits, int64_t row_stride, int n_tokens, int n_experts, int top, float* weights,
-                            int32_t* experts, int32_t* places, int32_t* rows, int32_t* offsets, int32_t* counts, void* stream) {
+                            int32_t* experts, int32_t* places, int32_t* rows, int32_t* offsets, int32_t* counts, float* place_weights,
+                            int score, void* stream) {
   if (n_tokens == 0) return ZP_OK;
   ZP_REQUIRE(logits && weights && experts && places && rows && offsets && counts, "zp_moe_route: null pointer");
   ZP_REQUIRE(n_experts > 0 && n_experts <= zp::RT_MAXE && top > 0 && top <= n_experts && row_stride >= n_experts,
              "zp_moe_route: %d of %d experts (at most %d)", top, n_experts, zp::RT_MAXE);
-  zp::RouteArgs a{logits, row_stride, n_tokens, n_experts, top, weights, experts, places, rows, offsets, counts};
+  ZP_REQUIRE(score == ZP_SCORE_SOFTMAX || score == ZP_SCORE_SIGMOID, "zp_moe_route: unknown score %d", score);
+  zp::RouteArgs a{logits, row_stride, n_tokens, n_experts, top, weights, experts, places, rows, offsets, counts, place_weights,
+                  score == ZP_SCORE_SIGMOID};
   cudaStream_t st = (cudaStream_t)stream;
   if (n_experts <= 32) return zp::launch_route<1>(a, st);
   if (n_experts <= 64) return zp::launch_route<2>(a, st);
@@ -229,14 +250,16 @@ extern "C" int zp_moe_route(const float* logits, int64_t row_stride, int n_token
 }
 
 extern "C" int zp_grouped_gemm(const void* x, int64_t x_stride, const int32_t* rows, int src_rows, const void* weight,
-                               const int32_t* offsets, void* out, int n_places, int n_experts, int n_out, int k, int act,
-                               int impl, int dtype, void* stream) {
+                               const int32_t* offsets, const float* row_scale, void* out, int n_places, int n_experts, int n_out, int k,
+                               int act, int impl, int dtype, void* stream) {
   if (n_places == 0) return ZP_OK;
   ZP_REQUIRE(x && weight && offsets && out, "zp_grouped_gemm: null pointer");
   ZP_REQUIRE(n_experts > 0 && n_out > 0 && k > 0 && src_rows > 0 && x_stride >= k, "zp_grouped_gemm: bad sizes");
-  ZP_REQUIRE(act == ZP_ACT_NONE || act == ZP_ACT_RELU_SQUARED, "zp_grouped_gemm: unknown activation %d", act);
+  ZP_REQUIRE(act == ZP_ACT_NONE || act == ZP_ACT_RELU_SQUARED || act == ZP_ACT_SILU_MUL, "zp_grouped_gemm: unknown activation %d", act);
+  ZP_REQUIRE(act == ZP_ACT_SILU_MUL ? n_out % 32 == 0 : !row_scale,
+             "zp_grouped_gemm: gated products take blocks of 16 + 16 rows, and only they take row factors");
   ZP_REQUIRE((n_out + zp::GS_T - 1) / zp::GS_T <= 65535, "zp_grouped_gemm: %d outputs", n_out);
-  zp::GroupedArgs a{x, rows, weight, offsets, out, x_stride, src_rows, n_places, n_experts, n_out, k, act};
+  zp::GroupedArgs a{x, rows, weight, offsets, row_scale, out, x_stride, src_rows, n_places, n_experts, n_out, k, act};
   cudaStream_t st = (cudaStream_t)stream;
   const bool tc = zp::grouped_tc_supports(a, dtype);
   if (impl == ZP_IMPL_TCGEN05 && !tc) {

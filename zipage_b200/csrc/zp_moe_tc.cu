@@ -12,6 +12,8 @@
 //   GT_TILE    one 128-row load (rows that already lie in the order of the places);
 //   GT_GATHER  four more warps copy the rows' 16-byte pieces with cp.async (a gather load fetches rows at a
 //              small part of a tile load's rate), publishing a stage two stages later, when its copies have landed.
+#include <type_traits>
+
 #include "zp_moe.cuh"
 #include "zp_tc.cuh"
 
@@ -75,7 +77,7 @@ template <int LEFT> __device__ __forceinline__ void gt_publish(uint64_t* bar, in
 
 template <int MODE> constexpr int gt_threads() { return MODE == GT_GATHER ? 320 : 192; }
 
-template <int BN, bool RELU2, int MODE>
+template <int BN, int ACT, int MODE>
 __global__ void __launch_bounds__(gt_threads<MODE>(), 1)
 grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW, const GtParams p) {
   constexpr int STAGE = GT_A + BN * 128;
@@ -222,6 +224,7 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_con
     const int q = warp & 3, row = q * 32 + lane;
     const uint32_t lane_base = tmem + (static_cast<uint32_t>(q * 32) << 16);
     const bool vec = p.a.Nout % 8 == 0;
+    constexpr bool GATED = ACT == ZP_ACT_SILU_MUL;
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.a.out);
     bool ok = true;
     int i = 0;
@@ -232,12 +235,32 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_con
       if (!ok) break;
       fence_after_sync();
       if (q * 32 < tl.count) {
-        __nv_bfloat16* o = out + (int64_t)(tl.first + row) * p.a.Nout + tl.n0;
+        __nv_bfloat16* o = GATED ? out + (int64_t)(tl.first + row) * (p.a.Nout >> 1) + (tl.n0 >> 1)
+                                 : out + (int64_t)(tl.first + row) * p.a.Nout + tl.n0;
+        const float scale = GATED && p.a.row_scale && row < tl.count ? p.a.row_scale[tl.first + row] : 1.f;
         const int cols = min(BN, p.a.Nout - tl.n0);
         for (int c0 = 0; c0 < cols; c0 += 32) {
           float v[32];
           tmem_ld32(lane_base + acc * BN + c0, v);
-          if (RELU2) {
+          if constexpr (GATED) {             // 16 gates, then the 16 entries of `up` that they meet
+            if (row < tl.count) {
+#pragma unroll
+              for (int c = 0; c < 16; c += 8) {
+                uint32_t w[4];
+#pragma unroll
+                for (int u = 0; u < 8; u += 2) {
+                  const float g0 = v[c + u] * scale, g1 = v[c + u + 1] * scale;
+                  const float y0 = __fdividef(g0, 1.f + __expf(fminf(-g0, 80.f))) * (v[16 + c + u] * scale);
+                  const float y1 = __fdividef(g1, 1.f + __expf(fminf(-g1, 80.f))) * (v[17 + c + u] * scale);
+                  const __nv_bfloat162 x = __floats2bfloat162_rn(y0, y1);
+                  w[u >> 1] = *reinterpret_cast<const uint32_t*>(&x);
+                }
+                st16(o + (c0 >> 1) + c, make_int4((int)w[0], (int)w[1], (int)w[2], (int)w[3]));
+              }
+            }
+            continue;
+          }
+          if (ACT == ZP_ACT_RELU_SQUARED) {
 #pragma unroll
             for (int u = 0; u < 32; ++u) { const float z = fmaxf(v[u], 0.f); v[u] = z * z; }
           }
@@ -279,7 +302,7 @@ bool grouped_tc_supports(const GroupedArgs& a, int dtype) {
          ((uintptr_t)a.x | (uintptr_t)a.w | (uintptr_t)a.out) % 16 == 0;
 }
 
-template <int BN, bool RELU2, int MODE> static int gt_launch(const GroupedArgs& a, cudaStream_t st) {
+template <int BN, int ACT, int MODE> static int gt_launch(const GroupedArgs& a, cudaStream_t st) {
   constexpr int STAGE = GT_A + BN * 128;
   GtParams p;
   p.a = a;
@@ -306,7 +329,7 @@ template <int BN, bool RELU2, int MODE> static int gt_launch(const GroupedArgs& 
     const uint32_t box[5] = {64, BN, 1, 1, 1};
     if (int rc = make_tensor_map_5d(&tmW, UmmaFmt<__nv_bfloat16>::tm, a.w, dims, strides, box, 2)) return rc;
   }
-  const auto kern = grouped_gemm_tc_kernel<BN, RELU2, MODE>;
+  const auto kern = grouped_gemm_tc_kernel<BN, ACT, MODE>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) { set_error("zp_grouped_gemm(tcgen05): %s", cudaGetErrorString(e)); return ZP_ERR_CUDA; }
   const int64_t most = ((int64_t)a.places / 128 + (a.places < a.E ? a.places : a.E)) * p.ntn;   // tiles, at most
@@ -314,16 +337,21 @@ template <int BN, bool RELU2, int MODE> static int gt_launch(const GroupedArgs& 
   return check_launch("zp_grouped_gemm(tcgen05)");
 }
 
-template <int BN, bool RELU2> static int gt_pick(const GroupedArgs& a, bool many, cudaStream_t st) {
-  if (!many) return gt_launch<BN, RELU2, GT_FEW>(a, st);
-  return a.rows ? gt_launch<BN, RELU2, GT_GATHER>(a, st) : gt_launch<BN, RELU2, GT_TILE>(a, st);
+template <int BN, int ACT> static int gt_pick(const GroupedArgs& a, bool many, cudaStream_t st) {
+  if (!many) return gt_launch<BN, ACT, GT_FEW>(a, st);
+  return a.rows ? gt_launch<BN, ACT, GT_GATHER>(a, st) : gt_launch<BN, ACT, GT_TILE>(a, st);
 }
 
 int grouped_gemm_tc(const GroupedArgs& a, cudaStream_t st) {
   // few places per expert: the weights stream through, and narrower tiles spread them better over the SMs
   const bool many = a.places >= 32 * (int64_t)a.E, wide = many && a.Nout > 128;
-  if (a.act == ZP_ACT_RELU_SQUARED) return wide ? gt_pick<256, true>(a, many, st) : gt_pick<128, true>(a, many, st);
-  return wide ? gt_pick<256, false>(a, many, st) : gt_pick<128, false>(a, many, st);
+  auto by_act = [&](auto act) {
+    constexpr int ACT = decltype(act)::value;
+    return wide ? gt_pick<256, ACT>(a, many, st) : gt_pick<128, ACT>(a, many, st);
+  };
+  if (a.act == ZP_ACT_SILU_MUL) return by_act(std::integral_constant<int, ZP_ACT_SILU_MUL>{});
+  if (a.act == ZP_ACT_RELU_SQUARED) return by_act(std::integral_constant<int, ZP_ACT_RELU_SQUARED>{});
+  return by_act(std::integral_constant<int, ZP_ACT_NONE>{});
 }
 
 }  // namespace zp

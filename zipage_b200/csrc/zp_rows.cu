@@ -152,7 +152,8 @@ gelu_tanh_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t n, int64_
 }
 
 // ---------------------------------------------------------------------------------------------
-// x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k w_k y[pos_k]);  out_i = T(layer norm of x with w_i, bias_i).
+// x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k w_k y[pos_k]);  out_i = T(norm of x with w_i, bias_i), the layer
+// norm or (rms) the one that takes no mean off.
 // Every part may be missing.  One block per row; VPT float4 per thread stay in registers (VPT = 0: any
 // row length, each thread reads back the entries of x that it wrote).
 // ---------------------------------------------------------------------------------------------
@@ -164,7 +165,7 @@ struct JoinArgs {
   const float *w1, *bias1, *w2, *bias2;
   void *out1, *out2;
   int64_t gate_stride, y_rows;
-  int top, H;
+  int top, H, rms;
   float eps;
 };
 
@@ -222,7 +223,7 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
   const int64_t row = blockIdx.x;
   if (p.top) {
     for (int k = threadIdx.x; k < p.top; k += blockDim.x) {
-      swts[k] = p.wts[row * p.top + k];
+      swts[k] = p.wts ? p.wts[row * p.top + k] : 1.f;
       spos[k] = (int32_t)min(max((int64_t)p.pos[row * p.top + k], (int64_t)0), p.y_rows - 1);
     }
     __syncthreads();
@@ -253,7 +254,7 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
       }
     }
     if (!norm) return;
-    const float mean = block_sum(s, red) / (float)p.H;
+    const float mean = p.rms ? 0.f : block_sum(s, red) / (float)p.H;
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
@@ -278,7 +279,7 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
       s += v;
     }
     if (!norm) return;
-    const float mean = block_sum(s, red) / (float)p.H;
+    const float mean = p.rms ? 0.f : block_sum(s, red) / (float)p.H;
     float ss = 0.f;
     for (int c = threadIdx.x; c < p.H; c += blockDim.x) { const float d = p.x[row * p.H + c] - mean; ss = fmaf(d, d, ss); }
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)p.H + p.eps);
@@ -383,15 +384,15 @@ extern "C" int zp_join_norms(float* x, const void* a, const float* ls_a, const v
                              const float* gate, int64_t gate_stride, const void* y, int64_t y_rows,
                              const int32_t* pos, const float* wts, int top, const float* w1, const float* bias1,
                              void* out1, const float* w2, const float* bias2, void* out2, int n_rows, int hidden,
-                             float eps, int dtype, void* stream) {
+                             float eps, int rms, int dtype, void* stream) {
   if (n_rows == 0) return ZP_OK;
   ZP_REQUIRE(x, "zp_join_norms: null pointer");
   ZP_REQUIRE(hidden > 0 && top >= 0 && top <= zp::JOIN_TOP, "zp_join_norms: bad sizes (%d experts a token, at most %d)", top, zp::JOIN_TOP);
-  ZP_REQUIRE(top == 0 || (y && pos && wts && y_rows > 0), "zp_join_norms: expert rows without places or weights");
+  ZP_REQUIRE(top == 0 || (y && pos && y_rows > 0), "zp_join_norms: expert rows without places");
   zp::JoinArgs p;
   p.x = x; p.a = a; p.b = b; p.y = top ? y : nullptr; p.ls_a = ls_a; p.ls_b = ls_b; p.gate = gate; p.wts = wts; p.pos = pos;
   p.w1 = w1; p.bias1 = bias1; p.w2 = w2; p.bias2 = bias2; p.out1 = out1; p.out2 = out2; p.gate_stride = gate_stride;
-  p.y_rows = y_rows; p.top = top; p.H = hidden; p.eps = eps;
+  p.y_rows = y_rows; p.top = top; p.H = hidden; p.eps = eps; p.rms = rms;
   const uintptr_t al = (uintptr_t)x | (uintptr_t)a | (uintptr_t)b | (uintptr_t)p.y | (uintptr_t)ls_a | (uintptr_t)ls_b | (uintptr_t)w1 |
                        (uintptr_t)bias1 | (uintptr_t)out1 | (uintptr_t)w2 | (uintptr_t)bias2 | (uintptr_t)out2;
   const bool vec = hidden % 4 == 0 && hidden <= 8192 && al % 16 == 0;

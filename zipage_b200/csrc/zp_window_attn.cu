@@ -99,11 +99,13 @@ __global__ void __launch_bounds__(WS_WARPS * 32) window_attn_simt_kernel(const W
       }
     }
   }
+  if (a.sink) l += expf(a.sink[h] - m);
+  const float f = l > 0.f ? win_head_factor<T>(a, sq_.row0 + r, h) / l : 0.f;
   T* op = reinterpret_cast<T*>(a.out) + (int64_t)(sq_.row0 + r) * a.out_stride + (int64_t)h * a.DV;
 #pragma unroll
   for (int j = 0; j < VPL; ++j) {
     const int d = lane + 32 * j;
-    if (d < a.DV) op[d] = Elem<T>::from_f32(l > 0.f ? o[j] / l : 0.f);
+    if (d < a.DV) op[d] = Elem<T>::from_f32(o[j] * f * win_entry_factor<T>(a, sq_.row0 + r, h, d));
   }
 }
 
@@ -156,7 +158,8 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
                                    const int32_t* cu_seqlens_q, const int32_t* context_lens,
                                    const int32_t* block_table, void* out, int B, int max_seqlen_q, int NBmax,
                                    int Hq, int Hkv, int D, int DV, int KP, int VP, int BS, int n_pages,
-                                   int64_t q_stride, int64_t out_stride, float scale, float softcap, int window,
+                                   int64_t q_stride, int64_t out_stride, float scale, float softcap, int window, int chunk,
+                                   const float* sink, const void* gate, int64_t gate_stride, int gate_mode, float out_scale,
                                    int total_q, int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream) {
   if (B == 0 || (cu_seqlens_q && max_seqlen_q == 0)) return ZP_OK;
   ZP_REQUIRE(q && k_cache && v_cache && context_lens && block_table && out, "zp_window_attention: null pointer");
@@ -166,25 +169,30 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
              "zp_window_attention: head sizes %d / %d (padded %d / %d) not supported", D, DV, KP, VP);
   ZP_REQUIRE(NBmax > 0 && n_pages > 0 && B <= 65535, "zp_window_attention: bad sizes");
   ZP_REQUIRE(((uintptr_t)k_cache | (uintptr_t)v_cache) % 16 == 0, "zp_window_attention: caches must be 16-byte aligned");
+  ZP_REQUIRE(chunk >= 0 && window >= 0 && gate_mode >= 0 && gate_mode <= 2 && (gate_mode == 0 || gate),
+             "zp_window_attention: bad mask or gate");
   zp::WinArgs a;
   a.q = q; a.k = k_cache; a.v = v_cache; a.cu_q = cu_seqlens_q; a.context_lens = context_lens; a.table = block_table;
   a.out = out; a.part = nullptr; a.B = B; a.NBmax = NBmax; a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.DV = DV; a.KP = KP;
   a.VP = VP; a.BS = BS; a.window = window; a.n_pages = n_pages; a.nsplit = 1; a.q_stride = q_stride;
-  a.out_stride = out_stride; a.scale = scale; a.softcap = softcap;
+  a.out_stride = out_stride; a.scale = scale; a.softcap = softcap; a.chunk = chunk; a.sink = sink; a.gate = gate;
+  a.gate_stride = gate_stride; a.gate_mode = gate_mode; a.out_scale = out_scale;
   cudaStream_t st = (cudaStream_t)stream;
   const bool half = dtype == ZP_DTYPE_BF16 || dtype == ZP_DTYPE_F16;
   // portions long enough to fill 128-row query tiles
   const bool tc = cu_seqlens_q && zp::window_tc_supports(a, total_q, dtype);
   if (impl == ZP_IMPL_TCGEN05 && !tc) {
-    zp::set_error("zp_window_attention: the tcgen05 kernel needs bf16 portions, head sizes of 128, 16-byte aligned rows "
-                  "and a soft cap of at most 34");
+    zp::set_error("zp_window_attention: the tcgen05 kernel needs bf16 portions, head sizes that are multiples of 8 up to 128, 16-byte "
+                  "aligned rows and no soft cap or one of at most 69");
     return ZP_ERR_UNSUPPORTED;
   }
-  if (tc && (impl == ZP_IMPL_TCGEN05 || (impl == ZP_IMPL_AUTO && max_seqlen_q >= 96)))
+  if (tc && (impl == ZP_IMPL_TCGEN05 || (impl == ZP_IMPL_AUTO && max_seqlen_q >= 96 && KP + VP > 128)))
     return zp::window_prefill_tc(a, max_seqlen_q, total_q, st);
   if (half && impl != ZP_IMPL_SIMT && zp::window_mma_supports(a)) {
     if (cu_seqlens_q) return zp::window_prefill_mma(a, max_seqlen_q, dtype, st);
-    const int reach = NBmax * BS, span = window > 0 && window < reach ? window : reach;
+    int span = NBmax * BS;
+    if (window > 0 && window < span) span = window;
+    if (chunk > 0 && chunk < span) span = chunk;
     a.nsplit = zp::window_decode_splits(B, Hkv, span);
     if (a.nsplit > 1) {
       const size_t need = (size_t)B * Hq * a.nsplit * (VP + 2) * sizeof(float);

@@ -10,7 +10,8 @@
 // operand (fp32's exponent range) the prefill kernel exponentiates against the bound c itself: no
 // running maximum, no rescaling of the accumulators, and, with E = exp(2 s / c),
 //   c tanh(s / c) - c = -2 c / (1 + E),
-// so a weight costs two exponentials and one reciprocal.
+// so a weight costs two exponentials and one reciprocal.  Caps up to c log2(e) = 100 do the same against 0: weights
+// within 2^-100 .. 2^100.
 #include "zp_mma.cuh"
 #include "zp_window_attn.cuh"
 
@@ -24,12 +25,13 @@ __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32
 __device__ __forceinline__ float rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
 // score in log2 units after scale and cap (c = cap * log2 e, y = 2 scale log2 e / cap)
-struct CapConst { float lin, y, c, cap; };
+struct CapConst { float lin, y, c, cap, ref; };
 __device__ __forceinline__ CapConst cap_const(const WinArgs& a) {
   CapConst k;
   k.lin = a.scale * WM_LOG2E; k.cap = a.softcap;
   k.y = a.softcap > 0.f ? 2.f * WM_LOG2E * a.scale / a.softcap : 0.f;
   k.c = a.softcap * WM_LOG2E;
+  k.ref = 2.f * k.c <= 100.f ? k.c : 0.f;
   return k;
 }
 __device__ __forceinline__ float capped(float s, const CapConst& k, float scale) {
@@ -157,7 +159,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
 #pragma unroll
         for (int nb = 0; nb < 8; ++nb) {
 #pragma unroll
-          for (int j = 0; j < 4; ++j) s[nb][j] = ex2(-2.f * cc.c * rcp(1.f + ex2(s[nb][j] * cc.y)));
+          for (int j = 0; j < 4; ++j) s[nb][j] = ex2(fmaf(-2.f * cc.c, rcp(1.f + ex2(s[nb][j] * cc.y)), cc.c - cc.ref));
           if (!whole) {
             const int key = key0 + nb * 8 + 2 * tq;
             if (key > pos0 || key < lo0) s[nb][0] = 0.f;
@@ -228,13 +230,26 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
   cp_async_wait<0>();
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
+  const int64_t grow = sq.row0 + qi0;
+  if (a.sink) {
+    const float s2 = win_sink2(a, h), r0 = BOUNDED ? cc.ref : m0, r1 = BOUNDED ? cc.ref : m1;
+    l0 += ex2(s2 - r0); l1 += ex2(s2 - r1);
+  }
+  const float i0 = l0 > 0.f && row0 < rows ? win_head_factor<T>(a, grow + row0, h) / l0 : 0.f;
+  const float i1 = l1 > 0.f && row0 + 8 < rows ? win_head_factor<T>(a, grow + row0 + 8, h) / l1 : 0.f;
   T* ob = reinterpret_cast<T*>(a.out) + (int64_t)(sq.row0 + qi0) * a.out_stride + (int64_t)h * a.DV;
   const bool pairs = a.DV % 2 == 0 && a.out_stride % 2 == 0;
 #pragma unroll
   for (int i = 0; i < 2 * NV16; ++i) {
     const int d = i * 8 + 2 * tq;
     if (d >= a.DV) continue;
+    if (a.gate_mode == WIN_GATE_ENTRY) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int r = row0 + (j >> 1) * 8;
+        if (r < rows && d + (j & 1) < a.DV) o[i][j] *= win_entry_factor<T>(a, grow + r, h, d + (j & 1));
+      }
+    }
     if (pairs) {
       if (row0 < rows) *reinterpret_cast<uint32_t*>(ob + row0 * a.out_stride + d) = pack2<T>(o[i][0] * i0, o[i][1] * i0);
       if (row0 + 8 < rows) *reinterpret_cast<uint32_t*>(ob + (row0 + 8) * a.out_stride + d) = pack2<T>(o[i][2] * i1, o[i][3] * i1);
@@ -396,8 +411,10 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
     }
     const int hq = hk * G + row;
     if (a.nsplit == 1) {
+      if (a.sink) den += ex2(win_sink2(a, hq) - M);
+      const float f = win_head_factor<T>(a, sq.row0, hq) * win_entry_factor<T>(a, sq.row0, hq, d);
       reinterpret_cast<T*>(a.out)[(int64_t)sq.row0 * a.out_stride + (int64_t)hq * a.DV + d] =
-          Elem<T>::from_f32(den > 0.f ? num / den : 0.f);
+          Elem<T>::from_f32(den > 0.f ? num / den * f : 0.f);
     } else {
       float* pp = a.part + (((int64_t)b * a.Hq + hq) * a.nsplit + split) * W;
       pp[d] = num;
@@ -423,8 +440,10 @@ __global__ void __launch_bounds__(128) window_decode_merge_kernel(const WinArgs 
       num = fmaf(w, rr[d], num);
       den = fmaf(w, rr[a.VP + 1], den);
     }
+    if (a.sink) den += ex2(win_sink2(a, hq) - M);
+    const float f = win_head_factor<T>(a, sq.row0, hq) * win_entry_factor<T>(a, sq.row0, hq, d);
     reinterpret_cast<T*>(a.out)[(int64_t)sq.row0 * a.out_stride + (int64_t)hq * a.DV + d] =
-        Elem<T>::from_f32(den > 0.f ? num / den : 0.f);
+        Elem<T>::from_f32(den > 0.f ? num / den * f : 0.f);
   }
 }
 
@@ -470,7 +489,7 @@ static int prefill_by_size(const WinArgs& a, int max_q, cudaStream_t st) {
   return launch_prefill<T, 16, BOUNDED>(a, max_q, st);
 }
 int window_prefill_mma(const WinArgs& a, int max_q, int dtype, cudaStream_t st) {
-  const bool bounded = a.softcap > 0.f && 2.f * a.softcap * WM_LOG2E <= 100.f;
+  const bool bounded = a.softcap > 0.f && a.softcap * WM_LOG2E <= 100.f;
   if (dtype == ZP_DTYPE_F16) return prefill_by_size<__half, false>(a, max_q, st);   // (2^-100 does not fit fp16)
   if (bounded) return prefill_by_size<__nv_bfloat16, true>(a, max_q, st);
   return prefill_by_size<__nv_bfloat16, false>(a, max_q, st);

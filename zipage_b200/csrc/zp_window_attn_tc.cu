@@ -1,20 +1,22 @@
-// Sliding-window, soft-capped prefill attention on tcgen05 tensor cores: bf16, key and value size 128,
-// paged caches (page size a multiple of 64).
+// Prefill attention with masks (sliding window, chunks), soft cap, sink and output gate on tcgen05 tensor cores:
+// bf16, key and value sizes up to 128, paged caches (page size a multiple of 64).
 //
-// The soft cap bounds every score, so the softmax is exponentiated against the bound itself (see
-// zp_window_attn_mma.cu): one pass over the visible 128-key tiles, no row maxima, no rescaling of the output
-// accumulator.  Per tile:
+// One pass over the visible 128-key tiles:
 //   S = Q K^T (M = 128 queries, N = 128 keys, K = 128 dims), accumulated in TMEM,
-//   p = exp(cap tanh(S scale / cap) - cap) in fp32, split into two bf16 numbers (hi + lo) in TMEM,
+//   p = exp(score - reference) in fp32, split into two bf16 numbers (hi + lo) in TMEM,
 //   O += P_hi V + P_lo V (V is the B operand as it lies in memory: MN-major), accumulated in TMEM,
-// and out = O / row sum.
+// and out = O / (row sum + sink's term) * gate.  The reference: a soft cap bounds every score, so it is fixed (the
+// cap, or 0; see zp_window_attn_mma.cu) and nothing is ever rescaled; without a cap it is one number per row
+// that moves, and O with it, only when a score exceeds it by more than 2^40, which fp32 sums and bf16 pairs
+// carry without loss, so nearly always in the first tile only.
 //
 // Roles (576 threads, one block per SM): warp 0 = TMA producer and TMEM owner, warp 1 = MMA issuer, warps
 // 2-17 = softmax (thread <-> TMEM lane <-> query row; the four warps of a lane quadrant split a tile's
 // 128 columns).  Shared memory: the Q tile and a ring of five 32 KB K/V stages; TMEM: two S
 // accumulators, O, P_hi and P_lo (all 512 columns).  A tile is two 64-key boxes per 64 dims, so its halves
-// may lie in different pages.  The softmax is bound by the special-function unit: two exponentials and
-// a reciprocal per score; four reciprocals share one instruction, 1/a = bcd / (abcd).
+// may lie in different pages; head sizes below 128 are filled with zeros by TMA.  The capped softmax is bound by the
+// special-function unit: two exponentials and a reciprocal per score; four reciprocals share one instruction,
+// 1/a = bcd / (abcd).
 // Every wait is bounded; after it the block raises the device error word and leaves.
 #include "zp_tc.cuh"
 #include "zp_window_attn.cuh"
@@ -62,9 +64,9 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16
 __device__ __forceinline__ float ex2_(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float rcp_(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
-// four raw products -> exp2(-2c / (1 + exp2(y s))).  The exponent is held at 30: beyond, 1 / (1 + E) is below
+// four raw products -> exp2(-2c / (1 + exp2(y s)) + off).  The exponent is held at 30: beyond, 1 / (1 + E) is below
 // 2^-30 and the weight is 1 to fp32 accuracy, and the product of four stays finite.
-__device__ __forceinline__ void weights4(const uint32_t* s, float y, float m2c, float (&p)[4]) {
+__device__ __forceinline__ void weights4(const uint32_t* s, float y, float m2c, float off, float (&p)[4]) {
   float a[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) a[i] = 1.f + ex2_(fminf(__uint_as_float(s[i]) * y, 30.f));
@@ -73,11 +75,32 @@ __device__ __forceinline__ void weights4(const uint32_t* s, float y, float m2c, 
   const float2 rr = fmul2(make_float2(ab_cd.y, ab_cd.x), make_float2(r, r));      // m2c / ab, m2c / cd
   const float2 lo = fmul2(make_float2(rr.x, rr.x), make_float2(a[1], a[0]));
   const float2 hi = fmul2(make_float2(rr.y, rr.y), make_float2(a[3], a[2]));
-  p[0] = ex2_(lo.x); p[1] = ex2_(lo.y); p[2] = ex2_(hi.x); p[3] = ex2_(hi.y);
+  p[0] = ex2_(lo.x + off); p[1] = ex2_(lo.y + off); p[2] = ex2_(hi.x + off); p[3] = ex2_(hi.y + off);
 }
+
+// meeting of the 128 threads of a lane quadrant (barriers 1-4); true when any of them brings true
+__device__ __forceinline__ bool wt_meet_any(int q, bool v) {
+  uint32_t out;
+  asm volatile(
+      "{\n\t.reg .pred p, r;\n\t"
+      "setp.ne.u32 p, %1, 0;\n\t"
+      "barrier.cta.red.or.pred r, %2, 128, p;\n\t"
+      "selp.u32 %0, 1, 0, r;\n\t}"
+      : "=r"(out) : "r"((uint32_t)v), "r"(q + 1) : "memory");
+  return out != 0;
+}
+__device__ __forceinline__ void wt_st32(uint32_t taddr, const uint32_t (&r)[32]) {
+  uint32_t x[16], y[16];
+#pragma unroll
+  for (int i = 0; i < 16; ++i) { x[i] = r[i]; y[i] = r[16 + i]; }
+  tmem_st16(taddr, x);
+  tmem_st16(taddr + 16, y);
+}
+constexpr float WT_LAZY = 40.f;    // log2 units
 
 struct WtParams { WinArgs a; int* error_word; };
 
+template <bool CAPPED>
 __global__ void __launch_bounds__(WT_THREADS, 1)
 window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                          const __grid_constant__ CUtensorMap tmV, const WtParams p) {
@@ -190,12 +213,101 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const int lo = r < rows ? win_first(a, p_first + r) : 0x7fffffff;
     const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(q * 32) << 16);
     const float log2e = 1.4426950408889634f;
-    const float y = 2.f * log2e * a.scale / a.softcap, m2c = -2.f * a.softcap * log2e;
+    const float y = 2.f * log2e * a.scale / a.softcap, m2c = -2.f * a.softcap * log2e;      // (CAPPED)
+    const float off = -2.f * m2c <= 200.f ? 0.f : -0.5f * m2c;                              // cap minus reference
+    const float sl2 = a.scale * log2e;
     bool ok = true;
     uint32_t ra[32];
-    float l0 = 0.f, l1 = 0.f;
-    for (int j = 0; ok && j < n; ++j) {
+    float l0 = 0.f, l1 = 0.f, ref = CAPPED ? -0.5f * m2c - off : -INFINITY;
+    for (int j = 0; CAPPED ? ok && j < n : j < n; ++j) {
       const int sb = j & 1;
+      if constexpr (!CAPPED) {      // (every thread reaches the meetings, whether or not a wait of its ran out)
+        const int key0 = (t0 + j) * 128 + cq * 32;
+        const bool whole = key0 >= lo && key0 + 31 <= lim;
+        float mx = -INFINITY;
+        if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&sh.sfull[sb], (j >> 1) & 1, abortp, p.error_word, 807));
+        if (ok) {
+          fence_after_sync();
+          tmem_ld32_issue(lane_base + sb * 128 + cq * 32, ra);
+          tmem_ld32_wait(ra);
+          fence_before_sync();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&sh.sempty[sb]);
+          if (!whole) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (key0 + i > lim || key0 + i < lo) ra[i] = 0xff800000u;      // -inf
+          }
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) mx = fmax3(mx, __uint_as_float(ra[i]), __uint_as_float(ra[i + 1]));
+          mx *= sl2;
+        }
+        if (wt_meet_any(q, mx > ref + WT_LAZY)) {           // some row's reference moves
+          sh.stat[cq][r] = mx;
+          wt_meet_any(q, false);
+          const float m = fmaxf(fmaxf(sh.stat[0][r], sh.stat[1][r]), fmaxf(sh.stat[2][r], sh.stat[3][r]));
+          float fac = 1.f;
+          if (m > ref + WT_LAZY) { fac = ex2_(ref - m); ref = m; }
+          l0 *= fac;
+          l1 *= fac;
+          if (j > 0) {
+            if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&sh.pempty, (j & 1) ^ 1, abortp, p.error_word, 812));
+            if (ok) {
+              fence_after_sync();
+              uint32_t o[32];
+              tmem_ld32_issue(lane_base + WT_O + cq * 32, o);
+              tmem_ld32_wait(o);
+#pragma unroll
+              for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * fac);
+              wt_st32(lane_base + WT_O + cq * 32, o);
+              asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+            }
+          }
+          wt_meet_any(q, false);                            // stat may be rewritten
+        }
+        if (ok) {
+          uint32_t hi[16], lw[16];
+          if (__any_sync(0xffffffffu, key0 + 31 >= lo && key0 <= lim)) {
+            const float mref = ref == -INFINITY ? 0.f : ref;   // (a row without keys so far: every weight is exp2(-inf))
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+              const float w0 = ex2_(fmaf(__uint_as_float(ra[i]), sl2, -mref)), w1 = ex2_(fmaf(__uint_as_float(ra[i + 1]), sl2, -mref));
+              l0 += w0;
+              l1 += w1;
+              const __nv_bfloat162 x = __floats2bfloat162_rn(w0, w1);
+              const float2 f = __bfloat1622float2(x);
+              const __nv_bfloat162 z = __floats2bfloat162_rn(w0 - f.x, w1 - f.y);
+              hi[i >> 1] = *reinterpret_cast<const uint32_t*>(&x);
+              lw[i >> 1] = *reinterpret_cast<const uint32_t*>(&z);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) hi[i] = lw[i] = 0u;
+          }
+          // rows of the V tile past the sequence become zeros (0 * garbage could be NaN)
+          const int first = sq.ctx - (t0 + j) * 128;
+          if (first < 128) {
+            const int t = 2 * j + 1, s = t % WT_NRING;
+            ok = __all_sync(0xffffffffu, mbar_wait(&sh.full[s], (t / WT_NRING) & 1, abortp, p.error_word, 808));
+            unsigned char* vt = ring + s * WT_TILE;
+            for (int idx = threadIdx.x - 64; ok && idx < (128 - first) * 16; idx += 512) {
+              const int row = first + (idx >> 4), c = idx & 15;
+              *reinterpret_cast<int4*>(vt + (c >> 3) * WT_BLK + row * 128 + ((c & 7) << 4)) = make_int4(0, 0, 0, 0);
+            }
+          }
+          if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&sh.pempty, (j & 1) ^ 1, abortp, p.error_word, 809));
+          if (ok) {
+            fence_after_sync();
+            tmem_st16(lane_base + WT_PHI + cq * 16, hi);
+            tmem_st16(lane_base + WT_PLO + cq * 16, lw);
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+            if (first < 128) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+          }
+        }
+        fence_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&sh.pfull);
+      } else {
       if (!mbar_wait(&sh.sfull[sb], (j >> 1) & 1, abortp, p.error_word, 807)) { ok = false; break; }
       fence_after_sync();
       tmem_ld32_issue(lane_base + sb * 128 + cq * 32, ra);
@@ -210,7 +322,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
 #pragma unroll
         for (int i = 0; i < 32; i += 4) {
           float w[4];
-          weights4(ra + i, y, m2c, w);
+          weights4(ra + i, y, m2c, off, w);
           if (!whole) {
 #pragma unroll
             for (int u = 0; u < 4; ++u)
@@ -251,6 +363,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&sh.pfull);
+      }
     }
     float l = l0 + l1;
     if (ok) {
@@ -261,14 +374,25 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     }
     if (ok) {
       l = (sh.stat[0][r] + sh.stat[1][r]) + (sh.stat[2][r] + sh.stat[3][r]);
+      if (a.sink) l += ex2_(win_sink2(a, h) - ref);
       fence_after_sync();
       tmem_ld32_issue(lane_base + WT_O + cq * 32, ra);
       tmem_ld32_wait(ra);
       if (r < rows) {
-        const float inv = l > 0.f ? 1.f / l : 0.f;
-        T* o = reinterpret_cast<T*>(a.out) + (int64_t)(sq.row0 + qi0 + r) * a.out_stride + (int64_t)h * 128 + cq * 32;
+        const int64_t row = sq.row0 + qi0 + r;
+        const float inv = l > 0.f ? win_head_factor<T>(a, row, h) / l : 0.f;
+        T* o = reinterpret_cast<T*>(a.out) + row * a.out_stride + (int64_t)h * a.DV + cq * 32;
+        const T* gate = reinterpret_cast<const T*>(a.gate) + row * a.gate_stride + (int64_t)h * a.DV + cq * 32;
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
+          if (cq * 32 + 8 * c >= a.DV) continue;
+          if (a.gate_mode == WIN_GATE_ENTRY) {
+            const int4 graw = ld16(gate + 8 * c);
+            const T* ge = reinterpret_cast<const T*>(&graw);
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              ra[8 * c + i] = __float_as_uint(__uint_as_float(ra[8 * c + i]) * win_sigmoid(__bfloat162float(ge[i])));
+          }
           uint32_t w[4];
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
@@ -291,8 +415,9 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
 
 // whether the kernel can run this call (total_q: rows of q)
 bool window_tc_supports(const WinArgs& a, int total_q, int dtype) {
-  return dtype == ZP_DTYPE_BF16 && a.D == 128 && a.DV == 128 && a.KP == 128 && a.VP == 128 && total_q > 0 &&
-         a.softcap > 0.f && 2.f * a.softcap * 1.4426950408889634f <= 100.f && a.q_stride % 8 == 0 && a.out_stride % 8 == 0 &&
+  return dtype == ZP_DTYPE_BF16 && a.KP <= 128 && a.VP <= 128 && a.D % 8 == 0 && a.DV % 8 == 0 && total_q > 0 &&
+         a.softcap * 1.4426950408889634f <= 100.f && a.q_stride % 8 == 0 && a.out_stride % 8 == 0 &&
+         (a.gate_mode != WIN_GATE_ENTRY || (a.gate_stride % 8 == 0 && (uintptr_t)a.gate % 16 == 0)) &&
          ((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.out) % 16 == 0;
 }
 
@@ -301,21 +426,23 @@ int window_prefill_tc(const WinArgs& a, int max_q, int total_q, cudaStream_t st)
   if (!p.error_word) { set_error("zp_window_attention(tcgen05): no device error word"); return ZP_ERR_CUDA; }
   CUtensorMap tmQ, tmK, tmV;
   {
-    const uint64_t dims[5] = {128, (uint64_t)a.Hq, (uint64_t)total_q, 1, 1};
-    const uint64_t strides[4] = {128, (uint64_t)a.q_stride, (uint64_t)a.q_stride, (uint64_t)a.q_stride};
+    const uint64_t dims[5] = {(uint64_t)a.D, (uint64_t)a.Hq, (uint64_t)total_q, 1, 1};
+    const uint64_t strides[4] = {(uint64_t)a.D, (uint64_t)a.q_stride, (uint64_t)a.q_stride, (uint64_t)a.q_stride};
     const uint32_t box[5] = {64, 1, 128, 1, 1};
     if (int rc = make_tensor_map_5d(&tmQ, UmmaFmt<__nv_bfloat16>::tm, a.q, dims, strides, box, 2)) return rc;
   }
-  const uint64_t page = (uint64_t)a.BS * a.Hkv * 128;
-  const uint64_t dims[5] = {128, (uint64_t)a.Hkv, (uint64_t)a.BS, (uint64_t)a.n_pages, 1};
-  const uint64_t strides[4] = {128, (uint64_t)a.Hkv * 128, page, page};
   const uint32_t box[5] = {64, 1, 64, 1, 1};
-  if (int rc = make_tensor_map_5d(&tmK, UmmaFmt<__nv_bfloat16>::tm, a.k, dims, strides, box, 2)) return rc;
-  if (int rc = make_tensor_map_5d(&tmV, UmmaFmt<__nv_bfloat16>::tm, a.v, dims, strides, box, 2)) return rc;
+  for (int kv = 0; kv < 2; ++kv) {
+    const uint64_t w = kv ? a.VP : a.KP, row = (uint64_t)a.Hkv * w, page = (uint64_t)a.BS * row;
+    const uint64_t dims[5] = {w, (uint64_t)a.Hkv, (uint64_t)a.BS, (uint64_t)a.n_pages, 1};
+    const uint64_t strides[4] = {w, row, page, page};
+    if (int rc = make_tensor_map_5d(kv ? &tmV : &tmK, UmmaFmt<__nv_bfloat16>::tm, kv ? a.v : a.k, dims, strides, box, 2)) return rc;
+  }
   const int smem = (1 + WT_NRING) * WT_TILE + (int)sizeof(WtShared) + 1024;
-  cudaError_t e = cudaFuncSetAttribute(window_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  const auto kern = a.softcap > 0.f ? window_prefill_tc_kernel<true> : window_prefill_tc_kernel<false>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) { set_error("zp_window_attention(tcgen05): %s", cudaGetErrorString(e)); return ZP_ERR_CUDA; }
-  window_prefill_tc_kernel<<<dim3((max_q + 127) / 128, a.Hq, a.B), WT_THREADS, smem, st>>>(tmQ, tmK, tmV, p);
+  kern<<<dim3((max_q + 127) / 128, a.Hq, a.B), WT_THREADS, smem, st>>>(tmQ, tmK, tmV, p);
   return check_launch("zp_window_attention(tcgen05)");
 }
 

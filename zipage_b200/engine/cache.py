@@ -63,6 +63,28 @@ class StateSpec:
         return slots * self.heads * (self.dim * ((self.vdim + 3) // 4 * 4) + self.dim + 1) * 4
 
 
+@dataclass(frozen=True)
+class DeltaSpec:
+    """What a gated delta rule keeps per slot: the fp32 matrix S [heads, dim, vdim padded to 4] and a ring of the last `taps`
+    inputs of its convolution, [taps, channels] in the model's dtype."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+
+    @property
+    def channels(self):
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    def allocate(self, pages, block_size, slots, dtype, device):
+        return (torch.zeros((slots, self.heads, self.dim, (self.vdim + 3) // 4 * 4), dtype=torch.float32, device=device),
+                torch.zeros((slots, self.taps, self.channels), dtype=dtype, device=device))
+
+    def bytes(self, pages, block_size, slots, itemsize):
+        return slots * (self.heads * self.dim * ((self.vdim + 3) // 4 * 4) * 4 + self.taps * self.channels * itemsize)
+
+
 class PagedStateCache:
     def __init__(self, specs, pages, block_size, slots, dtype, device):
         if block_size % 64:

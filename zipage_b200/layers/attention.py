@@ -13,6 +13,7 @@ from torch import nn
 from .. import _lib as L
 from ..kernel import _count, store_kvcache, store_query_cache
 from ..utils.context import get_context
+from .rotary import rotate_store
 
 _ws_cache: dict = {}
 _ws_kept: list = []   # outgrown buffers stay: a captured graph may still name them
@@ -122,13 +123,17 @@ class Attention(nn.Module):
 
 
 def window_attention(q, k_cache, v_cache, context_lens, block_table, num_heads, head_dim, v_dim, scale,
-                     window=0, softcap=0.0, cu_seqlens_q=None, max_seqlen_q=0, out=None, impl="auto"):
-    """Sliding-window, soft-capped attention over paged caches whose rows are padded to multiples of 16
+                     window=0, softcap=0.0, cu_seqlens_q=None, max_seqlen_q=0, out=None, impl="auto", chunk=0, sink=None,
+                     gate=None, gate_mode=None, out_scale=1.0):
+    """Attention with a sliding window or chunks, soft cap, sink [Hq] (fp32) and output gate (`gate_mode` "head": one
+    logit per head, "entry": one per entry of the result) over paged caches whose rows are padded to multiples of 16
     (k_cache [P, BS, Hkv, KP], v_cache [P, BS, Hkv, VP]).  q [rows, Hq * D] may be a column view of a
     projection.  One row per sequence without `cu_seqlens_q`."""
-    L.require_cuda(q, k_cache, v_cache, context_lens, block_table, cu_seqlens_q)
+    L.require_cuda(q, k_cache, v_cache, context_lens, block_table, cu_seqlens_q, sink, gate)
     P, BS, Hkv, KP = k_cache.shape
     VP = v_cache.shape[3]
+    assert sink is None or sink.dtype == torch.float32 and sink.is_contiguous()
+    assert gate is None or gate.dtype == q.dtype and gate.stride(1) == 1
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and q.stride(1) == 1 and block_table.stride(1) == 1
     if out is None:
         out = torch.empty((q.shape[0], num_heads * v_dim), dtype=q.dtype, device=q.device)
@@ -137,14 +142,15 @@ def window_attention(q, k_cache, v_cache, context_lens, block_table, num_heads, 
     lib = L.load()
     ws = None
     if cu_seqlens_q is None:
-        span = min(window, NB * BS) if window else NB * BS
+        span = min([NB * BS] + [n for n in (window, chunk) if n])
         need = lib.zp_window_attention_workspace_bytes(B, num_heads, Hkv, VP, span)
         ws = _workspace(q.device, need) if need else None
     L.check(lib.zp_window_attention(
         L.ptr(q), L.ptr(k_cache), L.ptr(v_cache), L.ptr(cu_seqlens_q), L.ptr(context_lens), L.ptr(block_table),
         L.ptr(out), B, int(max_seqlen_q), NB, num_heads, Hkv, head_dim, v_dim, KP, VP, BS, P, q.stride(0),
-        out.stride(0), float(scale), float(softcap or 0.0), int(window or 0), q.shape[0], L.IMPL[impl],
-        L.dtype_code(q),
+        out.stride(0), float(scale), float(softcap or 0.0), int(window or 0), int(chunk or 0),
+        L.ptr(sink), L.ptr(gate), 0 if gate is None else gate.stride(0), L.GATE[gate_mode], float(out_scale), q.shape[0],
+        L.IMPL[impl], L.dtype_code(q),
         L.ptr(ws), 0 if ws is None else ws.numel(), L.stream_ptr()), "window_attention")
     _count(1)
     return out
@@ -195,3 +201,51 @@ class WindowAttentionMixer(nn.Module):
             window_attention(q, kc, vc, ctx.context_lens[nd:], ctx.block_tables[nd:], *shape,
                              cu_seqlens_q=ctx.cu_seqlens_q[nd:], max_seqlen_q=ctx.max_seqlen_q, out=out)
         return out
+
+
+class RotaryHeads(nn.Module):
+    """The heads of grouped-query attention with rotary positions, from a projection's columns [q | k | v | gate] to
+    outputs; see `HeadsMixer`.  Optional: an RMS norm per head of queries and keys (`qk_norm`), values that are the keys as
+    projected (`shared_kv`: no columns of their own), a soft cap, chunks, a sink per head, an output gate per head or entry."""
+
+    def __init__(self, heads, kv_heads, dim, vdim, scale, rotary, eps, dtype, device, qk_norm=False, shared_kv=False, softcap=0.0,
+                 chunk=0, sink=False, gate=None, out_scale=1.0):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.rotary, self.eps, self.shared_kv, self.softcap, self.chunk = scale, rotary, eps, shared_kv, softcap, chunk
+        self.gate, self.out_scale = gate, out_scale
+        if shared_kv and dim != vdim:
+            raise ValueError(f"keys of {dim} entries as values of {vdim}")
+        self.nk, self.nv = kv_heads * dim, 0 if shared_kv else kv_heads * vdim
+        self.columns = heads * dim + self.nk + self.nv + {None: 0, "head": heads, "entry": heads * vdim}[gate]
+        self.out_columns = heads * vdim
+        e = lambda n: nn.Parameter(torch.empty(n, dtype=torch.float32, device=device), requires_grad=False)
+        self.q_norm, self.k_norm = (e(dim), e(dim)) if qk_norm else (None, None)
+        self.sink = e(heads) if sink else None
+        self.k_cache = self.v_cache = None                # bound by the cache
+
+    def load(self, get):
+        """-> rows of the projection."""
+        if self.q_norm is not None:
+            self.q_norm.copy_(get("q.norm"))
+            self.k_norm.copy_(get("k.norm"))
+        if self.sink is not None:
+            self.sink.copy_(get("sink"))
+        return torch.cat([get(n) for n in ("q", "k") + (() if self.shared_kv else ("v",)) + (("g",) if self.gate else ())], 0)
+
+    def forward(self, y, positions, out):
+        ctx = get_context()
+        nq = self.heads * self.dim
+        q, k = y[:, :nq], y[:, nq:nq + self.nk]
+        v = k if self.shared_kv else y[:, nq + self.nk:nq + self.nk + self.nv]
+        gate = y[:, nq + self.nk + self.nv:self.columns] if self.gate else None
+        rotate_store(q, k, v, positions, self.rotary, self.k_cache, self.v_cache, ctx.slot_mapping, self.dim, self.vdim,
+                     self.q_norm, self.k_norm, self.eps)
+        nd = ctx.decode_rows()
+        shape = (self.heads, self.dim, self.vdim, self.scale, 0, self.softcap)
+        kw = dict(out=out, chunk=self.chunk, sink=self.sink, gate=gate, gate_mode=self.gate, out_scale=self.out_scale)
+        if nd:
+            window_attention(q, self.k_cache, self.v_cache, ctx.context_lens[:nd], ctx.block_tables[:nd], *shape, **kw)
+        if ctx.is_prefill and nd < ctx.context_lens.shape[0]:
+            window_attention(q, self.k_cache, self.v_cache, ctx.context_lens[nd:], ctx.block_tables[nd:], *shape,
+                             cu_seqlens_q=ctx.cu_seqlens_q[nd:], max_seqlen_q=ctx.max_seqlen_q, **kw)

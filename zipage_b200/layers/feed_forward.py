@@ -33,30 +33,33 @@ def relu_squared_(x):
     return x
 
 
-def moe_route(logits, n_experts, top):
+def moe_route(logits, n_experts, top, score="softmax", by_place=False):
     """logits [N, >= n_experts] fp32 -> (weights [N, top] fp32, experts [N, top], places [N, top],
-    rows [N * top], offsets [n_experts + 1]): softmax over all experts, the `top` largest of a token, and
-    the (token, expert) pairs sorted by expert."""
+    rows [N * top], offsets [n_experts + 1]): scores (softmax over all experts, or sigmoid), the `top` largest of a
+    token, and the (token, expert) pairs sorted by expert.  `by_place`: the weights in that order instead, [N * top]."""
     L.require_cuda(logits)
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     N, dev = logits.shape[0], logits.device
     w = torch.empty((N, top), dtype=torch.float32, device=dev)
     ints = torch.empty(3 * N * top + 2 * n_experts + 1, dtype=torch.int32, device=dev)
     experts, places, rows, offsets, counts = ints.split([N * top] * 3 + [n_experts + 1, n_experts])
+    pw = torch.empty(N * top, dtype=torch.float32, device=dev) if by_place else None
     L.check(L.load().zp_moe_route(L.ptr(logits), logits.stride(0), N, n_experts, top, L.ptr(w), L.ptr(experts), L.ptr(places),
-                                  L.ptr(rows), L.ptr(offsets), L.ptr(counts), L.stream_ptr()), "moe_route")
+                                  L.ptr(rows), L.ptr(offsets), L.ptr(counts), L.ptr(pw), L.SCORE[score], L.stream_ptr()), "moe_route")
     _count(1 if N <= 512 and N * top <= 4096 else 2)
-    return w, experts.view(N, top), places.view(N, top), rows, offsets
+    return w if pw is None else pw, experts.view(N, top), places.view(N, top), rows, offsets
 
 
-def grouped_gemm(x, weight, offsets, n_places, rows=None, act=None, impl="auto"):
+def grouped_gemm(x, weight, offsets, n_places, rows=None, act=None, impl="auto", row_scale=None):
     """out[p] = act(x[rows[p]] @ weight[e].T) for the places p of every expert e; x [src, K] (rows None:
-    place p is row p), weight [E, n_out, K]."""
-    L.require_cuda(x, weight, offsets, rows)
+    place p is row p), weight [E, n_out, K].  act "silu_mul": weight as `interleave_gate_up` makes it, out [places, n_out / 2] =
+    silu(s gate) * (s up) with s = row_scale[p]."""
+    L.require_cuda(x, weight, offsets, rows, row_scale)
+    assert row_scale is None or row_scale.dtype == torch.float32 and row_scale.is_contiguous()
     E, n_out, K = weight.shape
     assert x.stride(1) == 1 and weight.is_contiguous() and x.dtype == weight.dtype and x.shape[1] == K
-    out = torch.empty((n_places, n_out), dtype=x.dtype, device=x.device)
-    L.check(L.load().zp_grouped_gemm(L.ptr(x), x.stride(0), L.ptr(rows), x.shape[0], L.ptr(weight), L.ptr(offsets), L.ptr(out),
+    out = torch.empty((n_places, n_out // 2 if act == "silu_mul" else n_out), dtype=x.dtype, device=x.device)
+    L.check(L.load().zp_grouped_gemm(L.ptr(x), x.stride(0), L.ptr(rows), x.shape[0], L.ptr(weight), L.ptr(offsets), L.ptr(row_scale), L.ptr(out),
                                      n_places, E, n_out, K, L.ACT[act], L.IMPL[impl], L.dtype_code(x), L.stream_ptr()),
             "grouped_gemm")
     _count(1)
@@ -114,3 +117,45 @@ class MixtureFF(nn.Module):
             out["b"] = project(relu_squared_(project(h, self.shared_up)), self.shared_down)
             out["gate"] = z[:, self.experts]
         return out
+
+
+def padded_ff(ff):
+    """Width that gated experts of width `ff` are stored with (whole blocks of 16)."""
+    return (ff + 15) // 16 * 16
+
+
+def interleave_gate_up(out, gate, up):
+    """out [2 * padded_ff, width]: blocks of 16 rows of gate and of up in turn, zeros past the last."""
+    ff, blocks = gate.shape[0], out.view(-1, 2, 16, out.shape[1])
+    out.zero_()
+    for i, w in enumerate((gate, up)):
+        whole = ff // 16
+        blocks[:whole, i].copy_(w[:whole * 16].view(whole, 16, -1))
+        if ff % 16:
+            blocks[whole, i, :ff % 16].copy_(w[whole * 16:])
+
+
+class GatedMixtureFF(nn.Module):
+    """`top` of `experts` SiLU-gated blocks per token, W_down (silu(W_gate z) * (W_up z)), each on z = s h with its
+    own score s (sigmoid by default, not renormalised): the score joins the gate and up products' epilogue."""
+
+    def __init__(self, width, experts, top, ff, dtype, device, score="sigmoid"):
+        super().__init__()
+        self.experts, self.top, self.ff, self.score = experts, top, ff, score
+        e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
+        self.router = e((experts + 7) // 8 * 8, width)      # (zero rows up to a multiple of 8: aligned rows of logits)
+        self.gate_up, self.down = e(experts, 2 * padded_ff(ff), width), e(experts, width, padded_ff(ff))
+
+    def load(self, get):
+        self.down.zero_()
+        for i in range(self.experts):
+            interleave_gate_up(self.gate_up[i], get(f"e{i}.gate"), get(f"e{i}.up"))
+            self.down[i, :, :self.ff].copy_(get(f"e{i}.down"))
+        self.router.zero_()
+        self.router[:self.experts].copy_(get("router"))
+
+    def forward(self, h):
+        places = h.shape[0] * self.top
+        w, _, pos, rows, offsets = moe_route(project(h, self.router, fp32=True), self.experts, self.top, self.score, by_place=True)
+        mid = grouped_gemm(h, self.gate_up, offsets, places, rows=rows, act="silu_mul", row_scale=w)
+        return {"y": grouped_gemm(mid, self.down, offsets, places), "pos": pos}

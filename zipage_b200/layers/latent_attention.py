@@ -10,8 +10,6 @@ Two forms of the same attention:
 """
 from __future__ import annotations
 
-import math
-
 import torch
 from torch import nn
 
@@ -19,13 +17,8 @@ from .. import _lib as L
 from ..kernel import _count
 from ..utils.context import get_context
 from .attention import _workspace
+from .rotary import rotary_turns
 from .row_ops import project
-
-
-def rotary_turns(dims, base, device):
-    """Frequencies of the pairs of a rotated vector in turns per position, fp64 [dims / 2]."""
-    i = torch.arange(dims // 2, dtype=torch.float64)
-    return (float(base) ** (-2.0 * i / dims) / (2.0 * math.pi)).to(device)
 
 
 def latent_prepare(y, positions, turns, q_weight, kv_weight, cache, slot_mapping, q_rank, kv_rank, rot, eps, dense=None):

@@ -45,10 +45,10 @@ def rms_norm_f32(x, weight, eps, dtype, offset=0.0):
     return out
 
 
-def join_norms(x, norms, eps, dtype, a=None, ls_a=None, b=None, ls_b=None, gate=None, y=None, pos=None, weights=None):
-    """The boundary between layers with parallel sublayers.  x fp32 [N, width], in place:
-    x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k weights[:, k] * y[pos[:, k]]); then one layer norm of x per
-    (weight, bias) of `norms` (at most two), each as `dtype`."""
+def join_norms(x, norms, eps, dtype, a=None, ls_a=None, b=None, ls_b=None, gate=None, y=None, pos=None, weights=None, rms=False):
+    """The boundary between sublayers.  x fp32 [N, width], in place:
+    x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k weights[:, k] * y[pos[:, k]]) (weights None: ones); then one layer
+    norm (`rms`: RMS norm) of x per (weight, bias) of `norms` (at most two), each as `dtype`."""
     L.require_cuda(x, a, ls_a, b, ls_b, gate, y, pos, weights, *(t for n in norms for t in n))
     assert x.dtype == torch.float32 and x.is_contiguous() and len(norms) <= 2
     assert all(t is None or t.dtype == dtype and t.is_contiguous() for t in (a, b, y))
@@ -58,7 +58,7 @@ def join_norms(x, norms, eps, dtype, a=None, ls_a=None, b=None, ls_b=None, gate=
     L.check(L.load().zp_join_norms(
         L.ptr(x), L.ptr(a), L.ptr(ls_a), L.ptr(b), L.ptr(ls_b), L.ptr(gate), 0 if gate is None else gate.stride(0), L.ptr(y),
         0 if y is None else y.shape[0], L.ptr(pos), L.ptr(weights), 0 if y is None else pos.shape[1], *flat, x.shape[0],
-        x.shape[1], float(eps), L.ZP_DTYPE[dtype], L.stream_ptr()), "join_norms")
+        x.shape[1], float(eps), int(rms), L.ZP_DTYPE[dtype], L.stream_ptr()), "join_norms")
     _count(1)
     return outs
 

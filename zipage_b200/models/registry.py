@@ -83,6 +83,15 @@ def _dobedra(config, weights, dtype, device):
     return LoadedModel("Dobedra", model, model.head, cfg.width, cfg.vocab, dtype, portions=True)
 
 
+@register("Tukarax", part="tukarax")
+def _tukarax(config, weights, dtype, device):
+    from .tukarax import TukaraxConfig, TukaraxModel
+    cfg = TukaraxConfig.from_dict(config)
+    model = TukaraxModel(cfg, dtype, device)
+    model.load_weights(weights)
+    return LoadedModel("Tukarax", model, model.head, cfg.width, cfg.vocab, dtype, portions=True)
+
+
 @register("Qwen3ForCausalLM")
 def _qwen3(config, weights, dtype, device):
     from ..engine.native_engine import full_state_from_hf
