@@ -130,7 +130,7 @@ def interleave_gate_up(out, gate, up):
     out.zero_()
     for i, w in enumerate((gate, up)):
         whole = ff // 16
-        blocks[:whole, i].copy_(w[:whole * 16].view(whole, 16, -1))
+        blocks[:whole, i].copy_(w[:whole * 16].view(whole, 16, w.shape[1]))
         if ff % 16:
             blocks[whole, i, :ff % 16].copy_(w[whole * 16:])
 
