@@ -51,7 +51,7 @@ def parse_args():
                     help="also run the reference ENGINE (baseline/_ref) on a synthetic Qwen3-8B-shaped model, as it "
                          "is and with this library's decode path bound, and report decode tokens/s (adds minutes)")
     ap.add_argument("--also-exact", action="store_true", help="time the exact variant as well")
-    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine", "similorn", "dobedra"],
+    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine", "similorn", "dobedra", "tukarax"],
                     help="compress (default, the headline op), decode (paged decode attention kernel) or "
                          "step_ops (the element-wise ops of a decoder layer step and the sampler) or "
                          "prefill (varlen causal prefill attention, one layer) or decode_step (the decode "
@@ -1464,6 +1464,215 @@ def run_dobedra(args):
     }))
 
 
+def tukarax_kernel_records(args, dev, peaks):
+    """Every kernel of the Tukarax decoder at sizes of an 8B-class model's layers (width 4096; attention 32 / 8 heads of 128; delta
+    rule 32 / 16 heads of 128 x 128, four taps; 64 experts of 1024, six a token; bf16) beside the like kernel of the closest
+    existing path at equal size: Qwen3's, Similorn's matrix memory, Dobedra's experts.  Inputs are larger than L2 wherever the
+    kernel streams."""
+    import torch
+    from zipage_b200.layers import attention as A
+    from zipage_b200.layers import feed_forward as F
+    from zipage_b200.layers import gated_delta as G
+    from zipage_b200.layers import row_ops as R
+    from zipage_b200.layers import step_ops as P
+    from zipage_b200.layers.mlstm import mlstm_step
+    from zipage_b200.layers.rotary import Rotary, rotate_store
+    bf, W = torch.bfloat16, 4096
+    rnd = lambda *s, dt=bf: torch.empty(s, dtype=dt, device=dev).normal_()
+    i32 = lambda t: t.to(torch.int32).to(dev)
+    rec = KernelTable(args, peaks)
+
+    # prompts: 4 x 4096 tokens
+    B, S = 4, 4096
+    T = B * S
+    cu, ctx, pos = i32(torch.arange(0, T + 1, S)), i32(torch.full((B,), S)), torch.arange(S, device=dev).repeat(B)
+    q, k, v = rnd(T, HQ, D), rnd(T, HKV, D), rnd(T, HKV, D)
+    pairs = B * S * S / 2
+    rec("qwen3 prefill attention", lambda: A.varlen_prefill_attention(q, k, v, S, cu, S, cu), 2.0 * T * D * (2 * HQ + 2 * HKV), 4.0 * D * HQ * pairs)
+    kc, vc = rnd(T // 64, 64, HKV, D), rnd(T // 64, 64, HKV, D)
+    table = i32(torch.arange(T // 64).view(B, -1))
+    q2, out = q.view(T, -1), torch.empty(T, HQ * D, dtype=bf, device=dev)
+    head_gate, gate, sink = rnd(T, HQ), rnd(T, HQ * D), torch.zeros(HQ, device=dev)
+    seen = lambda n, of: sum(p % n + 1 for p in range(of))
+    rec("window attention prefill, window 1024",
+        lambda: A.window_attention(q2, kc, vc, ctx, table, HQ, D, D, D ** -0.5, 1024, 30.0, cu_seqlens_q=cu, max_seqlen_q=S, out=out),
+        2.0 * T * D * (2 * HQ + 2 * HKV), 4.0 * D * HQ * B * sum(min(p + 1, 1024) for p in range(S)))
+    rec("chunked attention prefill, chunks of 1024",
+        lambda: A.window_attention(q2, kc, vc, ctx, table, HQ, D, D, D ** -0.5, 0, 50.0, cu_seqlens_q=cu, max_seqlen_q=S, out=out, chunk=1024,
+                                   sink=sink, gate=head_gate, gate_mode="head"),
+        2.0 * T * D * (2 * HQ + 2 * HKV), 4.0 * D * HQ * B * seen(1024, S), "window attention prefill, window 1024")
+    rec("gated attention prefill",
+        lambda: A.window_attention(q2, kc, vc, ctx, table, HQ, D, D, D ** -0.5, cu_seqlens_q=cu, max_seqlen_q=S, out=out, gate=gate, gate_mode="entry"),
+        2.0 * T * D * (3 * HQ + 2 * HKV), 4.0 * D * HQ * pairs, "qwen3 prefill attention")
+    del k, v, gate
+
+    mh, mk, mv = 16, 128, 256                    # a matrix memory whose state has the size of the delta rule's
+    norm, bias = torch.ones(mh * mv, device=dev), torch.zeros(2 * mh, device=dev)
+    bias[mh:] = 4.0
+
+    def memory(rows, n, cu=None, ctx=None):
+        x, gates, o = rnd(rows, 2 * mh * (mk + mv)), rnd(rows, 2 * mh, dt=torch.float32), torch.empty(rows, mh * mv, dtype=bf, device=dev)
+        st, slots = (torch.zeros(n, mh, mk, mv, device=dev), torch.zeros(n, mh, mk, device=dev), torch.zeros(n, mh, device=dev)), i32(torch.arange(n))
+        cols = x[:, :mh * mk], x[:, mh * mk:2 * mh * mk], x[:, 2 * mh * mk:2 * mh * mk + mh * mv], x[:, 2 * mh * mk + mh * mv:]
+        return lambda: mlstm_step(*cols, gates, bias, norm, st, o, ctx, slots, mh, mk, mv, 15.0, 1e-5, cu_seqlens_q=cu)
+    H, KV, dk, dv, taps = 32, 16, 128, 128, 4
+    C = 2 * KV * dk + H * dv
+    vec = [torch.zeros(H, device=dev), torch.full((H,), -2.0, device=dev), torch.ones(dv, device=dev)]
+    cw = rnd(taps, C, dt=torch.float32) * 0.5
+
+    def delta(rows, n, cu=None, ctx=None, raw=False):
+        x, z, ab, o = rnd(rows, C), rnd(rows, H * dv), rnd(rows, 2 * H, dt=torch.float32), torch.empty(rows, H * dv, dtype=bf, device=dev)
+        state, slots = torch.zeros(n, H, dk, dv, device=dev), i32(torch.arange(n))
+        kw = {"conv_weight": cw, "ring": rnd(n, taps, C)} if raw else {}
+        return lambda: G.gated_delta(x, z, ab, *vec, state, o, ctx, slots, H, KV, dk, dv, 1e-5, cu_seqlens_q=cu, **kw)
+    rec("mlstm prefill", memory(T, B, cu, ctx), 2.0 * T * mh * (2 * mk + 3 * mv) + 8.0 * T * mh, 2.0 * T * mh * (32 * (mk + mv) + 2 * mk * mv))
+    # products of the chunked form (64 tokens): scores of both kinds and their values (causal half), read-outs, update
+    rec("gated delta prefill", delta(T, B, cu, ctx), 2.0 * T * (C + 2 * H * dv) + 8.0 * T * H, 2.0 * T * H * (64 * (dk + dv) + 3 * dk * dv), "mlstm prefill")
+    up1, x, y, ring, slots = rnd(T, 12288), rnd(T, C), rnd(T, C), rnd(B, taps, C), i32(torch.arange(B))
+    rec("gelu", lambda: R.gelu_tanh(up1), 4.0 * T * 12288)
+    rec("short convolution", lambda: G.short_conv(x, cw, ring, ctx, slots, cu, S, y), 4.0 * T * C, 0.0, "gelu")
+    del up1, x, y
+    # decode: 256 sequences
+    n, NB = 256, 9
+    L = NB * 256 - 7
+    lens = i32(torch.full((n,), L))
+    qd, kq, vq = rnd(n, 1, HQ, D), rnd(n * NB, 256, HKV, D), rnd(n * NB, 256, HKV, D)
+    bt = i32(torch.randperm(n * NB).view(n, NB))
+    for seqs in (256, 64):
+        rec(f"qwen3 paged decode, {seqs} sequences", lambda: A.paged_decode_attention(qd[:seqs], kq, vq, lens[:seqs], bt[:seqs]), seqs * L * HKV * D * 4.0)
+    qf, og, oh, od = qd.view(n, -1), rnd(n, HQ * D), rnd(n, HQ), torch.empty(n, HQ * D, dtype=bf, device=dev)
+    for seqs in (256, 64):
+        rec(f"gated attention decode, {seqs} sequences", lambda: A.window_attention(
+            qf[:seqs], kq, vq, lens[:seqs], bt[:seqs], HQ, D, D, D ** -0.5, out=od[:seqs], gate=og[:seqs], gate_mode="entry"),
+            seqs * L * HKV * D * 4.0, 0.0, f"qwen3 paged decode, {seqs} sequences")
+    late = i32(torch.full((n,), 2041))           # 1017 keys of the second chunk
+    rec("window attention decode, window 1017", lambda: A.window_attention(qf, kq, vq, late, bt, HQ, D, D, D ** -0.5, 1017, 30.0), n * 1017 * HKV * D * 4.0)
+    rec("chunked attention decode, 1017 keys", lambda: A.window_attention(
+        qf, kq, vq, late, bt, HQ, D, D, D ** -0.5, 0, 50.0, out=od, chunk=1024, sink=sink, gate=oh, gate_mode="head"), n * 1017 * HKV * D * 4.0, 0.0,
+        "window attention decode, window 1017")
+    del kq, vq
+    five = i32(torch.full((n,), 5))
+    for seqs in (256, 64):
+        rec(f"mlstm decode, {seqs} sequences", memory(seqs, seqs, None, five[:seqs]), 8.0 * seqs * mh * mk * mv)
+        rec(f"gated delta decode, {seqs} sequences", delta(seqs, seqs, None, five[:seqs], raw=True), 8.0 * seqs * H * dk * dv + 2.0 * seqs * taps * C, 0.0,
+            f"mlstm decode, {seqs} sequences")
+    # row ops
+    xr, wr, res = rnd(T, W), torch.ones(W, dtype=bf, device=dev), rnd(T, W)
+    rec("qwen3 add + rms norm", lambda: P.rms_norm(xr, wr, 1e-6, res), 8.0 * T * W)
+    x, one, a = rnd(T, W, dt=torch.float32), torch.ones(W, device=dev), rnd(T, W)
+    rec("sublayer boundary", lambda: R.join_norms(x, [(one, None)], 1e-5, bf, a=a, rms=True), 12.0 * T * W, 0.0, "qwen3 add + rms norm")
+    E, top, ff = 64, 6, 1024
+    yy, places = rnd(T * top, W), i32(torch.randperm(T * top)).view(T, top)
+    rec("sublayer boundary, experts", lambda: R.join_norms(x, [(one, None)], 1e-5, bf, y=yy, pos=places, rms=True), (10.0 + 2 * top) * T * W, 0.0,
+        "qwen3 add + rms norm")
+    del yy, a, xr, res
+    tok, emb = torch.randint(0, 32768, (T,), device=dev), rnd(32768, W)
+    rec("embedding", lambda: R.embed_position(tok, pos, emb, 1.0), 6.0 * T * W, 0.0, "qwen3 add + rms norm")
+    qkv, slot = rnd(T, (HQ + 2 * HKV) * D), i32(torch.arange(T))
+    cs, w1 = P.rope_cos_sin_cache(D, S, 1e6, dev), torch.ones(D, dtype=bf, device=dev)
+    rec("qwen3 q/k norm, rotation and store", lambda: P.qk_norm_rope_store(
+        qkv, pos, cs, w1, w1, 1e-6, HQ, HKV, D, kc, vc, slot, return_k=False), 2.0 * T * D * (2 * HQ + 4 * HKV))
+    nq, nk = HQ * D, HKV * D
+    wd = torch.ones(D, device=dev)
+    like = "qwen3 q/k norm, rotation and store"
+    r1, r2 = Rotary.from_config({"dims": D, "base": 1e6}, True, dev), Rotary.from_config(
+        {"dims": D, "base": 1e6, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}, False, dev)
+    rec("norms, rotation and store, values = keys", lambda: rotate_store(
+        qkv[:, :nq], qkv[:, nq:nq + nk], qkv[:, nq:nq + nk], pos, r1, kc, vc, slot, D, D, wd, wd, 1e-5), 2.0 * T * D * (2 * HQ + 3 * HKV), 0.0, like)
+    rec("rotation and store", lambda: rotate_store(qkv[:, :nq], qkv[:, nq:nq + nk], qkv[:, nq + nk:], pos, r2, kc, vc, slot, D, D),
+        2.0 * T * D * (2 * HQ + 4 * HKV), 0.0, like)
+    del qkv
+    # experts
+    zl = rnd(T, E, dt=torch.float32)
+    for t, name in ((T, "prompts"), (64, "64 tokens")):
+        rec(f"routing by softmax, {name}", lambda: F.moe_route(zl[:t], E, top), 4.0 * t * E + t * top * 20.0, graph=True)
+        rec(f"routing by sigmoid, {name}", lambda: F.moe_route(zl[:t], E, top, "sigmoid", by_place=True), 4.0 * t * E + t * top * 24.0, 0.0,
+            f"routing by softmax, {name}", graph=True)
+    dn, wu, wg, wdn = rnd(T, W), rnd(E, ff, W), rnd(E, 2 * ff, W), rnd(E, W, ff)
+    pw, _, _, prow, off = F.moe_route(zl, E, top, "sigmoid", by_place=True)
+    M = T * top
+    mid = rnd(M, ff)
+    rec("experts up (squared relu), prompts", lambda: F.grouped_gemm(dn, wu, off, M, rows=prow, act="relu_squared"), 2.0 * (T * W + wu.numel() + M * ff),
+        2.0 * M * W * ff)
+    rec("experts gate and up, prompts", lambda: F.grouped_gemm(dn, wg, off, M, rows=prow, act="silu_mul", row_scale=pw),
+        2.0 * (T * W + wg.numel() + M * ff), 4.0 * M * W * ff, "experts up (squared relu), prompts")
+    rec("experts down, prompts", lambda: F.grouped_gemm(mid, wdn, off, M), 2.0 * (M * ff + wdn.numel() + M * W), 2.0 * M * W * ff,
+        "experts up (squared relu), prompts")
+    t = 64
+    pw2, _, _, prow2, off2 = F.moe_route(zl[:t], E, top, "sigmoid", by_place=True)
+    used = int((off2[1:] > off2[:-1]).sum())
+    sets, turn = [(wu, rnd(E, ff, W)), (wg, rnd(E, 2 * ff, W))], [0]
+
+    def decode(pair, **kw):
+        turn[0] ^= 1
+        F.grouped_gemm(dn[:t], pair[turn[0]], off2, t * top, rows=prow2, **kw)
+    rec("experts up (squared relu), 64 tokens", lambda: decode(sets[0], act="relu_squared"), 2.0 * (used * ff * W + t * W + t * top * ff))
+    rec("experts gate and up, 64 tokens", lambda: decode(sets[1], act="silu_mul", row_scale=pw2), 2.0 * (2 * used * ff * W + t * W + t * top * ff), 0.0,
+        "experts up (squared relu), 64 tokens")
+    return rec.recs, rec.launches
+
+
+def tukarax_of_size(dev, width, heads, kv, experts, top, eff, layers=12):
+    """A Tukarax decoder with random weights: parallel layers and chunked attention in turn, experts after each."""
+    import torch
+    from zipage_b200.models.registry import LoadedModel
+    from zipage_b200.models.tukarax import TukaraxConfig, TukaraxModel
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": eff}}
+    att = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    par = {"left": {**att, "rot": {"base": 1e6, "dims": 64}}, "left_scale": 0.5, "right_scale": 0.5,
+           "right": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    chunked = {**att, "mask": {"size": 1024}, "softcap": 50.0,
+               "rot": {"base": 1e6, "dims": 128, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    c = TukaraxConfig.from_dict({"vocab": 32768, "width": width, "norm": {"eps": 1e-5}, "layers": [
+        {"type": "attention", "mixer": chunked, "mlp": mlp} if i % 2 else {"type": "parallel", "mixer": par, "mlp": mlp} for i in range(layers)]})
+    m = TukaraxModel(c, torch.bfloat16, dev)
+    with torch.no_grad():
+        for n, p in m.named_parameters():
+            if p.dim() > 1:
+                p.normal_(0, p.shape[-1] ** -0.5)
+            else:
+                p.fill_(-2.0) if "dt_bias" in n else p.zero_() if "A_log" in n or "sink" in n else p.fill_(1.0)
+    return LoadedModel("Tukarax", m, m.head, width, 32768, torch.bfloat16, True)
+
+
+def run_tukarax(args):
+    """Prefill and decode throughput of the Tukarax decoder through the serving engine at two widths, random weights, beside
+    Dobedra decoders of equal width, depth, heads and experts and Qwen3 blocks whose feed-forward is as wide as what a token's
+    experts add up to; and the kernel table."""
+    import torch
+    dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
+    torch.cuda.set_device(dev)
+    pk = ROOT / "MEASURED_PEAKS.json"
+    peaks = json.loads(pk.read_text()) if pk.exists() else {}
+    torch.manual_seed(3)
+    R, PROMPT, GEN = SERVE
+    g = torch.Generator().manual_seed(1)
+    res = {}
+    with ClockSampler(dev.index or 0) as clocks:
+        kernels, launches = tukarax_kernel_records(args, dev, peaks)
+        torch.cuda.empty_cache()
+        for width, heads, kv, q_rank, experts, top, eff in ((4096, 32, 8, 1536, 64, 6, 1024), (2048, 16, 4, 768, 64, 6, 512)):
+            models = {"tukarax": lambda: tukarax_of_size(dev, width, heads, kv, experts, top, eff),
+                      "dobedra": lambda: dobedra_of_size(dev, width, heads, q_rank, top * eff, experts, top, eff),
+                      "qwen3": lambda: qwen_of_size(dev, width, heads, kv, top * eff, 12)}
+            row = res[f"width {width}"] = {"layers": 12}
+            for name, make in models.items():
+                row[name] = serve_model(make(), g)
+                torch.cuda.empty_cache()
+    head = res["width 4096"]["tukarax"]
+    print(json.dumps({
+        "metric": "tukarax_decode_tokens_per_s", "value": head["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+        "steps": args.steps, "warmup": args.warmup, "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True,
+        "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": f"serving engine, {R} requests, prompts of {PROMPT}, {GEN} sampled tokens each; random weights; 12 layers "
+                               "(attention and delta rule in parallel / chunked attention in turn; 64 experts, six a token) beside 12 "
+                               "Dobedra layers and 12 Qwen3 blocks",
+                   "l2": "inputs of the streaming kernels are larger than L2"},
+        "serving": res, "kernels": kernels, "gpu_launches": launches, "clocks": clocks.summary(),
+        "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")},
+    }))
+
+
 def run_host_control(args):
     """Host time per decode step of the control plane at `--requests` concurrent requests: the
     native scheduler's array calls (schedule, the runner's input arrays, postprocess) and, when an
@@ -1578,6 +1787,8 @@ def main():
         return run_similorn(args)
     if args.workload == "dobedra":
         return run_dobedra(args)
+    if args.workload == "tukarax":
+        return run_tukarax(args)
     if args.workload == "prefill":
         return run_prefill(args)
     if args.workload == "decode":
