@@ -587,7 +587,7 @@ int zp_short_conv(const void* x, int64_t x_stride, const float* weight, void* ri
  * its own row stride; A_log, dt_bias [H], norm_weight [vdim] fp32; state [n_slots, H, dim, VP] fp32 (VP >= vdim, a
  * multiple of 4).  cu_seqlens_q, context_lens, slots as in zp_mlstm.  taps > 0 (single rows only): x is the input of the
  * convolution of zp_short_conv, which is then part of the launch; taps 0: x has been through it.
- * bf16 portions with head sizes up to 128 (multiples of 8) and at least 8 rows per sequence on average take the chunked tcgen05
+ * bf16 portions with key sizes up to 128, value sizes up to 256 (multiples of 8) and at least 8 rows per sequence on average take the chunked tcgen05
  * kernels (ZP_IMPL_SIMT: never; ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED), which need a workspace. */
 size_t zp_gated_delta_workspace_bytes(int total_rows, int B, int H);
 int zp_gated_delta(const void* x, int64_t x_stride, const void* gate, int64_t gate_stride, const float* ab,

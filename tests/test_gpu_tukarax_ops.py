@@ -222,7 +222,7 @@ def _delta_want(cs, H, G, dk, dv, eps, x=None, S=None):
     return o.flatten(1), S
 
 
-SIZES = [(6, 2, 40, 56), (4, 4, 128, 128), (6, 3, 64, 120), (3, 3, 9, 7), (2, 1, 160, 200), (1, 1, 300, 33), (2, 2, 16, 300), (8, 1, 8, 8)]
+SIZES = [(6, 2, 40, 56), (4, 4, 128, 128), (6, 3, 64, 120), (3, 3, 9, 7), (2, 1, 160, 200), (1, 1, 300, 33), (2, 2, 16, 304), (8, 1, 8, 8), (2, 1, 96, 256), (3, 1, 128, 72)]
 
 
 @pytest.mark.parametrize("fast", [False, True])
@@ -234,7 +234,7 @@ def test_delta_portions(H, G, dk, dv, fast):
     plans = [[130, 64, 2], [2, 63, 70], [65, 1, 200]]
     cases = [_delta_case(H, G, dk, dv, sum(p), 10 + i, fast) for i, p in enumerate(plans)]
     impls = [(torch.float32, "auto"), (BF, "simt")]
-    if dk % 8 == dv % 8 == 0 and dk <= 128 and dv <= 128:
+    if dk % 8 == dv % 8 == 0 and dk <= 128 and dv <= 256:
         impls.append((BF, "tcgen05"))
     for dtype, impl in impls:
         for c in cases:

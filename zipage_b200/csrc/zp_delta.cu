@@ -13,20 +13,41 @@ namespace zp {
 
 constexpr int DR_THREADS = 256;
 
-// one channel of the convolution with its silu at position p: `now` is the current input
+// The inputs of one channel's convolution at a token, all loads in flight together (more than four taps: the rest in
+// `conv_finish`).
+template <typename T> struct ConvIn { T now, back[3]; float w[4]; };
+struct ConvPlace { int C, taps, row, seen; };          // row p % taps of the ring; how many earlier inputs there are
 template <typename T>
-__device__ __forceinline__ float conv_channel(const DeltaArgs& a, const T* ring, int c, int C, int p, float now) {
-  float acc = now * a.conv_w[(int64_t)(a.taps - 1) * C + c];
-  for (int j = 1; j < a.taps; ++j)
-    if (p - j >= 0) acc = fmaf(Elem<T>::to_f32(ring[(int64_t)((p - j) % a.taps) * C + c]), a.conv_w[(int64_t)(a.taps - 1 - j) * C + c], acc);
+__device__ __forceinline__ void conv_start(ConvIn<T>& v, const DeltaArgs& a, const ConvPlace& at, const T* xr, const T* ring, int c) {
+  v.now = xr[c];
+  v.w[0] = a.conv_w[(int64_t)(at.taps - 1) * at.C + c];
+#pragma unroll
+  for (int j = 1; j < 4; ++j) {
+    v.back[j - 1] = Elem<T>::from_f32(0.f);
+    v.w[j] = 0.f;
+    if (j <= at.seen) {
+      const int r = at.row - j;
+      v.back[j - 1] = ring[(int64_t)(r < 0 ? r + at.taps : r) * at.C + c];
+      v.w[j] = a.conv_w[(int64_t)(at.taps - 1 - j) * at.C + c];
+    }
+  }
+}
+template <typename T>
+__device__ __forceinline__ float conv_finish(const ConvIn<T>& v, const DeltaArgs& a, const ConvPlace& at, const T* ring, int c) {
+  float acc = Elem<T>::to_f32(v.now) * v.w[0];
+#pragma unroll
+  for (int j = 1; j < 4; ++j) acc = fmaf(Elem<T>::to_f32(v.back[j - 1]), v.w[j], acc);
+  for (int j = 4; j <= at.seen; ++j) {
+    const int r = at.row - j;
+    acc = fmaf(Elem<T>::to_f32(ring[(int64_t)(r < 0 ? r + at.taps : r) * at.C + c]), a.conv_w[(int64_t)(at.taps - 1 - j) * at.C + c], acc);
+  }
   return acc / (1.f + expf(-acc));
 }
 
 template <typename T, int RPT>   // RPT: state rows per thread
-__global__ void __launch_bounds__(DR_THREADS, 2) delta_recurrent_kernel(const DeltaArgs a) {
+__global__ void __launch_bounds__(DR_THREADS, RPT == 16 ? 2 : RPT == 8 ? 3 : 4) delta_recurrent_kernel(const DeltaArgs a) {
   extern __shared__ __align__(16) float sm[];
-  __shared__ float red[3][8];
-  __shared__ float red2[32];
+  __shared__ float red[3][8], red2[8];
   __shared__ float xsum[2];      // this block's sum of squares, by token parity
   const int vt = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const DeltaSeq sq = delta_seq(a, b);
@@ -35,10 +56,11 @@ __global__ void __launch_bounds__(DR_THREADS, 2) delta_recurrent_kernel(const De
   const int c0 = vt * a.VT, ncg = a.VT / 4, nrg = DR_THREADS / ncg;   // (powers of two; ncg <= 32)
   float* sq_ = sm;               // [dim] q
   float* sk = sq_ + a.dim;       // [dim] k
-  float* sv = sm + ((2 * a.dim + 3) & ~3);   // [VT] v, then the update's row u
-  float* part = sv + a.VT;       // [2][8 warps][VT]
+  float* sv = sm + ((2 * a.dim + 3) & ~3);   // [VT] v
+  float* su = sv + a.VT;         // [VT] the update's row
+  float* part = su + a.VT;       // [2][8 warps][VT]
   const int cg = tid & (ncg - 1), rg = tid / ncg, col = c0 + 4 * cg;
-  const bool mine = col < a.VP;
+  const bool mine = col < a.VP, out_col = tid < a.VT && c0 + tid < a.vdim;      // (VT <= 128)
   float* S = a.S + ((int64_t)sq.slot * a.H + h) * a.dim * a.VP + col;
   float4 s[RPT];
 #pragma unroll
@@ -48,37 +70,50 @@ __global__ void __launch_bounds__(DR_THREADS, 2) delta_recurrent_kernel(const De
   }
   const T* x = reinterpret_cast<const T*>(a.x);
   T* ring = reinterpret_cast<T*>(a.ring) + (int64_t)sq.slot * a.taps * C;
-  const float qscale = rsqrtf((float)a.dim);
+  const float qscale = rsqrtf((float)a.dim), nw = out_col ? a.norm_weight[c0 + tid] : 0.f;
+  const bool keeper = h % group == 0 && vt == 0;      // of the keys' and queries' inputs
 
   for (int t = 0; t < sq.count; ++t) {
     const int64_t row = sq.row0 + t;
     const int p = sq.ctx - sq.count + t;
     const T* xr = x + row * a.x_stride;
+    const float z = out_col ? Elem<T>::to_f32(reinterpret_cast<const T*>(a.gate)[row * a.gate_stride + (int64_t)h * a.vdim + c0 + tid]) : 0.f;
+    ConvPlace at{C, a.taps, 0, 0};
+    if (a.taps) { at.row = p % a.taps; at.seen = min(p, a.taps - 1); }
     float qq = 0.f, kk = 0.f, kq = 0.f;
-    for (int d = tid; d < a.dim; d += DR_THREADS) {
-      const int cq = hk * a.dim + d, ck = a.G * a.dim + cq;
-      float q = Elem<T>::to_f32(xr[cq]), k = Elem<T>::to_f32(xr[ck]);
-      if (a.taps) {
-        const T qr = xr[cq], kr = xr[ck];
-        q = conv_channel<T>(a, ring, cq, C, p, q);
-        k = conv_channel<T>(a, ring, ck, C, p, k);
-        if (h % group == 0 && vt == 0) {
-          ring[(int64_t)(p % a.taps) * C + cq] = qr;
-          ring[(int64_t)(p % a.taps) * C + ck] = kr;
+    if (tid < 128) {             // queries and keys; the other half brings the values
+#pragma unroll 1
+      for (int d = tid; d < a.dim; d += 128) {
+        const int cq = hk * a.dim + d, ck = a.G * a.dim + cq;
+        float q, k;
+        if (a.taps) {
+          ConvIn<T> vq, vk;
+          conv_start(vq, a, at, xr, ring, cq);
+          conv_start(vk, a, at, xr, ring, ck);
+          q = conv_finish(vq, a, at, ring, cq);
+          k = conv_finish(vk, a, at, ring, ck);
+          if (keeper) {
+            ring[(int64_t)at.row * C + cq] = vq.now;
+            ring[(int64_t)at.row * C + ck] = vk.now;
+          }
+        } else {
+          q = Elem<T>::to_f32(xr[cq]);
+          k = Elem<T>::to_f32(xr[ck]);
         }
+        sq_[d] = q; sk[d] = k;
+        qq = fmaf(q, q, qq); kk = fmaf(k, k, kk); kq = fmaf(k, q, kq);
       }
-      sq_[d] = q; sk[d] = k;
-      qq = fmaf(q, q, qq); kk = fmaf(k, k, kk); kq = fmaf(k, q, kq);
-    }
-    for (int c = tid; c < a.VT; c += DR_THREADS) {
+    } else if (tid - 128 < a.VT) {
+      const int c = tid - 128, cv = 2 * a.G * a.dim + h * a.vdim + c0 + c;
       float v = 0.f;
       if (c0 + c < a.vdim) {
-        const int cv = 2 * a.G * a.dim + h * a.vdim + c0 + c;
-        v = Elem<T>::to_f32(xr[cv]);
         if (a.taps) {
-          const T vr = xr[cv];
-          v = conv_channel<T>(a, ring, cv, C, p, v);
-          ring[(int64_t)(p % a.taps) * C + cv] = vr;
+          ConvIn<T> vv;
+          conv_start(vv, a, at, xr, ring, cv);
+          v = conv_finish(vv, a, at, ring, cv);
+          ring[(int64_t)at.row * C + cv] = vv.now;
+        } else {
+          v = Elem<T>::to_f32(xr[cv]);
         }
       }
       sv[c] = v;
@@ -87,10 +122,6 @@ __global__ void __launch_bounds__(DR_THREADS, 2) delta_recurrent_kernel(const De
     qq = warp_sum(qq); kk = warp_sum(kk); kq = warp_sum(kq);
     if (lane == 0) { red[0][warp] = qq; red[1][warp] = kk; red[2][warp] = kq; }
     __syncthreads();
-    qq = kk = kq = 0.f;
-#pragma unroll
-    for (int w = 0; w < 8; ++w) { qq += red[0][w]; kk += red[1][w]; kq += red[2][w]; }
-    const float rq = qscale / sqrtf(qq + DELTA_UNIT_EPS), rk = 1.f / sqrtf(kk + DELTA_UNIT_EPS);
     float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
@@ -112,53 +143,54 @@ __global__ void __launch_bounds__(DR_THREADS, 2) delta_recurrent_kernel(const De
       *reinterpret_cast<float4*>(part + (8 + warp) * a.VT + 4 * cg) = aq;
     }
     __syncthreads();
-    float o = 0.f;               // column tid of the tile (VT <= 128)
+    float o = 0.f;               // column tid of the tile
     if (tid < a.VT) {
+      qq = kk = kq = 0.f;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) { qq += red[0][w]; kk += red[1][w]; kq += red[2][w]; }
+      const float rq = qscale / sqrtf(qq + DELTA_UNIT_EPS), rk = 1.f / sqrtf(kk + DELTA_UNIT_EPS);
       float kS = 0.f, qS = 0.f;
 #pragma unroll
       for (int w = 0; w < 8; ++w) { kS += part[w * a.VT + tid]; qS += part[(8 + w) * a.VT + tid]; }
       const float u = beta * (sv[tid] - g * rk * kS);
       o = fmaf(g * rq, qS, rk * rq * kq * u);
-      sv[tid] = rk * u;
+      su[tid] = rk * u;
     }
-    const float ss0 = block_sum(o * o, red2);      // (its barriers also publish u)
+    float ss = warp_sum(o * o);
+    if (lane == 0) red2[warp] = ss;
+    __syncthreads();
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
       const int r = rg + i * nrg;
       if (r < a.dim) {
         const float kr = sk[r];
-        const float4 u = *reinterpret_cast<const float4*>(sv + 4 * cg);
+        const float4 u = *reinterpret_cast<const float4*>(su + 4 * cg);
         s[i].x = fmaf(kr, u.x, g * s[i].x); s[i].y = fmaf(kr, u.y, g * s[i].y);
         s[i].z = fmaf(kr, u.z, g * s[i].z); s[i].w = fmaf(kr, u.w, g * s[i].w);
+        if (t + 1 == sq.count && mine) *reinterpret_cast<float4*>(S + (int64_t)r * a.VP) = s[i];
       }
     }
-    float ss = ss0;
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) ss += red2[w];            // (columns: the first 128 threads)
     if (cluster_size() > 1) {
       if (tid == 0) xsum[t & 1] = ss;
       cluster_sync();
       ss = 0.f;
       for (uint32_t r = 0; r < cluster_size(); ++r) ss += ld_cluster(&xsum[t & 1], r);
     }
-    if (tid < a.VT && c0 + tid < a.vdim) {
+    if (out_col) {
       const float rr = a.out_scale / sqrtf(ss / (float)a.vdim + a.eps);
-      const int64_t e = (int64_t)h * a.vdim + c0 + tid;
-      const float z = Elem<T>::to_f32(reinterpret_cast<const T*>(a.gate)[row * a.gate_stride + e]);
-      reinterpret_cast<T*>(a.out)[row * a.out_stride + e] =
-          Elem<T>::from_f32(o * rr * a.norm_weight[c0 + tid] * (z / (1.f + expf(-z))));
+      reinterpret_cast<T*>(a.out)[row * a.out_stride + (int64_t)h * a.vdim + c0 + tid] = Elem<T>::from_f32(o * rr * nw * (z / (1.f + expf(-z))));
     }
     if (t + 1 < sq.count) __syncthreads();   // q, k and u are rewritten by the next token
-  }
-#pragma unroll
-  for (int i = 0; i < RPT; ++i) {
-    const int r = rg + i * nrg;
-    if (mine && r < a.dim) *reinterpret_cast<float4*>(S + (int64_t)r * a.VP) = s[i];
   }
   if (cluster_size() > 1) cluster_sync();   // peers may still be reading xsum
 }
 
 template <typename T, int RPT>
 static int launch_recurrent(const DeltaArgs& a, int tiles, cudaStream_t st) {
-  const size_t smem = sizeof(float) * (((2 * a.dim + 3) & ~3) + 17 * (size_t)a.VT);
+  const size_t smem = sizeof(float) * (((2 * a.dim + 3) & ~3) + 18 * (size_t)a.VT);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(tiles, a.H, a.B);
   cfg.blockDim = dim3(DR_THREADS);
@@ -196,8 +228,8 @@ static int delta_recurrent(DeltaArgs a, cudaStream_t st) {
 }
 
 // ---------------------------------------------------------------------------------------------
-// Short causal convolution over time, per channel, with silu: portions of prompts.  A thread owns V adjacent channels and
-// walks CV_RUN tokens with the last inputs in registers.
+// Short causal convolution over time, per channel, with silu: portions of prompts.  A thread owns V adjacent channels of
+// CV_RUN tokens, all loads in flight together; the warps of a block take runs that follow one another.
 // ---------------------------------------------------------------------------------------------
 struct ConvArgs {
   const void* x; const float* w; void* ring; void* out;
@@ -205,69 +237,68 @@ struct ConvArgs {
   int64_t x_stride, out_stride;
   int C, taps, n_slots;
 };
-constexpr int CV_RUN = 16, CV_MAX_TAPS = 8;
+constexpr int CV_RUN = 8, CV_WARPS = 8, CV_MAX_TAPS = 8;
 
-template <typename T, int V> struct ChanVec { T e[V]; };
-template <typename T, int V> __device__ __forceinline__ void cv_load(const T* p, float (&f)[V]) {
-  if constexpr (V == 1) f[0] = Elem<T>::to_f32(*p);
-  else {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);       // V * sizeof(T) = 8
-    const T* e = reinterpret_cast<const T*>(&raw);
+template <typename T, int V> struct __align__(V == 1 ? sizeof(T) : 8) ChanVec { T e[V]; };        // V * sizeof(T) = 8, or one entry
+template <typename T, int V> __device__ __forceinline__ ChanVec<T, V> cv_load(const T* p) {
+  ChanVec<T, V> r;
+  if constexpr (V == 1) r.e[0] = *p;
+  else *reinterpret_cast<uint2*>(&r) = *reinterpret_cast<const uint2*>(p);
+  return r;
+}
+template <typename T, int V> __device__ __forceinline__ void cv_floats(const ChanVec<T, V>& r, float (&f)[V]) {
 #pragma unroll
-    for (int i = 0; i < V; ++i) f[i] = Elem<T>::to_f32(e[i]);
-  }
+  for (int i = 0; i < V; ++i) f[i] = Elem<T>::to_f32(r.e[i]);
 }
 template <typename T, int V> __device__ __forceinline__ void cv_store(T* p, const float (&f)[V]) {
-  if constexpr (V == 1) *p = Elem<T>::from_f32(f[0]);
-  else {
-    uint2 raw;
-    T* e = reinterpret_cast<T*>(&raw);
+  ChanVec<T, V> r;
 #pragma unroll
-    for (int i = 0; i < V; ++i) e[i] = Elem<T>::from_f32(f[i]);
-    *reinterpret_cast<uint2*>(p) = raw;
-  }
+  for (int i = 0; i < V; ++i) r.e[i] = Elem<T>::from_f32(f[i]);
+  if constexpr (V == 1) *p = r.e[0];
+  else *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(&r);
 }
 
 template <typename T, int V, int TAPS>
-__global__ void __launch_bounds__(256) short_conv_kernel(const ConvArgs a) {
-  const int b = blockIdx.z, c = (blockIdx.y * 256 + threadIdx.x) * V;
+__global__ void __launch_bounds__(CV_WARPS * 32) short_conv_kernel(const ConvArgs a) {
+  const int b = blockIdx.z, c = (blockIdx.y * 32 + (threadIdx.x & 31)) * V;
   const int row0 = a.cu_q[b], count = a.cu_q[b + 1] - row0, ctx = a.context_lens[b], slot = a.slots[b];
-  const int t0 = blockIdx.x * CV_RUN, t1 = min(count, t0 + CV_RUN);
+  const int t0 = (blockIdx.x * CV_WARPS + (threadIdx.x >> 5)) * CV_RUN;
   if (c >= a.C || t0 >= count || ctx < count || slot < 0 || slot >= a.n_slots) return;
-  const T* x = reinterpret_cast<const T*>(a.x) + c;
-  const T* ring = reinterpret_cast<const T*>(a.ring) + (int64_t)slot * TAPS * a.C + c;
-  T* out = reinterpret_cast<T*>(a.out) + c;
+  const T* __restrict__ x = reinterpret_cast<const T*>(a.x) + (int64_t)row0 * a.x_stride + c;
+  const T* __restrict__ ring = reinterpret_cast<const T*>(a.ring) + (int64_t)slot * TAPS * a.C + c;
+  T* __restrict__ out = reinterpret_cast<T*>(a.out) + (int64_t)row0 * a.out_stride + c;
   const int pos0 = ctx - count;
-  float w[TAPS][V], hist[TAPS][V];           // hist[j]: the input j tokens back
+  ChanVec<T, V> in[CV_RUN + TAPS - 1];       // the inputs ahead of the run, then the run's
+#pragma unroll
+  for (int u = 0; u < CV_RUN + TAPS - 1; ++u) {
+    const int t = t0 + u - (TAPS - 1);
+#pragma unroll
+    for (int i = 0; i < V; ++i) in[u].e[i] = Elem<T>::from_f32(0.f);
+    if (t >= 0) { if (t < count) in[u] = cv_load<T, V>(x + (int64_t)t * a.x_stride); }
+    else if (pos0 + t >= 0) in[u] = cv_load<T, V>(ring + (int64_t)((pos0 + t) % TAPS) * a.C);
+  }
+  float w[TAPS][V];
 #pragma unroll
   for (int j = 0; j < TAPS; ++j)
 #pragma unroll
-    for (int i = 0; i < V; ++i) w[j][i] = a.w[(int64_t)(TAPS - 1 - j) * a.C + c + i];
+    for (int i = 0; i < V; ++i) w[j][i] = a.w[(int64_t)j * a.C + c + i];
+  float f[TAPS][V];                          // inputs of the current token, in a circle
 #pragma unroll
-  for (int j = 1; j < TAPS; ++j) {           // the inputs ahead of the run: hist[j - 1] before the first shift
-    const int t = t0 - j;
+  for (int j = 0; j < TAPS - 1; ++j) cv_floats(in[j], f[j]);
 #pragma unroll
-    for (int i = 0; i < V; ++i) hist[j - 1][i] = 0.f;
-    if (t >= 0) cv_load<T, V>(x + (int64_t)(row0 + t) * a.x_stride, hist[j - 1]);
-    else if (pos0 + t >= 0) cv_load<T, V>(ring + (int64_t)((pos0 + t) % TAPS) * a.C, hist[j - 1]);
-  }
-#pragma unroll 4
-  for (int t = t0; t < t1; ++t) {
-#pragma unroll
-    for (int j = TAPS - 1; j > 0; --j)
-#pragma unroll
-      for (int i = 0; i < V; ++i) hist[j][i] = hist[j - 1][i];
-    cv_load<T, V>(x + (int64_t)(row0 + t) * a.x_stride, hist[0]);
+  for (int u = 0; u < CV_RUN; ++u) {
+    if (t0 + u >= count) break;
+    cv_floats(in[u + TAPS - 1], f[(u + TAPS - 1) % TAPS]);
     float y[V];
 #pragma unroll
     for (int i = 0; i < V; ++i) {
       float acc = 0.f;
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j][i], hist[j][i], acc);
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j][i], f[(u + j) % TAPS][i], acc);
       if constexpr (sizeof(T) == 4) y[i] = acc / (1.f + expf(-acc));
       else y[i] = __fdividef(acc, 1.f + __expf(fminf(-acc, 80.f)));
     }
-    cv_store<T, V>(out + (int64_t)(row0 + t) * a.out_stride, y);
+    cv_store<T, V>(out + (int64_t)(t0 + u) * a.out_stride, y);
   }
 }
 
@@ -283,7 +314,7 @@ template <typename T> __global__ void __launch_bounds__(256) conv_keep_kernel(co
 
 template <typename T, int V> static int conv_by_taps(const ConvArgs& a, dim3 grid, cudaStream_t st) {
   switch (a.taps) {
-#define ZP_CONV(n) case n: short_conv_kernel<T, V, n><<<grid, 256, 0, st>>>(a); break
+#define ZP_CONV(n) case n: short_conv_kernel<T, V, n><<<grid, CV_WARPS * 32, 0, st>>>(a); break
     ZP_CONV(1); ZP_CONV(2); ZP_CONV(3); ZP_CONV(4); ZP_CONV(5); ZP_CONV(6); ZP_CONV(7); ZP_CONV(8);
 #undef ZP_CONV
     default: return ZP_ERR_UNSUPPORTED;
@@ -306,8 +337,9 @@ extern "C" int zp_short_conv(const void* x, int64_t x_stride, const float* weigh
   ZP_DISPATCH_DTYPE(dtype, T, {
     constexpr int V = 8 / sizeof(T);
     const bool vec = channels % V == 0 && x_stride % V == 0 && out_stride % V == 0 && ((uintptr_t)x | (uintptr_t)ring | (uintptr_t)out) % 8 == 0;
-    const int per = 256 * (vec ? V : 1);
-    const dim3 grid((max_seqlen_q + zp::CV_RUN - 1) / zp::CV_RUN, (channels + per - 1) / per, B);
+    const int per = 32 * (vec ? V : 1), run = zp::CV_RUN * zp::CV_WARPS;
+    ZP_REQUIRE((channels + per - 1) / per <= 65535, "zp_short_conv: %d channels", channels);
+    const dim3 grid((max_seqlen_q + run - 1) / run, (channels + per - 1) / per, B);
     rc = vec ? zp::conv_by_taps<T, V>(a, grid, st) : zp::conv_by_taps<T, 1>(a, grid, st);
     if (rc == ZP_OK) {
       zp::conv_keep_kernel<T><<<dim3((channels + 255) / 256, B), 256, 0, st>>>(a);
@@ -342,8 +374,8 @@ extern "C" int zp_gated_delta(const void* x, int64_t x_stride, const void* gate,
   cudaStream_t st = (cudaStream_t)stream;
   const bool tc = cu_seqlens_q && total_rows > 0 && zp::delta_chunk_supports(a, dtype);
   if (impl == ZP_IMPL_TCGEN05 && !tc) {
-    zp::set_error("zp_gated_delta: the tcgen05 kernels need bf16 portions, head sizes that are multiples of 8 up to 128 and "
-                  "16-byte aligned rows");
+    zp::set_error("zp_gated_delta: the tcgen05 kernels need bf16 portions, head sizes that are multiples of 8, keys up to 128, values up to 256, "
+                  "and 16-byte aligned rows");
     return ZP_ERR_UNSUPPORTED;
   }
   if (tc && (impl == ZP_IMPL_TCGEN05 || (impl == ZP_IMPL_AUTO && total_rows >= 8 * B))) {

@@ -119,21 +119,6 @@ __device__ __forceinline__ bool mt_wait_cluster(uint64_t* bar, uint32_t parity, 
   return false;
 }
 
-// 4 x 4 transpose of 16-byte chunks within groups of four lanes: v[i] of lane t <- v[t] of lane i.  Turns
-// "one row per lane" into "four lanes per row", so that global accesses touch whole 64-byte row pieces.
-__device__ __forceinline__ void mt_transpose4(int4 (&v)[4], int lane) {
-  auto swap = [&](int4& x, int4& y, int mask, bool upper) {
-    int4 snd = upper ? x : y, rcv;
-    rcv.x = __shfl_xor_sync(0xffffffffu, snd.x, mask); rcv.y = __shfl_xor_sync(0xffffffffu, snd.y, mask);
-    rcv.z = __shfl_xor_sync(0xffffffffu, snd.z, mask); rcv.w = __shfl_xor_sync(0xffffffffu, snd.w, mask);
-    if (upper) x = rcv; else y = rcv;
-  };
-  swap(v[0], v[1], 1, lane & 1);
-  swap(v[2], v[3], 1, lane & 1);
-  swap(v[0], v[2], 2, lane & 2);
-  swap(v[1], v[3], 2, lane & 2);
-}
-
 struct MtParams { MlstmArgs a; int* error_word; };
 
 __global__ void __launch_bounds__(MT_THREADS, 1)
@@ -499,7 +484,7 @@ mlstm_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         ss = all;
       }
       const float rr = rsqrtf(ss / (float)a.vdim + a.eps);
-      mt_transpose4(gt, lane);                     // to this thread's own row
+      transpose4(gt, lane);                     // to this thread's own row
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int gg[4] = {gt[i].x, gt[i].y, gt[i].z, gt[i].w};
@@ -515,7 +500,7 @@ mlstm_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
         gt[i] = make_int4((int)w[0], (int)w[1], (int)w[2], (int)w[3]);
       }
-      mt_transpose4(gt, lane);
+      transpose4(gt, lane);
 #pragma unroll
       for (int i = 0; i < 4; ++i)
         if (lrow + i < n) st16(reinterpret_cast<T*>(a.out) + (lrow0 + i) * a.out_stride + lcol, gt[i]);

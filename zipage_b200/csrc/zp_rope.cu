@@ -2,8 +2,10 @@
 // first `dims` entries of each head (interleaved or half-split pairs), queries in place, keys and values into padded
 // paged caches.  The values may be the keys themselves, as projected.
 //
-// One block per token: its cosines and sines are made once (fp64 turns, reduced before the sine) and shared by all heads; a
-// warp takes a head at a time, holding the row in shared memory because pairs lie in different lanes.
+// One block per token: its cosines and sines are made once (fp64 turns, reduced before the sine) and shared by all heads.
+// 16-bit rows of whole 16-byte pieces: a half warp (or, above 128 entries, a warp) takes a head, eight entries a lane, several
+// heads in flight, and pairs that lie in different lanes meet by shuffles.  Other rows: a warp takes a head at a time
+// and holds the row in shared memory.
 #include "zp_common.cuh"
 
 namespace zp {
@@ -119,6 +121,119 @@ __global__ void __launch_bounds__(RO_THREADS) rotate_store_kernel(const RotateAr
   }
 }
 
+// LANES: lanes of a head; NI: heads of a group of lanes in flight
+template <typename T, int LANES, int NI>
+__global__ void __launch_bounds__(RO_THREADS) rotate_store_vec_kernel(const RotateArgs a) {
+  extern __shared__ __align__(16) float ro_sm[];   // cos [dims / 2], sin [dims / 2]
+  constexpr int GROUPS = RO_THREADS / LANES;
+  const int64_t n = blockIdx.x;
+  const int grp = threadIdx.x / LANES, l = threadIdx.x & (LANES - 1), half = a.dims >> 1, e0 = 8 * l;
+  float *cs = ro_sm, *sn = cs + half;
+  const int64_t slot = a.slots[n];
+  const bool stored = slot >= 0 && slot < a.n_slots;
+  const int total = a.Hq + 2 * a.Hkv;
+  auto row_of = [&](int item) -> const T* {
+    if (item < a.Hq) return reinterpret_cast<const T*>(a.q) + n * a.row_stride + (int64_t)item * a.D;
+    item -= a.Hq;
+    if (item < a.Hkv) return reinterpret_cast<const T*>(a.k) + n * a.row_stride + (int64_t)item * a.D;
+    return reinterpret_cast<const T*>(a.v) + n * a.row_stride + (int64_t)(item - a.Hkv) * a.DV;
+  };
+  auto width_of = [&](int item) { return item < a.Hq + a.Hkv ? a.D : a.DV; };
+  int4 raw[NI];
+  auto fetch = [&](int first) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int item = first + i * GROUPS;
+      raw[i] = item < total && e0 < width_of(item) ? ld16(row_of(item) + e0) : make_int4(0, 0, 0, 0);
+    }
+  };
+  fetch(grp);
+  const double p = (double)a.positions[n];
+  for (int i = threadIdx.x; i < half; i += RO_THREADS) {
+    const double t = p * a.turns[i];
+    float s, c;
+    sincospif(2.f * (float)(t - rint(t)), &s, &c);
+    cs[i] = c * a.mul;
+    sn[i] = s * a.mul;
+  }
+  __syncthreads();
+  // where this lane's pairs are: in the lane itself, or eight entries of another lane
+  const bool turns_here = e0 < a.dims, second = !a.interleaved && e0 >= half;
+  const int lane0 = (threadIdx.x & 31) - l, mate = lane0 + (a.interleaved || !turns_here ? l : (second ? l - (half >> 3) : l + (half >> 3)));
+  for (int base = grp; base - grp < total; base += NI * GROUPS) {      // (the same number of rounds in every lane)
+    if (base != grp) fetch(base);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int item = base + i * GROUPS;
+      const bool is_q = item < a.Hq, is_k = !is_q && item < a.Hq + a.Hkv, live = item < total && e0 < width_of(item);
+      float f[8];
+      const T* e = reinterpret_cast<const T*>(&raw[i]);
+#pragma unroll
+      for (int u = 0; u < 8; ++u) f[u] = Elem<T>::to_f32(e[u]);
+      const float* w = is_q ? a.q_weight : is_k ? a.k_weight : nullptr;
+      float ss = 0.f;
+#pragma unroll
+      for (int u = 0; u < 8; ++u) ss = fmaf(f[u], f[u], ss);
+#pragma unroll
+      for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      float r = 1.f;
+      if (w && live) {
+        r = 1.f / sqrtf(ss / (float)a.D + a.eps);
+        const float4 w0 = *reinterpret_cast<const float4*>(w + e0), w1 = *reinterpret_cast<const float4*>(w + e0 + 4);
+        f[0] *= w0.x; f[1] *= w0.y; f[2] *= w0.z; f[3] *= w0.w; f[4] *= w1.x; f[5] *= w1.y; f[6] *= w1.z; f[7] *= w1.w;
+      }
+      float y[8];
+      if (a.interleaved) {
+        if (turns_here && (is_q || is_k)) {
+#pragma unroll
+          for (int u = 0; u < 8; u += 2) {
+            if (e0 + u >= a.dims) continue;
+            const float c = cs[(e0 + u) >> 1], s = sn[(e0 + u) >> 1], x0 = f[u], x1 = f[u + 1];
+            f[u] = fmaf(x0, c, -x1 * s);
+            f[u + 1] = fmaf(x1, c, x0 * s);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int u = 0; u < 8; ++u) y[u] = __shfl_sync(0xffffffffu, f[u], mate);
+        if (turns_here && (is_q || is_k)) {
+          const int at = second ? e0 - half : e0;
+#pragma unroll
+          for (int u = 0; u < 8; ++u) f[u] = fmaf(f[u], cs[at + u], (second ? y[u] : -y[u]) * sn[at + u]);
+        }
+      }
+      if (live && (is_q || stored)) {
+        int4 o;
+        T* oe = reinterpret_cast<T*>(&o);
+#pragma unroll
+        for (int u = 0; u < 8; ++u) oe[u] = Elem<T>::from_f32(f[u] * r);
+        T* dst = is_q ? const_cast<T*>(row_of(item))
+                      : is_k ? reinterpret_cast<T*>(a.k_cache) + (slot * a.Hkv + item - a.Hq) * a.KP
+                             : reinterpret_cast<T*>(a.v_cache) + (slot * a.Hkv + item - a.Hq - a.Hkv) * a.VP;
+        st16(dst + e0, o);
+      }
+    }
+  }
+}
+
+template <typename T> static int launch_rotate(const RotateArgs& a, int n_tokens, cudaStream_t st) {
+  const uintptr_t al = (uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache |
+                       (uintptr_t)a.q_weight | (uintptr_t)a.k_weight;
+  const int widest = a.D > a.DV ? a.D : a.DV;
+  if (sizeof(T) == 2 && a.D % 8 == 0 && a.DV % 8 == 0 && a.KP % 8 == 0 && a.VP % 8 == 0 && a.row_stride % 8 == 0 && widest <= 256 &&
+      (a.interleaved || a.dims % 16 == 0) && al % 16 == 0) {
+    const size_t smem = sizeof(float) * a.dims;
+    if (widest <= 128) rotate_store_vec_kernel<T, 16, 3><<<n_tokens, RO_THREADS, smem, st>>>(a);
+    else rotate_store_vec_kernel<T, 32, 3><<<n_tokens, RO_THREADS, smem, st>>>(a);
+  } else {
+    const bool vec = a.D % 4 == 0 && a.DV % 4 == 0 && a.KP % 4 == 0 && a.VP % 4 == 0 && a.row_stride % 4 == 0 && al % 16 == 0;
+    const size_t smem = sizeof(float) * (((a.dims + 3) & ~3) + RO_WARPS * ((a.D + 3) & ~3));
+    if (vec) rotate_store_kernel<T, 4><<<n_tokens, RO_THREADS, smem, st>>>(a);
+    else rotate_store_kernel<T, 1><<<n_tokens, RO_THREADS, smem, st>>>(a);
+  }
+  return check_launch("zp_rotate_store");
+}
+
 }  // namespace zp
 
 extern "C" int zp_rotate_store(void* q, const void* k, const void* v, int64_t row_stride, const int64_t* positions,
@@ -132,12 +247,6 @@ extern "C" int zp_rotate_store(void* q, const void* k, const void* v, int64_t ro
              "zp_rotate_store: bad sizes (heads of %d with %d rotated entries)", D, dims);
   zp::RotateArgs a{q, k, v, row_stride, positions, turns, q_weight, k_weight, k_cache, v_cache, slot_mapping, n_slots,
                    Hq, Hkv, D, DV, KP, VP, dims, interleaved, mul, eps};
-  const bool vec = D % 4 == 0 && DV % 4 == 0 && KP % 4 == 0 && VP % 4 == 0 && row_stride % 4 == 0 &&
-                   ((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16 == 0;
-  const size_t smem = sizeof(float) * (((dims + 3) & ~3) + zp::RO_WARPS * ((D + 3) & ~3));
-  ZP_DISPATCH_DTYPE(dtype, T, {
-    if (vec) zp::rotate_store_kernel<T, 4><<<n_tokens, zp::RO_THREADS, smem, (cudaStream_t)stream>>>(a);
-    else zp::rotate_store_kernel<T, 1><<<n_tokens, zp::RO_THREADS, smem, (cudaStream_t)stream>>>(a);
-  });
-  return zp::check_launch("zp_rotate_store");
+  ZP_DISPATCH_DTYPE(dtype, T, { return zp::launch_rotate<T>(a, n_tokens, (cudaStream_t)stream); });
+  return ZP_OK;
 }

@@ -200,6 +200,21 @@ template <> struct Pair<__half> {
   static __device__ __forceinline__ float2 unpack(V v) { return __half22float2(v); }
 };
 
+// 4 x 4 transpose of 16-byte chunks within groups of four lanes: v[i] of lane t <- v[t] of lane i.  Turns
+// "one row per lane" into "four lanes per row", so that global accesses touch whole 64-byte row pieces.
+__device__ __forceinline__ void transpose4(int4 (&v)[4], int lane) {
+  auto swap = [&](int4& x, int4& y, int mask, bool upper) {
+    int4 snd = upper ? x : y, rcv;
+    rcv.x = __shfl_xor_sync(0xffffffffu, snd.x, mask); rcv.y = __shfl_xor_sync(0xffffffffu, snd.y, mask);
+    rcv.z = __shfl_xor_sync(0xffffffffu, snd.z, mask); rcv.w = __shfl_xor_sync(0xffffffffu, snd.w, mask);
+    if (upper) x = rcv; else y = rcv;
+  };
+  swap(v[0], v[1], 1, lane & 1);
+  swap(v[2], v[3], 1, lane & 1);
+  swap(v[0], v[2], 2, lane & 2);
+  swap(v[1], v[3], 2, lane & 2);
+}
+
 // ---- descriptors ----------------------------------------------------------------------------------
 // K-major operand tile in shared memory, 128-byte swizzle: rows of 128 bytes, 8-row groups 1024
 // bytes apart (stride byte offset 1024), leading byte offset unused (1), descriptor version 1.
