@@ -256,7 +256,7 @@ __global__ void __launch_bounds__(DP_THREADS, 3) delta_prepare_kernel(const Delt
     for (int d = 1; d < 4; ++d) {
       if (warp < 4 - d) {
         const int j = warp, i = warp + d;
-        float x[2][4] = {};                      // the sum, transposed: it is the next product's right operand as it lies
+        float x[2][4] = {}, xa[2][4] = {}, xb[2][4] = {};      // the sum, transposed: it is the next product's right operand as it lies
 #pragma unroll
         for (int k0 = 0; k0 < d; ++k0) {
           const int k = j + k0;
@@ -268,13 +268,15 @@ __global__ void __launch_bounds__(DP_THREADS, 3) delta_prepare_kernel(const Delt
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             mma16816<T>(x[e], wh, ah[2 * e], ah[2 * e + 1]);
-            mma16816<T>(x[e], wh, al[2 * e], al[2 * e + 1]);
-            mma16816<T>(x[e], wl, ah[2 * e], ah[2 * e + 1]);
+            mma16816<T>(xa[e], wh, al[2 * e], al[2 * e + 1]);
+            mma16816<T>(xb[e], wl, ah[2 * e], ah[2 * e + 1]);
           }
         }
         uint32_t xh[2][2], xl[2][2];             // [column block][half of k]
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
+#pragma unroll
+          for (int u = 0; u < 4; ++u) x[e][u] += xa[e][u] + xb[e][u];
           dc_split(x[e][0], x[e][1], xh[0][e], xl[0][e]);
           dc_split(x[e][2], x[e][3], xh[1][e], xl[1][e]);
         }
@@ -284,10 +286,12 @@ __global__ void __launch_bounds__(DP_THREADS, 3) delta_prepare_kernel(const Delt
         ldmatrix_x4(tl, tLo + tr);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          float y[4] = {};
+          float y[4] = {}, ya[4] = {}, yb[4] = {};
           mma16816<T>(y, th, xh[e][0], xh[e][1]);
-          mma16816<T>(y, th, xl[e][0], xl[e][1]);
-          mma16816<T>(y, tl, xh[e][0], xh[e][1]);
+          mma16816<T>(ya, th, xl[e][0], xl[e][1]);
+          mma16816<T>(yb, tl, xh[e][0], xh[e][1]);
+#pragma unroll
+          for (int u = 0; u < 4; ++u) y[u] += ya[u] + yb[u];
           uint32_t hi, lo;
           const int oa = dp_piece(i * 16 + g, 2 * j + e) + tq * 4, ob = dp_piece(i * 16 + g + 8, 2 * j + e) + tq * 4;
           dc_split(-y[0], -y[1], hi, lo);
@@ -319,12 +323,12 @@ __global__ void __launch_bounds__(DP_THREADS, 3) delta_prepare_kernel(const Delt
           uint32_t bh[4], bl[4];
           ldmatrix_x4_trans(bh, wHi + off);
           ldmatrix_x4_trans(bl, wLo + off);
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            mma16816<T>(m[2 * np + e], ph, bh[2 * e], bh[2 * e + 1]);
-            mma16816<T>(m[2 * np + e], ph, bl[2 * e], bl[2 * e + 1]);
-            mma16816<T>(m[2 * np + e], pl, bh[2 * e], bh[2 * e + 1]);
-          }
+          mma16816<T>(m[2 * np], ph, bh[0], bh[1]);
+          mma16816<T>(m[2 * np + 1], ph, bh[2], bh[3]);
+          mma16816<T>(m[2 * np], ph, bl[0], bl[1]);
+          mma16816<T>(m[2 * np + 1], ph, bl[2], bl[3]);
+          mma16816<T>(m[2 * np], pl, bh[0], bh[1]);
+          mma16816<T>(m[2 * np + 1], pl, bh[2], bh[3]);
         }
       }
 #pragma unroll
@@ -390,17 +394,16 @@ __device__ __forceinline__ void ds_ld16(uint32_t taddr, float (&v)[16]) {   // l
   for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
 }
 __device__ __forceinline__ float ds_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
-// push a float into / arrive on a barrier of another block of the cluster
+// a float into the shared memory of a block of the cluster (the same place), counted by that block's barrier: no release
+// that would wait for the warp's stores to global memory
 __device__ __forceinline__ uint32_t ds_map(const void* p, uint32_t rank) {
   uint32_t ra;
   asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(p)), "r"(rank));
   return ra;
 }
-__device__ __forceinline__ void ds_push(const float* p, uint32_t rank, float v) {
-  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(ds_map(p, rank)), "f"(v) : "memory");
-}
-__device__ __forceinline__ void ds_arrive_peer(const uint64_t* bar, uint32_t rank) {
-  asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(ds_map(bar, rank)) : "memory");
+__device__ __forceinline__ void ds_push(const float* p, const uint64_t* bar, uint32_t rank, float v) {
+  asm volatile("st.async.weak.shared::cluster.mbarrier::complete_tx::bytes.b32 [%0], %1, [%2];"
+               ::"r"(ds_map(p, rank)), "r"(__float_as_uint(v)), "r"(ds_map(bar, rank)) : "memory");
 }
 __device__ __forceinline__ bool ds_wait_cluster(uint64_t* bar, uint32_t parity, volatile int* abort_flag, int* error_word, int where) {
   for (uint32_t i = 0; i < WAIT_LIMIT; ++i) {
@@ -448,7 +451,7 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     mbar_init(&sh.full, 2); mbar_init(&sh.vfull, 1); mbar_init(&sh.ifull, 1); mbar_init(&sh.sready, 8); mbar_init(&sh.zfull, 1);
     mbar_init(&sh.rready, 4); mbar_init(&sh.yfull, 1); mbar_init(&sh.uready, 4); mbar_init(&sh.dfull, 1);
     mbar_init(&sh.oread, 4);
-    for (int i = 0; i < 2; ++i) { mbar_init(&sh.ffull[i], 1); mbar_init(&sh.xbar[i], 4 * tiles); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&sh.ffull[i], 1); mbar_init(&sh.xbar[i], 1); }
     sh.abort_flag = 0;
     fence_mbar_init();
   }
@@ -677,12 +680,10 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         }
       }
       fence_before_sync();
-      for (int k = 0; k < tiles; ++k) ds_push(&sh.xs[ph][2 * vt + cq][t], k, ss);
+      if (warp == 0 && lane == 0) mbar_arrive_expect_tx(&sh.xbar[ph], 2 * tiles * 64 * 4);
+      for (int k = 0; k < tiles; ++k) ds_push(&sh.xs[ph][2 * vt + cq][t], &sh.xbar[ph], k, ss);
       __syncwarp();
-      if (lane == 0) {
-        mbar_arrive(&sh.oread);
-        for (int k = 0; k < tiles; ++k) ds_arrive_peer(&sh.xbar[ph], k);
-      }
+      if (lane == 0) mbar_arrive(&sh.oread);
       // the output gate, four lanes per row (lane u of a group: chunk u of the group's rows)
       int4 in[4];
 #pragma unroll
