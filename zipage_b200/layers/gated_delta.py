@@ -12,7 +12,6 @@ from torch import nn
 from .. import _lib as L
 from ..kernel import _count
 from ..utils.context import get_context
-from .attention import _workspace
 
 
 def short_conv(x, weight, ring, context_lens, slots, cu_seqlens_q, max_seqlen_q, out):
@@ -36,9 +35,9 @@ def gated_delta(x, gate, ab, A_log, dt_bias, norm_weight, state, out, context_le
     assert x.stride(1) == gate.stride(1) == ab.stride(1) == out.stride(1) == 1 and ab.dtype == state.dtype == torch.float32
     assert state.is_contiguous() and state.shape[1:3] == (heads, dim) and x.dtype == gate.dtype == out.dtype
     lib, B = L.load(), context_lens.shape[0]
-    ws = None
+    ws = None                # (portions never run inside a graph: an allocation of this call's size)
     if cu_seqlens_q is not None and x.dtype == torch.bfloat16 and impl != "simt":
-        ws = _workspace(x.device, lib.zp_gated_delta_workspace_bytes(x.shape[0], B, heads))
+        ws = torch.empty(lib.zp_gated_delta_workspace_bytes(x.shape[0], B, heads), dtype=torch.uint8, device=x.device)
     L.check(lib.zp_gated_delta(
         L.ptr(x), x.stride(0), L.ptr(gate), gate.stride(0), L.ptr(ab), ab.stride(0), L.ptr(A_log), L.ptr(dt_bias), L.ptr(norm_weight),
         L.ptr(conv_weight), L.ptr(ring), 0 if conv_weight is None else conv_weight.shape[0], L.ptr(cu_seqlens_q), L.ptr(context_lens),
