@@ -53,6 +53,7 @@ extern "C" {
 #define ZP_ACT_SILU_MUL 2
 #define ZP_SCORE_SOFTMAX 0
 #define ZP_SCORE_SIGMOID 1
+#define ZP_SCORE_SOFTMAX_TOP 2   /* softmax over the chosen logits alone */
 
 const char* zp_last_error(void);
 int zp_version(void);
@@ -406,9 +407,10 @@ int zp_sample_sharded_emulated(zp_comm* const* comms, int world, const void* con
 
 /* x[n, :] = table[tokens[n], :] * scale + position vector, fp32, and its copy x_t as T (may be NULL).
  * Position vector: entries 2i / 2i + 1 = sin / cos of 2 pi positions[n] turns[i]; turns [(hidden + 1)
- * / 2] fp64 on the device, NULL = no position vector.  Ids outside [0, vocab) are clamped. */
+ * / 2] fp64 on the device, NULL = none.  learned [n_learned, hidden] of T (instead of turns): row positions[n] is
+ * added (positions past the table are clamped).  Ids outside [0, vocab) are clamped. */
 int zp_embed_position(const int64_t* tokens, const int64_t* positions, const void* table, const double* turns,
-                      float scale, float* x, void* x_t, int n_tokens, int hidden, int64_t vocab, int dtype,
+                      float scale, const void* learned, int64_t n_learned, float* x, void* x_t, int n_tokens, int hidden, int64_t vocab, int dtype,
                       void* stream);
 
 /* out = T(x * rsqrt(mean(x^2) + eps) * (weight + weight_offset)) over fp32 rows x [n_rows, hidden]
@@ -429,7 +431,8 @@ int zp_store_kv_padded(const void* k, const void* v, void* k_cache, void* v_cach
 /* Softmax attention of a step's queries over paged keys, with masks, a soft cap, a sink and an output gate:
  * score = q . k * scale; softcap > 0: score = softcap * tanh(score / softcap); the query at position p
  * sees the keys j <= p, of these with window > 0 only p - j < window, with chunk > 0 only floor(j / chunk) =
- * floor(p / chunk).  sink [Hq] (or NULL): the softmax's denominator also has exp(sink[h]).  The result is
+ * floor(p / chunk), and with keep > 0 the keys j < keep in any case.  slopes [Hq] fp32 (or NULL): slopes[h] * (p - j) is taken
+ * off the (capped) score.  sink [Hq] (or NULL): the softmax's denominator also has exp(sink[h]).  The result is
  * multiplied by out_scale and, with gate_mode 1 (2), by sigmoid(gate), gate [rows, Hq] ([rows, Hq * DV]) of T
  * with its own row stride.
  * q [rows, Hq, D] (row stride), caches [n_pages, BS, Hkv, KP | VP] as zp_store_kv_padded leaves them,
@@ -446,7 +449,7 @@ int zp_window_attention(const void* q, const void* k_cache, const void* v_cache,
                         const int32_t* context_lens, const int32_t* block_table, void* out, int B,
                         int max_seqlen_q, int NBmax, int Hq, int Hkv, int D, int DV, int KP, int VP, int BS,
                         int n_pages, int64_t q_stride, int64_t out_stride, float scale, float softcap,
-                        int window, int chunk, const float* sink, const void* gate, int64_t gate_stride, int gate_mode,
+                        int window, int chunk, int keep, const float* slopes, const float* sink, const void* gate, int64_t gate_stride, int gate_mode,
                         float out_scale, int total_q, int impl, int dtype, void* workspace, size_t workspace_bytes,
                         void* stream);
 
@@ -475,6 +478,7 @@ int zp_mlstm(const void* q, const void* k, const void* v, const void* g, const f
 
 /* The boundary between two layers, per fp32 row of x [n_rows, hidden], in place:
  *   x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k weights[k] * y[pos[k]])
+ *        + pair_scale * (rms(m1) * mw1 + rms(m2) * mw2)      (each row over its root mean square; m1, m2 both NULL: none)
  *   out1 = T(norm of x * w1 + bias1), out2 likewise  (layer norm: variance = mean of the squared deviations; rms 1: no
  *   mean taken off)
  * a, b [n_rows, hidden] of T, ls_* [hidden] fp32 (NULL = ones), gate: one fp32 number per row at stride
@@ -482,7 +486,7 @@ int zp_mlstm(const void* q, const void* k, const void* v, const void* g, const f
  * a, b, out1 and out2 may be NULL; with no summand x is only read. */
 int zp_join_norms(float* x, const void* a, const float* ls_a, const void* b, const float* ls_b, const float* gate,
                   int64_t gate_stride, const void* y, int64_t y_rows, const int32_t* pos, const float* weights,
-                  int top, const float* w1, const float* bias1, void* out1, const float* w2, const float* bias2,
+                  int top, const void* m1, const float* mw1, const void* m2, const float* mw2, float pair_scale, const float* w1, const float* bias1, void* out1, const float* w2, const float* bias2,
                   void* out2, int n_rows, int hidden, float eps, int rms, int dtype, void* stream);
 
 /* gate | up [n_rows, 2 width] -> T(gelu_tanh(gate) * up) [n_rows, width] */
@@ -538,12 +542,12 @@ int zp_latent_prefill(const void* q, int64_t q_stride, const void* kv, const voi
 int zp_gather_rows(const void* cache, const int32_t* block_table, const int32_t* cu_seqlens_k, void* dense, int B,
                    int NBmax, int BS, int n_pages, int row_bytes, int total, void* stream);
 
-/* Routing: logits [n_tokens, n_experts] fp32 (row stride, at most 1024 experts), s = softmax over all
- * experts (ZP_SCORE_SOFTMAX) or sigmoid (ZP_SCORE_SIGMOID); the top largest of a token (ties: the lower expert) with weights s, not renormalised.
+/* Routing: logits [n_tokens, n_experts] fp32 (row stride, at most 1024 experts) + bias [n_experts] (or NULL), s = softmax over all
+ * experts (ZP_SCORE_SOFTMAX) or over the chosen ones (ZP_SCORE_SOFTMAX_TOP), or sigmoid (ZP_SCORE_SIGMOID); the top largest of a token (ties: the lower expert) with weights s, not renormalised.
  * weights, experts, places [n_tokens, top]; the n_tokens * top pairs sorted by expert: expert e has the places
  * offsets[e] .. offsets[e + 1] ([n_experts + 1]), rows[place] = its token.  counts [n_experts]: scratch.
  * place_weights [n_tokens * top] (may be NULL): the weights in the order of the places. */
-int zp_moe_route(const float* logits, int64_t row_stride, int n_tokens, int n_experts, int top, float* weights,
+int zp_moe_route(const float* logits, int64_t row_stride, const float* bias, int n_tokens, int n_experts, int top, float* weights,
                  int32_t* experts, int32_t* places, int32_t* rows, int32_t* offsets, int32_t* counts, float* place_weights,
                  int score, void* stream);
 
@@ -571,11 +575,11 @@ int zp_rotate_store(void* q, const void* k, const void* v, int64_t row_stride, c
                     int n_tokens, int Hq, int Hkv, int D, int DV, int KP, int VP, int64_t n_slots, int dtype,
                     void* stream);
 
-/* out[t, c] = silu(sum_j weight[taps - 1 - j, c] x[t - j, c]) over the portions of a step: sequence b has the rows
+/* out[t, c] = silu(bias[c] + sum_j weight[taps - 1 - j, c] x[t - j, c]) (bias NULL = 0) over the portions of a step: sequence b has the rows
  * cu_seqlens_q[b] .. of x [rows, channels] (row stride) and out; earlier inputs come from ring [n_slots, taps, channels], where
  * position p lies in row p % taps, and are zero before position 0.  The portion's last inputs go into the ring.
  * weight [taps, channels] fp32, at most 8 taps; context_lens counts each sequence's tokens including these. */
-int zp_short_conv(const void* x, int64_t x_stride, const float* weight, void* ring, const int32_t* cu_seqlens_q,
+int zp_short_conv(const void* x, int64_t x_stride, const float* weight, const float* bias, void* ring, const int32_t* cu_seqlens_q,
                   const int32_t* context_lens, const int32_t* slots, void* out, int64_t out_stride, int B,
                   int max_seqlen_q, int channels, int taps, int n_slots, int dtype, void* stream);
 
@@ -596,6 +600,53 @@ int zp_gated_delta(const void* x, int64_t x_stride, const void* gate, int64_t ga
                    const int32_t* context_lens, const int32_t* slots, float* state, void* out, int64_t out_stride,
                    int B, int H, int G, int dim, int vdim, int VP, int n_slots, float eps, float out_scale,
                    int total_rows, int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream);
+
+/* ---- Linear attention with decaying states, group norms with gates ------------------------------------
+ * No counterpart in the reference.  The Dinatar decoder runs on these; each takes its constants as parameters. */
+
+/* Where a linear-attention state's decays come from (a per head and key channel, or per head), with z = gate + gate_bias:
+ *   FORGET: a = l + (1 - l) sigmoid(z), key 1 - a, query silu(q);          l = lower
+ *   POWER:  a = sigmoid(z)^rtau, key k, query q qscale
+ *   SCALAR: dt = softplus(z), a = exp(-exp(A_log) dt), key dt k, query q; D v joins the output */
+#define ZP_LINEAR_FORGET 0
+#define ZP_LINEAR_POWER 1
+#define ZP_LINEAR_SCALAR 2
+
+typedef struct zp_linear_state_params {
+  int32_t kind, B, H, G;        /* G: heads of q and k (SCALAR; head h uses h / (H / G)), else H    */
+  int32_t dim, vdim, VP, n_slots, taps, total_rows;
+  const void *q, *k, *v;        /* [rows, G dim | G dim | H vdim] of T, one row stride; k unused by FORGET */
+  int64_t x_stride;
+  const float* gate;            /* [rows, H dim], SCALAR: [rows, H]                                  */
+  int64_t gate_stride;
+  const float *gate_bias;       /* [H dim], SCALAR: [H]                                              */
+  const float *lower;           /* FORGET: [H dim]                                                   */
+  const float *A_log, *D;       /* SCALAR: [H]                                                       */
+  const float *conv_weight, *conv_bias;   /* taps > 0: [taps, channels], [channels]                  */
+  void* ring;                   /* taps > 0: [n_slots, taps, channels] of T                          */
+  const int32_t *cu_seqlens_q, *context_lens, *slots;
+  float* state;                 /* [n_slots, H, dim, VP], VP >= vdim, a multiple of 4                */
+  void* out;                    /* [rows, H vdim] of T, row stride out_stride                        */
+  int64_t out_stride;
+  float rtau, qscale;
+  void* workspace;
+  size_t workspace_bytes;
+} zp_linear_state_params;
+
+/* One step of S <- diag(a) S + k v^T, o = S^T q over a batch of sequences, token after token of each; S fp32, in place, in
+ * the sequences' slots.  Rows, contexts and slots as in zp_mlstm.  taps > 0 (SCALAR, single rows only): q, k and v are
+ * columns of the input of the convolution of zp_short_conv with channels v | k | q, which is then part of the launch.
+ * bf16 portions with key sizes up to 128, key and value sizes that are multiples of 8 and at least 8 rows per sequence on average
+ * take the chunked tcgen05 kernels (ZP_IMPL_SIMT: never; ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED), which need a workspace. */
+size_t zp_linear_state_workspace_bytes(int total_rows, int B, int H, int dim);
+int zp_linear_state(const zp_linear_state_params* params, int impl, int dtype, void* stream);
+
+/* out [n_rows, parts * width] = T(rms(pre * x) * weight * post), each of the `parts` equal parts of a row over its own root mean
+ * square; x [n_rows, parts * width] of T; pre = silu(pre_gate), post = silu(post_gate), each with a row stride of its own (NULL = 1);
+ * weight fp32 [width], or [parts * width] with weight_per_part.  out may be x. */
+int zp_group_norm_gate(const void* x, int64_t x_stride, const void* pre_gate, int64_t pre_stride, const void* post_gate,
+                       int64_t post_stride, const float* weight, int weight_per_part, void* out, int64_t out_stride, int n_rows,
+                       int parts, int width, float eps, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

@@ -79,7 +79,7 @@ def test_argument_errors_come_back_as_errors():
     build()
     lib = L.load()
     one = L.C.c_void_p(16)
-    assert lib.zp_moe_route(one, 8, 4, 8, 9, one, one, one, one, one, one, None, 0, None) == -1      # more chosen than there are
+    assert lib.zp_moe_route(one, 8, None, 4, 8, 9, one, one, one, one, one, one, None, 0, None) == -1      # more chosen than there are
     assert lib.zp_grouped_gemm(one, 8, None, 4, one, one, None, one, 4, 2, 8, 9, 0, 0, 1, None) == -1   # rows shorter than k
     assert lib.zp_latent_attention(one, one, None, one, one, one, 1, 1, 1, 1, 2, 1100, 1104, 64, 1, 1.0, 0, 0, None, 0, None) == -1
     assert lib.zp_latent_prefill_supported(128, 64, 128, 512, 576, 0) == 1

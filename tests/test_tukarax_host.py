@@ -86,7 +86,7 @@ def test_argument_errors_come_back_as_errors():
     build()
     lib = L.load()
     one = L.C.c_void_p(16)
-    conv = lambda taps: lib.zp_short_conv(one, 8, one, one, one, one, one, one, 8, 1, 1, 8, taps, 1, 0, None)
+    conv = lambda taps: lib.zp_short_conv(one, 8, one, None, one, one, one, one, one, 8, 1, 1, 8, taps, 1, 0, None)
     assert conv(9) == -1 and conv(0) == -1
     delta = lambda taps, cu, H, G, impl, dim: lib.zp_gated_delta(one, 64, one, 64, one, 8, one, one, one, one, one, taps, cu, one, one, one,
                                                                  one, 64, 1, H, G, dim, 8, 8, 1, 1e-5, 1.0, 4, impl, 0, None, 0, None)
@@ -99,7 +99,7 @@ def test_argument_errors_come_back_as_errors():
     assert rot(10, 8) == -1 and rot(3, 8) == -1 and rot(8, 24) == -1
     grouped = lambda n_out, act, scale: lib.zp_grouped_gemm(one, 8, None, 4, one, one, scale, one, 4, 2, n_out, 8, act, 0, 1, None)
     assert grouped(48, 2, None) == -1 and grouped(64, 1, one) == -1
-    assert lib.zp_moe_route(one, 8, 4, 8, 2, one, one, one, one, one, one, None, 7, None) == -1
+    assert lib.zp_moe_route(one, 8, None, 4, 8, 2, one, one, one, one, one, one, None, 7, None) == -1
     assert lib.zp_gated_delta_workspace_bytes(0, 1, 1) == 0 and lib.zp_gated_delta_workspace_bytes(200, 2, 3) > 0
 
 

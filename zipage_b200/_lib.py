@@ -15,7 +15,7 @@ LIB_PATH = _PKG / "libzipage_b200.so"
 
 ZP_DTYPE = {torch.bfloat16: 0, torch.float32: 1, torch.float16: 2}
 ACT = {None: 0, "relu_squared": 1, "silu_mul": 2}
-SCORE = {"softmax": 0, "sigmoid": 1}
+SCORE = {"softmax": 0, "sigmoid": 1, "softmax_top": 2}
 GATE = {None: 0, "head": 1, "entry": 2}
 IMPL = {"auto": 0, "simt": 1, "tcgen05": 2}
 
@@ -43,6 +43,14 @@ class CompressParams(C.Structure):
         ("redundancy_temperature", C.c_float), ("redundancy_threshold", C.c_float),
         ("softmax_scale", C.c_float),
     ]
+
+
+class LinearStateParams(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("kind", "B", "H", "G", "dim", "vdim", "VP", "n_slots", "taps", "total_rows")] + [
+        ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("x_stride", C.c_int64), ("gate", C.c_void_p), ("gate_stride", C.c_int64)] + [
+        (n, C.c_void_p) for n in ("gate_bias", "lower", "A_log", "D", "conv_weight", "conv_bias", "ring", "cu_seqlens_q", "context_lens",
+                                  "slots", "state", "out")] + [
+        ("out_stride", C.c_int64), ("rtau", C.c_float), ("qscale", C.c_float), ("workspace", C.c_void_p), ("workspace_bytes", C.c_size_t)]
 
 
 _P, _I, _L, _F, _Z = C.c_void_p, C.c_int, C.c_int64, C.c_float, C.c_size_t
@@ -80,14 +88,14 @@ SIGNATURES = {
     "zp_qk_norm_rope_store": (_I, [_P] * 5 + [_F] + [_P] * 7 + [_I, _P] + [_I] * 4 + [_L] * 3 + [_I, _P]),
     "zp_sample": (_I, [_P, _P, _P, _P, _I, _I, C.c_uint64, _I, _P]),
     "zp_prepare_decode": (_I, [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P]),
-    "zp_embed_position": (_I, [_P] * 4 + [_F, _P, _P, _I, _I, _L, _I, _P]),
+    "zp_embed_position": (_I, [_P] * 4 + [_F, _P, _L, _P, _P, _I, _I, _L, _I, _P]),
     "zp_rms_norm_f32": (_I, [_P, _P, _F, _P, _I, _I, _F, _I, _P]),
     "zp_gelu_tanh": (_I, [_P, _P, _L, _I, _P]),
     "zp_store_kv_padded": (_I, [_P] * 5 + [_I] * 6 + [_L, _L, _I, _P]),
     "zp_window_attention_workspace_bytes": (_Z, [_I] * 5),
-    "zp_window_attention": (_I, [_P] * 7 + [_I] * 11 + [_L, _L, _F, _F, _I, _I, _P, _P, _L, _I, _F, _I, _I, _I, _P, _Z, _P]),
+    "zp_window_attention": (_I, [_P] * 7 + [_I] * 11 + [_L, _L, _F, _F, _I, _I, _I, _P, _P, _P, _L, _I, _F, _I, _I, _I, _P, _Z, _P]),
     "zp_mlstm": (_I, [_P] * 14 + [_I] * 6 + [_L] * 3 + [_F] * 3 + [_I, _I, _I, _P]),
-    "zp_join_norms": (_I, [_P] * 6 + [_L, _P, _L, _P, _P, _I] + [_P] * 6 + [_I, _I, _F, _I, _I, _P]),
+    "zp_join_norms": (_I, [_P] * 6 + [_L, _P, _L, _P, _P, _I] + [_P] * 4 + [_F] + [_P] * 6 + [_I, _I, _F, _I, _I, _P]),
     "zp_gelu_tanh_and_mul": (_I, [_P, _P, _I, _I, _I, _P]),
     "zp_relu_squared": (_I, [_P, _P, _L, _I, _P]),
     "zp_soft_cap": (_I, [_P, _L, _F, _P]),
@@ -98,12 +106,15 @@ SIGNATURES = {
     "zp_latent_prefill_supported": (_I, [_I] * 6),
     "zp_latent_prefill": (_I, [_P, _L] + [_P] * 5 + [_L] + [_I] * 10 + [_F, _I, _P]),
     "zp_gather_rows": (_I, [_P] * 4 + [_I] * 6 + [_P]),
-    "zp_moe_route": (_I, [_P, _L, _I, _I, _I] + [_P] * 7 + [_I, _P]),
+    "zp_moe_route": (_I, [_P, _L, _P, _I, _I, _I] + [_P] * 7 + [_I, _P]),
     "zp_grouped_gemm": (_I, [_P, _L, _P, _I, _P, _P, _P, _P] + [_I] * 7 + [_P]),
     "zp_rotate_store": (_I, [_P, _P, _P, _L, _P, _P, _I, _I, _F, _P, _P, _F, _P, _P, _P] + [_I] * 7 + [_L, _I, _P]),
-    "zp_short_conv": (_I, [_P, _L] + [_P] * 6 + [_L] + [_I] * 6 + [_P]),
+    "zp_short_conv": (_I, [_P, _L] + [_P] * 7 + [_L] + [_I] * 6 + [_P]),
     "zp_gated_delta_workspace_bytes": (_Z, [_I] * 3),
     "zp_gated_delta": (_I, [_P, _L, _P, _L, _P, _L] + [_P] * 5 + [_I] + [_P] * 5 + [_L] + [_I] * 7 + [_F, _F, _I, _I, _I, _P, _Z, _P]),
+    "zp_linear_state_workspace_bytes": (_Z, [_I] * 4),
+    "zp_linear_state": (_I, [C.POINTER(LinearStateParams), _I, _I, _P]),
+    "zp_group_norm_gate": (_I, [_P, _L, _P, _L, _P, _L, _P, _I, _P, _L, _I, _I, _I, _F, _I, _P]),
     "zp_comm_create": (_I, [_I, _I, _Z, _I, C.POINTER(_P)]),
     "zp_comm_segment": (_I, [_P, C.POINTER(_P), C.POINTER(_Z)]),
     "zp_comm_ipc_handle": (_I, [_P, _P]),

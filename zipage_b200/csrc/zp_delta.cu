@@ -6,6 +6,7 @@
 // correction needs (S^T k) and the update are one pass over memory: with S^T k and S^T q of the old state,
 //   u = b (v - g S^T k),   o = g S^T q + (k . q) u,   S <- g S + k u^T.
 // The blocks of a head form a cluster when there are several: the output norm spans all value dims.
+#include "zp_conv.cuh"
 #include "zp_delta.cuh"
 #include "zp_mlstm.cuh"    // cluster helpers
 #include "zp_tc.cuh"       // packed fp32 pairs
@@ -13,37 +14,6 @@
 namespace zp {
 
 constexpr int DR_THREADS = 256;
-
-// The inputs of one channel's convolution at a token, all loads in flight together (more than four taps: the rest in
-// `conv_finish`).
-template <typename T> struct ConvIn { T now, back[3]; float w[4]; };
-struct ConvPlace { int C, taps, row, seen; };          // row p % taps of the ring; how many earlier inputs there are
-template <typename T>
-__device__ __forceinline__ void conv_start(ConvIn<T>& v, const DeltaArgs& a, const ConvPlace& at, const T* xr, const T* ring, int c) {
-  v.now = xr[c];
-  v.w[0] = a.conv_w[(int64_t)(at.taps - 1) * at.C + c];
-#pragma unroll
-  for (int j = 1; j < 4; ++j) {
-    v.back[j - 1] = Elem<T>::from_f32(0.f);
-    v.w[j] = 0.f;
-    if (j <= at.seen) {
-      const int r = at.row - j;
-      v.back[j - 1] = ring[(int64_t)(r < 0 ? r + at.taps : r) * at.C + c];
-      v.w[j] = a.conv_w[(int64_t)(at.taps - 1 - j) * at.C + c];
-    }
-  }
-}
-template <typename T>
-__device__ __forceinline__ float conv_finish(const ConvIn<T>& v, const DeltaArgs& a, const ConvPlace& at, const T* ring, int c) {
-  float acc = Elem<T>::to_f32(v.now) * v.w[0];
-#pragma unroll
-  for (int j = 1; j < 4; ++j) acc = fmaf(Elem<T>::to_f32(v.back[j - 1]), v.w[j], acc);
-  for (int j = 4; j <= at.seen; ++j) {
-    const int r = at.row - j;
-    acc = fmaf(Elem<T>::to_f32(ring[(int64_t)(r < 0 ? r + at.taps : r) * at.C + c]), a.conv_w[(int64_t)(at.taps - 1 - j) * at.C + c], acc);
-  }
-  return acc / (1.f + expf(-acc));
-}
 
 template <typename T, int RPT>   // RPT: state rows per thread
 __global__ void __launch_bounds__(DR_THREADS, RPT == 16 ? 2 : RPT == 8 ? 3 : 4) delta_recurrent_kernel(const DeltaArgs a) {
@@ -70,7 +40,7 @@ __global__ void __launch_bounds__(DR_THREADS, RPT == 16 ? 2 : RPT == 8 ? 3 : 4) 
     s[i] = (mine && r < a.dim && !sq.fresh) ? *reinterpret_cast<const float4*>(S + (int64_t)r * a.VP) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   const T* x = reinterpret_cast<const T*>(a.x);
-  T* ring = reinterpret_cast<T*>(a.ring) + (int64_t)sq.slot * a.taps * C;
+  ConvSource<T> cv{a.conv_w, nullptr, reinterpret_cast<T*>(a.ring) + (int64_t)sq.slot * a.taps * C, C, a.taps, 0, 0};
   const float qscale = rsqrtf((float)a.dim), nw = out_col ? a.norm_weight[c0 + tid] : 0.f;
   const bool keeper = h % group == 0 && vt == 0;      // of the keys' and queries' inputs
 
@@ -79,8 +49,7 @@ __global__ void __launch_bounds__(DR_THREADS, RPT == 16 ? 2 : RPT == 8 ? 3 : 4) 
     const int p = sq.ctx - sq.count + t;
     const T* xr = x + row * a.x_stride;
     const float z = out_col ? Elem<T>::to_f32(reinterpret_cast<const T*>(a.gate)[row * a.gate_stride + (int64_t)h * a.vdim + c0 + tid]) : 0.f;
-    ConvPlace at{C, a.taps, 0, 0};
-    if (a.taps) { at.row = p % a.taps; at.seen = min(p, a.taps - 1); }
+    if (a.taps) { cv.row = p % a.taps; cv.seen = min(p, a.taps - 1); }
     float qq = 0.f, kk = 0.f, kq = 0.f;
     if (tid < 128) {             // queries and keys; the other half brings the values
 #pragma unroll 1
@@ -89,14 +58,11 @@ __global__ void __launch_bounds__(DR_THREADS, RPT == 16 ? 2 : RPT == 8 ? 3 : 4) 
         float q, k;
         if (a.taps) {
           ConvIn<T> vq, vk;
-          conv_start(vq, a, at, xr, ring, cq);
-          conv_start(vk, a, at, xr, ring, ck);
-          q = conv_finish(vq, a, at, ring, cq);
-          k = conv_finish(vk, a, at, ring, ck);
-          if (keeper) {
-            ring[(int64_t)at.row * C + cq] = vq.now;
-            ring[(int64_t)at.row * C + ck] = vk.now;
-          }
+          conv_start(vq, cv, xr[cq], cq);
+          conv_start(vk, cv, xr[ck], ck);
+          q = conv_finish(vq, cv, cq);
+          k = conv_finish(vk, cv, ck);
+          if (keeper) { conv_keep(vq, cv, cq); conv_keep(vk, cv, ck); }
         } else {
           q = Elem<T>::to_f32(xr[cq]);
           k = Elem<T>::to_f32(xr[ck]);
@@ -105,16 +71,16 @@ __global__ void __launch_bounds__(DR_THREADS, RPT == 16 ? 2 : RPT == 8 ? 3 : 4) 
         qq = fmaf(q, q, qq); kk = fmaf(k, k, kk); kq = fmaf(k, q, kq);
       }
     } else if (tid - 128 < a.VT) {
-      const int c = tid - 128, cv = 2 * a.G * a.dim + h * a.vdim + c0 + c;
+      const int c = tid - 128, ch = 2 * a.G * a.dim + h * a.vdim + c0 + c;
       float v = 0.f;
       if (c0 + c < a.vdim) {
         if (a.taps) {
           ConvIn<T> vv;
-          conv_start(vv, a, at, xr, ring, cv);
-          v = conv_finish(vv, a, at, ring, cv);
-          ring[(int64_t)at.row * C + cv] = vv.now;
+          conv_start(vv, cv, xr[ch], ch);
+          v = conv_finish(vv, cv, ch);
+          conv_keep(vv, cv, ch);
         } else {
-          v = Elem<T>::to_f32(xr[cv]);
+          v = Elem<T>::to_f32(xr[ch]);
         }
       }
       sv[c] = v;
@@ -233,7 +199,7 @@ static int delta_recurrent(DeltaArgs a, cudaStream_t st) {
 // walks a run of tokens in batches, the next batch's loads in flight.
 // ---------------------------------------------------------------------------------------------
 struct ConvArgs {
-  const void* x; const float* w; void* ring; void* out;
+  const void* x; const float* w; const float* bias; void* ring; void* out;
   const int32_t *cu_q, *context_lens, *slots;
   int64_t x_stride, out_stride;
   int C, taps, n_slots;
@@ -281,7 +247,9 @@ __global__ void __launch_bounds__(CV_THREADS, TAPS <= 4 ? 3 : 2) short_conv_kern
       if (t + u < t1) next[u] = cv_load<T, V>(x + (int64_t)(t + u) * a.x_stride);
   };
   fetch(t0);
-  float w[TAPS][V], f[TAPS][V];              // f: inputs of the current token, in a circle
+  float w[TAPS][V], f[TAPS][V], bias[V];     // f: inputs of the current token, in a circle
+#pragma unroll
+  for (int i = 0; i < V; ++i) bias[i] = a.bias ? a.bias[c + i] : 0.f;
 #pragma unroll
   for (int j = 0; j < TAPS - 1; ++j) {       // those ahead of the run
     const int t = t0 + j - (TAPS - 1);
@@ -313,7 +281,7 @@ __global__ void __launch_bounds__(CV_THREADS, TAPS <= 4 ? 3 : 2) short_conv_kern
       cv_floats(cur[u], f[(u + TAPS - 1) % TAPS]);
       float y[V];
       if constexpr (V == 4 && sizeof(T) == 2) {
-        float2 lo = make_float2(0.f, 0.f), hi = lo;      // pairs of channels
+        float2 lo = make_float2(bias[0], bias[1]), hi = make_float2(bias[2], bias[3]);      // pairs of channels
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) {
           const float* g = f[(u + j) % TAPS];
@@ -330,7 +298,7 @@ __global__ void __launch_bounds__(CV_THREADS, TAPS <= 4 ? 3 : 2) short_conv_kern
       } else {
 #pragma unroll
         for (int i = 0; i < V; ++i) {
-          float acc = 0.f;
+          float acc = bias[i];
 #pragma unroll
           for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j][i], f[(u + j) % TAPS][i], acc);
           y[i] = acc / (1.f + expf(-acc));
@@ -363,14 +331,14 @@ template <typename T, int V> static int conv_by_taps(const ConvArgs& a, dim3 gri
 
 }  // namespace zp
 
-extern "C" int zp_short_conv(const void* x, int64_t x_stride, const float* weight, void* ring, const int32_t* cu_seqlens_q,
+extern "C" int zp_short_conv(const void* x, int64_t x_stride, const float* weight, const float* bias, void* ring, const int32_t* cu_seqlens_q,
                              const int32_t* context_lens, const int32_t* slots, void* out, int64_t out_stride, int B,
                              int max_seqlen_q, int channels, int taps, int n_slots, int dtype, void* stream) {
   if (B == 0 || max_seqlen_q == 0) return ZP_OK;
   ZP_REQUIRE(x && weight && ring && cu_seqlens_q && context_lens && slots && out, "zp_short_conv: null pointer");
   ZP_REQUIRE(channels > 0 && taps > 0 && taps <= zp::CV_MAX_TAPS && n_slots > 0 && B <= 65535 && x_stride >= channels && out_stride >= channels,
              "zp_short_conv: bad sizes (%d taps, at most %d)", taps, zp::CV_MAX_TAPS);
-  zp::ConvArgs a{x, weight, ring, out, cu_seqlens_q, context_lens, slots, x_stride, out_stride, channels, taps, n_slots};
+  zp::ConvArgs a{x, weight, bias, ring, out, cu_seqlens_q, context_lens, slots, x_stride, out_stride, channels, taps, n_slots};
   cudaStream_t st = (cudaStream_t)stream;
   int rc = ZP_OK;
   ZP_DISPATCH_DTYPE(dtype, T, {

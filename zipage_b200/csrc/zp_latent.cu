@@ -208,6 +208,6 @@ extern "C" int zp_latent_attention(const void* q, const void* cache, const int32
   }
   // one shared key/value head whose values are the first R entries of its keys
   return zp_window_attention(q, cache, cache, cu_seqlens_q, context_lens, block_table, out, B, max_seqlen_q, NBmax, H, 1, KP, R, KP,
-                             KP, BS, n_pages, (int64_t)H * KP, (int64_t)H * R, scale, 0.f, 0, 0, nullptr, nullptr, 0, 0, 1.f, total_rows, ZP_IMPL_SIMT, dtype,
+                             KP, BS, n_pages, (int64_t)H * KP, (int64_t)H * R, scale, 0.f, 0, 0, 0, nullptr, nullptr, nullptr, 0, 0, 1.f, total_rows, ZP_IMPL_SIMT, dtype,
                              nullptr, 0, stream);
 }

@@ -1,4 +1,4 @@
-// Mixture of experts: routing (softmax scores over all experts or sigmoid scores, the largest `top` of a token) with the
+// Mixture of experts: routing (softmax scores over all experts or over the chosen ones, or sigmoid scores, the largest `top` of a token) with the
 // bookkeeping that sorts (token, expert) pairs by expert, and matrix products of the sorted rows with their
 // expert's weights.  This file has the routing kernels, the SIMT product for fp32 and odd sizes, and the entry
 // points; zp_moe_tc.cu has the tensor-core product.
@@ -20,15 +20,16 @@ __device__ __forceinline__ unsigned order_key(float v) {
 // The `top` largest of one token's logits by one warp: lane holds experts lane, lane + 32, ...  Ties: the lower
 // expert.  Choice k is returned by lane k % 32 of round k / 32 (emit(k, expert, score) is called by that lane,
 // all lanes of a round at once).
+// Returns the sum that ZP_SCORE_SOFTMAX_TOP divides by (its scores are emitted without).
 template <int VPL, typename F>
-__device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, int top, bool sigmoid, F&& emit) {
+__device__ __forceinline__ float top_experts(const float* __restrict__ z, const float* __restrict__ bias, int E, int top, int score_kind, F&& emit) {
   const int lane = threadIdx.x & 31;
   float v[VPL], mx = -INFINITY;
   unsigned key[VPL];                        // 0: taken, or no expert
 #pragma unroll
   for (int i = 0; i < VPL; ++i) {
     const bool in = lane + 32 * i < E;
-    v[i] = in ? z[lane + 32 * i] : -INFINITY;
+    v[i] = in ? z[lane + 32 * i] + (bias ? bias[lane + 32 * i] : 0.f) : -INFINITY;
     key[i] = in ? max(order_key(v[i]), 1u) : 0u;
     mx = fmaxf(mx, v[i]);
   }
@@ -36,7 +37,8 @@ __device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, 
   float sum = 0.f;
 #pragma unroll
   for (int i = 0; i < VPL; ++i) sum += lane + 32 * i < E ? expf(v[i] - mx) : 0.f;
-  sum = warp_sum(sum);
+  sum = score_kind == ZP_SCORE_SOFTMAX ? warp_sum(sum) : 1.f;
+  float chosen = 0.f;
   for (int k0 = 0; k0 < top; k0 += 32) {
     int mine = 0;
     float score = 0.f;
@@ -49,6 +51,7 @@ __device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, 
       const unsigned best = __reduce_max_sync(0xffffffffu, bk);
       const unsigned at = __reduce_min_sync(0xffffffffu, bk == best ? bi : 0xffffffffu);
       bv = __shfl_sync(0xffffffffu, bv, at & 31);
+      chosen += expf(bv - mx);
       if ((int)(at & 31) == lane) {
 #pragma unroll
         for (int i = 0; i < VPL; ++i)
@@ -56,8 +59,9 @@ __device__ __forceinline__ void top_experts(const float* __restrict__ z, int E, 
       }
       if (lane == k - k0) { mine = (int)at; score = bv; }
     }
-    if (lane < top - k0) emit(k0 + lane, mine, sigmoid ? 1.f / (1.f + expf(-score)) : expf(score - mx) / sum);
+    if (lane < top - k0) emit(k0 + lane, mine, score_kind == ZP_SCORE_SIGMOID ? 1.f / (1.f + expf(-score)) : expf(score - mx) / sum);
   }
+  return chosen;
 }
 
 // exclusive scan of counts[0 .. E) into offs[0 .. E] by the first warp of the block
@@ -87,7 +91,8 @@ struct RouteArgs {
   int32_t *idx, *pos;  // [N, top]; between the two kernels pos holds ranks within the expert
   int32_t *rows, *offsets, *counts;
   float* place_wts;    // [N * top] or NULL: the weights in the order of the places
-  int sigmoid;
+  int score;
+  const float* bias;   // [E] or NULL
 };
 
 // One block does everything (ONE; at most RT_ONE pairs), or several blocks choose and count and route_place_kernel places.
@@ -100,8 +105,8 @@ __global__ void __launch_bounds__(ONE ? 1024 : 256) route_kernel(const RouteArgs
   __syncthreads();
   const int nw = blockDim.x >> 5, per = ONE ? a.N : 32;        // tokens of a block
   const int t0 = blockIdx.x * per, t1 = min(a.N, t0 + per);
-  for (int t = t0 + (threadIdx.x >> 5); t < t1; t += nw)
-    top_experts<VPL>(a.logits + (int64_t)t * a.ld, a.E, a.top, a.sigmoid != 0, [&](int k, int e, float s) {
+  for (int t = t0 + (threadIdx.x >> 5); t < t1; t += nw) {
+    const float chosen = top_experts<VPL>(a.logits + (int64_t)t * a.ld, a.bias, a.E, a.top, a.score, [&](int k, int e, float s) {
       const int64_t at = (int64_t)t * a.top + k;
       a.wts[at] = s;
       a.idx[at] = e;
@@ -109,6 +114,9 @@ __global__ void __launch_bounds__(ONE ? 1024 : 256) route_kernel(const RouteArgs
       if constexpr (ONE) picks[at] = make_int2(e, rank);
       else a.pos[at] = rank;
     });
+    if (a.score == ZP_SCORE_SOFTMAX_TOP)       // (a lane divides what it has written)
+      for (int k = threadIdx.x & 31; k < a.top; k += 32) a.wts[(int64_t)t * a.top + k] /= chosen;
+  }
   __syncthreads();
   if constexpr (ONE) {
     scan_counts(hist, offs, a.E);
@@ -231,16 +239,16 @@ template <typename T> __global__ void __launch_bounds__(256) grouped_gemm_simt_k
 
 }  // namespace zp
 
-extern "C" int zp_moe_route(const float* logits, int64_t row_stride, int n_tokens, int n_experts, int top, float* weights,
+extern "C" int zp_moe_route(const float* logits, int64_t row_stride, const float* bias, int n_tokens, int n_experts, int top, float* weights,
                             int32_t* experts, int32_t* places, int32_t* rows, int32_t* offsets, int32_t* counts, float* place_weights,
                             int score, void* stream) {
   if (n_tokens == 0) return ZP_OK;
   ZP_REQUIRE(logits && weights && experts && places && rows && offsets && counts, "zp_moe_route: null pointer");
   ZP_REQUIRE(n_experts > 0 && n_experts <= zp::RT_MAXE && top > 0 && top <= n_experts && row_stride >= n_experts,
              "zp_moe_route: %d of %d experts (at most %d)", top, n_experts, zp::RT_MAXE);
-  ZP_REQUIRE(score == ZP_SCORE_SOFTMAX || score == ZP_SCORE_SIGMOID, "zp_moe_route: unknown score %d", score);
+  ZP_REQUIRE(score == ZP_SCORE_SOFTMAX || score == ZP_SCORE_SIGMOID || score == ZP_SCORE_SOFTMAX_TOP, "zp_moe_route: unknown score %d", score);
   zp::RouteArgs a{logits, row_stride, n_tokens, n_experts, top, weights, experts, places, rows, offsets, counts, place_weights,
-                  score == ZP_SCORE_SIGMOID};
+                  score, bias};
   cudaStream_t st = (cudaStream_t)stream;
   if (n_experts <= 32) return zp::launch_route<1>(a, st);
   if (n_experts <= 64) return zp::launch_route<2>(a, st);

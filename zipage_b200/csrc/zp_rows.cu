@@ -1,10 +1,10 @@
 // Row ops of decoders that keep the residual stream in fp32 between 16-bit matrix products:
-//   * token embedding, scaled, plus a sinusoidal position vector (and its copy as T),
+//   * token embedding, scaled, plus a sinusoidal or a learned position vector (and its copy as T),
 //   * RMSNorm of an fp32 row to T with the weight stored as an offset (out = x * r * (w + offset)),
 //     or, without a weight, the plain conversion of the row,
 //   * the boundary between two layers whose mixer and feed-forward read the same x: both results (with
-//     their layer scales, the experts' weights and a gate) join x, and the next layer's two layer norms
-//     follow from the row while it is in registers,
+//     their layer scales, the experts' weights and a gate; the mixer's also as the mean of two that are normed first) join x, and
+//     the next layer's norms follow from the row while it is in registers,
 //   * activations: tanh-form GELU, its gated form, squared ReLU; the soft cap of the logits.
 // All are streams over HBM with fp32 maths and one rounding to T at the end.
 #include "zp_common.cuh"
@@ -36,21 +36,26 @@ template <> __device__ __forceinline__ float4 ldf4<float>(const float* p) { retu
 // ---------------------------------------------------------------------------------------------
 // x[n, 2i] = E[tok, 2i] * scale + sin(p w_i),  x[n, 2i + 1] = E[tok, 2i + 1] * scale + cos(p w_i).
 // `turns[i]` = w_i / (2 pi) in fp64: p * turns is reduced to a fraction of a turn before the
-// conversion to fp32, so the angle keeps its accuracy at any position.
+// conversion to fp32, so the angle keeps its accuracy at any position.  `learned`: row p of that table is added instead.
 // ---------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
 embed_position_kernel(const int64_t* __restrict__ tokens, const int64_t* __restrict__ positions,
                       const T* __restrict__ table, const double* __restrict__ turns, float scale,
-                      float* __restrict__ x, T* __restrict__ x_t, int H, int64_t vocab) {
+                      const T* __restrict__ learned, int64_t n_learned, float* __restrict__ x, T* __restrict__ x_t, int H, int64_t vocab) {
   const int64_t n = blockIdx.x;
   const int64_t tok = min(max(tokens[n], (int64_t)0), vocab - 1);   // (the host rejects ids outside the table)
   const double p = (double)positions[n];
+  const int64_t at = min(max(positions[n], (int64_t)0), n_learned - 1);
   for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
     float s = 0.f, c = 0.f;
     if (turns) {
       const double t = p * turns[i];
       sincospif(2.f * (float)(t - rint(t)), &s, &c);
+    }
+    if (learned) {
+      s = Elem<T>::to_f32(learned[at * H + 2 * i]);
+      c = 2 * i + 1 < H ? Elem<T>::to_f32(learned[at * H + 2 * i + 1]) : 0.f;
     }
     const float a = fmaf(Elem<T>::to_f32(table[tok * H + 2 * i]), scale, s);
     x[n * H + 2 * i] = a;
@@ -152,7 +157,7 @@ gelu_tanh_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t n, int64_
 }
 
 // ---------------------------------------------------------------------------------------------
-// x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k w_k y[pos_k]);  out_i = T(norm of x with w_i, bias_i), the layer
+// x += ls_a * a + ls_b * (sigmoid(gate) * b + sum_k w_k y[pos_k]) + pair_scale * (rms(m1) * mw1 + rms(m2) * mw2);  out_i = T(norm of x with w_i, bias_i), the layer
 // norm or (rms) the one that takes no mean off.
 // Every part may be missing.  One block per row; VPT float4 per thread stay in registers (VPT = 0: any
 // row length, each thread reads back the entries of x that it wrote).
@@ -164,9 +169,11 @@ struct JoinArgs {
   const int32_t* pos;
   const float *w1, *bias1, *w2, *bias2;
   void *out1, *out2;
+  const void *m1, *m2;        // both or none
+  const float *mw1, *mw2;
   int64_t gate_stride, y_rows;
   int top, H, rms;
-  float eps;
+  float eps, pair_scale;
 };
 
 template <typename T, int V> struct JoinVec;      // V consecutive entries of a row
@@ -190,12 +197,17 @@ __device__ __forceinline__ float4 splat4(float s) { return make_float4(s, s, s, 
 // What joins x at entry c of a row: `add` gathers it, so that the loads of all of a thread's entries can be in
 // flight before the first of them is stored.
 template <typename T, int V>
-__device__ __forceinline__ float4 join_add(const JoinArgs& p, int64_t row, int c, const float* swts, const int32_t* spos, float g) {
+__device__ __forceinline__ float4 join_add(const JoinArgs& p, int64_t row, int c, const float* swts, const int32_t* spos, float g, float2 rp) {
   using L = JoinVec<T, V>;
   float4 add = splat4(0.f);
+  if (p.m1) {
+    const float4 u = L::ld(p.m1, row * p.H + c), v = L::ld(p.m2, row * p.H + c), s = L::ldf(p.mw1, c), t = L::ldf(p.mw2, c);
+    add = make_float4(u.x * rp.x * s.x + v.x * rp.y * t.x, u.y * rp.x * s.y + v.y * rp.y * t.y, u.z * rp.x * s.z + v.z * rp.y * t.z,
+                      u.w * rp.x * s.w + v.w * rp.y * t.w);
+  }
   if (p.a) {
-    add = L::ld(p.a, row * p.H + c);
-    if (p.ls_a) { const float4 s = L::ldf(p.ls_a, c); add = make_float4(add.x * s.x, add.y * s.y, add.z * s.z, add.w * s.w); }
+    const float4 a = L::ld(p.a, row * p.H + c);
+    add = fma4(p.ls_a ? L::ldf(p.ls_a, c) : splat4(1.f), a, add);
   }
   if (p.b || p.y) {
     float4 f = splat4(0.f);
@@ -229,7 +241,20 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
     __syncthreads();
   }
   const float g = p.gate ? 1.f / (1.f + expf(-p.gate[row * p.gate_stride])) : 1.f;
-  const bool norm = p.out1 || p.out2, any = p.a || p.b || p.y;
+  const bool norm = p.out1 || p.out2, any = p.a || p.b || p.y || p.m1;
+  float2 rp = make_float2(0.f, 0.f);        // pair_scale over the root mean squares of the pair's rows
+  if (p.m1) {
+    constexpr int V = VPT > 0 ? 4 : 1;
+    using L = JoinVec<T, V>;
+    float s1 = 0.f, s2 = 0.f;
+    for (int c = threadIdx.x * V; c < p.H; c += blockDim.x * V) {
+      const float4 u = L::ld(p.m1, row * p.H + c), v = L::ld(p.m2, row * p.H + c);
+      s1 = fmaf(u.x, u.x, s1); s1 = fmaf(u.y, u.y, s1); s1 = fmaf(u.z, u.z, s1); s1 = fmaf(u.w, u.w, s1);
+      s2 = fmaf(v.x, v.x, s2); s2 = fmaf(v.y, v.y, s2); s2 = fmaf(v.z, v.z, s2); s2 = fmaf(v.w, v.w, s2);
+    }
+    rp.x = p.pair_scale / sqrtf(block_sum(s1, red) / (float)p.H + p.eps);
+    rp.y = p.pair_scale / sqrtf(block_sum(s2, red) / (float)p.H + p.eps);
+  }
   if constexpr (VPT > 0) {
     const int nvec = p.H / 4;
     using L = JoinVec<T, 4>;
@@ -241,7 +266,7 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
       if (c < nvec) {
         const float4 x = L::ldf(p.x, row * p.H + 4 * c);
         if (!any) { v[i] = x; continue; }
-        const float4 d = join_add<T, 4>(p, row, 4 * c, swts, spos, g);
+        const float4 d = join_add<T, 4>(p, row, 4 * c, swts, spos, g, rp);
         v[i] = make_float4(x.x + d.x, x.y + d.y, x.z + d.z, x.w + d.w);
       }
     }
@@ -275,7 +300,7 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
     float s = 0.f;
     for (int c = threadIdx.x; c < p.H; c += blockDim.x) {
       float v = p.x[row * p.H + c];
-      if (any) p.x[row * p.H + c] = v += join_add<T, 1>(p, row, c, swts, spos, g).x;
+      if (any) p.x[row * p.H + c] = v += join_add<T, 1>(p, row, c, swts, spos, g, rp).x;
       s += v;
     }
     if (!norm) return;
@@ -337,14 +362,14 @@ static int stream_grid(int64_t n) {
 }  // namespace zp
 
 extern "C" int zp_embed_position(const int64_t* tokens, const int64_t* positions, const void* table,
-                                 const double* turns, float scale, float* x, void* x_t, int n_tokens,
+                                 const double* turns, float scale, const void* learned, int64_t n_learned, float* x, void* x_t, int n_tokens,
                                  int hidden, int64_t vocab, int dtype, void* stream) {
   if (n_tokens == 0) return ZP_OK;
   ZP_REQUIRE(tokens && positions && table && x, "zp_embed_position: null pointer");
-  ZP_REQUIRE(hidden > 0 && vocab > 0, "zp_embed_position: bad sizes");
+  ZP_REQUIRE(hidden > 0 && vocab > 0 && (!learned || (n_learned > 0 && !turns)), "zp_embed_position: bad sizes, or two kinds of positions");
   ZP_DISPATCH_DTYPE(dtype, T, {
     zp::embed_position_kernel<T><<<n_tokens, 256, 0, (cudaStream_t)stream>>>(
-        tokens, positions, (const T*)table, turns, scale, x, (T*)x_t, hidden, vocab);
+        tokens, positions, (const T*)table, turns, scale, (const T*)learned, n_learned, x, (T*)x_t, hidden, vocab);
   });
   return zp::check_launch("zp_embed_position");
 }
@@ -382,18 +407,21 @@ extern "C" int zp_gelu_tanh(const void* x, void* out, int64_t n, int dtype, void
 
 extern "C" int zp_join_norms(float* x, const void* a, const float* ls_a, const void* b, const float* ls_b,
                              const float* gate, int64_t gate_stride, const void* y, int64_t y_rows,
-                             const int32_t* pos, const float* wts, int top, const float* w1, const float* bias1,
+                             const int32_t* pos, const float* wts, int top, const void* m1, const float* mw1, const void* m2,
+                             const float* mw2, float pair_scale, const float* w1, const float* bias1,
                              void* out1, const float* w2, const float* bias2, void* out2, int n_rows, int hidden,
                              float eps, int rms, int dtype, void* stream) {
   if (n_rows == 0) return ZP_OK;
   ZP_REQUIRE(x, "zp_join_norms: null pointer");
   ZP_REQUIRE(hidden > 0 && top >= 0 && top <= zp::JOIN_TOP, "zp_join_norms: bad sizes (%d experts a token, at most %d)", top, zp::JOIN_TOP);
   ZP_REQUIRE(top == 0 || (y && pos && y_rows > 0), "zp_join_norms: expert rows without places");
+  ZP_REQUIRE(!m1 == !m2 && (!m1 || (mw1 && mw2)), "zp_join_norms: a pair takes two rows and two weights");
   zp::JoinArgs p;
+  p.m1 = m1; p.m2 = m2; p.mw1 = mw1; p.mw2 = mw2; p.pair_scale = pair_scale;
   p.x = x; p.a = a; p.b = b; p.y = top ? y : nullptr; p.ls_a = ls_a; p.ls_b = ls_b; p.gate = gate; p.wts = wts; p.pos = pos;
   p.w1 = w1; p.bias1 = bias1; p.w2 = w2; p.bias2 = bias2; p.out1 = out1; p.out2 = out2; p.gate_stride = gate_stride;
   p.y_rows = y_rows; p.top = top; p.H = hidden; p.eps = eps; p.rms = rms;
-  const uintptr_t al = (uintptr_t)x | (uintptr_t)a | (uintptr_t)b | (uintptr_t)p.y | (uintptr_t)ls_a | (uintptr_t)ls_b | (uintptr_t)w1 |
+  const uintptr_t al = (uintptr_t)x | (uintptr_t)a | (uintptr_t)b | (uintptr_t)p.y | (uintptr_t)m1 | (uintptr_t)m2 | (uintptr_t)mw1 | (uintptr_t)mw2 | (uintptr_t)ls_a | (uintptr_t)ls_b | (uintptr_t)w1 |
                        (uintptr_t)bias1 | (uintptr_t)out1 | (uintptr_t)w2 | (uintptr_t)bias2 | (uintptr_t)out2;
   const bool vec = hidden % 4 == 0 && hidden <= 8192 && al % 16 == 0;
   cudaStream_t st = (cudaStream_t)stream;

@@ -63,9 +63,12 @@ __global__ void __launch_bounds__(WS_WARPS * 32) window_attn_simt_kernel(const W
 #pragma unroll
   for (int j = 0; j < VPL; ++j) o[j] = 0.f;
   constexpr int EPV = 16 / sizeof(T);
-  for (int k0 = win_first(a, pos) & ~31; k0 <= pos; k0 += 32) {
+  const int lo = win_first(a, pos), near = lo & ~31;
+  const float slope = a.slopes ? a.slopes[h] : 0.f;
+  for (int k0 = min(near, a.keep > 0 ? 0 : near); k0 <= pos; k0 += 32) {
+    if (k0 >= a.keep && k0 < near) k0 = near;      // between the kept keys and the window
     const int key = k0 + lane;
-    const bool seen = key >= win_first(a, pos) && key <= pos;
+    const bool seen = (key >= lo || key < a.keep) && key <= pos;
     // the page size is a multiple of 32: the 32 keys share a page
     const int64_t slot0 = (int64_t)win_page(a, b, k0) * a.BS + k0 % a.BS;
     float s = -INFINITY;
@@ -80,6 +83,7 @@ __global__ void __launch_bounds__(WS_WARPS * 32) window_attn_simt_kernel(const W
       }
       s = acc * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+      s = fmaf(-slope, (float)(pos - key), s);
     }
     const float mx = fmaxf(m, warp_max(s));
     const float corr = m == -INFINITY ? 0.f : expf(m - mx);
@@ -88,9 +92,10 @@ __global__ void __launch_bounds__(WS_WARPS * 32) window_attn_simt_kernel(const W
     m = mx;
 #pragma unroll
     for (int j = 0; j < VPL; ++j) o[j] *= corr;
-    const int first = max(win_first(a, pos) - k0, 0), last = min(pos - k0, 31);
+    const int first = k0 < a.keep ? 0 : max(lo - k0, 0), last = min(pos - k0, 31);
     for (int t = first; t <= last; ++t) {
       const float pt = __shfl_sync(0xffffffffu, p, t);
+      if (pt == 0.f) continue;
       const T* vr = vc + ((slot0 + t) * a.Hkv + hk) * a.VP;
 #pragma unroll
       for (int j = 0; j < VPL; ++j) {
@@ -158,8 +163,8 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
                                    const int32_t* cu_seqlens_q, const int32_t* context_lens,
                                    const int32_t* block_table, void* out, int B, int max_seqlen_q, int NBmax,
                                    int Hq, int Hkv, int D, int DV, int KP, int VP, int BS, int n_pages,
-                                   int64_t q_stride, int64_t out_stride, float scale, float softcap, int window, int chunk,
-                                   const float* sink, const void* gate, int64_t gate_stride, int gate_mode, float out_scale,
+                                   int64_t q_stride, int64_t out_stride, float scale, float softcap, int window, int chunk, int keep,
+                                   const float* slopes, const float* sink, const void* gate, int64_t gate_stride, int gate_mode, float out_scale,
                                    int total_q, int impl, int dtype, void* workspace, size_t workspace_bytes, void* stream) {
   if (B == 0 || (cu_seqlens_q && max_seqlen_q == 0)) return ZP_OK;
   ZP_REQUIRE(q && k_cache && v_cache && context_lens && block_table && out, "zp_window_attention: null pointer");
@@ -169,13 +174,13 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
              "zp_window_attention: head sizes %d / %d (padded %d / %d) not supported", D, DV, KP, VP);
   ZP_REQUIRE(NBmax > 0 && n_pages > 0 && B <= 65535, "zp_window_attention: bad sizes");
   ZP_REQUIRE(((uintptr_t)k_cache | (uintptr_t)v_cache) % 16 == 0, "zp_window_attention: caches must be 16-byte aligned");
-  ZP_REQUIRE(chunk >= 0 && window >= 0 && gate_mode >= 0 && gate_mode <= 2 && (gate_mode == 0 || gate),
+  ZP_REQUIRE(chunk >= 0 && window >= 0 && keep >= 0 && gate_mode >= 0 && gate_mode <= 2 && (gate_mode == 0 || gate),
              "zp_window_attention: bad mask or gate");
   zp::WinArgs a;
   a.q = q; a.k = k_cache; a.v = v_cache; a.cu_q = cu_seqlens_q; a.context_lens = context_lens; a.table = block_table;
   a.out = out; a.part = nullptr; a.B = B; a.NBmax = NBmax; a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.DV = DV; a.KP = KP;
   a.VP = VP; a.BS = BS; a.window = window; a.n_pages = n_pages; a.nsplit = 1; a.q_stride = q_stride;
-  a.out_stride = out_stride; a.scale = scale; a.softcap = softcap; a.chunk = chunk; a.sink = sink; a.gate = gate;
+  a.out_stride = out_stride; a.scale = scale; a.softcap = softcap; a.chunk = chunk; a.keep = keep; a.slopes = slopes; a.sink = sink; a.gate = gate;
   a.gate_stride = gate_stride; a.gate_mode = gate_mode; a.out_scale = out_scale;
   cudaStream_t st = (cudaStream_t)stream;
   const bool half = dtype == ZP_DTYPE_BF16 || dtype == ZP_DTYPE_F16;
@@ -183,7 +188,7 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
   const bool tc = cu_seqlens_q && zp::window_tc_supports(a, total_q, dtype);
   if (impl == ZP_IMPL_TCGEN05 && !tc) {
     zp::set_error("zp_window_attention: the tcgen05 kernel needs bf16 portions, head sizes that are multiples of 8 up to 128, 16-byte "
-                  "aligned rows and no soft cap or one of at most 69");
+                  "aligned rows and no soft cap or one of at most 69 without slopes");
     return ZP_ERR_UNSUPPORTED;
   }
   if (tc && (impl == ZP_IMPL_TCGEN05 || (impl == ZP_IMPL_AUTO && max_seqlen_q >= 96 && KP + VP > 128)))
@@ -191,8 +196,8 @@ extern "C" int zp_window_attention(const void* q, const void* k_cache, const voi
   if (half && impl != ZP_IMPL_SIMT && zp::window_mma_supports(a)) {
     if (cu_seqlens_q) return zp::window_prefill_mma(a, max_seqlen_q, dtype, st);
     int span = NBmax * BS;
-    if (window > 0 && window < span) span = window;
-    if (chunk > 0 && chunk < span) span = chunk;
+    if (window > 0 && window + keep < span) span = window + keep;
+    if (chunk > 0 && chunk + keep < span) span = chunk + keep;
     a.nsplit = zp::window_decode_splits(B, Hkv, span);
     if (a.nsplit > 1) {
       const size_t need = (size_t)B * Hq * a.nsplit * (VP + 2) * sizeof(float);

@@ -1,4 +1,4 @@
-// Arguments shared by the attention kernels with masks, soft caps, sinks and output gates (SIMT, mma.sync, tcgen05).
+// Arguments shared by the attention kernels with masks, soft caps, distance biases, sinks and output gates (SIMT, mma.sync, tcgen05).
 #pragma once
 #include "zp_common.cuh"
 
@@ -8,7 +8,8 @@ namespace zp {
 // cu_q[b] .. cu_q[b + 1] (absolute rows of q / out), or row b alone when cu_q is NULL; its context
 // (keys up to and including this step's tokens) is context_lens[b], so row r sits at position
 // context - count + r and sees the keys j <= position with position - j < window (window > 0) and, with chunk > 0,
-// those of its own chunk, floor(j / chunk) = floor(position / chunk).  A head's sink is one more term of its softmax's
+// those of its own chunk, floor(j / chunk) = floor(position / chunk); the keys j < keep are seen in any case.  With slopes,
+// slopes[h] * (position - j) is taken off a score.  A head's sink is one more term of its softmax's
 // denominator, exp(sink[h]).  The result is multiplied by out_scale and by sigmoid(gate), one gate per head or per entry.
 struct WinArgs {
   const void* q; const void* k; const void* v;   // q [rows, Hq, D] with a row stride; paged caches [P, BS, Hkv, KP | VP]
@@ -19,6 +20,8 @@ struct WinArgs {
   int64_t out_stride;    // elements between rows of out
   float scale, softcap;  // softcap 0 = none
   int chunk;             // 0 = none
+  int keep;              // first keys that every later query sees
+  const float* slopes;   // [Hq] or NULL
   const float* sink;     // [Hq] or NULL
   const void* gate;      // rows of T: [Hq] (WIN_GATE_HEAD) or [Hq, DV] (WIN_GATE_ENTRY)
   int64_t gate_stride;
@@ -42,6 +45,21 @@ __device__ __forceinline__ int win_first(const WinArgs& a, int pos) {
   const int w = a.window > 0 ? max(0, pos - a.window + 1) : 0;
   return a.chunk > 0 ? max(w, pos - pos % a.chunk) : w;
 }
+// Tiles of `tk` keys that queries from position `first_pos` to `last_pos` see: `kept` tiles with the kept keys, then those
+// from t0 on.
+struct WinTiles {
+  int kept, t0, n;
+  __device__ __forceinline__ int tile(int j) const { return j < kept ? j : t0 + j - kept; }
+};
+__device__ __forceinline__ WinTiles win_tiles(const WinArgs& a, int first_pos, int last_pos, int tk) {
+  WinTiles w;
+  w.t0 = win_first(a, first_pos) / tk;
+  w.kept = min((a.keep + tk - 1) / tk, w.t0);
+  w.n = w.kept + last_pos / tk - w.t0 + 1;
+  return w;
+}
+// slope of head h in log2 units
+__device__ __forceinline__ float win_slope2(const WinArgs& a, int h) { return a.slopes ? a.slopes[h] * 1.4426950408889634f : 0.f; }
 enum { WIN_GATE_NONE = 0, WIN_GATE_HEAD = 1, WIN_GATE_ENTRY = 2 };
 __device__ __forceinline__ float win_sigmoid(float z) { return 1.f / (1.f + __expf(-z)); }
 // what the output of head h in `row` (absolute) is multiplied by: the factor of all entries, ...

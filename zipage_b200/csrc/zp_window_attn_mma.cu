@@ -24,7 +24,7 @@ constexpr float WM_LOG2E = 1.4426950408889634f;
 __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
-// score in log2 units after scale and cap (c = cap * log2 e, y = 2 scale log2 e / cap)
+// score in log2 units after scale and cap, the distance's bias not yet taken off (c = cap * log2 e, y = 2 scale log2 e / cap)
 struct CapConst { float lin, y, c, cap, ref; };
 __device__ __forceinline__ CapConst cap_const(const WinArgs& a) {
   CapConst k;
@@ -90,7 +90,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
   const int stage_bytes = WM_TK * (rbk + rbv);
   const int rows = min(WM_TQ, sq.count - qi0);
   const int p_first = sq.pos0 + qi0, p_last = p_first + rows - 1;   // positions of the tile's rows
-  const int t0 = win_first(a, p_first) / WM_TK, t1 = p_last / WM_TK;
+  const WinTiles wt = win_tiles(a, p_first, p_last, WM_TK);
 
   auto load_tile = [&](int t, int stage) {
     const int key0 = t * WM_TK;
@@ -100,7 +100,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
     load_page_rows(ks, reinterpret_cast<const char*>(a.k), slot0, a.Hkv, hk, KP, n_valid);
     load_page_rows(ks + WM_TK * rbk, reinterpret_cast<const char*>(a.v), slot0, a.Hkv, hk, VP, n_valid);
   };
-  load_tile(t0, 0);
+  load_tile(wt.tile(0), 0);
   cp_async_commit();
   {  // the query tile, its padding columns and missing rows zero
     const T* qp = reinterpret_cast<const T*>(a.q) + (int64_t)(sq.row0 + qi0) * a.q_stride + (int64_t)h * a.D;
@@ -130,15 +130,17 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
   for (int i = 0; i < 2 * NV16; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
-  for (int t = t0; t <= t1; ++t) {
-    if (t + 1 <= t1) load_tile(t + 1, (t + 1 - t0) & 1);
+  const float slope = win_slope2(a, h);
+  for (int ti = 0; ti < wt.n; ++ti) {
+    if (ti + 1 < wt.n) load_tile(wt.tile(ti + 1), (ti + 1) & 1);
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
-    const unsigned char* ks = sKV + ((t - t0) & 1) * stage_bytes;
+    const unsigned char* ks = sKV + (ti & 1) * stage_bytes;
     const unsigned char* vs = ks + WM_TK * rbk;
-    const int key0 = t * WM_TK;
-    if (key0 <= wp1 && key0 + WM_TK > win_first(a, wp0)) {   // else the warp's rows see none of these keys
+    const int key0 = wt.tile(ti) * WM_TK;
+    auto hidden = [&](int key, int pos, int lo) { return key > pos || (key < lo && key >= a.keep); };
+    if (key0 <= wp1 && (key0 + WM_TK > win_first(a, wp0) || key0 < a.keep)) {   // else the warp's rows see none of these keys
       float s[8][4];
 #pragma unroll
       for (int nb = 0; nb < 8; ++nb) { s[nb][0] = s[nb][1] = s[nb][2] = s[nb][3] = 0.f; }
@@ -154,7 +156,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
           mma16816<T>(s[2 * np + 1], qa, bf[2], bf[3]);
         }
       }
-      const bool whole = key0 + WM_TK - 1 <= wp0 && key0 >= win_first(a, wp1);   // no masking in this tile
+      const bool whole = key0 + WM_TK - 1 <= wp0 && (key0 >= win_first(a, wp1) || key0 + WM_TK <= a.keep);   // no masking in this tile
       if constexpr (BOUNDED) {
 #pragma unroll
         for (int nb = 0; nb < 8; ++nb) {
@@ -162,10 +164,10 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
           for (int j = 0; j < 4; ++j) s[nb][j] = ex2(fmaf(-2.f * cc.c, rcp(1.f + ex2(s[nb][j] * cc.y)), cc.c - cc.ref));
           if (!whole) {
             const int key = key0 + nb * 8 + 2 * tq;
-            if (key > pos0 || key < lo0) s[nb][0] = 0.f;
-            if (key + 1 > pos0 || key + 1 < lo0) s[nb][1] = 0.f;
-            if (key > pos1 || key < lo1) s[nb][2] = 0.f;
-            if (key + 1 > pos1 || key + 1 < lo1) s[nb][3] = 0.f;
+            if (hidden(key, pos0, lo0)) s[nb][0] = 0.f;
+            if (hidden(key + 1, pos0, lo0)) s[nb][1] = 0.f;
+            if (hidden(key, pos1, lo1)) s[nb][2] = 0.f;
+            if (hidden(key + 1, pos1, lo1)) s[nb][3] = 0.f;
           }
           l0 += s[nb][0] + s[nb][1];
           l1 += s[nb][2] + s[nb][3];
@@ -176,12 +178,13 @@ __global__ void __launch_bounds__(WM_THREADS) window_prefill_mma_kernel(const Wi
         for (int nb = 0; nb < 8; ++nb) {
           const int key = key0 + nb * 8 + 2 * tq;
 #pragma unroll
-          for (int j = 0; j < 4; ++j) s[nb][j] = capped(s[nb][j], cc, a.scale);
+          for (int j = 0; j < 4; ++j)
+            s[nb][j] = fmaf(-slope, (float)((j < 2 ? pos0 : pos1) - key - (j & 1)), capped(s[nb][j], cc, a.scale));
           if (!whole) {
-            if (key > pos0 || key < lo0) s[nb][0] = -INFINITY;
-            if (key + 1 > pos0 || key + 1 < lo0) s[nb][1] = -INFINITY;
-            if (key > pos1 || key < lo1) s[nb][2] = -INFINITY;
-            if (key + 1 > pos1 || key + 1 < lo1) s[nb][3] = -INFINITY;
+            if (hidden(key, pos0, lo0)) s[nb][0] = -INFINITY;
+            if (hidden(key + 1, pos0, lo0)) s[nb][1] = -INFINITY;
+            if (hidden(key, pos1, lo1)) s[nb][2] = -INFINITY;
+            if (hidden(key + 1, pos1, lo1)) s[nb][3] = -INFINITY;
           }
           mx0 = fmaxf(mx0, fmaxf(s[nb][0], s[nb][1]));
           mx1 = fmaxf(mx1, fmaxf(s[nb][2], s[nb][3]));
@@ -283,9 +286,9 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
   unsigned char* sKV = smem + 16 * rbk;
   const int stage_bytes = WM_TK * (rbk + rbv);
   const int pos = sq.ctx - 1, lo = win_first(a, pos);
-  const int first = lo / WM_TK, nt_all = pos / WM_TK - first + 1;
-  const int per = (nt_all + a.nsplit - 1) / a.nsplit;
-  const int t0 = first + split * per, t1 = min(first + (split + 1) * per, first + nt_all);   // tiles [t0, t1)
+  const WinTiles wt = win_tiles(a, pos, pos, WM_TK);
+  const int per = (wt.n + a.nsplit - 1) / a.nsplit;
+  const int t0 = split * per, t1 = min(t0 + per, wt.n);   // tiles [t0, t1) of the list
 
   auto load_tile = [&](int t, int stage) {
     const int key0 = t * WM_TK;
@@ -295,7 +298,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
     load_page_rows(ks, reinterpret_cast<const char*>(a.k), slot0, a.Hkv, hk, KP, n_valid);
     load_page_rows(ks + WM_TK * rbk, reinterpret_cast<const char*>(a.v), slot0, a.Hkv, hk, VP, n_valid);
   };
-  if (t0 < t1) load_tile(t0, 0);
+  if (t0 < t1) load_tile(wt.tile(t0), 0);
   cp_async_commit();
   {
     const T* qp = reinterpret_cast<const T*>(a.q) + (int64_t)sq.row0 * a.q_stride + (int64_t)hk * G * a.D;
@@ -310,9 +313,10 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
 #pragma unroll
   for (int i = 0; i < 2 * NV16; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;   // rows g and g + 8
+  const float slope0 = g < G ? win_slope2(a, hk * G + g) : 0.f, slope1 = g + 8 < G ? win_slope2(a, hk * G + g + 8) : 0.f;
 
   for (int t = t0; t < t1; ++t) {
-    if (t + 1 < t1) load_tile(t + 1, (t + 1 - t0) & 1);
+    if (t + 1 < t1) load_tile(wt.tile(t + 1), (t + 1 - t0) & 1);
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
@@ -333,11 +337,12 @@ __global__ void __launch_bounds__(WM_THREADS) window_decode_mma_kernel(const Win
     float mx0 = m0, mx1 = m1;
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb) {
-      const int key = t * WM_TK + kw + nb * 8 + 2 * tq;
+      const int key = wt.tile(t) * WM_TK + kw + nb * 8 + 2 * tq;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int kj = key + (j & 1);
-        s[nb][j] = (kj <= pos && kj >= lo) ? capped(s[nb][j], cc, a.scale) : -INFINITY;
+        const float sc = fmaf(-((j < 2) ? slope0 : slope1), (float)(pos - kj), capped(s[nb][j], cc, a.scale));
+        s[nb][j] = (kj <= pos && (kj >= lo || kj < a.keep)) ? sc : -INFINITY;
       }
       mx0 = fmaxf(mx0, fmaxf(s[nb][0], s[nb][1]));
       mx1 = fmaxf(mx1, fmaxf(s[nb][2], s[nb][3]));
@@ -489,7 +494,7 @@ static int prefill_by_size(const WinArgs& a, int max_q, cudaStream_t st) {
   return launch_prefill<T, 16, BOUNDED>(a, max_q, st);
 }
 int window_prefill_mma(const WinArgs& a, int max_q, int dtype, cudaStream_t st) {
-  const bool bounded = a.softcap > 0.f && a.softcap * WM_LOG2E <= 100.f;
+  const bool bounded = a.softcap > 0.f && a.softcap * WM_LOG2E <= 100.f && !a.slopes;
   if (dtype == ZP_DTYPE_F16) return prefill_by_size<__half, false>(a, max_q, st);   // (2^-100 does not fit fp16)
   if (bounded) return prefill_by_size<__nv_bfloat16, true>(a, max_q, st);
   return prefill_by_size<__nv_bfloat16, false>(a, max_q, st);

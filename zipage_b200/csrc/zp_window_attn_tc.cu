@@ -100,7 +100,7 @@ constexpr float WT_LAZY = 40.f;    // log2 units
 
 struct WtParams { WinArgs a; int* error_word; };
 
-template <bool CAPPED>
+template <bool CAPPED, bool SLOPED>   // (not both)
 __global__ void __launch_bounds__(WT_THREADS, 1)
 window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                          const __grid_constant__ CUtensorMap tmV, const WtParams p) {
@@ -114,7 +114,8 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   const int hk = h / (a.Hq / a.Hkv);
   const int rows = min(128, sq.count - qi0);
   const int p_first = sq.pos0 + qi0, p_last = p_first + rows - 1;
-  const int t0 = win_first(a, p_first) >> 7, n = (p_last >> 7) - t0 + 1;   // 128-key tiles t0 .. t0 + n - 1
+  const WinTiles wt = win_tiles(a, p_first, p_last, 128);
+  const int n = wt.n;                                // 128-key tiles
 
   extern __shared__ unsigned char smem_raw[];
   unsigned char* qbuf = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -155,7 +156,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       tma_load_5d(qbuf + WT_BLK, &tmQ, &sh.qfull, 64, h, sq.row0 + qi0, 0, 0);
       bool ok = true;
       for (int j = 0; ok && j < n; ++j) {
-        const int key0 = (t0 + j) * 128;
+        const int key0 = wt.tile(j) * 128;
         const int pg0 = win_page(a, b, key0), pg1 = win_page(a, b, key0 + 64);
         for (int kv = 0; kv < 2; ++kv) {
           const int t = 2 * j + kv, s = t % WT_NRING, k = t / WT_NRING;
@@ -215,15 +216,16 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const float log2e = 1.4426950408889634f;
     const float y = 2.f * log2e * a.scale / a.softcap, m2c = -2.f * a.softcap * log2e;      // (CAPPED)
     const float off = -2.f * m2c <= 200.f ? 0.f : -0.5f * m2c;                              // cap minus reference
-    const float sl2 = a.scale * log2e;
+    const float sl2 = a.scale * log2e, slope = SLOPED ? win_slope2(a, h) : 0.f;
     bool ok = true;
     uint32_t ra[32];
     float l0 = 0.f, l1 = 0.f, ref = CAPPED ? -0.5f * m2c - off : -INFINITY;
     for (int j = 0; CAPPED ? ok && j < n : j < n; ++j) {
       const int sb = j & 1;
       if constexpr (!CAPPED) {      // (every thread reaches the meetings, whether or not a wait of its ran out)
-        const int key0 = (t0 + j) * 128 + cq * 32;
-        const bool whole = key0 >= lo && key0 + 31 <= lim;
+        const int key0 = wt.tile(j) * 128 + cq * 32;
+        const bool whole = (key0 >= lo || key0 + 32 <= a.keep) && key0 + 31 <= lim;
+        const float at = SLOPED ? slope * (float)(key0 - (p_first + r)) : 0.f;      // bias of the first column
         float mx = -INFINITY;
         if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&sh.sfull[sb], (j >> 1) & 1, abortp, p.error_word, 807));
         if (ok) {
@@ -236,11 +238,16 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           if (!whole) {
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              if (key0 + i > lim || key0 + i < lo) ra[i] = 0xff800000u;      // -inf
+              if (key0 + i > lim || (key0 + i < lo && key0 + i >= a.keep)) ra[i] = 0xff800000u;      // -inf
+          }
+          if constexpr (SLOPED) {                           // scores in log2 units
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              ra[i] = __float_as_uint(fmaf(__uint_as_float(ra[i]), sl2, fmaf(slope, (float)i, at)));
           }
 #pragma unroll
           for (int i = 0; i < 32; i += 2) mx = fmax3(mx, __uint_as_float(ra[i]), __uint_as_float(ra[i + 1]));
-          mx *= sl2;
+          if constexpr (!SLOPED) mx *= sl2;
         }
         if (wt_meet_any(q, mx > ref + WT_LAZY)) {           // some row's reference moves
           sh.stat[cq][r] = mx;
@@ -267,11 +274,12 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         }
         if (ok) {
           uint32_t hi[16], lw[16];
-          if (__any_sync(0xffffffffu, key0 + 31 >= lo && key0 <= lim)) {
+          if (__any_sync(0xffffffffu, (key0 + 31 >= lo || key0 < a.keep) && key0 <= lim)) {
             const float mref = ref == -INFINITY ? 0.f : ref;   // (a row without keys so far: every weight is exp2(-inf))
 #pragma unroll
             for (int i = 0; i < 32; i += 2) {
-              const float w0 = ex2_(fmaf(__uint_as_float(ra[i]), sl2, -mref)), w1 = ex2_(fmaf(__uint_as_float(ra[i + 1]), sl2, -mref));
+              const float w0 = ex2_(SLOPED ? __uint_as_float(ra[i]) - mref : fmaf(__uint_as_float(ra[i]), sl2, -mref));
+              const float w1 = ex2_(SLOPED ? __uint_as_float(ra[i + 1]) - mref : fmaf(__uint_as_float(ra[i + 1]), sl2, -mref));
               l0 += w0;
               l1 += w1;
               const __nv_bfloat162 x = __floats2bfloat162_rn(w0, w1);
@@ -285,7 +293,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
             for (int i = 0; i < 16; ++i) hi[i] = lw[i] = 0u;
           }
           // rows of the V tile past the sequence become zeros (0 * garbage could be NaN)
-          const int first = sq.ctx - (t0 + j) * 128;
+          const int first = sq.ctx - wt.tile(j) * 128;
           if (first < 128) {
             const int t = 2 * j + 1, s = t % WT_NRING;
             ok = __all_sync(0xffffffffu, mbar_wait(&sh.full[s], (t / WT_NRING) & 1, abortp, p.error_word, 808));
@@ -315,10 +323,10 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&sh.sempty[sb]);
-      const int key0 = (t0 + j) * 128 + cq * 32;
-      const bool whole = key0 >= lo && key0 + 31 <= lim;
+      const int key0 = wt.tile(j) * 128 + cq * 32;
+      const bool whole = (key0 >= lo || key0 + 32 <= a.keep) && key0 + 31 <= lim;
       uint32_t hi[16], lw[16];
-      if (__any_sync(0xffffffffu, key0 + 31 >= lo && key0 <= lim)) {
+      if (__any_sync(0xffffffffu, (key0 + 31 >= lo || key0 < a.keep) && key0 <= lim)) {
 #pragma unroll
         for (int i = 0; i < 32; i += 4) {
           float w[4];
@@ -326,7 +334,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           if (!whole) {
 #pragma unroll
             for (int u = 0; u < 4; ++u)
-              if (key0 + i + u < lo || key0 + i + u > lim) w[u] = 0.f;
+              if ((key0 + i + u < lo && key0 + i + u >= a.keep) || key0 + i + u > lim) w[u] = 0.f;
           }
           l0 += w[0] + w[1];
           l1 += w[2] + w[3];
@@ -344,7 +352,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         for (int i = 0; i < 16; ++i) hi[i] = lw[i] = 0u;
       }
       // rows of the V tile past the sequence become zeros (0 * garbage could be NaN)
-      const int first = sq.ctx - (t0 + j) * 128;
+      const int first = sq.ctx - wt.tile(j) * 128;
       if (first < 128) {
         const int t = 2 * j + 1, s = t % WT_NRING;
         if (!mbar_wait(&sh.full[s], (t / WT_NRING) & 1, abortp, p.error_word, 808)) { ok = false; break; }
@@ -416,7 +424,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
 // whether the kernel can run this call (total_q: rows of q)
 bool window_tc_supports(const WinArgs& a, int total_q, int dtype) {
   return dtype == ZP_DTYPE_BF16 && a.KP <= 128 && a.VP <= 128 && a.D % 8 == 0 && a.DV % 8 == 0 && total_q > 0 &&
-         a.softcap * 1.4426950408889634f <= 100.f && a.q_stride % 8 == 0 && a.out_stride % 8 == 0 &&
+         a.softcap * 1.4426950408889634f <= 100.f && !(a.slopes && a.softcap > 0.f) && a.q_stride % 8 == 0 && a.out_stride % 8 == 0 &&
          (a.gate_mode != WIN_GATE_ENTRY || (a.gate_stride % 8 == 0 && (uintptr_t)a.gate % 16 == 0)) &&
          ((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.out) % 16 == 0;
 }
@@ -439,7 +447,8 @@ int window_prefill_tc(const WinArgs& a, int max_q, int total_q, cudaStream_t st)
     if (int rc = make_tensor_map_5d(kv ? &tmV : &tmK, UmmaFmt<__nv_bfloat16>::tm, kv ? a.v : a.k, dims, strides, box, 2)) return rc;
   }
   const int smem = (1 + WT_NRING) * WT_TILE + (int)sizeof(WtShared) + 1024;
-  const auto kern = a.softcap > 0.f ? window_prefill_tc_kernel<true> : window_prefill_tc_kernel<false>;
+  const auto kern = a.softcap > 0.f ? window_prefill_tc_kernel<true, false> : a.slopes ? window_prefill_tc_kernel<false, true>
+                                                                                         : window_prefill_tc_kernel<false, false>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) { set_error("zp_window_attention(tcgen05): %s", cudaGetErrorString(e)); return ZP_ERR_CUDA; }
   kern<<<dim3((max_q + 127) / 128, a.Hq, a.B), WT_THREADS, smem, st>>>(tmQ, tmK, tmV, p);

@@ -85,6 +85,24 @@ class DeltaSpec:
         return slots * (self.heads * self.dim * ((self.vdim + 3) // 4 * 4) * 4 + self.taps * self.channels * itemsize)
 
 
+@dataclass(frozen=True)
+class LinearStateSpec:
+    """What a linear-attention mixer keeps per slot: the fp32 matrix S [heads, dim, vdim padded to 4] and, with a convolution
+    (taps > 0), a ring of its last `taps` inputs, [taps, channels] in the model's dtype."""
+    heads: int
+    dim: int
+    vdim: int
+    channels: int = 0
+    taps: int = 0
+
+    def allocate(self, pages, block_size, slots, dtype, device):
+        out = (torch.zeros((slots, self.heads, self.dim, (self.vdim + 3) // 4 * 4), dtype=torch.float32, device=device),)
+        return out + ((torch.zeros((slots, self.taps, self.channels), dtype=dtype, device=device),) if self.taps else ())
+
+    def bytes(self, pages, block_size, slots, itemsize):
+        return slots * (self.heads * self.dim * ((self.vdim + 3) // 4 * 4) * 4 + self.taps * self.channels * itemsize)
+
+
 class PagedStateCache:
     def __init__(self, specs, pages, block_size, slots, dtype, device):
         if block_size % 64:

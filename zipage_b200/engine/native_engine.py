@@ -74,6 +74,7 @@ class NativeEngine:
         if graph:
             self.runner.capture()
         self.greedy, self.seed, self.step_no = greedy, seed, 0
+        self._fed = {}              # tokens of the sequences that are fed (replayed)
         self.forced = None          # optional iterator of token lists (teacher forcing in tests)
         self.argmax_log = None      # optional list: own arg-max of every step
         self.time_record = defaultdict(float)
@@ -89,7 +90,14 @@ class NativeEngine:
         self._temps_view = self._temps_host.numpy()
 
     # -- requests -------------------------------------------------------------------------------
+    def _check_length(self, tokens):
+        """Models with a table of positions serve sequences up to its length."""
+        limit = getattr(self.model, "max_positions", None)
+        if limit is not None and tokens > limit:
+            raise ValueError(f"a sequence of {tokens} tokens, the model has {limit} positions")
+
     def add_request(self, seq):
+        self._check_length(len(seq._prompt) + seq._params.max_tokens)
         self.scheduler.add(seq)
         return seq._h
 
@@ -257,7 +265,11 @@ class NativeEngine:
 
     # given tokens instead of sampled ones
     def feed(self, tokens, handle=-1):
-        return self.scheduler.feed(tokens, handle)
+        held = self._fed.get(handle, 0) + len(tokens)
+        self._check_length(held)
+        handle = self.scheduler.feed(tokens, handle)
+        self._fed[handle] = held
+        return handle
 
     @torch.inference_mode()
     def run_fed(self, handles, counts, want):
@@ -275,6 +287,7 @@ class NativeEngine:
 
     def close(self, handle):
         self.scheduler.close(handle)
+        self._fed.pop(handle, None)
 
     def generate(self, seqs):
         """Runs the requests to completion; -> {handle: completion token ids}."""

@@ -124,15 +124,16 @@ class Attention(nn.Module):
 
 def window_attention(q, k_cache, v_cache, context_lens, block_table, num_heads, head_dim, v_dim, scale,
                      window=0, softcap=0.0, cu_seqlens_q=None, max_seqlen_q=0, out=None, impl="auto", chunk=0, sink=None,
-                     gate=None, gate_mode=None, out_scale=1.0):
-    """Attention with a sliding window or chunks, soft cap, sink [Hq] (fp32) and output gate (`gate_mode` "head": one
+                     gate=None, gate_mode=None, out_scale=1.0, keep=0, slopes=None):
+    """Attention with a sliding window or chunks, `keep` first tokens that are always seen, soft cap, distance biases
+    (`slopes` [Hq] fp32 times the distance, off the scores), sink [Hq] (fp32) and output gate (`gate_mode` "head": one
     logit per head, "entry": one per entry of the result) over paged caches whose rows are padded to multiples of 16
     (k_cache [P, BS, Hkv, KP], v_cache [P, BS, Hkv, VP]).  q [rows, Hq * D] may be a column view of a
     projection.  One row per sequence without `cu_seqlens_q`."""
-    L.require_cuda(q, k_cache, v_cache, context_lens, block_table, cu_seqlens_q, sink, gate)
+    L.require_cuda(q, k_cache, v_cache, context_lens, block_table, cu_seqlens_q, sink, gate, slopes)
     P, BS, Hkv, KP = k_cache.shape
     VP = v_cache.shape[3]
-    assert sink is None or sink.dtype == torch.float32 and sink.is_contiguous()
+    assert all(t is None or t.dtype == torch.float32 and t.is_contiguous() and t.numel() == num_heads for t in (sink, slopes))
     assert gate is None or gate.dtype == q.dtype and gate.stride(1) == 1
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and q.stride(1) == 1 and block_table.stride(1) == 1
     if out is None:
@@ -142,14 +143,14 @@ def window_attention(q, k_cache, v_cache, context_lens, block_table, num_heads, 
     lib = L.load()
     ws = None
     if cu_seqlens_q is None:
-        span = min([NB * BS] + [n for n in (window, chunk) if n])
+        span = min([NB * BS] + [n + int(keep) for n in (window, chunk) if n])
         need = lib.zp_window_attention_workspace_bytes(B, num_heads, Hkv, VP, span)
         ws = _workspace(q.device, need) if need else None
     L.check(lib.zp_window_attention(
         L.ptr(q), L.ptr(k_cache), L.ptr(v_cache), L.ptr(cu_seqlens_q), L.ptr(context_lens), L.ptr(block_table),
         L.ptr(out), B, int(max_seqlen_q), NB, num_heads, Hkv, head_dim, v_dim, KP, VP, BS, P, q.stride(0),
         out.stride(0), float(scale), float(softcap or 0.0), int(window or 0), int(chunk or 0),
-        L.ptr(sink), L.ptr(gate), 0 if gate is None else gate.stride(0), L.GATE[gate_mode], float(out_scale), q.shape[0],
+        int(keep), L.ptr(slopes), L.ptr(sink), L.ptr(gate), 0 if gate is None else gate.stride(0), L.GATE[gate_mode], float(out_scale), q.shape[0],
         L.IMPL[impl], L.dtype_code(q),
         L.ptr(ws), 0 if ws is None else ws.numel(), L.stream_ptr()), "window_attention")
     _count(1)
@@ -167,27 +168,38 @@ def store_kv_padded(k, v, k_cache, v_cache, slot_mapping, head_dim, v_dim):
     _count(1)
 
 
+def distance_slopes(heads):
+    """Slopes of linear distance biases, a geometric sequence that ends at 2^-8."""
+    return [2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)]
+
+
 class WindowAttentionMixer(nn.Module):
     """Grouped-query attention without rotation, with a sliding window and a soft cap on the scores;
     h -> head outputs [rows, heads * vdim] before the output projection.  `run` selects the cache of
-    this pass when the layer runs several times."""
+    this pass when the layer runs several times.  Optional: `keep` first tokens that stay visible behind the window, distance
+    biases (`slopes`, one per head), biases of the projections (named as their weights with '.b' added)."""
 
-    def __init__(self, width, heads, kv_heads, dim, vdim, scale, softcap, window, dtype, device):
+    def __init__(self, width, heads, kv_heads, dim, vdim, scale, softcap, window, dtype, device, keep=0, slopes=None, bias=False):
         super().__init__()
+        self.keep = keep
+        self.slopes = None if slopes is None else nn.Parameter(torch.tensor(slopes, dtype=torch.float32, device=device), requires_grad=False)
         self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
         self.scale, self.softcap, self.window = scale, softcap, window
         e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
         self.qkv = e(heads * dim + kv_heads * (dim + vdim), width)
+        self.qkv_bias = e(heads * dim + kv_heads * (dim + vdim)) if bias else None
         self.out_proj = e(width, heads * vdim)
         self.caches = []                                       # one (k_cache, v_cache) per pass
 
     def load(self, get):
         self.qkv.copy_(torch.cat([get(n) for n in "qkv"], 0))
+        if self.qkv_bias is not None:
+            self.qkv_bias.copy_(torch.cat([get(n + ".b") for n in "qkv"], 0))
         self.out_proj.copy_(get("o"))
 
     def forward(self, h, run):
         ctx = get_context()
-        x = torch.mm(h, self.qkv.t())
+        x = torch.mm(h, self.qkv.t()) if self.qkv_bias is None else torch.addmm(self.qkv_bias, h, self.qkv.t())
         nq, nk = self.heads * self.dim, self.kv_heads * self.dim
         q, k, v = x[:, :nq], x[:, nq:nq + nk], x[:, nq + nk:]
         kc, vc = self.caches[run]
@@ -195,11 +207,12 @@ class WindowAttentionMixer(nn.Module):
         out = torch.empty((h.shape[0], self.heads * self.vdim), dtype=h.dtype, device=h.device)
         nd = ctx.decode_rows()
         shape = (self.heads, self.dim, self.vdim, self.scale, self.window, self.softcap)
+        kw = dict(out=out, keep=self.keep, slopes=self.slopes)
         if nd:
-            window_attention(q, kc, vc, ctx.context_lens[:nd], ctx.block_tables[:nd], *shape, out=out)
+            window_attention(q, kc, vc, ctx.context_lens[:nd], ctx.block_tables[:nd], *shape, **kw)
         if ctx.is_prefill and nd < ctx.context_lens.shape[0]:
             window_attention(q, kc, vc, ctx.context_lens[nd:], ctx.block_tables[nd:], *shape,
-                             cu_seqlens_q=ctx.cu_seqlens_q[nd:], max_seqlen_q=ctx.max_seqlen_q, out=out)
+                             cu_seqlens_q=ctx.cu_seqlens_q[nd:], max_seqlen_q=ctx.max_seqlen_q, **kw)
         return out
 
 

@@ -12,6 +12,7 @@ from torch import nn
 from .. import _lib as L
 from ..kernel import _count
 from .row_ops import project
+from .step_ops import silu_and_mul
 
 
 def gelu_tanh_and_mul(x):
@@ -33,18 +34,20 @@ def relu_squared_(x):
     return x
 
 
-def moe_route(logits, n_experts, top, score="softmax", by_place=False):
+def moe_route(logits, n_experts, top, score="softmax", by_place=False, bias=None):
     """logits [N, >= n_experts] fp32 -> (weights [N, top] fp32, experts [N, top], places [N, top],
-    rows [N * top], offsets [n_experts + 1]): scores (softmax over all experts, or sigmoid), the `top` largest of a
+    rows [N * top], offsets [n_experts + 1]): scores of logits + bias (softmax over all experts or, "softmax_top", over the
+    chosen ones; or sigmoid), the `top` largest of a
     token, and the (token, expert) pairs sorted by expert.  `by_place`: the weights in that order instead, [N * top]."""
-    L.require_cuda(logits)
+    L.require_cuda(logits, bias)
+    assert bias is None or bias.dtype == torch.float32 and bias.is_contiguous()
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     N, dev = logits.shape[0], logits.device
     w = torch.empty((N, top), dtype=torch.float32, device=dev)
     ints = torch.empty(3 * N * top + 2 * n_experts + 1, dtype=torch.int32, device=dev)
     experts, places, rows, offsets, counts = ints.split([N * top] * 3 + [n_experts + 1, n_experts])
     pw = torch.empty(N * top, dtype=torch.float32, device=dev) if by_place else None
-    L.check(L.load().zp_moe_route(L.ptr(logits), logits.stride(0), N, n_experts, top, L.ptr(w), L.ptr(experts), L.ptr(places),
+    L.check(L.load().zp_moe_route(L.ptr(logits), logits.stride(0), L.ptr(bias), N, n_experts, top, L.ptr(w), L.ptr(experts), L.ptr(places),
                                   L.ptr(rows), L.ptr(offsets), L.ptr(counts), L.ptr(pw), L.SCORE[score], L.stream_ptr()), "moe_route")
     _count(1 if N <= 512 and N * top <= 4096 else 2)
     return w if pw is None else pw, experts.view(N, top), places.view(N, top), rows, offsets
@@ -80,6 +83,22 @@ class GatedFF(nn.Module):
 
     def forward(self, h):
         return {"b": project(gelu_tanh_and_mul(project(h, self.gate_up)), self.down)}
+
+
+class SquaredReluFF(nn.Module):
+    """W_down max(W_up h, 0)^2."""
+
+    def __init__(self, width, ff, dtype, device):
+        super().__init__()
+        e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
+        self.up, self.down = e(ff, width), e(width, ff)
+
+    def load(self, get):
+        self.up.copy_(get("up"))
+        self.down.copy_(get("down"))
+
+    def forward(self, h):
+        return {"b": project(relu_squared_(project(h, self.up)), self.down)}
 
 
 class MixtureFF(nn.Module):
@@ -136,15 +155,19 @@ def interleave_gate_up(out, gate, up):
 
 
 class GatedMixtureFF(nn.Module):
-    """`top` of `experts` SiLU-gated blocks per token, W_down (silu(W_gate z) * (W_up z)), each on z = s h with its
-    own score s (sigmoid by default, not renormalised): the score joins the gate and up products' epilogue."""
+    """`top` of `experts` SiLU-gated blocks per token, W_down (silu(W_gate z) * (W_up z)).  weigh "input": each on z = s h with
+    its own score s (the score joins the gate and up products' epilogue); "output": on z = h, and the scores weight the sum.
+    `score` as in `moe_route`.  Optional: a bias of the router's logits, a shared block of the same form that every token takes."""
 
-    def __init__(self, width, experts, top, ff, dtype, device, score="sigmoid"):
+    def __init__(self, width, experts, top, ff, dtype, device, score="sigmoid", weigh="input", bias=False, shared_ff=0):
         super().__init__()
-        self.experts, self.top, self.ff, self.score = experts, top, ff, score
+        self.experts, self.top, self.ff, self.score, self.weigh, self.shared_ff = experts, top, ff, score, weigh, shared_ff
+        self.bias = nn.Parameter(torch.empty(experts, dtype=torch.float32, device=device), requires_grad=False) if bias else None
         e = lambda *s: nn.Parameter(torch.empty(*s, dtype=dtype, device=device), requires_grad=False)
         self.router = e((experts + 7) // 8 * 8, width)      # (zero rows up to a multiple of 8: aligned rows of logits)
         self.gate_up, self.down = e(experts, 2 * padded_ff(ff), width), e(experts, width, padded_ff(ff))
+        if shared_ff:                                       # (gate rows, then up rows, each with zeros past the last)
+            self.shared_gate_up, self.shared_down = e(2, padded_ff(shared_ff), width), e(width, padded_ff(shared_ff))
 
     def load(self, get):
         self.down.zero_()
@@ -153,9 +176,23 @@ class GatedMixtureFF(nn.Module):
             self.down[i, :, :self.ff].copy_(get(f"e{i}.down"))
         self.router.zero_()
         self.router[:self.experts].copy_(get("router"))
+        if self.bias is not None:
+            self.bias.copy_(get("router.b"))
+        if self.shared_ff:
+            self.shared_gate_up.zero_()
+            self.shared_down.zero_()
+            for i, n in enumerate(("gate", "up")):
+                self.shared_gate_up[i, :self.shared_ff].copy_(get("shared." + n))
+            self.shared_down[:, :self.shared_ff].copy_(get("shared.down"))
 
     def forward(self, h):
-        places = h.shape[0] * self.top
-        w, _, pos, rows, offsets = moe_route(project(h, self.router, fp32=True), self.experts, self.top, self.score, by_place=True)
-        mid = grouped_gemm(h, self.gate_up, offsets, places, rows=rows, act="silu_mul", row_scale=w)
-        return {"y": grouped_gemm(mid, self.down, offsets, places), "pos": pos}
+        places, early = h.shape[0] * self.top, self.weigh == "input"
+        w, _, pos, rows, offsets = moe_route(project(h, self.router, fp32=True), self.experts, self.top, self.score, by_place=early,
+                                             bias=self.bias)
+        mid = grouped_gemm(h, self.gate_up, offsets, places, rows=rows, act="silu_mul", row_scale=w if early else None)
+        out = {"y": grouped_gemm(mid, self.down, offsets, places), "pos": pos}
+        if not early:
+            out["weights"] = w
+        if self.shared_ff:
+            out["b"] = project(silu_and_mul(project(h, self.shared_gate_up.view(-1, h.shape[1]))), self.shared_down)
+        return out

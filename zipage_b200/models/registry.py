@@ -92,6 +92,15 @@ def _tukarax(config, weights, dtype, device):
     return LoadedModel("Tukarax", model, model.head, cfg.width, cfg.vocab, dtype, portions=True)
 
 
+@register("Dinatar", part="dinatar")
+def _dinatar(config, weights, dtype, device):
+    from .dinatar import DinatarConfig, DinatarModel
+    cfg = DinatarConfig.from_dict(config)
+    model = DinatarModel(cfg, dtype, device, DinatarModel.ranks_of(weights))
+    model.load_weights(weights)
+    return LoadedModel("Dinatar", model, model.head, cfg.width, cfg.vocab, dtype, portions=True)
+
+
 @register("Qwen3ForCausalLM")
 def _qwen3(config, weights, dtype, device):
     from ..engine.native_engine import full_state_from_hf
