@@ -51,7 +51,7 @@ def parse_args():
                     help="also run the reference ENGINE (baseline/_ref) on a synthetic Qwen3-8B-shaped model, as it "
                          "is and with this library's decode path bound, and report decode tokens/s (adds minutes)")
     ap.add_argument("--also-exact", action="store_true", help="time the exact variant as well")
-    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine", "similorn", "dobedra", "tukarax"],
+    ap.add_argument("--workload", default="compress", choices=["compress", "decode", "step_ops", "prefill", "decode_step", "tp_allreduce", "engine_decode", "long_prompt", "host_control", "native_engine", "similorn", "dobedra", "tukarax", "dinatar"],
                     help="compress (default, the headline op), decode (paged decode attention kernel) or "
                          "step_ops (the element-wise ops of a decoder layer step and the sampler) or "
                          "prefill (varlen causal prefill attention, one layer) or decode_step (the decode "
@@ -1056,7 +1056,7 @@ class KernelTable:
     products at the measured cuBLAS rate) and how many times farther from it than the like kernel."""
 
     def __init__(self, args, peaks):
-        self.args, self.recs, self.launches = args, {}, 0
+        self.args, self.recs, self.launches, self.share = args, {}, 0, {}
         self.hbm, self.tf = peaks.get("hbm_gbs", 6650.0) * 1e9, peaks.get("bf16_tflops", 1590.0) * 1e12
 
     def __call__(self, name, fn, nbytes, flops=0.0, like=None, graph=False):
@@ -1084,12 +1084,13 @@ class KernelTable:
         ms = e0.elapsed_time(e1) / self.args.steps
         self.launches += self.args.steps
         roof = max(nbytes / self.hbm, flops / self.tf)
+        self.share[name] = roof / (ms * 1e-3)
         r = self.recs[name] = {"ms": round(ms, 4), "bound": "hbm" if nbytes / self.hbm >= flops / self.tf else "tensor",
-                               "frac": round(roof / (ms * 1e-3), 3), "gbs": round(nbytes / ms / 1e6, 1),
+                               "frac": round(self.share[name], 3), "gbs": round(nbytes / ms / 1e6, 1),
                                "tflops": round(flops / ms / 1e9, 1)}
         if like:
             r["like"] = like
-            r["distance_ratio"] = round(self.recs[like]["frac"] / r["frac"], 2)
+            r["distance_ratio"] = round(self.share[like] / self.share[name], 2)
 
 
 def qwen_of_size(dev, width, heads, kv, ff, blocks):
@@ -1673,6 +1674,217 @@ def run_tukarax(args):
     }))
 
 
+def dinatar_kernel_records(args, dev, peaks):
+    """Every kernel of the Dinatar decoder at sizes of an 8B-class model's layers (width 4096; linear attention with 16 states of
+    128 x 256 or 32 of 128 x 128; attention 32 / 8 heads of 128, window 1024 behind 64 kept tokens; 64 experts of 1024, six a token;
+    bf16) beside the like kernel of the closest existing path at equal size: Similorn's matrix memory and attention, Tukarax's
+    convolution, boundaries and experts.  Inputs are larger than L2 wherever the kernel streams."""
+    import torch
+    from zipage_b200.layers import attention as A
+    from zipage_b200.layers import feed_forward as F
+    from zipage_b200.layers import gated_delta as G
+    from zipage_b200.layers import linear_state as S_
+    from zipage_b200.layers import row_ops as R
+    from zipage_b200.layers import step_ops as P
+    from zipage_b200.layers.mlstm import mlstm_step
+    bf, f32, W = torch.bfloat16, torch.float32, 4096
+    rnd = lambda *s, dt=bf: torch.empty(s, dtype=dt, device=dev).normal_()
+    i32 = lambda t: t.to(torch.int32).to(dev)
+    rec = KernelTable(args, peaks)
+
+    # prompts: 4 x 4096 tokens
+    B, S = 4, 4096
+    T = B * S
+    cu, ctx, pos = i32(torch.arange(0, T + 1, S)), i32(torch.full((B,), S)), torch.arange(S, device=dev).repeat(B)
+    q, kc, vc = rnd(T, HQ * D), rnd(T // 64, 64, HKV, D), rnd(T // 64, 64, HKV, D)
+    table, out = i32(torch.arange(T // 64).view(B, -1)), torch.empty(T, HQ * D, dtype=bf, device=dev)
+    slopes = torch.tensor(A.distance_slopes(HQ), device=dev)
+    io = 2.0 * T * D * (2 * HQ + 2 * HKV)
+    rec("window attention prefill, window 1024",
+        lambda: A.window_attention(q, kc, vc, ctx, table, HQ, D, D, D ** -0.5, 1024, 30.0, cu_seqlens_q=cu, max_seqlen_q=S, out=out),
+        io, 4.0 * D * HQ * B * sum(min(p + 1, 1024) for p in range(S)))
+    rec("biased attention prefill, window 1024 and 64 kept",
+        lambda: A.window_attention(q, kc, vc, ctx, table, HQ, D, D, D ** -0.5, 1024, cu_seqlens_q=cu, max_seqlen_q=S, out=out, keep=64, slopes=slopes),
+        io, 4.0 * D * HQ * B * sum(min(p + 1, 1024 + min(64, max(0, p - 1023))) for p in range(S)), "window attention prefill, window 1024")
+    kv, slot = rnd(T, HQ * D + 2 * HKV * D), i32(torch.arange(T))
+    rec("key/value store", lambda: A.store_kv_padded(kv[:, HQ * D:HQ * D + HKV * D], kv[:, HQ * D + HKV * D:], kc, vc, slot, D, D), 8.0 * T * HKV * D)
+    del q, kv, out
+
+    mh, mk, mv = 16, 128, 256
+    mnorm, mbias = torch.ones(mh * mv, device=dev), torch.zeros(2 * mh, device=dev)
+    mbias[mh:] = 4.0
+
+    def memory(rows, n, cu=None, ctx=None):
+        x, gates, o = rnd(rows, 2 * mh * (mk + mv)), rnd(rows, 2 * mh, dt=f32), torch.empty(rows, mh * mv, dtype=bf, device=dev)
+        st, slots = (torch.zeros(n, mh, mk, mv, device=dev), torch.zeros(n, mh, mk, device=dev), torch.zeros(n, mh, device=dev)), i32(torch.arange(n))
+        cols = x[:, :mh * mk], x[:, mh * mk:2 * mh * mk], x[:, 2 * mh * mk:2 * mh * mk + mh * mv], x[:, 2 * mh * mk + mh * mv:]
+        return lambda: mlstm_step(*cols, gates, mbias, mnorm, st, o, ctx, slots, mh, mk, mv, 15.0, 1e-5, cu_seqlens_q=cu)
+    H, G_, N, V, taps = 32, 2, 128, 128, 4       # the state-space mixer
+    C = H * V + 2 * G_ * N
+    cw, cb = rnd(taps, C, dt=f32) * 0.5, rnd(C, dt=f32)
+
+    def linear(kind, rows, n, cu=None, ctx=None, norm=True):
+        """Recurrence and the norm with its gate, as the layers call them."""
+        slots = i32(torch.arange(n))
+        if kind == "scalar":
+            x, z, g = rnd(rows, C), rnd(rows, H * V), rnd(rows, H, dt=f32)
+            vec = {"A_log": torch.zeros(H, device=dev), "D": torch.ones(H, device=dev)}
+            if cu is None:
+                vec |= {"conv_weight": cw, "conv_bias": cb, "ring": rnd(n, taps, C)}
+            st, o, w, bias = torch.zeros(n, H, N, V, device=dev), torch.empty(rows, H * V, dtype=bf, device=dev), torch.ones(H * V, device=dev), \
+                torch.full((H,), -2.0, device=dev)
+
+            def run():
+                S_.linear_state(kind, x[:, H * V + G_ * N:], x[:, H * V:H * V + G_ * N], x[:, :H * V], g, bias, st, o, ctx, slots, H, G_, N, V,
+                                cu_seqlens_q=cu, **vec)
+                if norm:
+                    S_.group_norm_gate(o, w, G_, 1e-5, pre_gate=z, out=o)
+            return run
+        nk, nv = mh * mk, mh * mv
+        x, g = rnd(rows, 2 * nk + 2 * nv), rnd(rows, nk, dt=f32)
+        vec = {"lower": torch.full((nk,), 0.5, device=dev)} if kind == "forget" else {"rtau": 1 / 16, "qscale": mk ** -0.5}
+        st, o, w, bias = torch.zeros(n, mh, mk, mv, device=dev), torch.empty(rows, nv, dtype=bf, device=dev), torch.ones(mv, device=dev), \
+            torch.ones(nk, device=dev)
+
+        def run():
+            S_.linear_state(kind, x[:, :nk], None if kind == "forget" else x[:, nk:2 * nk], x[:, 2 * nk:2 * nk + nv], g, bias, st, o, ctx, slots, mh, mh,
+                            mk, mv, cu_seqlens_q=cu, **vec)
+            if norm:
+                S_.group_norm_gate(o, w, mh, 1e-5, post_gate=None if kind == "forget" else x[:, 2 * nk + nv:], out=o)
+        return run
+    # products of the chunked form (64 tokens): scores and their values (causal half), read-out, update
+    rec("mlstm prefill", memory(T, B, cu, ctx), 2.0 * T * mh * (2 * mk + 3 * mv) + 8.0 * T * mh, 2.0 * T * mh * (32 * (mk + mv) + 2 * mk * mv))
+    chunked = lambda h, dk, dv: 2.0 * T * h * (32 * (dk + dv) + 2 * dk * dv)
+    rec("hgrn2 prefill", linear("forget", T, B, cu, ctx), T * mh * (2.0 * (mk + 2 * mv) + 4.0 * mk), chunked(mh, mk, mv), "mlstm prefill")
+    rec("gla prefill", linear("power", T, B, cu, ctx), T * mh * (2.0 * (2 * mk + 3 * mv) + 4.0 * mk), chunked(mh, mk, mv), "mlstm prefill")
+    rec("ssd prefill", linear("scalar", T, B, cu, ctx), T * (2.0 * (3 * H * V + 2 * G_ * N) + 4.0 * H), chunked(H, N, V), "mlstm prefill")
+    x, y, w0, w1 = rnd(T, W), torch.empty(T, W, dtype=bf, device=dev), torch.ones(mv, device=dev), torch.ones(W, device=dev)
+    gate, wr, res = rnd(T, W), torch.ones(W, dtype=bf, device=dev), rnd(T, W)
+    rec("qwen3 add + rms norm", lambda: P.rms_norm(x, wr, 1e-6, res), 8.0 * T * W)
+    rec("norm per head", lambda: S_.group_norm_gate(x, w0, mh, 1e-5, out=y), 4.0 * T * W, 0.0, "qwen3 add + rms norm")
+    rec("norm per head, gate after", lambda: S_.group_norm_gate(x, w0, mh, 1e-5, post_gate=gate, out=y), 6.0 * T * W, 0.0, "qwen3 add + rms norm")
+    rec("norm of two parts, gate before", lambda: S_.group_norm_gate(x, w1, 2, 1e-5, pre_gate=gate, out=y), 6.0 * T * W, 0.0, "qwen3 add + rms norm")
+    xc, yc, ring, slots = rnd(T, C), rnd(T, C), rnd(B, taps, C), i32(torch.arange(B))
+    rec("short convolution", lambda: G.short_conv(xc, cw, ring, ctx, slots, cu, S, yc), 4.0 * T * C)
+    rec("short convolution with a bias", lambda: G.short_conv(xc, cw, ring, ctx, slots, cu, S, yc, bias=cb), 4.0 * T * C, 0.0, "short convolution")
+    del xc, yc, gate, res
+    # decode: 256 sequences
+    n, NB = 256, 9
+    lens, qd = i32(torch.full((n,), NB * 256 - 7)), rnd(n, HQ * D)
+    kq, vq = rnd(n * NB, 256, HKV, D), rnd(n * NB, 256, HKV, D)
+    bt = i32(torch.randperm(n * NB).view(n, NB))
+    for seqs in (256, 64):
+        a = qd[:seqs], kq, vq, lens[:seqs], bt[:seqs], HQ, D, D, D ** -0.5
+        rec(f"window attention decode, window 1024, {seqs} sequences", lambda: A.window_attention(*a, 1024, 30.0), seqs * 1024 * HKV * D * 4.0)
+        rec(f"biased attention decode, window 1024 and 64 kept, {seqs} sequences", lambda: A.window_attention(*a, 1024, keep=64, slopes=slopes),
+            seqs * 1088 * HKV * D * 4.0, 0.0, f"window attention decode, window 1024, {seqs} sequences")
+    del kq, vq
+    five = i32(torch.full((n,), 5))
+    for seqs in (256, 64):
+        rec(f"mlstm decode, {seqs} sequences", memory(seqs, seqs, None, five[:seqs]), 8.0 * seqs * mh * mk * mv)
+        for name, kind in (("hgrn2", "forget"), ("gla", "power"), ("ssd", "scalar")):
+            rec(f"{name} decode, {seqs} sequences", linear(kind, seqs, seqs, None, five[:seqs], norm=False),
+                8.0 * seqs * mh * mk * mv + (2.0 * seqs * taps * C if kind == "scalar" else 0.0), 0.0, f"mlstm decode, {seqs} sequences")
+    # boundaries
+    xf, a, b, m1, m2 = rnd(T, W, dt=f32), *(rnd(T, W) for _ in range(4))
+    norms = [(torch.ones(W, device=dev), torch.zeros(W, device=dev))]
+    E, top, ff = 64, 6, 1024
+    yy, places, wt = rnd(T * top, W), i32(torch.randperm(T * top)).view(T, top), torch.rand(T, top, device=dev)
+    pair = ((m1, w1), (m2, w1))
+    like = "layer boundary, mixer and feed-forward"
+    rec(like, lambda: R.join_norms(xf, norms, 1e-5, bf, a=a, b=b), 14.0 * T * W, 0.0, "qwen3 add + rms norm")
+    rec("layer boundary, normed pair and feed-forward", lambda: R.join_norms(xf, norms, 1e-5, bf, b=b, pair=pair), 16.0 * T * W, 0.0, like)
+    rec("layer boundary, mixer, experts and shared", lambda: R.join_norms(xf, norms, 1e-5, bf, a=a, b=b, y=yy, pos=places, weights=wt),
+        (14.0 + 2 * top) * T * W, 0.0, like)
+    rec("layer boundary, normed pair, experts and shared", lambda: R.join_norms(xf, norms, 1e-5, bf, b=b, pair=pair, y=yy, pos=places, weights=wt),
+        (16.0 + 2 * top) * T * W, 0.0, like)
+    del yy, a, b, m1, m2, pair
+    tok, emb, learned = torch.randint(0, 32768, (T,), device=dev), rnd(32768, W), rnd(S, W)
+    rec("embedding", lambda: R.embed_position(tok, pos, emb, 1.0), 6.0 * T * W)
+    rec("embedding and learned position", lambda: R.embed_position(tok, pos, emb, 12.0, learned=learned), 6.0 * T * W + 2.0 * S * W, 0.0, "embedding")
+    up = rnd(T, 2 * 12288)
+    rec("qwen3 silu and mul", lambda: P.silu_and_mul(up), 6.0 * T * 12288)
+    rec("squared relu", lambda: F.relu_squared_(up), 8.0 * T * 12288, 0.0, "qwen3 silu and mul")
+    del up
+    # experts
+    zl, rb = rnd(T, E, dt=f32), rnd(E, dt=f32)
+    for t, name in ((T, "prompts"), (64, "64 tokens")):
+        rec(f"routing by softmax, {name}", lambda: F.moe_route(zl[:t], E, top), 4.0 * t * E + t * top * 20.0, graph=True)
+        rec(f"routing by softmax over the chosen, {name}", lambda: F.moe_route(zl[:t], E, top, "softmax_top", bias=rb), 4.0 * t * E + t * top * 20.0, 0.0,
+            f"routing by softmax, {name}", graph=True)
+    dn, wg, wdn = rnd(T, W), rnd(E, 2 * ff, W), rnd(E, W, ff)
+    s = torch.rand(T * top, device=dev)
+    _, _, _, prow, off = F.moe_route(zl, E, top)
+    M = T * top
+    fl = 2.0 * (T * W + wg.numel() + M * ff), 4.0 * M * W * ff
+    rec("experts gate and up, scaled inputs", lambda: F.grouped_gemm(dn, wg, off, M, rows=prow, act="silu_mul", row_scale=s), *fl)
+    rec("experts gate and up", lambda: F.grouped_gemm(dn, wg, off, M, rows=prow, act="silu_mul"), *fl, "experts gate and up, scaled inputs")
+    return rec.recs, rec.launches
+
+
+def dinatar_of_size(dev, width, heads, kv, experts, top, eff, layers=12):
+    """A Dinatar decoder with random weights: its three kinds of layers in turn, experts and a shared one after each."""
+    import torch
+    from zipage_b200.models.dinatar import DinatarConfig, DinatarModel
+    from zipage_b200.models.registry import LoadedModel
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": eff}, "shared": {"ff": eff}}
+    kinds = [{"type": "hgrn2", "mixer": {"heads": heads, "dim": 128, "vdim": 128}},
+             {"type": "gla", "mixer": {"heads": heads // 2, "dim": 128, "vdim": 256, "tau": 16.0}},
+             {"type": "parallel", "mixer": {
+                 "left": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024, "keep_first": 64}},
+                 "right": {"heads": heads, "groups": 2, "state": 128, "vdim": 128, "conv": 4, "norm_groups": 2}}}]
+    c = DinatarConfig.from_dict({"vocab": 32768, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "logit_scale": 1.0,
+                                 "max_positions": 4096, "layers": [{**kinds[i % 3], "mlp": mlp} for i in range(layers)]})
+    m = DinatarModel(c, torch.bfloat16, dev, {i: 16 for i in range(layers) if i % 3 == 1})
+    with torch.no_grad():
+        for n, p in m.named_parameters():
+            if n.endswith("slopes"):
+                continue
+            if p.dim() > 1:
+                p.normal_(0, p.shape[-1] ** -0.5)
+            else:
+                p.fill_(0.5) if "lower" in n else p.zero_() if "bias" in n or "A_log" in n else p.fill_(1.0)
+    return LoadedModel("Dinatar", m, m.head, width, 32768, torch.bfloat16, True)
+
+
+def run_dinatar(args):
+    """Prefill and decode throughput of the Dinatar decoder through the serving engine at two widths, random weights, beside
+    Tukarax decoders of equal width, depth, heads and experts and Qwen3 blocks whose feed-forward is as wide as what a token's
+    experts add up to; and the kernel table."""
+    import torch
+    dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
+    torch.cuda.set_device(dev)
+    pk = ROOT / "MEASURED_PEAKS.json"
+    peaks = json.loads(pk.read_text()) if pk.exists() else {}
+    torch.manual_seed(3)
+    R, PROMPT, GEN = SERVE
+    g = torch.Generator().manual_seed(1)
+    res = {}
+    with ClockSampler(dev.index or 0) as clocks:
+        kernels, launches = dinatar_kernel_records(args, dev, peaks)
+        torch.cuda.empty_cache()
+        for width, heads, kv, experts, top, eff in ((4096, 32, 8, 64, 6, 1024), (2048, 16, 4, 64, 6, 512)):
+            models = {"dinatar": lambda: dinatar_of_size(dev, width, heads, kv, experts, top, eff),
+                      "tukarax": lambda: tukarax_of_size(dev, width, heads, kv, experts, top, eff),
+                      "qwen3": lambda: qwen_of_size(dev, width, heads, kv, top * eff, 12)}
+            row = res[f"width {width}"] = {"layers": 12}
+            for name, make in models.items():
+                row[name] = serve_model(make(), g)
+                torch.cuda.empty_cache()
+    head = res["width 4096"]["dinatar"]
+    print(json.dumps({
+        "metric": "dinatar_decode_tokens_per_s", "value": head["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+        "steps": args.steps, "warmup": args.warmup, "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True,
+        "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": f"serving engine, {R} requests, prompts of {PROMPT}, {GEN} sampled tokens each; random weights; 12 layers "
+                               "(HGRN2, gated linear attention, windowed attention beside a state-space mixer in turn; 64 experts, six a "
+                               "token, and a shared one) beside 12 Tukarax layers and 12 Qwen3 blocks",
+                   "l2": "inputs of the streaming kernels are larger than L2"},
+        "serving": res, "kernels": kernels, "gpu_launches": launches, "clocks": clocks.summary(),
+        "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")},
+    }))
+
+
 def run_host_control(args):
     """Host time per decode step of the control plane at `--requests` concurrent requests: the
     native scheduler's array calls (schedule, the runner's input arrays, postprocess) and, when an
@@ -1787,6 +1999,8 @@ def main():
         return run_similorn(args)
     if args.workload == "dobedra":
         return run_dobedra(args)
+    if args.workload == "dinatar":
+        return run_dinatar(args)
     if args.workload == "tukarax":
         return run_tukarax(args)
     if args.workload == "prefill":

@@ -267,7 +267,7 @@ def test_linear_state_portions(H, G, dk, dv, kind, span):
                 z[at:at + m] = c["z"][d:d + m]
                 at += m
             x, done = _dev(x), [d + m for d, m in zip(done, n)]
-            out = torch.full((total, H * dv + 2), 9.0, dtype=dtype, device="cuda")
+            out = torch.full((total, (H * dv + 15) // 8 * 8), 9.0, dtype=dtype, device="cuda")
             cu = _i32([lead] + [lead + v for v in torch.tensor(n).cumsum(0).tolist()])
             linear_state(kind, x[:, :G * dk], None if kind == "forget" else x[:, nq:nq + G * dk], x[:, 2 * nq:2 * nq + H * dv], _dev(z),
                          _dev(cases[0]["bias"]), state, out[:, :H * dv], _i32(done), _i32(slots), H, G, dk, dv, cu_seqlens_q=cu, impl=impl, **shared)

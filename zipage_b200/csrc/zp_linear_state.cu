@@ -6,6 +6,7 @@
 // while keys, queries and decays are made.
 #include "zp_conv.cuh"
 #include "zp_linear_state.cuh"
+#include "zp_mma.cuh"       // packed 16-bit pairs
 
 namespace zp {
 
@@ -164,102 +165,136 @@ struct GroupNormArgs {
   int parts, width, per_part;
   float eps;
 };
+__device__ __forceinline__ float gn_ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float gn_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 template <typename T> __device__ __forceinline__ float gn_gate(float z) {
   if constexpr (sizeof(T) == 4) return z / (1.f + expf(-z));
-  else return __fdividef(z, 1.f + __expf(-z));      // (the fast forms' last bits disappear in the rounding to T)
+  else return z * gn_rcp(1.f + gn_ex2(-1.4426950408889634f * z));      // (the fast forms' last bits disappear in the rounding to T)
+}
+// a 16-byte piece as fp32 and back
+template <typename T> __device__ __forceinline__ void gn_unpack(const int4& raw, float (&v)[16 / sizeof(T)]) {
+  if constexpr (sizeof(T) == 4) {
+    v[0] = __int_as_float(raw.x); v[1] = __int_as_float(raw.y); v[2] = __int_as_float(raw.z); v[3] = __int_as_float(raw.w);
+  } else {
+    const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = Elem<T>::to_f32(e[j]);
+  }
+}
+template <typename T> __device__ __forceinline__ int4 gn_pack(const float (&v)[16 / sizeof(T)]) {
+  if constexpr (sizeof(T) == 4) return make_int4(__float_as_int(v[0]), __float_as_int(v[1]), __float_as_int(v[2]), __float_as_int(v[3]));
+  else return make_int4((int)pack2<T>(v[0], v[1]), (int)pack2<T>(v[2], v[3]), (int)pack2<T>(v[4], v[5]), (int)pack2<T>(v[6], v[7]));
 }
 
-template <typename T, int VPL, int TPP>   // TPP: threads of a part (32 or 256)
+template <typename T, int VPL, int TPP, int IT>   // TPP: threads of a part (32 or 256); IT: parts that a warp or block takes at a time
 __global__ void __launch_bounds__(256) group_norm_gate_kernel(const GroupNormArgs a) {
   __shared__ float red[32];
   constexpr int EPV = 16 / sizeof(T);
-  const int64_t item = TPP == 32 ? (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x;
-  if (item >= a.n) return;                       // (a whole warp or block)
+  const uint32_t first = (TPP == 32 ? blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x) * IT, count = (uint32_t)a.n;   // (below 2^31)
+  if (first >= count) return;                    // (a whole warp or block)
   const int lane = TPP == 32 ? threadIdx.x & 31 : threadIdx.x;
-  const int64_t row = item / a.parts;
-  const int part = (int)(item - row * a.parts), c0 = part * a.width;
-  const T* x = reinterpret_cast<const T*>(a.x) + row * a.x_stride + c0;
-  const T* pre = a.pre ? reinterpret_cast<const T*>(a.pre) + row * a.pre_stride + c0 : nullptr;
-  const T* post = a.post ? reinterpret_cast<const T*>(a.post) + row * a.post_stride + c0 : nullptr;
-  const float* w = a.w + (a.per_part ? c0 : 0);
-  T* out = reinterpret_cast<T*>(a.out) + row * a.out_stride + c0;
-  float ss = 0.f;
+  struct Part { int64_t row; int c0; };
+  const uint32_t row0 = first / (uint32_t)a.parts, part0 = first - row0 * a.parts;
+  auto at = [&](int t) {                         // the t-th of this warp's or block's parts
+    uint32_t row = row0, part = part0 + t;
+    while (part >= (uint32_t)a.parts) { part -= a.parts; ++row; }
+    return Part{(int64_t)row, (int)part * a.width};
+  };
+  const T *x = reinterpret_cast<const T*>(a.x), *pre = reinterpret_cast<const T*>(a.pre), *post = reinterpret_cast<const T*>(a.post);
+  T* out = reinterpret_cast<T*>(a.out);
   if constexpr (VPL > 0) {
     const int nvec = a.width / EPV;
-    int4 raw[VPL], g[VPL];
-    float v[VPL][EPV];
+    int4 raw[IT][VPL], g[IT][VPL];
 #pragma unroll
-    for (int i = 0; i < VPL; ++i)
-      if (lane + i * TPP < nvec) {
-        raw[i] = ld16(x + (lane + i * TPP) * EPV);
-        if (pre) g[i] = ld16(pre + (lane + i * TPP) * EPV);
-        else if (post) g[i] = ld16(post + (lane + i * TPP) * EPV);
-      }
+    for (int t = 0; t < IT; ++t) {
+      const Part p = at(min((uint32_t)t, count - 1 - first));
 #pragma unroll
-    for (int i = 0; i < VPL; ++i)
-      if (lane + i * TPP < nvec) {
-        const T *e = reinterpret_cast<const T*>(&raw[i]), *f = reinterpret_cast<const T*>(&g[i]);
-#pragma unroll
-        for (int j = 0; j < EPV; ++j) {
-          v[i][j] = Elem<T>::to_f32(e[j]);
-          if (pre) v[i][j] *= gn_gate<T>(Elem<T>::to_f32(f[j]));
-          ss = fmaf(v[i][j], v[i][j], ss);
+      for (int i = 0; i < VPL; ++i)
+        if (lane + i * TPP < nvec) {
+          const int c = p.c0 + (lane + i * TPP) * EPV;
+          raw[t][i] = ld16(x + p.row * a.x_stride + c);
+          if (pre) g[t][i] = ld16(pre + p.row * a.pre_stride + c);
+          else if (post) g[t][i] = ld16(post + p.row * a.post_stride + c);
         }
-      }
-    ss = TPP == 32 ? warp_sum(ss) : block_sum(ss, red);
-    const float r = 1.f / sqrtf(ss / (float)a.width + a.eps);
-#pragma unroll
-    for (int i = 0; i < VPL; ++i)
-      if (lane + i * TPP < nvec) {
-        const int c = (lane + i * TPP) * EPV;
-        if (pre && post) g[i] = ld16(post + c);
-        const T* f = reinterpret_cast<const T*>(&g[i]);
-        int4 res;
-        T* o = reinterpret_cast<T*>(&res);
-#pragma unroll
-        for (int j = 0; j < EPV; j += 4) {
-          const float4 wv = *reinterpret_cast<const float4*>(w + c + j);
-          const float ww[4] = {wv.x, wv.y, wv.z, wv.w};
-#pragma unroll
-          for (int u = 0; u < 4; ++u) {
-            float y = v[i][j + u] * r * ww[u];
-            if (post) y *= gn_gate<T>(Elem<T>::to_f32(f[j + u]));
-            o[j + u] = Elem<T>::from_f32(y);
-          }
-        }
-        st16(out + c, res);
-      }
-  } else {
-    for (int c = lane; c < a.width; c += TPP) {
-      float y = Elem<T>::to_f32(x[c]);
-      if (pre) y *= gn_gate<T>(Elem<T>::to_f32(pre[c]));
-      ss = fmaf(y, y, ss);
     }
+#pragma unroll
+    for (int t = 0; t < IT; ++t) {
+      if (first + t >= count) break;
+      const Part p = at(t);
+      float v[VPL][EPV], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < VPL; ++i)
+        if (lane + i * TPP < nvec) {
+          gn_unpack<T>(raw[t][i], v[i]);
+          if (pre) {
+            float z[EPV];
+            gn_unpack<T>(g[t][i], z);
+#pragma unroll
+            for (int j = 0; j < EPV; ++j) v[i][j] *= gn_gate<T>(z[j]);
+          }
+#pragma unroll
+          for (int j = 0; j < EPV; ++j) ss = fmaf(v[i][j], v[i][j], ss);
+        }
+      ss = TPP == 32 ? warp_sum(ss) : block_sum(ss, red);
+      const float r = 1.f / sqrtf(ss / (float)a.width + a.eps);
+      const float* w = a.w + (a.per_part ? p.c0 : 0);
+#pragma unroll
+      for (int i = 0; i < VPL; ++i)
+        if (lane + i * TPP < nvec) {
+          const int c = (lane + i * TPP) * EPV;
+          if (pre && post) g[t][i] = ld16(post + p.row * a.post_stride + p.c0 + c);
+#pragma unroll
+          for (int j = 0; j < EPV; j += 4) {
+            const float4 wv = *reinterpret_cast<const float4*>(w + c + j);
+            v[i][j] *= r * wv.x; v[i][j + 1] *= r * wv.y; v[i][j + 2] *= r * wv.z; v[i][j + 3] *= r * wv.w;
+          }
+          if (post) {
+            float z[EPV];
+            gn_unpack<T>(g[t][i], z);
+#pragma unroll
+            for (int j = 0; j < EPV; ++j) v[i][j] *= gn_gate<T>(z[j]);
+          }
+          st16(out + p.row * a.out_stride + p.c0 + c, gn_pack<T>(v[i]));
+        }
+    }
+  } else {
+    const Part p = at(0);
+    const float* w = a.w + (a.per_part ? p.c0 : 0);
+    auto entry = [&](int c) {
+      const float y = Elem<T>::to_f32(x[p.row * a.x_stride + p.c0 + c]);
+      return pre ? y * gn_gate<T>(Elem<T>::to_f32(pre[p.row * a.pre_stride + p.c0 + c])) : y;
+    };
+    float ss = 0.f;
+    for (int c = lane; c < a.width; c += TPP) { const float y = entry(c); ss = fmaf(y, y, ss); }
     ss = TPP == 32 ? warp_sum(ss) : block_sum(ss, red);
     const float r = 1.f / sqrtf(ss / (float)a.width + a.eps);
     for (int c = lane; c < a.width; c += TPP) {
-      float y = Elem<T>::to_f32(x[c]);
-      if (pre) y *= gn_gate<T>(Elem<T>::to_f32(pre[c]));
-      y *= r * w[c];
-      if (post) y *= gn_gate<T>(Elem<T>::to_f32(post[c]));
-      out[c] = Elem<T>::from_f32(y);
+      float y = entry(c) * r * w[c];
+      if (post) y *= gn_gate<T>(Elem<T>::to_f32(post[p.row * a.post_stride + p.c0 + c]));
+      out[p.row * a.out_stride + p.c0 + c] = Elem<T>::from_f32(y);
     }
   }
 }
 
+template <typename T, int VPL, int TPP, int IT> static void group_norm_items(const GroupNormArgs& a, cudaStream_t st) {
+  const int64_t per = (TPP == 32 ? 8 : 1) * IT;
+  group_norm_gate_kernel<T, VPL, TPP, IT><<<(unsigned)((a.n + per - 1) / per), 256, 0, st>>>(a);
+}
 template <typename T> static void launch_group_norm(const GroupNormArgs& a, bool vec, cudaStream_t st) {
-  constexpr int EPV = 16 / sizeof(T);
-  const unsigned warps = (unsigned)((a.n + 7) / 8), blocks = (unsigned)a.n;
-  const int nv = a.width / EPV;
+  const int nv = a.width / (int)(16 / sizeof(T));
+  const bool many = a.n >= 148 * 8 * 8 * 4;      // (few parts: spread over the SMs instead)
   if (!vec) {
-    if (a.width <= 1024) group_norm_gate_kernel<T, 0, 32><<<warps, 256, 0, st>>>(a);
-    else group_norm_gate_kernel<T, 0, 256><<<blocks, 256, 0, st>>>(a);
-  } else if (nv <= 32) group_norm_gate_kernel<T, 1, 32><<<warps, 256, 0, st>>>(a);
-  else if (nv <= 64) group_norm_gate_kernel<T, 2, 32><<<warps, 256, 0, st>>>(a);
-  else if (nv <= 256) group_norm_gate_kernel<T, 1, 256><<<blocks, 256, 0, st>>>(a);
-  else if (nv <= 512) group_norm_gate_kernel<T, 2, 256><<<blocks, 256, 0, st>>>(a);
-  else if (nv <= 1024) group_norm_gate_kernel<T, 4, 256><<<blocks, 256, 0, st>>>(a);
-  else group_norm_gate_kernel<T, 0, 256><<<blocks, 256, 0, st>>>(a);
+    if (a.width <= 1024) group_norm_items<T, 0, 32, 1>(a, st);
+    else group_norm_items<T, 0, 256, 1>(a, st);
+  } else if (nv <= 32) {
+    if (many) group_norm_items<T, 1, 32, 4>(a, st); else group_norm_items<T, 1, 32, 1>(a, st);
+  } else if (nv <= 64) {
+    if (many) group_norm_items<T, 2, 32, 2>(a, st); else group_norm_items<T, 2, 32, 1>(a, st);
+  } else if (nv <= 256) {
+    if (many) group_norm_items<T, 1, 256, 2>(a, st); else group_norm_items<T, 1, 256, 1>(a, st);
+  } else if (nv <= 512) group_norm_items<T, 2, 256, 1>(a, st);
+  else if (nv <= 1024) group_norm_items<T, 4, 256, 1>(a, st);
+  else group_norm_items<T, 0, 256, 1>(a, st);
 }
 
 }  // namespace zp
