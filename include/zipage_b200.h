@@ -442,7 +442,7 @@ int zp_store_kv_padded(const void* k, const void* v, void* k_cache, void* v_cach
  * 16-bit caches with KP, VP <= 256 and Hq / Hkv <= 16 take the tensor-core kernels (ZP_IMPL_SIMT: never), whose
  * one-row form may need a workspace (zp_window_attention_workspace_bytes, span = the most keys a row
  * sees).  With total_q (rows of q; 0 = not told), bf16 portions with head sizes up to 128 (multiples of 8) and no
- * soft cap or one of at most 69 take the tcgen05 kernel (ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED).  Scores and
+ * soft cap or one of at most 69 (no slopes beside a cap) take the tcgen05 kernel (ZP_IMPL_TCGEN05: always, or ZP_ERR_UNSUPPORTED).  Scores and
  * softmax weights are fp32 in all of them. */
 size_t zp_window_attention_workspace_bytes(int B, int Hq, int Hkv, int VP, int span);
 int zp_window_attention(const void* q, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens_q,

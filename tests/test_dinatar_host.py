@@ -121,6 +121,7 @@ def test_the_family_library_has_what_it_needs():
     used = {"zp_embed_position", "zp_join_norms", "zp_window_attention", "zp_store_kv_padded", "zp_prepare_decode", "zp_sample", "zp_last_error",
             "zp_device_error_async", "zp_moe_route", "zp_grouped_gemm", "zp_short_conv", "zp_silu_and_mul", "zp_relu_squared"}
     used |= set(re.findall(r"\.(zp_[a-z0-9_]+)\(", (B.PKG / "layers/linear_state.py").read_text()))
+    used |= set(re.findall(r"\.(zp_[a-z0-9_]+)\(", (B.PKG / "layers/short_conv.py").read_text()))
     assert "zp_linear_state" in used and "zp_group_norm_gate" in used
     missing = [n for n in used if not re.search(r"extern \"C\"[^\n]*\b" + n + r"\(", text)]
     assert not missing, missing

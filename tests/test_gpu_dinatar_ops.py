@@ -384,7 +384,7 @@ def test_linear_state_decoding(H, dk, dv, kind, dtype):
 def test_scalar_state_convolution_prompts_and_decoding(H, G, dk, dv, taps, dtype):
     """Prompts through the convolution, then single rows with the convolution in the launch, then portions again: outputs, state and
     the convolution's memory carry over; a batch of two sequences out of step, and a padding row."""
-    from zipage_b200.layers.gated_delta import short_conv
+    from zipage_b200.layers.short_conv import short_conv
     from zipage_b200.layers.linear_state import linear_state
     g = _gen(taps)
     T, nv, nk = [41, 30], H * dv, G * dk
@@ -445,7 +445,7 @@ def test_scalar_state_convolution_prompts_and_decoding(H, G, dk, dv, taps, dtype
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("C,taps", [(96, 2), (100, 3), (37, 4), (2056, 4), (40, 8), (16, 1)])
 def test_short_convolution_with_a_bias(C, taps, dtype):
-    from zipage_b200.layers.gated_delta import short_conv
+    from zipage_b200.layers.short_conv import short_conv
     g = _gen(C)
     plan = [2, 1, 16, 17, 3, 33, 5]
     x, w, b = _r(g, sum(plan), C).to(dtype), _r(g, C, taps), _r(g, C)

@@ -72,7 +72,7 @@ def test_the_family_library_has_what_it_needs():
     text = "".join((B.CSRC / f"{n}.cu").read_text() for n in B.PARTS["tukarax"])
     used = {"zp_embed_position", "zp_join_norms", "zp_window_attention", "zp_prepare_decode", "zp_sample", "zp_last_error",
             "zp_device_error_async"}
-    for f in ("layers/gated_delta.py", "layers/rotary.py"):
+    for f in ("layers/gated_delta.py", "layers/short_conv.py", "layers/rotary.py"):
         used |= set(re.findall(r"\.(zp_[a-z0-9_]+)\(", (B.PKG / f).read_text()))
     used |= {"zp_moe_route", "zp_grouped_gemm"}
     assert "zp_gated_delta" in used and "zp_rotate_store" in used

@@ -34,9 +34,9 @@ PARTS = {
                  "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
     "dobedra": ("zp_api", "zp_host_sched", "zp_latent", "zp_latent_decode_tc", "zp_latent_prefill_tc", "zp_moe", "zp_moe_tc", "zp_rows", "zp_step", "zp_tc",
                 "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
-    "tukarax": ("zp_api", "zp_delta", "zp_delta_tc", "zp_host_sched", "zp_moe", "zp_moe_tc", "zp_rope", "zp_rows", "zp_step", "zp_tc",
+    "tukarax": ("zp_api", "zp_conv", "zp_delta", "zp_delta_tc", "zp_host_sched", "zp_moe", "zp_moe_tc", "zp_rope", "zp_rows", "zp_step", "zp_tc",
                 "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
-    "dinatar": ("zp_api", "zp_delta", "zp_delta_tc", "zp_host_sched", "zp_linear_state", "zp_linear_state_tc", "zp_moe", "zp_moe_tc", "zp_rows",
+    "dinatar": ("zp_api", "zp_conv", "zp_host_sched", "zp_linear_state", "zp_linear_state_tc", "zp_moe", "zp_moe_tc", "zp_rows",
                 "zp_step", "zp_tc", "zp_window_attn", "zp_window_attn_mma", "zp_window_attn_tc"),
 }
 

@@ -62,7 +62,7 @@ __device__ __forceinline__ float2 lc_unpack(uint32_t v) { return __bfloat1622flo
 __device__ __forceinline__ int linear_first_slot(const LinearArgs& a, int b) { return (a.cu_seqlens_q[b] - a.cu_seqlens_q[0]) / LC_C + b; }
 static int linear_slots(int total_rows, int B) { return total_rows / LC_C + B; }
 
-// fp32 elementary functions on the special-function unit, with errors of a few 2^-24 of the result
+// fp32 functions on the special-function unit (relative errors of a few 2^-23; the logarithm near 1: absolute)
 __device__ __forceinline__ float lc_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float lc_lg2(float x) { float y; asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float lc_sigmoid(float z) { return lc_rcp(1.f + lc_ex2(-LC_LOG2E * z)); }
@@ -705,6 +705,9 @@ linear_scan_tc_kernel(const __grid_constant__ CUtensorMap tmV, const LsParams p)
         if (t < n && there) st16(o + t * a.out_stride, ld16(tile + t * LS_VT + cl));
       }
     }
+  }
+  if (*abortp) {                                           // a wait ran out: copies that are still on their way land first
+    for (int i = 0; i < 64; ++i) __nanosleep(4000);
   }
   fence_before_sync();
   __syncthreads();

@@ -12,19 +12,7 @@ from torch import nn
 from .. import _lib as L
 from ..kernel import _count
 from ..utils.context import get_context
-
-
-def short_conv(x, weight, ring, context_lens, slots, cu_seqlens_q, max_seqlen_q, out, bias=None):
-    """Causal convolution with silu over portions; x [rows, >= channels] (column view), weight [taps, channels] and bias [channels] fp32,
-    ring [slots, taps, channels], out [rows, channels]."""
-    L.require_cuda(x, weight, ring, context_lens, slots, cu_seqlens_q, out, bias)
-    taps, C = weight.shape
-    assert x.stride(1) == out.stride(1) == 1 and ring.is_contiguous() and ring.shape[1:] == (taps, C) and x.dtype == ring.dtype == out.dtype
-    L.check(L.load().zp_short_conv(
-        L.ptr(x), x.stride(0), L.ptr(weight), L.ptr(bias), L.ptr(ring), L.ptr(cu_seqlens_q), L.ptr(context_lens), L.ptr(slots), L.ptr(out),
-        out.stride(0), context_lens.shape[0], int(max_seqlen_q), C, taps, ring.shape[0], L.dtype_code(x), L.stream_ptr()), "short_conv")
-    _count(2)
-    return out
+from .short_conv import short_conv
 
 
 def gated_delta(x, gate, ab, A_log, dt_bias, norm_weight, state, out, context_lens, slots, heads, kv_heads, dim, vdim, eps,

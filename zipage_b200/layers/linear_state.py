@@ -13,8 +13,8 @@ from torch import nn
 from .. import _lib as L
 from ..kernel import _count
 from ..utils.context import get_context
-from .gated_delta import short_conv
 from .row_ops import project
+from .short_conv import short_conv
 
 KIND = {"forget": 0, "power": 1, "scalar": 2}
 
