@@ -1801,7 +1801,7 @@ def dinatar_kernel_records(args, dev, peaks):
     del yy, a, b, m1, m2, pair
     tok, emb, learned = torch.randint(0, 32768, (T,), device=dev), rnd(32768, W), rnd(S, W)
     rec("embedding", lambda: R.embed_position(tok, pos, emb, 1.0), 6.0 * T * W)
-    rec("embedding and learned position", lambda: R.embed_position(tok, pos, emb, 12.0, learned=learned), 6.0 * T * W + 2.0 * S * W, 0.0, "embedding")
+    rec("embedding and learned position", lambda: R.embed_position(tok, pos, emb, 3.0, learned=learned), 6.0 * T * W + 2.0 * S * W, 0.0, "embedding")
     up = rnd(T, 2 * 12288)
     rec("qwen3 silu and mul", lambda: P.silu_and_mul(up), 6.0 * T * 12288)
     rec("squared relu", lambda: F.relu_squared_(up), 8.0 * T * 12288, 0.0, "qwen3 silu and mul")

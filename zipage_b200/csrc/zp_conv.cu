@@ -35,7 +35,7 @@ template <typename T, int V> __device__ __forceinline__ void cv_store(T* p, cons
   else *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(&r);
 }
 
-template <typename T, int V, int TAPS>
+template <typename T, int V, int TAPS, bool BIAS>
 __global__ void __launch_bounds__(CV_THREADS, TAPS <= 4 ? 3 : 2) short_conv_kernel(const ConvArgs a) {
   constexpr int BATCH = cv_batch(TAPS), RUN = cv_run(TAPS);
   const int b = blockIdx.z, c = (blockIdx.x * CV_THREADS + threadIdx.x) * V;
@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(CV_THREADS, TAPS <= 4 ? 3 : 2) short_conv_kern
   fetch(t0);
   float w[TAPS][V], f[TAPS][V], bias[V];     // f: inputs of the current token, in a circle
 #pragma unroll
-  for (int i = 0; i < V; ++i) bias[i] = a.bias ? a.bias[c + i] : 0.f;
+  for (int i = 0; i < V; ++i) bias[i] = BIAS ? a.bias[c + i] : 0.f;
 #pragma unroll
   for (int j = 0; j < TAPS - 1; ++j) {       // those ahead of the run
     const int t = t0 + j - (TAPS - 1);
@@ -125,9 +125,9 @@ template <typename T> __global__ void __launch_bounds__(256) conv_keep_kernel(co
     ring[(int64_t)((ctx - 1 - j) % a.taps) * a.C] = reinterpret_cast<const T*>(a.x)[(int64_t)(row0 + count - 1 - j) * a.x_stride + c];
 }
 
-template <typename T, int V> static int conv_by_taps(const ConvArgs& a, dim3 grid, cudaStream_t st) {
+template <typename T, int V, bool BIAS> static int conv_by_taps(const ConvArgs& a, dim3 grid, cudaStream_t st) {
   switch (a.taps) {
-#define ZP_CONV(n) case n: short_conv_kernel<T, V, n><<<grid, CV_THREADS, 0, st>>>(a); break
+#define ZP_CONV(n) case n: short_conv_kernel<T, V, n, BIAS><<<grid, CV_THREADS, 0, st>>>(a); break
     ZP_CONV(1); ZP_CONV(2); ZP_CONV(3); ZP_CONV(4); ZP_CONV(5); ZP_CONV(6); ZP_CONV(7); ZP_CONV(8);
 #undef ZP_CONV
     default: return ZP_ERR_UNSUPPORTED;
@@ -154,7 +154,8 @@ extern "C" int zp_short_conv(const void* x, int64_t x_stride, const float* weigh
     const int per = zp::CV_THREADS * (vec ? V : 1), run = zp::cv_run(taps), runs = (max_seqlen_q + run - 1) / run;
     ZP_REQUIRE(runs <= 65535, "zp_short_conv: portions of %d tokens", max_seqlen_q);
     const dim3 grid((channels + per - 1) / per, runs, B);
-    rc = vec ? zp::conv_by_taps<T, V>(a, grid, st) : zp::conv_by_taps<T, 1>(a, grid, st);
+    if (bias) rc = vec ? zp::conv_by_taps<T, V, true>(a, grid, st) : zp::conv_by_taps<T, 1, true>(a, grid, st);
+    else rc = vec ? zp::conv_by_taps<T, V, false>(a, grid, st) : zp::conv_by_taps<T, 1, false>(a, grid, st);
     if (rc == ZP_OK) {
       zp::conv_keep_kernel<T><<<dim3((channels + 255) / 256, B), 256, 0, st>>>(a);
       rc = zp::check_launch("zp_short_conv(keep)");

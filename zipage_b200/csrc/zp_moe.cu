@@ -51,7 +51,7 @@ __device__ __forceinline__ float top_experts(const float* __restrict__ z, const 
       const unsigned best = __reduce_max_sync(0xffffffffu, bk);
       const unsigned at = __reduce_min_sync(0xffffffffu, bk == best ? bi : 0xffffffffu);
       bv = __shfl_sync(0xffffffffu, bv, at & 31);
-      chosen += expf(bv - mx);
+      if (score_kind == ZP_SCORE_SOFTMAX_TOP) chosen += expf(bv - mx);
       if ((int)(at & 31) == lane) {
 #pragma unroll
         for (int i = 0; i < VPL; ++i)

@@ -196,18 +196,19 @@ __device__ __forceinline__ float4 splat4(float s) { return make_float4(s, s, s, 
 
 // What joins x at entry c of a row: `add` gathers it, so that the loads of all of a thread's entries can be in
 // flight before the first of them is stored.
-template <typename T, int V>
+template <typename T, int V, bool PAIR>
 __device__ __forceinline__ float4 join_add(const JoinArgs& p, int64_t row, int c, const float* swts, const int32_t* spos, float g, float2 rp) {
   using L = JoinVec<T, V>;
   float4 add = splat4(0.f);
-  if (p.m1) {
+  if constexpr (PAIR) {
     const float4 u = L::ld(p.m1, row * p.H + c), v = L::ld(p.m2, row * p.H + c), s = L::ldf(p.mw1, c), t = L::ldf(p.mw2, c);
     add = make_float4(u.x * rp.x * s.x + v.x * rp.y * t.x, u.y * rp.x * s.y + v.y * rp.y * t.y, u.z * rp.x * s.z + v.z * rp.y * t.z,
                       u.w * rp.x * s.w + v.w * rp.y * t.w);
   }
   if (p.a) {
-    const float4 a = L::ld(p.a, row * p.H + c);
-    add = fma4(p.ls_a ? L::ldf(p.ls_a, c) : splat4(1.f), a, add);
+    float4 a = L::ld(p.a, row * p.H + c);
+    if (p.ls_a) { const float4 s = L::ldf(p.ls_a, c); a = make_float4(a.x * s.x, a.y * s.y, a.z * s.z, a.w * s.w); }
+    add = PAIR ? make_float4(add.x + a.x, add.y + a.y, add.z + a.z, add.w + a.w) : a;
   }
   if (p.b || p.y) {
     float4 f = splat4(0.f);
@@ -227,7 +228,7 @@ __device__ __forceinline__ void join_norm(const JoinArgs& p, int64_t row, int c,
 }
 
 constexpr int JOIN_TOP = 64;
-template <typename T, int VPT>
+template <typename T, int VPT, bool PAIR>
 __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
   __shared__ float red[32];
   __shared__ float swts[JOIN_TOP];
@@ -241,9 +242,9 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
     __syncthreads();
   }
   const float g = p.gate ? 1.f / (1.f + expf(-p.gate[row * p.gate_stride])) : 1.f;
-  const bool norm = p.out1 || p.out2, any = p.a || p.b || p.y || p.m1;
+  const bool norm = p.out1 || p.out2, any = PAIR || p.a || p.b || p.y;
   float2 rp = make_float2(0.f, 0.f);        // pair_scale over the root mean squares of the pair's rows
-  if (p.m1) {
+  if constexpr (PAIR) {
     constexpr int V = VPT > 0 ? 4 : 1;
     using L = JoinVec<T, V>;
     float s1 = 0.f, s2 = 0.f;
@@ -266,7 +267,7 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
       if (c < nvec) {
         const float4 x = L::ldf(p.x, row * p.H + 4 * c);
         if (!any) { v[i] = x; continue; }
-        const float4 d = join_add<T, 4>(p, row, 4 * c, swts, spos, g, rp);
+        const float4 d = join_add<T, 4, PAIR>(p, row, 4 * c, swts, spos, g, rp);
         v[i] = make_float4(x.x + d.x, x.y + d.y, x.z + d.z, x.w + d.w);
       }
     }
@@ -300,7 +301,7 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
     float s = 0.f;
     for (int c = threadIdx.x; c < p.H; c += blockDim.x) {
       float v = p.x[row * p.H + c];
-      if (any) p.x[row * p.H + c] = v += join_add<T, 1>(p, row, c, swts, spos, g, rp).x;
+      if (any) p.x[row * p.H + c] = v += join_add<T, 1, PAIR>(p, row, c, swts, spos, g, rp).x;
       s += v;
     }
     if (!norm) return;
@@ -310,6 +311,14 @@ __global__ void __launch_bounds__(256) join_norms_kernel(const JoinArgs p) {
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)p.H + p.eps);
     for (int c = threadIdx.x; c < p.H; c += blockDim.x) join_norm<T, 1>(p, row, c, make_float4(p.x[row * p.H + c] - mean, 0.f, 0.f, 0.f), r);
   }
+}
+
+template <typename T, bool PAIR> static void launch_join(const JoinArgs& p, int n_rows, bool vec, cudaStream_t st) {
+  if (!vec) join_norms_kernel<T, 0, PAIR><<<n_rows, 256, 0, st>>>(p);
+  else if (p.H <= 1024) join_norms_kernel<T, 1, PAIR><<<n_rows, 256, 0, st>>>(p);
+  else if (p.H <= 2048) join_norms_kernel<T, 2, PAIR><<<n_rows, 256, 0, st>>>(p);
+  else if (p.H <= 4096) join_norms_kernel<T, 4, PAIR><<<n_rows, 256, 0, st>>>(p);
+  else join_norms_kernel<T, 8, PAIR><<<n_rows, 256, 0, st>>>(p);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -426,11 +435,8 @@ extern "C" int zp_join_norms(float* x, const void* a, const float* ls_a, const v
   const bool vec = hidden % 4 == 0 && hidden <= 8192 && al % 16 == 0;
   cudaStream_t st = (cudaStream_t)stream;
   ZP_DISPATCH_DTYPE(dtype, T, {
-    if (!vec) zp::join_norms_kernel<T, 0><<<n_rows, 256, 0, st>>>(p);
-    else if (hidden <= 1024) zp::join_norms_kernel<T, 1><<<n_rows, 256, 0, st>>>(p);
-    else if (hidden <= 2048) zp::join_norms_kernel<T, 2><<<n_rows, 256, 0, st>>>(p);
-    else if (hidden <= 4096) zp::join_norms_kernel<T, 4><<<n_rows, 256, 0, st>>>(p);
-    else zp::join_norms_kernel<T, 8><<<n_rows, 256, 0, st>>>(p);
+    if (m1) zp::launch_join<T, true>(p, n_rows, vec, st);
+    else zp::launch_join<T, false>(p, n_rows, vec, st);
   });
   return zp::check_launch("zp_join_norms");
 }

@@ -114,7 +114,7 @@ class LinearMixer(nn.Module):
 
 
 class HGRN2Mixer(LinearMixer):
-    """Forget gates with a lower bound that also decide what is written (HGRN2)."""
+    """HGRN2: forget gates, bounded below, whose complement is the key."""
 
     def __init__(self, width, heads, dim, vdim, eps, dtype, device):
         super().__init__(width, {"q": heads * dim, "v": heads * vdim}, heads, dim, vdim, eps, dtype, device)
